@@ -38,6 +38,8 @@ class CacheNeed:
     that several key heads share).  `block_state` is a second float32 area per sequence, of that many values, for
     what the layer's block keeps from token to token beside its mixer's state (empty: 0).  `keep_first` (kind 'window'):
     every query also reads the first so many keys of its sequence, whose pages are therefore never given back.
+    `pool` (kind 'window'): beside the tokens, one key and one value is kept for every whole block of so many tokens, in
+    pages of their own (a second group); `window` then has to reach over an unfinished block too.
     """
     kind: str = "none"
     num_kv_heads: int = 0
@@ -48,6 +50,7 @@ class CacheNeed:
     value_heads: Optional[int] = None
     block_state: int = 0
     keep_first: int = 0
+    pool: int = 0
 
     def __post_init__(self):
         if self.kind not in ("full", "window", "chunk", "none"):
@@ -56,11 +59,13 @@ class CacheNeed:
             raise ValueError("a window or chunk group needs a positive size")
         if self.kind != "none" and (self.num_kv_heads <= 0 or self.head_dim <= 0):
             raise ValueError("a key/value group needs num_kv_heads and head_dim")
+        if self.pool and (self.kind != "window" or not 0 < self.pool <= self.window):
+            raise ValueError("pooled blocks go with a window that is at least as long as a block")
 
     def group_key(self):
         return (self.kind, self.num_kv_heads, self.head_dim, self.window if self.kind in ("window", "chunk") else None,
                 self.value_dim or self.head_dim, self.value_heads or self.num_kv_heads,
-                self.keep_first if self.kind == "window" else 0)
+                self.keep_first if self.kind == "window" else 0, self.pool)
 
 
 class CacheError(RuntimeError):
@@ -96,6 +101,7 @@ def _host():
         lib.q3_book_pages_held.argtypes = [ctypes.c_void_p]
         lib.q3_book_table.argtypes = [ctypes.c_void_p, ctypes.c_int]
         lib.q3_book_table.restype = i32p
+        lib.q3_book_group_pages.argtypes = [ctypes.c_void_p, ctypes.c_int]
         lib.q3_book_free_pages.argtypes = [ctypes.c_void_p, ctypes.c_int, ctypes.c_void_p]
         lib.q3_step_layout.argtypes = [ctypes.c_int] * 5 + [ctypes.c_void_p]
         lib.q3_pack_step.argtypes = [ctypes.c_void_p, ctypes.c_void_p, ctypes.c_void_p, ctypes.c_int, ctypes.c_void_p, ctypes.c_int64,
@@ -133,11 +139,12 @@ class _Slots:
 
 
 class PageGroup:
-    """The pages of the layers that share one `CacheNeed`: a view of the book's group."""
+    """The pages of the layers that share one `CacheNeed`: a view of the book's group.  `pooled`: the group holds the
+    need's blocks, one entry each, and not its tokens."""
 
-    def __init__(self, book: "CacheBook", index: int, need: CacheNeed, layers: List[int]):
-        self._book, self._index, self.need, self.layers = book, index, need, layers
-        self.n_pages = book.n_pages
+    def __init__(self, book: "CacheBook", index: int, need: CacheNeed, layers: List[int], pooled: bool = False):
+        self._book, self._index, self.need, self.layers, self.pooled = book, index, need, layers, pooled
+        self.n_pages = int(_host().q3_book_group_pages(book._handle, index))
         pointer = _host().q3_book_table(book._handle, index)
         self.table = np.ctypeslib.as_array(pointer, shape=(book.n_slots, book.pages_per_slot))   # -1: no page
 
@@ -172,11 +179,13 @@ class CacheBook:
             raise ValueError("max_tokens and max_seq_len must be positive")
         self.page_tokens = PAGE_TOKENS
         self.group_of_layer: Dict[int, int] = {}
+        self.pool_group_of_layer: Dict[int, int] = {}
         self.state_layers: Dict[int, Tuple[int, ...]] = {}
         self.block_state_layers: Dict[int, int] = {}
         by_key: Dict[tuple, int] = {}
         group_needs: List[CacheNeed] = []
         group_layers: List[List[int]] = []
+        pooled: List[bool] = []
         for layer, need in enumerate(needs):
             if need is None:
                 continue
@@ -187,16 +196,19 @@ class CacheBook:
             if need.kind == "none":
                 continue
             key = need.group_key()
-            if key not in by_key:
-                by_key[key] = len(group_needs)
-                group_needs.append(need)
-                group_layers.append([])
-            group_layers[by_key[key]].append(layer)
-            self.group_of_layer[layer] = by_key[key]
+            for blocks in ((False, True) if need.pool else (False,)):      # the tokens' group, then the blocks' group
+                if (key, blocks) not in by_key:
+                    by_key[key, blocks] = len(group_needs)
+                    group_needs.append(need)
+                    group_layers.append([])
+                    pooled.append(blocks)
+                group_layers[by_key[key, blocks]].append(layer)
+                (self.pool_group_of_layer if blocks else self.group_of_layer)[layer] = by_key[key, blocks]
         G = len(group_needs)
-        kinds = (ctypes.c_int32 * max(G, 1))(*[{"window": 1, "chunk": 2}.get(n.kind, 0) for n in group_needs])
-        windows = (ctypes.c_int32 * max(G, 1))(*[int(n.window or 0) for n in group_needs])
-        keeps = (ctypes.c_int32 * max(G, 1))(*[int(n.keep_first or 0) for n in group_needs])
+        kinds = (ctypes.c_int32 * max(G, 1))(*[3 if blocks else {"window": 1, "chunk": 2}.get(n.kind, 0)
+                                               for n, blocks in zip(group_needs, pooled)])
+        windows = (ctypes.c_int32 * max(G, 1))(*[int((n.pool if blocks else n.window) or 0) for n, blocks in zip(group_needs, pooled)])
+        keeps = (ctypes.c_int32 * max(G, 1))(*[0 if blocks else int(n.keep_first or 0) for n, blocks in zip(group_needs, pooled)])
         handle = ctypes.c_void_p()
         code = _host().q3_book_create(kinds, windows, G, int(max_tokens), int(max_seq_len), int(n_slots or 0), PAGE_TOKENS,
                                       ctypes.byref(handle), keeps)
@@ -208,7 +220,7 @@ class CacheBook:
         self.n_pages, self.n_slots, self.pages_per_slot = int(info[0]), int(info[1]), int(info[2])
         self.lengths = np.ctypeslib.as_array(_host().q3_book_lengths(self._handle), shape=(self.n_slots,))
         self.slots = _Slots(self)
-        self.groups: List[PageGroup] = [PageGroup(self, g, group_needs[g], group_layers[g]) for g in range(G)]
+        self.groups: List[PageGroup] = [PageGroup(self, g, group_needs[g], group_layers[g], pooled[g]) for g in range(G)]
 
     def __del__(self):
         handle, self._handle = getattr(self, "_handle", None), None

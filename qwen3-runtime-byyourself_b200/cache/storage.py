@@ -10,6 +10,8 @@ streams whole panels and a 2-D bulk copy can fetch one.  State rows are float32
 a second such area (`block_state`, [slot, n]).  Every group
 has one page more than its pool hands out: page number `n_pages` belongs to no
 sequence and takes the writes of the padding rows of a fixed-size decode batch.
+A layer whose need says `pool` has a second pair of areas of the same layout, in a
+group of their own, whose entries are blocks of that many tokens.
 """
 from __future__ import annotations
 
@@ -32,6 +34,9 @@ class LayerCache:
     window: Optional[int] = None
     shared: bool = False              # the view of a layer that reads another layer's cache: it must not write
     block_state: Optional[torch.Tensor] = None   # [n_slots + 1, n] float32: what the layer's block keeps per sequence
+    pool_group: Optional[int] = None             # the group of the pooled blocks, with their keys and values
+    pool_keys: Optional[torch.Tensor] = None
+    pool_values: Optional[torch.Tensor] = None
 
 
 class KVCache(CacheBook):
@@ -57,17 +62,22 @@ class KVCache(CacheBook):
         for layer, need in enumerate(needs):
             if need is None:
                 continue
-            gi = self.group_of_layer.get(layer)
-            keys = values = None
-            if gi is not None:
-                li = self.groups[gi].layers.index(layer)
-                store = self.stores[gi]
-                keys, values = (store[0][li], store[1][li]) if isinstance(store, tuple) else (store[li, 0], store[li, 1])
+            gi, pi = self.group_of_layer.get(layer), self.pool_group_of_layer.get(layer)
+            keys, values = self._areas(gi, layer)
+            pool_keys, pool_values = self._areas(pi, layer)
             self._views[layer] = LayerCache(gi, keys, values, self.states.get(layer),
                                             need.window if need.kind == "window" else None,
-                                            block_state=self.block_states.get(layer))
+                                            block_state=self.block_states.get(layer),
+                                            pool_group=pi, pool_keys=pool_keys, pool_values=pool_values)
         for layer, src in (cache_from or {}).items():
             self._views[layer] = dataclasses.replace(self._views[src], shared=True)
+
+    def _areas(self, group: Optional[int], layer: int):
+        """The keys and the values of `layer` in a group (None, None without one)."""
+        if group is None:
+            return None, None
+        li, store = self.groups[group].layers.index(layer), self.stores[group]
+        return (store[0][li], store[1][li]) if isinstance(store, tuple) else (store[li, 0], store[li, 1])
 
     def _on_alloc(self, slot: int) -> None:
         for state in list(self.states.values()) + list(self.block_states.values()):
@@ -80,4 +90,4 @@ class KVCache(CacheBook):
         item = torch.empty((), dtype=self.dtype).element_size()
         return sum(len(g.layers) * (g.need.num_kv_heads * g.need.head_dim
                                     + (g.need.value_heads or g.need.num_kv_heads) * (g.need.value_dim or g.need.head_dim)) * item
-                   for g in self.groups)
+                   // (g.need.pool if g.pooled else 1) for g in self.groups)

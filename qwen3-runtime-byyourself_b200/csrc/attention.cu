@@ -16,7 +16,10 @@
 // rotation; values of another size than keys (`vd`); scores capped smoothly,
 // s <- cap * tanh(s / cap); a window of the last keys, or the keys of the query's own chunk
 // of positions (chunks of `chunk` positions counted from 0); and a sink, one more term
-// exp(0) in the softmax's denominator that carries no value.
+// exp(0) in the softmax's denominator that carries no value.  Further: values that are the projected keys (no value
+// columns in the projection), values rotated by their own position (the caller turns the outputs back), and pooled
+// blocks beside a window: every block of `size` tokens that lies wholly before a query's window is seen as one key and
+// one value, the means of the block's cached keys and values, which `pool_blocks` makes when a block is complete.
 //
 // Cache layout: pages [page, kv head, PAGE tokens, head_dim]; `page_table[seq]` lists
 // the pages of a sequence in order.  Keys are visited page by page in ascending
@@ -42,6 +45,18 @@ template <typename T> __device__ __forceinline__ void store_pack_f32(T* p, const
     store_pack<T>(p, k);
 }
 
+template <typename T> __device__ __forceinline__ float normed(float unit, float w, int once) {
+    return once ? unit * w : round_to<T>(round_to<T>(unit) * w);
+}
+
+struct PrepareOptions {
+    int64_t row;            // values from one row of the projection to the next
+    int tied;               // the values are the projected keys: the projection has no value columns
+    int norm_once;          // a normed value is rounded once, when it is stored (else after the division and the weight too)
+    const float* v_cos;     // [positions, vd / 2] or null: values are rotated by their position, over the whole head
+    const float* v_sin;
+};
+
 template <typename T>
 __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages,
                                    T* __restrict__ v_pages, const float* __restrict__ q_norm_w,
@@ -49,7 +64,7 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_
                                    const float* __restrict__ sin_tab, const int* __restrict__ token_seq,
                                    const int* __restrict__ token_pos, const int* __restrict__ page_table,
                                    int pages_per_seq, int nq, int nkv, int d, float eps, int write_kv, int rot,
-                                   const float* __restrict__ bias, int vd, int nv) {
+                                   const float* __restrict__ bias, int vd, int nv, const PrepareOptions opt) {
     pdl_launch_dependents();
     pdl_wait();
     const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -58,9 +73,9 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_
     const int64_t t = blockIdx.y;
     const int pos = token_pos[t];
     // a row of the projection: nq query heads and nkv key heads of d values, then nv value heads of vd values
-    const int64_t row = (int64_t)(nq + nkv) * d + (int64_t)nv * vd;
-    const int64_t col0 = head < nq + nkv ? (int64_t)head * d : (int64_t)(nq + nkv) * d + (int64_t)(head - nq - nkv) * vd;
-    const T* src = qkv + t * row + col0;
+    int64_t col0 = head < nq + nkv ? (int64_t)head * d : (int64_t)(nq + nkv) * d + (int64_t)(head - nq - nkv) * vd;
+    if (opt.tied && head >= nq + nkv) col0 = (int64_t)(head - nkv) * d;
+    const T* src = qkv + t * opt.row + col0;
     if (bias != nullptr) bias += col0;
 
     T* dst;
@@ -78,7 +93,10 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_
         rotate = rotate && !is_v;
         if (is_v) {                                     // a value head: vd values that pass through
             d = vd;
-            rot = 0;
+            cos_tab = opt.v_cos;
+            sin_tab = opt.v_sin;
+            rotate = cos_tab != nullptr;
+            rot = rotate ? vd : 0;
         }
     }
 
@@ -119,15 +137,15 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_
         for (int n = 0; n < MAX_HEAD_DIM / 64; ++n) {
             const int i = lane + 32 * n;
             if (i < rhalf) {
-                a[n] = round_to<T>(round_to<T>(a[n] * inv) * norm_w[i]);
-                b[n] = round_to<T>(round_to<T>(b[n] * inv) * norm_w[i + rhalf]);
+                a[n] = normed<T>(a[n] * inv, norm_w[i], opt.norm_once);
+                b[n] = normed<T>(b[n] * inv, norm_w[i + rhalf], opt.norm_once);
             }
         }
         if (rot < d) {
 #pragma unroll
             for (int n = 0; n < MAX_HEAD_DIM / 32; ++n) {
                 const int i = rot + lane + 32 * n;
-                if (i < d) c[n] = round_to<T>(round_to<T>(c[n] * inv) * norm_w[i]);
+                if (i < d) c[n] = normed<T>(c[n] * inv, norm_w[i], opt.norm_once);
             }
         }
     }
@@ -154,22 +172,22 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_
     }
 }
 
-// The same with 16-byte accesses: a head is shared by half/VEC lanes, each of which owns VEC
-// consecutive elements of the first half and the matching VEC of the second half (the two members
-// of every rotation pair), so a warp works on several heads at once.  One warp per group of
-// consecutive (token, head) pairs.
+// The same with 16-byte accesses: a head is shared by (d/2)/VEC lanes.  The lanes of the rotated stretch own VEC
+// consecutive elements of its first half and the matching VEC of its second half (the two members of every rotation
+// pair), the lanes behind them 2 VEC consecutive elements that pass through; a warp works on several heads at once.
+// One warp per group of consecutive (token, head) pairs.
 template <typename T>
 __global__ void qkv_prepare_vec_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* __restrict__ k_pages,
                                        T* __restrict__ v_pages, const float* __restrict__ q_norm_w,
                                        const float* __restrict__ k_norm_w, const float* __restrict__ cos_tab,
                                        const float* __restrict__ sin_tab, const int* __restrict__ token_seq,
                                        const int* __restrict__ token_pos, const int* __restrict__ page_table,
-                                       int pages_per_seq, int nq, int nkv, int d, float eps, int write_kv,
-                                       int64_t n_tokens, const float* __restrict__ bias) {
+                                       int pages_per_seq, int nq, int nkv, int d, float eps, int write_kv, int rot,
+                                       int64_t n_tokens, const float* __restrict__ bias, const PrepareOptions opt) {
     constexpr int VEC = Pack<T>::N;
     pdl_launch_dependents();
     pdl_wait();
-    const int half = d >> 1, lph = half / VEC, hpw = 32 / lph;       // lanes per head, heads per warp
+    const int lph = (d >> 1) / VEC, hpw = 32 / lph;                   // lanes per head, heads per warp
     const int lane = threadIdx.x & 31, sub = lane % lph, grp = lane / lph;
     const int heads = nq + 2 * nkv;
     const int64_t warp = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -180,19 +198,26 @@ __global__ void qkv_prepare_vec_kernel(const T* __restrict__ qkv, T* __restrict_
     const bool is_q = head < nq, is_v = head >= nq + nkv;
     const bool live = active && (is_q || write_kv);
     const int pos = token_pos[t];
-    const T* src = qkv + (t * heads + head) * (int64_t)d + sub * VEC;
+    const float* cs_tab = is_v ? opt.v_cos : cos_tab;
+    const float* sn_tab = is_v ? opt.v_sin : sin_tab;
+    const int rhalf = (is_v ? d : rot) >> 1, turning = rhalf / VEC;    // a value head is rotated as a whole, or not at all
+    const bool rotate = cs_tab != nullptr && sub < turning;
+    const int a_at = sub < turning ? sub * VEC : 2 * rhalf + (sub - turning) * 2 * VEC;
+    const int b_at = sub < turning ? rhalf + sub * VEC : a_at + VEC;
+    const int col = (opt.tied && is_v ? head - nkv : head) * d;        // the head's columns in a row of the projection
+    const T* src = qkv + t * opt.row + col;
     float a[VEC], b[VEC];
 #pragma unroll
     for (int i = 0; i < VEC; ++i) a[i] = b[i] = 0.0f;
     if (live) {
-        load_pack_f32<T>(src, a);
-        load_pack_f32<T>(src + half, b);
+        load_pack_f32<T>(src + a_at, a);
+        load_pack_f32<T>(src + b_at, b);
         if (bias != nullptr) {                       // one value per column of the projection, added before anything else
-            const float* bh = bias + (int64_t)head * d + sub * VEC;
+            const float* bh = bias + col;
 #pragma unroll
             for (int i = 0; i < VEC; ++i) {
-                a[i] = round_to<T>(a[i] + bh[i]);
-                b[i] = round_to<T>(b[i] + bh[half + i]);
+                a[i] = round_to<T>(a[i] + bh[a_at + i]);
+                b[i] = round_to<T>(b[i] + bh[b_at + i]);
             }
         }
     }
@@ -208,14 +233,14 @@ __global__ void qkv_prepare_vec_kernel(const T* __restrict__ qkv, T* __restrict_
         const float inv = rsqrtf(total / (float)d + eps);
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
-            a[i] = round_to<T>(round_to<T>(a[i] * inv) * norm_w[sub * VEC + i]);
-            b[i] = round_to<T>(round_to<T>(b[i] * inv) * norm_w[half + sub * VEC + i]);
+            a[i] = normed<T>(a[i] * inv, norm_w[a_at + i], opt.norm_once);
+            b[i] = normed<T>(b[i] * inv, norm_w[b_at + i], opt.norm_once);
         }
     }
     if (!live) return;
-    if (cos_tab != nullptr && !is_v) {
-        const float* c = cos_tab + (int64_t)pos * half + sub * VEC;
-        const float* sn = sin_tab + (int64_t)pos * half + sub * VEC;
+    if (rotate) {
+        const float* c = cs_tab + (int64_t)pos * rhalf + a_at;
+        const float* sn = sn_tab + (int64_t)pos * rhalf + a_at;
 #pragma unroll
         for (int i = 0; i < VEC; ++i) {
             const float x = a[i] * c[i] - b[i] * sn[i], y = b[i] * c[i] + a[i] * sn[i];
@@ -231,9 +256,49 @@ __global__ void qkv_prepare_vec_kernel(const T* __restrict__ qkv, T* __restrict_
         const int page = page_table[(int64_t)token_seq[t] * pages_per_seq + pos / PAGE];
         dst = (is_v ? v_pages : k_pages) + (((int64_t)page * nkv + kvh) * PAGE + pos % PAGE) * d;
     }
-    store_pack_f32<T>(dst + sub * VEC, a);
-    store_pack_f32<T>(dst + half + sub * VEC, b);
+    store_pack_f32<T>(dst + a_at, a);
+    store_pack_f32<T>(dst + b_at, b);
 }
+
+// The pooled blocks that the step completes: block b of a sequence holds the tokens b size .. b size + size - 1, all of
+// them in the cache by now; its key and value are the means of theirs, and go to entry b of the sequence's pool pages.
+// One block of threads per (block of tokens, key/value head, sequence); thread i owns one key or value channel.
+template <typename T>
+__global__ void pool_blocks_kernel(const T* __restrict__ k_pages, const T* __restrict__ v_pages, const int* __restrict__ page_table,
+                                   T* __restrict__ pool_k, T* __restrict__ pool_v, const int* __restrict__ pool_table,
+                                   const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, int pages_per_seq, int nkv,
+                                   int d, int vd, int size) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int kvh = blockIdx.y, seq = blockIdx.z;
+    const int64_t pos0 = seq_pos0[seq], end = pos0 + seq_start[seq + 1] - seq_start[seq];
+    const int64_t b = pos0 / size + blockIdx.x;
+    if ((b + 1) * size > end) return;
+    const int* pages = page_table + (int64_t)seq * pages_per_seq;
+    const int64_t to = ((int64_t)pool_table[(int64_t)seq * pages_per_seq + b / PAGE] * nkv + kvh) * PAGE + b % PAGE;
+    const float inv = 1.0f / (float)size;
+    for (int i = threadIdx.x; i < d + vd; i += blockDim.x) {
+        const bool is_v = i >= d;
+        const int c = is_v ? i - d : i, width = is_v ? vd : d;
+        const T* from = (is_v ? v_pages : k_pages) + c;
+        float sum = 0.0f;
+#pragma unroll 4
+        for (int j = 0; j < size; ++j) {
+            const int64_t p = b * size + j;
+            sum += to_f32<T>(from[(((int64_t)pages[p / PAGE] * nkv + kvh) * PAGE + p % PAGE) * width]);
+        }
+        (is_v ? pool_v : pool_k)[to * width + c] = from_f32<T>(sum * inv);
+    }
+}
+
+// Pooled blocks beside a window (size 0: none): entry b of a sequence's pool pages is seen by a query whose window
+// starts at `lo` if the block's last token lies before it, that is if b < lo / size.
+template <typename T> struct PoolView {
+    const T* k;
+    const T* v;
+    const int* table;           // [sequences, pages_per_seq]
+    int size;
+};
 
 // One block per (query head, token).  128 threads: the four warps share the keys of a
 // page for the scores; thread t owns output dims t, t + 128, t + 256 and t + 384.  Keys up to GENERIC_KEY_DIM and
@@ -244,7 +309,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
                          T* __restrict__ out, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                          const int* __restrict__ page_table, int pages_per_seq, int nq, int nkv, int d, float scale,
                          int window, int vd, float softcap, int chunk, int sink, int nv, int out_f32,
-                         const float* __restrict__ sink_values, int keep_first) {
+                         const float* __restrict__ sink_values, int keep_first, const PoolView<T> pool) {
     __shared__ float q_s[GENERIC_KEY_DIM];
     __shared__ float score[PAGE];
     __shared__ float prob[PAGE];
@@ -267,13 +332,20 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
     const float inv_cap = softcap > 0.0f ? 1.0f / softcap : 0.0f;
     // with a window, the first `keep_first` keys of the sequence stay visible: their pages come first, then the window's
     const int keep = window > 0 ? keep_first : 0;
-    for (int pg = 0; pg <= pos / PAGE; ++pg) {
-        if (pg < lo / PAGE && pg * PAGE >= keep) continue;          // nothing of this page is seen (it may be given back)
-        const T* kp = k_pages + ((int64_t)pages[pg] * nkv + kvh) * PAGE * d;
-        const T* vp = v_pages + ((int64_t)pages[pg] * nv + vh) * PAGE * vd;
-        const int j_hi = min(pos - pg * PAGE, PAGE - 1);            // inclusive, in-page
-        const int j_lo = pg * PAGE < keep ? 0 : max(lo - pg * PAGE, 0);
-        const int gap_lo = keep - pg * PAGE, gap_hi = lo - pg * PAGE;   // keys j with gap_lo <= j < gap_hi are not seen
+    // the pooled blocks' pages come first of all
+    const int n_blocks = pool.size > 0 ? lo / pool.size : 0, pool_pages = (n_blocks + PAGE - 1) / PAGE;
+    const int* pool_list = pool.size > 0 ? pool.table + (int64_t)token_seq[t] * pages_per_seq : nullptr;
+    for (int x = 0; x <= pool_pages + pos / PAGE; ++x) {
+        const bool pooled = x < pool_pages;
+        const int pg = pooled ? x : x - pool_pages;
+        if (!pooled && pg < lo / PAGE && pg * PAGE >= keep) continue;   // nothing of this page is seen (it may be given back)
+        const int page = pooled ? pool_list[pg] : pages[pg];
+        const T* kp = (pooled ? pool.k : k_pages) + ((int64_t)page * nkv + kvh) * PAGE * d;
+        const T* vp = (pooled ? pool.v : v_pages) + ((int64_t)page * nv + vh) * PAGE * vd;
+        const int j_hi = min((pooled ? n_blocks - 1 : pos) - pg * PAGE, PAGE - 1);            // inclusive, in-page
+        const int j_lo = pooled || pg * PAGE < keep ? 0 : max(lo - pg * PAGE, 0);
+        const int gap_lo = pooled ? PAGE : keep - pg * PAGE;            // keys j with gap_lo <= j < gap_hi are not seen
+        const int gap_hi = pooled ? PAGE : lo - pg * PAGE;
         for (int j = warp; j < PAGE; j += 4) {
             float dot = 0.0f;
             if (j >= j_lo && j <= j_hi && !(j >= gap_lo && j < gap_hi)) {
@@ -320,7 +392,7 @@ template <typename T>
 int qkv_prepare_launch(const T* qkv, T* q_out, T* k_pages, T* v_pages, const float* q_norm_w, const float* k_norm_w,
                        const float* cos_tab, const float* sin_tab, const int* token_seq, const int* token_pos,
                        const int* page_table, int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d, float eps,
-                       int write_kv, int rot, const float* bias, int vd, int nv, cudaStream_t stream) {
+                       int write_kv, int rot, const float* bias, int vd, int nv, PrepareOptions opt, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (nv <= 0) nv = nkv;                       // as many value heads as key heads
     if (d <= 0 || d > MAX_HEAD_DIM || nq <= 0 || nkv <= 0 || nkv % nv != 0) return Q3_ERR_BAD_SIZE;
@@ -329,31 +401,38 @@ int qkv_prepare_launch(const T* qkv, T* q_out, T* k_pages, T* v_pages, const flo
     if (rot % 2 != 0) rot = 0;                   // an odd head without tables: every value passes through
     if (vd <= 0) vd = d;                         // values as wide as keys
     if (vd > MAX_HEAD_DIM) return Q3_ERR_BAD_SIZE;
+    const int64_t columns = (int64_t)(nq + nkv) * d + (opt.tied ? 0 : (int64_t)nv * vd);
+    if (opt.row <= 0) opt.row = columns;
+    if (opt.row < columns || (opt.tied && (vd != d || nv != nkv)) || (opt.v_cos == nullptr) != (opt.v_sin == nullptr) ||
+        (opt.v_cos != nullptr && vd % 2 != 0))
+        return Q3_ERR_BAD_SIZE;
     constexpr int VEC = Pack<T>::N;
-    if (rot == d && vd == d && nv == nkv && n_tokens >= 64 && (d / 2) % VEC == 0 && (d / 2) / VEC <= 32 && aligned16(qkv) && aligned16(q_out) &&
-        aligned16(k_pages) && aligned16(v_pages)) {
+    if ((rot / 2) % VEC == 0 && (d - rot) % (2 * VEC) == 0 && rot % 2 == 0 && vd == d && nv == nkv && n_tokens >= 64 && (d / 2) % VEC == 0 &&
+        (d / 2) / VEC <= 32 && opt.row % VEC == 0 && aligned16(qkv) && aligned16(q_out) && aligned16(k_pages) && aligned16(v_pages)) {
         const int hpw = 32 / ((d / 2) / VEC);
         const int64_t n_warps = (n_tokens * (nq + 2 * nkv) + hpw - 1) / hpw;
         const int64_t blocks = (n_warps + 7) / 8;
         if (blocks > 0x7fffffffLL) return Q3_ERR_TOO_LARGE;
         return (int)q3_launch(qkv_prepare_vec_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, qkv, q_out, k_pages,
                               v_pages, q_norm_w, k_norm_w, cos_tab, sin_tab, token_seq, token_pos, page_table, pages_per_seq,
-                              nq, nkv, d, eps, write_kv, n_tokens, bias);
+                              nq, nkv, d, eps, write_kv, rot, n_tokens, bias, opt);
     }
     if (n_tokens > 65535) return Q3_ERR_TOO_LARGE;
     const int warps = 4;
     const dim3 grid((nq + nkv + nv + warps - 1) / warps, (unsigned)n_tokens);
     return (int)q3_launch(qkv_prepare_kernel<T>, grid, dim3(warps * 32), 0, stream, qkv, q_out, k_pages, v_pages, q_norm_w,
                           k_norm_w, cos_tab, sin_tab, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, d, eps, write_kv, rot,
-                          bias, vd, nv);
+                          bias, vd, nv, opt);
 }
 
 template <typename T>
 int attention_generic_launch(const T* q, const T* k_pages, const T* v_pages, T* out, const int* token_seq,
                              const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq,
                              int nkv, int d, float scale, int window, int vd, float softcap, int chunk, int sink, int nv,
-                             int out_f32, const float* sink_values, int keep_first, cudaStream_t stream) {
+                             int out_f32, const float* sink_values, int keep_first, PoolView<T> pool, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (pool.size < 0 || (pool.size > 0 && (window <= 0 || keep_first > 0 || pool.k == nullptr || pool.v == nullptr || pool.table == nullptr)))
+        return Q3_ERR_BAD_SIZE;
     if (vd <= 0) vd = d;
     if (nv <= 0) nv = nkv;
     if (nkv <= 0 || nkv % nv != 0) return Q3_ERR_BAD_SIZE;
@@ -363,7 +442,20 @@ int attention_generic_launch(const T* q, const T* k_pages, const T* v_pages, T* 
     const dim3 grid(nq, (unsigned)n_tokens);
     return (int)q3_launch(attention_generic_kernel<T>, grid, dim3(128), 0, stream, q, k_pages, v_pages, out, token_seq,
                           token_pos, page_table, pages_per_seq, nq, nkv, d, scale, window, vd, softcap, chunk, sink, nv, out_f32, sink_values,
-                          keep_first);
+                          keep_first, pool);
+}
+
+template <typename T>
+int pool_blocks_launch(const T* k_pages, const T* v_pages, const int* page_table, T* pool_k, T* pool_v, const int* pool_table,
+                       const int* seq_start, const int* seq_pos0, int pages_per_seq, int n_seqs, int max_new, int nkv, int d, int vd,
+                       int size, cudaStream_t stream) {
+    if (n_seqs <= 0 || max_new <= 0) return 0;
+    if (nkv <= 0 || d <= 0 || vd <= 0 || size <= 0) return Q3_ERR_BAD_SIZE;
+    if (n_seqs > 65535 || nkv > 65535) return Q3_ERR_TOO_LARGE;
+    // a step of n tokens completes at most n / size blocks, and one more that an earlier step began
+    const int threads = d + vd <= 64 ? 64 : (d + vd <= 128 ? 128 : 256);
+    return (int)q3_launch(pool_blocks_kernel<T>, dim3((unsigned)(max_new / size + 1), nkv, n_seqs), dim3(threads), 0, stream, k_pages, v_pages,
+                          page_table, pool_k, pool_v, pool_table, seq_start, seq_pos0, pages_per_seq, nkv, d, vd, size);
 }
 
 // Values blended across layers, on the value columns of a projection's rows (in place): v <- v + bias first (if
@@ -418,6 +510,64 @@ __global__ void head_gate_kernel(T* __restrict__ x, const T* __restrict__ gate, 
     }
 }
 
+// The heads of an attention's output, in place: turned back by the query's position (pairs (i, i + vd/2), tables
+// [positions, vd/2]; null: not turned) and multiplied value by value by sigmoid(gate) (null: no gate).
+template <typename T, int VEC>
+__global__ void turn_back_gate_kernel(T* __restrict__ x, const float* __restrict__ cos_tab, const float* __restrict__ sin_tab,
+                                      const int* __restrict__ token_pos, const T* __restrict__ gate, int64_t gate_row, int heads, int vd,
+                                      int64_t n_tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int half = vd >> 1, per_head = half / VEC;
+    const int64_t total = n_tokens * heads * per_head;
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+        const int64_t th = i / per_head, t = th / heads;
+        const int c = (int)(i % per_head) * VEC, h = (int)(th % heads);
+        T* at = x + th * vd + c;
+        float a[VEC], b[VEC];
+        if constexpr (VEC == 1) {
+            a[0] = to_f32<T>(at[0]);
+            b[0] = to_f32<T>(at[half]);
+        } else {
+            load_pack_f32<T>(at, a);
+            load_pack_f32<T>(at + half, b);
+        }
+        if (cos_tab != nullptr) {
+            const float* cs = cos_tab + (int64_t)token_pos[t] * half + c;
+            const float* sn = sin_tab + (int64_t)token_pos[t] * half + c;
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) {
+                const float u = a[k] * cs[k] + b[k] * sn[k], v = b[k] * cs[k] - a[k] * sn[k];
+                a[k] = u;
+                b[k] = v;
+            }
+        }
+        if (gate != nullptr) {
+            const T* g = gate + t * gate_row + (int64_t)h * vd + c;
+            float ga[VEC], gb[VEC];
+            if constexpr (VEC == 1) {
+                ga[0] = to_f32<T>(g[0]);
+                gb[0] = to_f32<T>(g[half]);
+            } else {
+                load_pack_f32<T>(g, ga);
+                load_pack_f32<T>(g + half, gb);
+            }
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) {
+                a[k] *= 1.0f / (1.0f + expf(-ga[k]));
+                b[k] *= 1.0f / (1.0f + expf(-gb[k]));
+            }
+        }
+        if constexpr (VEC == 1) {
+            at[0] = from_f32<T>(a[0]);
+            at[half] = from_f32<T>(b[0]);
+        } else {
+            store_pack_f32<T>(at, a);
+            store_pack_f32<T>(at + half, b);
+        }
+    }
+}
+
 template <typename Kernel, typename... Args>
 int launch_flat(Kernel kernel, int64_t work, cudaStream_t stream, Args... args) {
     int64_t blocks = (work + 255) / 256;
@@ -434,21 +584,49 @@ int launch_flat(Kernel kernel, int64_t work, cudaStream_t stream, Args... args) 
                                           const float* sin_tab, const int* token_seq, const int* token_pos,           \
                                           const int* page_table, int pages_per_seq, int64_t n_tokens, int nq,         \
                                           int nkv, int d, float eps, int write_kv, int rotary_dim,           \
-                                          const float* bias, int value_dim, int value_heads, void* stream) {          \
+                                          const float* bias, int value_dim, int value_heads, int64_t row,             \
+                                          int tied_values, int norm_once, const float* v_cos, const float* v_sin,     \
+                                          void* stream) {                                                             \
+        PrepareOptions opt;                                                                                           \
+        opt.row = row; opt.tied = tied_values; opt.norm_once = norm_once; opt.v_cos = v_cos; opt.v_sin = v_sin;       \
         return qkv_prepare_launch<T>((const T*)qkv, (T*)q_out, (T*)k_pages, (T*)v_pages, q_norm_w, k_norm_w, cos_tab, \
                                      sin_tab, token_seq, token_pos, page_table, pages_per_seq, n_tokens, nq, nkv, d,  \
-                                     eps, write_kv, rotary_dim, bias, value_dim, value_heads, (cudaStream_t)stream);  \
+                                     eps, write_kv, rotary_dim, bias, value_dim, value_heads, opt,                    \
+                                     (cudaStream_t)stream);                                                           \
+    }                                                                                                                 \
+    Q3_EXPORT int q3_pool_blocks_##SUFFIX(const void* k_pages, const void* v_pages, const int* page_table, void* pool_k, \
+                                          void* pool_v, const int* pool_table, const int* seq_start,                  \
+                                          const int* seq_pos0, int pages_per_seq, int n_seqs, int max_new, int nkv,   \
+                                          int d, int value_dim, int size, void* stream) {                             \
+        return pool_blocks_launch<T>((const T*)k_pages, (const T*)v_pages, page_table, (T*)pool_k, (T*)pool_v,        \
+                                     pool_table, seq_start, seq_pos0, pages_per_seq, n_seqs, max_new, nkv, d,         \
+                                     value_dim, size, (cudaStream_t)stream);                                          \
+    }                                                                                                                 \
+    Q3_EXPORT int q3_turn_back_gate_##SUFFIX(void* x, const float* cos_tab, const float* sin_tab, const int* token_pos, \
+                                             const void* gate, int64_t gate_row, int heads, int vd, int64_t n_tokens, \
+                                             void* stream) {                                                          \
+        if (n_tokens <= 0) return 0;                                                                                  \
+        if (heads <= 0 || vd <= 0 || vd % 2 != 0 || (cos_tab == nullptr) != (sin_tab == nullptr)) return Q3_ERR_BAD_SIZE; \
+        constexpr int V = Pack<T>::N;                                                                                 \
+        if ((vd / 2) % V == 0 && aligned16(x) && (gate == nullptr || (gate_row % V == 0 && aligned16(gate))))         \
+            return launch_flat(turn_back_gate_kernel<T, V>, n_tokens * heads * (vd / 2 / V), (cudaStream_t)stream,    \
+                               (T*)x, cos_tab, sin_tab, token_pos, (const T*)gate, gate_row, heads, vd, n_tokens);    \
+        return launch_flat(turn_back_gate_kernel<T, 1>, n_tokens * heads * (vd / 2), (cudaStream_t)stream, (T*)x,     \
+                           cos_tab, sin_tab, token_pos, (const T*)gate, gate_row, heads, vd, n_tokens);               \
     }                                                                                                                 \
     Q3_EXPORT int q3_attention_generic_##SUFFIX(const void* q, const void* k_pages, const void* v_pages, void* out,   \
                                                 const int* token_seq, const int* token_pos, const int* page_table,    \
                                                 int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d,          \
                                                 float scale, int window, int value_dim, float softcap,     \
                                                 int chunk, int sink, int value_heads, int out_f32,                   \
-                                                const float* sink_values, int keep_first, void* stream) {             \
+                                                const float* sink_values, int keep_first, const void* pool_k,         \
+                                                const void* pool_v, const int* pool_table, int pool_size,             \
+                                                void* stream) {                                                       \
+        const PoolView<T> pool = {(const T*)pool_k, (const T*)pool_v, pool_table, pool_size};                         \
         return attention_generic_launch<T>((const T*)q, (const T*)k_pages, (const T*)v_pages, (T*)out, token_seq,     \
                                            token_pos, page_table, pages_per_seq, n_tokens, nq, nkv, d, scale, window, \
                                            value_dim, softcap, chunk, sink, value_heads, out_f32, sink_values,        \
-                                           keep_first, (cudaStream_t)stream);                                         \
+                                           keep_first, pool, (cudaStream_t)stream);                                   \
     }                                                                                                                 \
     Q3_EXPORT int q3_value_mix_##SUFFIX(void* rows, int64_t row, int64_t v_off, int width, const float* bias,         \
                                         void* first, int save, float lambda, int64_t n_tokens, void* stream) {        \

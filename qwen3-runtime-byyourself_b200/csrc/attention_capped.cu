@@ -6,6 +6,10 @@
 //     j visible from i:  j <= i  and  floor(j / chunk) == floor(i / chunk)       (chunk = 0: j <= i)
 //                        or, with a window: j <= i  and  (i - j < window  or  j < keep), keep the number of first keys
 //                        of a sequence that stay visible (their pages are walked before the window's)
+//                        and, with pooled blocks of P tokens beside a window, one key and one value for every block that
+//                        ends before the window: block b = the tokens bP .. bP + P - 1 is seen from i if b < lo / P with
+//                        lo the window's first key; its key and value, the means of its tokens', lie in pages of
+//                        their own, which are walked before the window's
 //     p_j = exp(s_j) / (sink + sum_visible exp(s_j)),  sink = 1 or 0
 //     o   = sum_j p_j v_j
 //
@@ -95,6 +99,14 @@ __device__ __forceinline__ int chunk_start(int pos, int chunk) {
     return chunk > 0 ? pos / chunk * chunk : (chunk < 0 ? max(pos + chunk + 1, 0) : 0);
 }
 
+// Pooled blocks beside a window (size 0: none): entry b of a sequence's pages in `table` is block b.
+struct PoolArgs {
+    const bf16* k;
+    const bf16* v;
+    const int* table;           // [sequences, pages_per_seq]
+    int size;
+};
+
 template <typename TO> __device__ __forceinline__ void store_pair(TO* p, float a, float b);
 template <> __device__ __forceinline__ void store_pair<bf16>(bf16* p, float a, float b) {
     *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b);
@@ -118,12 +130,12 @@ constexpr int BM = 64;
 constexpr int K_TILE = PAGE * K_ROW, V_TILE = PAGE * V_ROW;
 constexpr int PREFILL_SMEM = 2 * (K_TILE + V_TILE);
 
-template <typename TO>
+template <typename TO, bool POOL>
 __global__ void __launch_bounds__(WARPS * 32)
 prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                       TO* __restrict__ out, const int* __restrict__ seq_start, const int* __restrict__ seq_pos0,
                       const int* __restrict__ page_table, int pages_per_seq, int nq, int nkv, float scale, float cap, int chunk,
-                      int sink, int nv, const float* __restrict__ sink_values, int keep) {
+                      int sink, int nv, const float* __restrict__ sink_values, int keep, const PoolArgs pool) {
     extern __shared__ __align__(16) unsigned char smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -164,19 +176,26 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
     const int pg_begin = chunk_start(pos0 + tile * BM, chunk) / PAGE, pg_end = (pos0 + last_row) / PAGE + 1;
     // with a window, the first `keep` keys of the sequence stay visible: the pages that hold them and lie before the
     // window's come first; step i of the walk is page i if i < n_keep, else page pg_begin + i - n_keep
-    const int n_keep = min((keep + PAGE - 1) / PAGE, pg_begin), n_walk = n_keep + pg_end - pg_begin;
+    // (or the pages of the pooled blocks that the tile's last row sees: these hold blocks, not tokens)
+    constexpr bool pooling = POOL;
+    const int last_block = pooling ? chunk_start(pos0 + last_row, chunk) / pool.size : 0;
+    const int n_keep = pooling ? (last_block + PAGE - 1) / PAGE : min((keep + PAGE - 1) / PAGE, pg_begin), n_walk = n_keep + pg_end - pg_begin;
+    const int b_lo = pooling ? c_lo / pool.size : 0, b_hi = pooling ? c_hi / pool.size : 0;    // blocks that each row sees
+    const int* pool_list = pooling ? pool.table + (int64_t)seq * pages_per_seq : pages;
     const int warp_first_pos = pos0 + tile * BM + warp * 16;                   // lowest position of the warp's rows
     const int warp_first_key = chunk_start(warp_first_pos, chunk);             // no row of the warp sees a key before it
     const int warp_last_start = chunk_start(warp_first_pos + 15, chunk);       // from here on every row of the warp may see
+    const int warp_first_block = pooling ? warp_first_key / pool.size : 0, warp_last_block = pooling ? warp_last_start / pool.size : 0;
     const uint32_t base = smem_u32(smem);
 
     auto issue = [&](int i) {
         if (i < n_walk) {
-            const int pg = i < n_keep ? i : pg_begin + i - n_keep;
-            const int64_t k_at = ((int64_t)pages[pg] * nkv + kvh) * PAGE, v_at = ((int64_t)pages[pg] * nv + vh) * PAGE;
+            const bool blocks = pooling && i < n_keep;
+            const int page = i < n_keep ? pool_list[i] : pages[pg_begin + i - n_keep];
+            const int64_t k_at = ((int64_t)page * nkv + kvh) * PAGE, v_at = ((int64_t)page * nv + vh) * PAGE;
             const uint32_t dst = base + (i & 1) * (K_TILE + V_TILE);
-            load_rows<PAGE, D, K_ROW, WARPS * 32>(dst, k_pages + k_at * D, threadIdx.x);
-            load_rows<PAGE, VD, V_ROW, WARPS * 32>(dst + K_TILE, v_pages + v_at * VD, threadIdx.x);
+            load_rows<PAGE, D, K_ROW, WARPS * 32>(dst, (blocks ? pool.k : k_pages) + k_at * D, threadIdx.x);
+            load_rows<PAGE, VD, V_ROW, WARPS * 32>(dst + K_TILE, (blocks ? pool.v : v_pages) + v_at * VD, threadIdx.x);
         }
         cp_async_commit();
     };
@@ -190,7 +209,10 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
         const int key_base = pg * PAGE;
         // a warp whose rows all lie before this page, or whose chunks all start behind it, has nothing to see in it
         // (but for the kept keys)
-        if (key_base <= warp_first_pos + 15 && (key_base + PAGE > warp_first_key || key_base < keep)) {
+        const bool blocks = pooling && i < n_keep;             // the page's entries are pooled blocks
+        const bool needed = blocks ? key_base < warp_last_block
+                                   : key_base <= warp_first_pos + 15 && (key_base + PAGE > warp_first_key || key_base < keep);
+        if (needed) {
             float s[8][4];
 #pragma unroll
             for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
@@ -205,7 +227,7 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
                     mma_bf16(s[2 * jp + 1], qa[kt], b[2], b[3]);
                 }
             }
-            const bool edge = key_base + PAGE - 1 > warp_first_pos || key_base < warp_last_start;
+            const bool edge = blocks ? key_base + PAGE > warp_first_block : key_base + PAGE - 1 > warp_first_pos || key_base < warp_last_start;
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int j = 0; j < 8; ++j)
@@ -214,7 +236,7 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
                     float v = score_log2(s[j][e], scale, cap, inv_cap);
                     if (edge) {
                         const int key = key_base + j * 8 + tq * 2 + (e & 1);
-                        const bool seen = (e >> 1) ? (key <= p_hi && (key >= c_hi || key < keep)) : (key <= p_lo && (key >= c_lo || key < keep));
+                        const bool seen = blocks ? key < ((e >> 1) ? b_hi : b_lo) : (e >> 1) ? (key <= p_hi && (key >= c_hi || key < keep)) : (key <= p_lo && (key >= c_lo || key < keep));
                         v = seen ? v : -INFINITY;
                     }
                     s[j][e] = v;
@@ -329,12 +351,12 @@ __device__ __forceinline__ void prepare_head(const bf16* __restrict__ src, const
 
 // part: [tokens, nq, splits, VD + 2] float32: the unnormalised sums, then the maximum (base-2 scale) and the denominator.
 // FUSED: `q` is unused; the pages are written by the block that holds the token's own page.
-template <bool FUSED>
+template <bool FUSED, bool POOL>
 __global__ void __launch_bounds__(WARPS * 32)
 decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, const bf16* v_pages,
                            float* __restrict__ part, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                            const int* __restrict__ page_table, int pages_per_seq, int nq, int nkv, float scale, float cap,
-                           int chunk, const FusedArgs fused, int nv, int keep) {
+                           int chunk, const FusedArgs fused, int nv, int keep, const PoolArgs pool) {
     extern __shared__ __align__(16) unsigned char smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -347,7 +369,11 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
     const int lo = chunk_start(pos, chunk);
     // with a window, the pages of the first `keep` keys that lie before the window's pages are walked first: step x of
     // the walk is page x if x < n_keep, else page first_page + x - n_keep; the splits share the steps
-    const int first_page = lo / PAGE, n_keep = min((keep + PAGE - 1) / PAGE, first_page);
+    // (or the pages of the pooled blocks, whose entries are blocks)
+    constexpr bool pooling = POOL;
+    const int n_blocks = pooling ? lo / pool.size : 0;
+    const int first_page = lo / PAGE, n_keep = pooling ? (n_blocks + PAGE - 1) / PAGE : min((keep + PAGE - 1) / PAGE, first_page);
+    const int* pool_list = pooling ? pool.table + (int64_t)token_seq[t] * pages_per_seq : pages;
     const int n_pages = n_keep + pos / PAGE + 1 - first_page;
     const int per_split = (n_pages + n_splits - 1) / n_splits;
     const int pg_begin = split * per_split;
@@ -358,12 +384,13 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
     const uint32_t pipe = smem_u32(smem) + warp * (STAGES * (K_PANEL + V_PANEL));
     auto issue = [&](int i) {
         if (i < count) {
-            const int page = pages[page_of(pg_begin + i)];
+            const bool blocks = pooling && pg_begin + i < n_keep;
+            const int page = (blocks ? pool_list : pages)[page_of(pg_begin + i)];
             const int64_t at = ((int64_t)page * nkv + kvh) * PAGE + warp * KEYS_PER_WARP;
             const int64_t v_at = ((int64_t)page * nv + kvh / (nkv / nv)) * PAGE + warp * KEYS_PER_WARP;
             const uint32_t dst = pipe + (i % STAGES) * (K_PANEL + V_PANEL);
-            load_rows<KEYS_PER_WARP, D, K_ROW, 32>(dst, k_pages + at * D, lane);
-            load_rows<KEYS_PER_WARP, VD, V_ROW, 32>(dst + K_PANEL, v_pages + v_at * VD, lane);
+            load_rows<KEYS_PER_WARP, D, K_ROW, 32>(dst, (blocks ? pool.k : k_pages) + at * D, lane);
+            load_rows<KEYS_PER_WARP, VD, V_ROW, 32>(dst + K_PANEL, (blocks ? pool.v : v_pages) + v_at * VD, lane);
         }
         cp_async_commit();
     };
@@ -443,15 +470,17 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
             mma_bf16(s[0], qa[kt], b[0], b[1]);
             mma_bf16(s[1], qa[kt], b[2], b[3]);
         }
-        // key index of s[j][e]: page*64 + warp*16 + j*8 + tq*2 + (e & 1); keys outside [lo, pos] are not seen
+        // key index of s[j][e]: page*64 + warp*16 + j*8 + tq*2 + (e & 1); keys outside [lo, pos] (blocks from n_blocks on) are not seen
         const int key0 = page_of(pg_begin + i) * PAGE + warp * KEYS_PER_WARP + tq * 2;
+        const bool blocks = pooling && pg_begin + i < n_keep;
+        const int seen_from = blocks ? 0 : lo, seen_to = blocks ? n_blocks - 1 : last_key;
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
         for (int j = 0; j < 2; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = key0 + j * 8 + (e & 1);
-                const float v = ((key >= lo || key < keep) && key <= last_key) ? score_log2(s[j][e], scale, cap, inv_cap) : -INFINITY;
+                const float v = ((key >= seen_from || key < keep) && key <= seen_to) ? score_log2(s[j][e], scale, cap, inv_cap) : -INFINITY;
                 s[j][e] = v;
                 mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }
@@ -577,6 +606,11 @@ __global__ void decode_capped_merge_kernel(const float* __restrict__ part, TO* _
 
 }  // namespace
 
+static bool pool_fits(const void* k, const void* v, const int* table, int size, int window, int keep_first) {
+    if (size == 0) return true;
+    return size > 0 && k != nullptr && v != nullptr && table != nullptr && window > 0 && keep_first == 0;
+}
+
 Q3_EXPORT int q3_attention_capped_head_dim() { return D; }
 Q3_EXPORT int q3_attention_capped_value_dim() { return VD; }
 
@@ -585,29 +619,32 @@ Q3_EXPORT int q3_attention_capped_prefill_bf16(const void* q, const void* k_page
                                                const int* seq_start, const int* seq_pos0, const int* page_table,
                                                int pages_per_seq, int n_seqs, int max_new, int nq, int nkv, float scale,
                                                float softcap, int chunk, int sink, int window, int value_heads, int out_f32,
-                                               const float* sink_values, int keep_first, void* stream) {
+                                               const float* sink_values, int keep_first, const void* pool_k, const void* pool_v,
+                                               const int* pool_table, int pool_size, void* stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
-    if (keep_first < 0 || (keep_first > 0 && window <= 0)) return Q3_ERR_BAD_SIZE;
+    if (keep_first < 0 || (keep_first > 0 && window <= 0) || !pool_fits(pool_k, pool_v, pool_table, pool_size, window, keep_first))
+        return Q3_ERR_BAD_SIZE;
+    const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size};
     if (value_heads <= 0) value_heads = nkv;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nkv % value_heads != 0 || softcap < 0.0f || chunk < 0 || window < 0 ||
         (chunk > 0 && window > 0))
         return Q3_ERR_BAD_SIZE;
     if (n_seqs > 65535 || nq > 65535) return Q3_ERR_TOO_LARGE;
     const int span = window > 0 ? -window : chunk;             // see chunk_start
-    static Q3PerDevice configured[2];
+    static Q3PerDevice configured[4];
     const dim3 grid((max_new + BM - 1) / BM, nq, n_seqs);
-    if (out_f32) {
-        cudaError_t e = q3_allow_shared_memory(prefill_capped_kernel<float>, PREFILL_SMEM, configured[1]);
+    auto launch = [&](auto kernel, auto* to, Q3PerDevice& state) {
+        const cudaError_t e = q3_allow_shared_memory(kernel, PREFILL_SMEM, state);
         if (e != cudaSuccess) return (int)e;
-        return (int)q3_launch(prefill_capped_kernel<float>, grid, dim3(WARPS * 32), PREFILL_SMEM, (cudaStream_t)stream, (const bf16*)q,
-                              (const bf16*)k_pages, (const bf16*)v_pages, (float*)out, seq_start, seq_pos0, page_table,
-                              pages_per_seq, nq, nkv, scale, softcap, span, sink, value_heads, sink_values, keep_first);
-    }
-    cudaError_t e = q3_allow_shared_memory(prefill_capped_kernel<bf16>, PREFILL_SMEM, configured[0]);
-    if (e != cudaSuccess) return (int)e;
-    return (int)q3_launch(prefill_capped_kernel<bf16>, grid, dim3(WARPS * 32), PREFILL_SMEM, (cudaStream_t)stream, (const bf16*)q,
-                          (const bf16*)k_pages, (const bf16*)v_pages, (bf16*)out, seq_start, seq_pos0, page_table,
-                          pages_per_seq, nq, nkv, scale, softcap, span, sink, value_heads, sink_values, keep_first);
+        return (int)q3_launch(kernel, grid, dim3(WARPS * 32), PREFILL_SMEM, (cudaStream_t)stream, (const bf16*)q, (const bf16*)k_pages,
+                              (const bf16*)v_pages, to, seq_start, seq_pos0, page_table, pages_per_seq, nq, nkv, scale, softcap, span,
+                              sink, value_heads, sink_values, keep_first, pool);
+    };
+    if (pool_size > 0)
+        return out_f32 ? launch(prefill_capped_kernel<float, true>, (float*)out, configured[3])
+                       : launch(prefill_capped_kernel<bf16, true>, (bf16*)out, configured[2]);
+    return out_f32 ? launch(prefill_capped_kernel<float, false>, (float*)out, configured[1])
+                   : launch(prefill_capped_kernel<bf16, false>, (bf16*)out, configured[0]);
 }
 
 // One new token per sequence: scratch holds n_tokens * nq * n_splits * (VD + 2) float32.
@@ -615,24 +652,29 @@ Q3_EXPORT int q3_attention_capped_decode_bf16(const void* q, const void* k_pages
                                               const int* token_seq, const int* token_pos, const int* page_table,
                                               int pages_per_seq, int64_t n_tokens, int nq, int nkv, float scale, float softcap,
                                               int chunk, int sink, int n_splits, int window, int value_heads, int out_f32,
-                                              const float* sink_values, int keep_first, void* stream) {
+                                              const float* sink_values, int keep_first, const void* pool_k, const void* pool_v,
+                                              const int* pool_table, int pool_size, void* stream) {
     if (n_tokens <= 0) return 0;
-    if (keep_first < 0 || (keep_first > 0 && window <= 0)) return Q3_ERR_BAD_SIZE;
+    if (keep_first < 0 || (keep_first > 0 && window <= 0) || !pool_fits(pool_k, pool_v, pool_table, pool_size, window, keep_first))
+        return Q3_ERR_BAD_SIZE;
+    const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size};
     if (value_heads <= 0) value_heads = nkv;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || nkv % value_heads != 0 || softcap < 0.0f || chunk < 0 ||
         window < 0 || (chunk > 0 && window > 0) || n_splits <= 0)
         return Q3_ERR_BAD_SIZE;
     const int span = window > 0 ? -window : chunk;             // see chunk_start
     if (n_tokens > 65535 || nkv > 65535 || nq > 0x7fffffff / 2) return Q3_ERR_TOO_LARGE;
-    static Q3PerDevice configured;
-    {
-        cudaError_t e = q3_allow_shared_memory(decode_capped_split_kernel<false>, DECODE_SMEM, configured);
-        if (e != cudaSuccess) return (int)e;
-    }
-    FusedArgs none = {};
-    cudaError_t e = q3_launch(decode_capped_split_kernel<false>, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32), DECODE_SMEM,
-                              (cudaStream_t)stream, (const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, scratch, token_seq,
-                              token_pos, page_table, pages_per_seq, nq, nkv, scale, softcap, span, none, value_heads, keep_first);
+    static Q3PerDevice configured[2];
+    const FusedArgs none = {};
+    auto launch = [&](auto kernel, Q3PerDevice& state) {
+        const cudaError_t e = q3_allow_shared_memory(kernel, DECODE_SMEM, state);
+        if (e != cudaSuccess) return e;
+        return q3_launch(kernel, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32), DECODE_SMEM, (cudaStream_t)stream, (const bf16*)q,
+                         (const bf16*)k_pages, (const bf16*)v_pages, scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv,
+                         scale, softcap, span, none, value_heads, keep_first, pool);
+    };
+    const cudaError_t e = pool_size > 0 ? launch(decode_capped_split_kernel<false, true>, configured[1])
+                                        : launch(decode_capped_split_kernel<false, false>, configured[0]);
     if (e != cudaSuccess) return (int)e;
     if (out_f32)
         return (int)q3_launch(decode_capped_merge_kernel<float>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
@@ -655,15 +697,15 @@ Q3_EXPORT int q3_attention_capped_decode_fused_bf16(const void* qkv, void* k_pag
     if (n_tokens > 65535 || nkv > 65535 || nq > 0x7fffffff / 2) return Q3_ERR_TOO_LARGE;
     static Q3PerDevice configured;
     {
-        cudaError_t e = q3_allow_shared_memory(decode_capped_split_kernel<true>, DECODE_SMEM_FUSED, configured);
+        cudaError_t e = q3_allow_shared_memory(decode_capped_split_kernel<true, false>, DECODE_SMEM_FUSED, configured);
         if (e != cudaSuccess) return (int)e;
     }
     FusedArgs fused;
     fused.qkv = (const bf16*)qkv; fused.bias = bias; fused.cos_tab = cos_tab; fused.sin_tab = sin_tab;
     fused.rot = rotary_dim > 0 ? rotary_dim : D;
-    cudaError_t e = q3_launch(decode_capped_split_kernel<true>, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32),
+    cudaError_t e = q3_launch(decode_capped_split_kernel<true, false>, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32),
                               DECODE_SMEM_FUSED, (cudaStream_t)stream, (const bf16*)nullptr, (const bf16*)k_pages, (const bf16*)v_pages,
-                              scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, scale, softcap, chunk, fused, nkv, 0);
+                              scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, scale, softcap, chunk, fused, nkv, 0, PoolArgs{});
     if (e != cudaSuccess) return (int)e;
     return (int)q3_launch(decode_capped_merge_kernel<bf16>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
                           (cudaStream_t)stream, (const float*)scratch, (bf16*)out, nq, n_splits, sink, (const float*)nullptr);

@@ -51,6 +51,7 @@ struct CapArgs {
     float cap;         // 0: no cap
     int chunk;         // 0: every earlier key is seen
     int sink;          // 1: one more term exp(0) in the denominator
+    const float* sink_values;   // one score per query head instead of that 0 (may be null)
 };
 
 constexpr int D = Q3_HEAD_DIM;
@@ -290,6 +291,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         const int c_last = (CAPPED && capped.chunk > 0) ? (pos0 + tile * BM + BM - 1) / capped.chunk * capped.chunk : 0;
         const float cap_l2 = capped.cap * 1.4426950408889634f;                       // the cap in log2 units
         const float tanh_k = capped.cap > 0.0f ? 2.0f * capped.scale * 1.4426950408889634f / capped.cap : 0.0f;
+        const float sink_score = CAPPED && capped.sink_values != nullptr ? capped.sink_values[head] * 1.4426950408889634f : 0.0f;
         for (int j = 0; j < n_pages && ok; ++j) {
             ok = mbar_wait(bar_s_full, (uint32_t)j & 1u);
             if (!ok) { if (lane == 0) atomicExch(status, 15); break; }
@@ -327,9 +329,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             if (j == 0) {
                 if (CAPPED) {
                     // a row may see nothing of its tile's first page (its chunk starts later): a maximum below every
-                    // score then lets the next page raise it; the sink is a key of score 0 that is always seen
-                    m_run = capped.sink ? fmaxf(m_page, 0.0f) : (m_page == -INFINITY ? -1.0e30f : m_page);
-                    l_run = capped.sink ? ex2_approx(-m_run) : 0.0f;
+                    // score then lets the next page raise it; the sink is a key of score 0, or of the head's own, that is always seen
+                    m_run = capped.sink ? fmaxf(m_page, sink_score) : (m_page == -INFINITY ? -1.0e30f : m_page);
+                    l_run = capped.sink ? ex2_approx(sink_score - m_run) : 0.0f;
                 } else {
                     m_run = m_page == -INFINITY ? 0.0f : m_page;             // the first page overwrites O: nothing to rescale
                 }
@@ -489,10 +491,10 @@ Q3_EXPORT int q3_attention_capped_prefill_tc_bf16(const void* q, const void* k_p
                                                   const int* seq_start, const int* seq_pos0, const int* page_table,
                                                   int pages_per_seq, int n_seqs, int max_new, int64_t n_tokens,
                                                   int64_t n_cache_pages, int nq, int nkv, float scale, float softcap, int chunk,
-                                                  int sink, int* status, void* stream) {
+                                                  int sink, const float* sink_values, int* status, void* stream) {
     if (softcap < 0.0f || chunk < 0) return Q3_ERR_BAD_SIZE;
     CapArgs capped;
-    capped.scale = scale; capped.cap = softcap; capped.chunk = chunk; capped.sink = sink ? 1 : 0;
+    capped.scale = scale; capped.cap = softcap; capped.chunk = chunk; capped.sink = sink ? 1 : 0; capped.sink_values = sink_values;
     return launch_prefill_tc(q, k_pages, v_pages, out, seq_start, seq_pos0, page_table, pages_per_seq, n_seqs, max_new, n_tokens,
                              n_cache_pages, nq, nkv, scale, status, stream, capped);
 }

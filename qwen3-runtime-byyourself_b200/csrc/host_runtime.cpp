@@ -42,13 +42,15 @@ qwen3::GenerationProgress* progress_of(void* h) { return static_cast<qwen3::Gene
 
 Q3_HOST_EXPORT const char* q3_host_last_error() { return g_error.c_str(); }
 
-// kinds[g]: 0 = every key, 1 = a window of windows[g] keys, 2 = the keys of the query's own chunk of windows[g] positions.
+// kinds[g]: 0 = every key, 1 = a window of windows[g] keys, 2 = the keys of the query's own chunk of windows[g] positions,
+// 3 = one entry for every whole block of windows[g] tokens.
 Q3_HOST_EXPORT int q3_book_create(const int* kinds, const int* windows, int n_groups, int64_t max_tokens, int64_t max_seq_len,
                                   int n_slots, int page_tokens, void** out, const int* keep_first) {
     return guarded([&] {
         std::vector<qwen3::GroupNeed> needs(n_groups);
         for (int g = 0; g < n_groups; ++g) {
-            needs[g].kind = kinds[g] == 2 ? qwen3::GroupKind::Chunk : kinds[g] ? qwen3::GroupKind::Window : qwen3::GroupKind::Full;
+            if (kinds[g] < 0 || kinds[g] > 3) throw std::invalid_argument("unknown kind of cache group");
+            needs[g].kind = (qwen3::GroupKind)kinds[g];
             needs[g].window = windows[g];
             needs[g].keep_first = keep_first != nullptr ? keep_first[g] : 0;
         }
@@ -78,6 +80,7 @@ Q3_HOST_EXPORT int q3_book_is_held(void* h, int slot) { return book_of(h)->is_he
 Q3_HOST_EXPORT int q3_book_free_slots(void* h) { return book_of(h)->n_free_slots(); }
 Q3_HOST_EXPORT int q3_book_pages_held(void* h) { return book_of(h)->pages_held(); }
 Q3_HOST_EXPORT int32_t* q3_book_table(void* h, int group) { return book_of(h)->group(group).table(); }
+Q3_HOST_EXPORT int q3_book_group_pages(void* h, int group) { return book_of(h)->group(group).n_pages(); }
 Q3_HOST_EXPORT int q3_book_free_pages(void* h, int group, int32_t* out) {      // out: n_pages elements at most; returns the count
     const std::vector<int32_t>& f = book_of(h)->group(group).free_pages();
     if (out != nullptr && !f.empty()) std::memcpy(out, f.data(), f.size() * sizeof(int32_t));

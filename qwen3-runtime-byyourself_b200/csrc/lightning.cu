@@ -6,6 +6,9 @@
 // with q, k, v = SiLU of the projection output.  A row of the projection holds, head by head, the H*d
 // values of q, the H*d of k, the H*vd of v and the H*vd of the output gate g.
 //
+// Retention is the same recurrence on other inputs (`Input`): no activation, the first `rot` values of every head of q
+// and k rotated by their position in pairs (i, i + rot/2), k multiplied by a constant.
+//
 //   lightning_scan  : one block per (head, sequence, tile of up to 64 columns of the state: columns do not
 //                     depend on one another) walks the sequence's new tokens in order with its share of the
 //                     state in registers: thread (j, r) owns column j of the tile and the rows r, r + R,
@@ -24,13 +27,34 @@ namespace {
 
 __device__ __forceinline__ float silu_f32(float z) { return z / (1.0f + expf(-z)); }
 
+// What becomes of q, k and v before the recurrence, all of it in 32-bit, and where the state's rows lie.
+struct Input {
+    int silu;                  // q, k and v go through SiLU
+    float k_scale;
+    const float* cos_tab;      // [positions, rot / 2] or null
+    const float* sin_tab;
+    int rot;
+    const int* token_pos;
+    int64_t slot_stride;       // of the state: values from one slot's row to the next
+};
+__device__ __forceinline__ float activated(float z, int silu) { return silu ? silu_f32(z) : z; }
+// Value `i` of a head of q or k of token `t`.
+template <typename T> __device__ __forceinline__ float query_or_key(const T* head, int i, int64_t t, const Input& in) {
+    const float z = activated(to_f32<T>(head[i]), in.silu);
+    if (in.cos_tab == nullptr || i >= in.rot) return z;
+    const int half = in.rot >> 1, j = i < half ? i : i - half;
+    const int64_t at = (int64_t)in.token_pos[t] * half + j;
+    const float other = activated(to_f32<T>(head[i < half ? i + half : j]), in.silu), c = in.cos_tab[at], s = in.sin_tab[at];
+    return i < half ? z * c - other * s : z * c + other * s;
+}
+
 constexpr int COL_TILE = 64;      // columns of the state per block
 constexpr int MAX_THREADS = 512;
 
 template <typename T, int ROWS>
 __global__ void __launch_bounds__(MAX_THREADS) lightning_scan_kernel(const T* __restrict__ proj, float* __restrict__ state, const float* __restrict__ decay,
                                       const int* __restrict__ seq_start, const int* __restrict__ seq_slots,
-                                      float* __restrict__ out, int H, int d, int vd, int R, int vt) {
+                                      float* __restrict__ out, int H, int d, int vd, int R, int vt, const Input in) {
     extern __shared__ float smem[];
     float* q_s = smem;                 // [d]
     float* k_s = q_s + d;              // [d]
@@ -43,7 +67,7 @@ __global__ void __launch_bounds__(MAX_THREADS) lightning_scan_kernel(const T* __
     const bool live = r < R && j < vd;
     const float lam = decay[head];
     const int64_t cols = 2 * (int64_t)H * d + 2 * (int64_t)H * vd;
-    float* S_g = state + ((int64_t)seq_slots[seq] * H + head) * d * vd;
+    float* S_g = state + (int64_t)seq_slots[seq] * in.slot_stride + (int64_t)head * d * vd;
     float S[ROWS];
 #pragma unroll
     for (int n = 0; n < ROWS; ++n) {
@@ -53,11 +77,11 @@ __global__ void __launch_bounds__(MAX_THREADS) lightning_scan_kernel(const T* __
     for (int t = seq_start[seq]; t < seq_start[seq + 1]; ++t) {
         const T* row = proj + t * cols;
         for (int i = tid; i < d; i += blockDim.x) {
-            q_s[i] = silu_f32(to_f32<T>(row[(int64_t)head * d + i]));
-            k_s[i] = silu_f32(to_f32<T>(row[(int64_t)(H + head) * d + i]));
+            q_s[i] = query_or_key<T>(row + (int64_t)head * d, i, t, in);
+            k_s[i] = query_or_key<T>(row + (int64_t)(H + head) * d, i, t, in) * in.k_scale;
         }
         for (int i = tid; i < vt; i += blockDim.x)
-            v_s[i] = col0 + i < vd ? silu_f32(to_f32<T>(row[2 * (int64_t)H * d + (int64_t)head * vd + col0 + i])) : 0.0f;
+            v_s[i] = col0 + i < vd ? activated(to_f32<T>(row[2 * (int64_t)H * d + (int64_t)head * vd + col0 + i]), in.silu) : 0.0f;
         __syncthreads();
         if (live) {
             const float v = v_s[jt];
@@ -90,7 +114,7 @@ __global__ void __launch_bounds__(MAX_THREADS) lightning_scan_kernel(const T* __
 
 template <typename T>
 int lightning_scan_launch(const T* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots, float* out,
-                          int n_seqs, int H, int d, int vd, cudaStream_t stream) {
+                          int n_seqs, int H, int d, int vd, const Input& in, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (H <= 0 || d <= 0 || vd <= 0 || d > 256 || vd > 256 || n_seqs > 65535) return Q3_ERR_BAD_SIZE;
     const int vt = min(vd, COL_TILE);
@@ -101,7 +125,7 @@ int lightning_scan_launch(const T* proj, float* state, const float* decay, const
     const dim3 grid(H, n_seqs, (vd + vt - 1) / vt);
 #define Q3_SCAN(ROWS)                                                                                                    \
     return (int)q3_launch(lightning_scan_kernel<T, ROWS>, grid, dim3(threads), smem, stream, proj, state, decay, seq_start, \
-                          seq_slots, out, H, d, vd, R, vt)
+                          seq_slots, out, H, d, vd, R, vt, in)
     if (rows <= 1) Q3_SCAN(1);
     if (rows <= 2) Q3_SCAN(2);
     if (rows <= 4) Q3_SCAN(4);
@@ -120,7 +144,7 @@ constexpr int CHUNK = 32;
 template <typename T, int ROWS>
 __global__ void __launch_bounds__(MAX_THREADS) lightning_chunks_kernel(const T* __restrict__ proj, float* __restrict__ state, const float* __restrict__ decay,
                                         const int* __restrict__ seq_start, const int* __restrict__ seq_slots,
-                                        float* __restrict__ out, int H, int d, int vd, int R, int vt) {
+                                        float* __restrict__ out, int H, int d, int vd, int R, int vt, const Input in) {
     extern __shared__ float smem[];
     float* q_s = smem;                         // [C][d + 1]
     float* k_s = q_s + CHUNK * (d + 1);        // [C][d + 1]
@@ -138,7 +162,7 @@ __global__ void __launch_bounds__(MAX_THREADS) lightning_chunks_kernel(const T* 
     for (int n = tid; n <= CHUNK; n += nthreads) pw[n] = n == 0 ? 1.0f : (lam > 0.0f ? exp2f((float)n * l2) : 0.0f);
     const int64_t cols = 2 * (int64_t)H * d + 2 * (int64_t)H * vd;
     const int dp = d + 1;
-    float* S_g = state + ((int64_t)seq_slots[seq] * H + head) * d * vd;
+    float* S_g = state + (int64_t)seq_slots[seq] * in.slot_stride + (int64_t)head * d * vd;
     float S[ROWS];
 #pragma unroll
     for (int n = 0; n < ROWS; ++n) {
@@ -152,12 +176,12 @@ __global__ void __launch_bounds__(MAX_THREADS) lightning_chunks_kernel(const T* 
         for (int x = tid; x < C * d; x += nthreads) {
             const int i = x / d, c = x % d;
             const T* row = proj + (int64_t)(t0 + i) * cols;
-            q_s[i * dp + c] = silu_f32(to_f32<T>(row[(int64_t)head * d + c]));
-            k_s[i * dp + c] = silu_f32(to_f32<T>(row[(int64_t)(H + head) * d + c]));
+            q_s[i * dp + c] = query_or_key<T>(row + (int64_t)head * d, c, t0 + i, in);
+            k_s[i * dp + c] = query_or_key<T>(row + (int64_t)(H + head) * d, c, t0 + i, in) * in.k_scale;
         }
         for (int x = tid; x < C * vt; x += nthreads) {
             const int i = x / vt, c = col0 + x % vt;
-            v_s[x] = c < vd ? silu_f32(to_f32<T>(proj[(int64_t)(t0 + i) * cols + 2 * (int64_t)H * d + (int64_t)head * vd + c])) : 0.0f;
+            v_s[x] = c < vd ? activated(to_f32<T>(proj[(int64_t)(t0 + i) * cols + 2 * (int64_t)H * d + (int64_t)head * vd + c]), in.silu) : 0.0f;
         }
         __syncthreads();
         // scores inside the chunk
@@ -217,7 +241,7 @@ __global__ void __launch_bounds__(MAX_THREADS) lightning_chunks_kernel(const T* 
 
 template <typename T>
 int lightning_chunks_launch(const T* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
-                            float* out, int n_seqs, int H, int d, int vd, cudaStream_t stream) {
+                            float* out, int n_seqs, int H, int d, int vd, const Input& in, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (H <= 0 || d <= 0 || vd <= 0 || d > 256 || vd > 256 || n_seqs > 65535) return Q3_ERR_BAD_SIZE;
     // narrower column tiles while the blocks are fewer than the multiprocessors: a prompt of one sequence has only
@@ -238,7 +262,7 @@ int lightning_chunks_launch(const T* proj, float* state, const float* decay, con
             if (e != cudaSuccess) return (int)e;                                                                          \
         }                                                                                                                 \
         return (int)q3_launch(lightning_chunks_kernel<T, ROWS>, grid, dim3(threads), smem, stream, proj, state, decay,     \
-                              seq_start, seq_slots, out, H, d, vd, R, vt);                                                \
+                              seq_start, seq_slots, out, H, d, vd, R, vt, in);                                                \
     }
     if (rows <= 1) Q3_CHUNKS(1, 0)
     if (rows <= 2) Q3_CHUNKS(2, 1)
@@ -310,7 +334,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state, const float* __restrict__ decay,
                            const int* __restrict__ seq_start, const int* __restrict__ seq_slots, float* __restrict__ out, int H, int d,
-                           int vd, int vt) {
+                           int vd, int vt, const Input in) {
     extern __shared__ float smem[];
     const int dp = (d + 15) & ~15;                      // rows of the state in whole 16-row tiles; the padding stays zero
     const int ldq = dp + 4, ldv = vt + 8, lda = C + 4;  // row lengths that spread the fragments' rows over the banks
@@ -328,7 +352,7 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
     const float l2 = lam > 0.0f ? log2f(lam) : 0.0f;
     for (int n = tid; n <= C; n += 256) pw[n] = n == 0 ? 1.0f : (lam > 0.0f ? exp2f((float)n * l2) : 0.0f);
     const int64_t cols = 2 * (int64_t)H * d + 2 * (int64_t)H * vd;
-    float* S_g = state + ((int64_t)seq_slots[seq] * H + head) * d * vd;
+    float* S_g = state + (int64_t)seq_slots[seq] * in.slot_stride + (int64_t)head * d * vd;
     for (int x = tid; x < dp * ldv; x += 256) {
         const int i = x / ldv, c = x % ldv;
         S_s[x] = (i < d && c < vt && col0 + c < vd) ? S_g[(int64_t)i * vd + col0 + c] : 0.0f;
@@ -347,10 +371,31 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
             if (i < Cn) {
                 const T* row = proj + (int64_t)(t0 + i) * cols;
                 const Pack<T> qp = load_pack<T>(row + (int64_t)head * d + c), kp = load_pack<T>(row + (int64_t)(H + head) * d + c);
+                const int half = in.rot >> 1;
+                const bool turns = in.cos_tab != nullptr && c < in.rot;
+                if (!turns) {
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) {
-                    qv[e] = silu_f32(qp.get(e));
-                    kv[e] = silu_f32(kp.get(e));
+                    for (int e = 0; e < VEC; ++e) {
+                        qv[e] = activated(qp.get(e), in.silu);
+                        kv[e] = activated(kp.get(e), in.silu) * in.k_scale;
+                    }
+                } else if (half % VEC == 0) {             // a packet and the packet of its pairs' other members
+                    const int j = c < half ? c : c - half, other = c < half ? c + half : j;
+                    const Pack<T> qo = load_pack<T>(row + (int64_t)head * d + other), ko = load_pack<T>(row + (int64_t)(H + head) * d + other);
+                    const int64_t at = (int64_t)in.token_pos[t0 + i] * half + j;
+                    const float sign = c < half ? -1.0f : 1.0f;
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        const float cs = in.cos_tab[at + e], sn = sign * in.sin_tab[at + e];
+                        qv[e] = activated(qp.get(e), in.silu) * cs + activated(qo.get(e), in.silu) * sn;
+                        kv[e] = (activated(kp.get(e), in.silu) * cs + activated(ko.get(e), in.silu) * sn) * in.k_scale;
+                    }
+                } else {
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) {
+                        qv[e] = query_or_key<T>(row + (int64_t)head * d, c + e, t0 + i, in);
+                        kv[e] = query_or_key<T>(row + (int64_t)(H + head) * d, c + e, t0 + i, in) * in.k_scale;
+                    }
                 }
             } else {
 #pragma unroll
@@ -370,7 +415,7 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
             if (i < Cn && col0 + c < vd) {
                 const Pack<T> vp = load_pack<T>(proj + (int64_t)(t0 + i) * cols + 2 * (int64_t)H * d + (int64_t)head * vd + col0 + c);
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) vv[e] = silu_f32(vp.get(e));
+                for (int e = 0; e < VEC; ++e) vv[e] = activated(vp.get(e), in.silu);
             }
 #pragma unroll
             for (int e = 0; e < VEC; ++e) v_s[i * ldv + c + e] = vv[e];
@@ -438,7 +483,7 @@ static inline size_t smem_bytes(int d, int vt) {
 
 template <typename T>
 int launch(const T* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots, float* out, int n_seqs, int H,
-           int d, int vd, cudaStream_t stream) {
+           int d, int vd, const Input& in, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (H <= 0 || d <= 0 || vd <= 0 || d > 256 || vd > 256 || d % 8 != 0 || vd % 8 != 0 || n_seqs > 65535) return Q3_ERR_BAD_SIZE;
     if (!aligned16(proj)) return Q3_ERR_MISALIGNED;
@@ -452,7 +497,7 @@ int launch(const T* proj, float* state, const float* decay, const int* seq_start
     const cudaError_t e = q3_allow_shared_memory(lightning_chunks_tc_kernel<T>, 200 * 1024, allowed);
     if (e != cudaSuccess) return (int)e;
     return (int)q3_launch(lightning_chunks_tc_kernel<T>, dim3(H, n_seqs, (vd + vt - 1) / vt), dim3(256), smem, stream, proj, state, decay,
-                          seq_start, seq_slots, out, H, d, vd, vt);
+                          seq_start, seq_slots, out, H, d, vd, vt, in);
 }
 }  // namespace tc
 
@@ -474,20 +519,31 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const T* __restri
     }
 }
 
+static inline bool input_fits(const Input& in, int d) {
+    if ((in.cos_tab == nullptr) != (in.sin_tab == nullptr)) return false;
+    return in.cos_tab == nullptr || (in.rot > 0 && in.rot % 2 == 0 && in.rot <= d && in.token_pos != nullptr);
+}
+
 }  // namespace
 
 #define Q3_LIGHTNING_EXPORTS(SUFFIX, T)                                                                                   \
     Q3_EXPORT int q3_lightning_scan_##SUFFIX(const void* proj, float* state, const float* decay, const int* seq_start,    \
                                              const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd,      \
-                                             void* stream) {                                                              \
+                                             int silu, float k_scale, const float* cos_tab, const float* sin_tab,         \
+                                             int rot, const int* token_pos, int64_t slot_stride, void* stream) {                            \
+        const Input in = {silu, k_scale, cos_tab, sin_tab, rot, token_pos, slot_stride};                                               \
+        if (!input_fits(in, d)) return Q3_ERR_BAD_SIZE;                                                                   \
         return lightning_scan_launch<T>((const T*)proj, state, decay, seq_start, seq_slots, out, n_seqs, heads, d, vd,    \
-                                        (cudaStream_t)stream);                                                            \
+                                        in, (cudaStream_t)stream);                                                            \
     }                                                                                                                     \
     Q3_EXPORT int q3_lightning_chunks_##SUFFIX(const void* proj, float* state, const float* decay, const int* seq_start,  \
                                                const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd,    \
-                                               void* stream) {                                                            \
+                                               int silu, float k_scale, const float* cos_tab, const float* sin_tab,       \
+                                               int rot, const int* token_pos, int64_t slot_stride, void* stream) {                          \
+        const Input in = {silu, k_scale, cos_tab, sin_tab, rot, token_pos, slot_stride};                                               \
+        if (!input_fits(in, d)) return Q3_ERR_BAD_SIZE;                                                                   \
         return lightning_chunks_launch<T>((const T*)proj, state, decay, seq_start, seq_slots, out, n_seqs, heads, d, vd,  \
-                                          (cudaStream_t)stream);                                                          \
+                                          in, (cudaStream_t)stream);                                                          \
     }                                                                                                                     \
     Q3_EXPORT int q3_gated_norm_##SUFFIX(const float* o, const void* gate, int64_t gate_stride, const float* w, float eps, \
                                          void* out, int64_t n_tokens, int size, void* stream) {                           \
@@ -500,8 +556,12 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, const T* __restri
 // The chunked form with its products on the tensor cores (operands split into TF32 hi + lo terms): for a compute type of
 // bfloat16, head sizes in steps of 8.
 Q3_EXPORT int q3_lightning_chunks_tc_bf16(const void* proj, float* state, const float* decay, const int* seq_start,
-                                          const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, void* stream) {
-    return tc::launch<bf16>((const bf16*)proj, state, decay, seq_start, seq_slots, out, n_seqs, heads, d, vd, (cudaStream_t)stream);
+                                          const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale,
+                                          const float* cos_tab, const float* sin_tab, int rot, const int* token_pos,
+                                          int64_t slot_stride, void* stream) {
+    const Input in = {silu, k_scale, cos_tab, sin_tab, rot, token_pos, slot_stride};
+    if (!input_fits(in, d)) return Q3_ERR_BAD_SIZE;
+    return tc::launch<bf16>((const bf16*)proj, state, decay, seq_start, seq_slots, out, n_seqs, heads, d, vd, in, (cudaStream_t)stream);
 }
 
 Q3_LIGHTNING_EXPORTS(f32, float)

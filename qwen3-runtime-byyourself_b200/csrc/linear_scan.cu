@@ -28,7 +28,7 @@
 //                  scan over the warp, and writes keep = exp(f + m_(t-1) - m_t), write = exp(i - m_t) and low = exp(-m_t).
 //   head_gated_norm : per (token, head): x = o (divided by max(|n . q|, low) + floor if the state has the normaliser
 //                  column), y = x / sqrt(mean(x^2) + eps) * w * act(gate), act = sigmoid or SiLU; w one vector per
-//                  head or one for all heads.
+//                  head, one for all heads, or none.
 //
 // Decays, gates, state and outputs are 32-bit whatever T; T is the type of q, k, v, the output gate and the result.
 #include "common.cuh"
@@ -367,12 +367,12 @@ __global__ void head_gated_norm_kernel(const float* __restrict__ o, const float*
         sq += y * y;
     }
     const float inv = rsqrtf(warp_sum(sq) / (float)vd + eps);
-    const float* wh = w + (w_per_head ? (int64_t)head * vd : 0);
+    const float* wh = w == nullptr ? nullptr : w + (w_per_head ? (int64_t)head * vd : 0);
     const T* g = gate + t * gate_row + (int64_t)head * vd;
     for (int c = lane; c < vd; c += 32) {
         const float z = to_f32<T>(g[c]);
         const float s = 1.0f / (1.0f + expf(-z));
-        out[row * vd + c] = from_f32<T>(x[c] * inv_den * inv * wh[c] * (act ? z * s : s));
+        out[row * vd + c] = from_f32<T>(x[c] * inv_den * inv * (wh != nullptr ? wh[c] : 1.0f) * (act ? z * s : s));
     }
 }
 

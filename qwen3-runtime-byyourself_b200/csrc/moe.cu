@@ -16,9 +16,11 @@
 //   moe_up      : act[slot] = f(W_gate x, W_up x) for the pairs of each expert, a tile of TM pairs x 64
 //                 columns per block; g = min(gate, limit), u = clamp(up, -limit, limit),
 //                 f = g sigmoid(alpha g) (u + up_offset)  (limit = infinity, alpha = 1, up_offset = 0: SiLU(gate) * up).
+//                 Experts without a gate: act[slot] = max(W_up x, 0)^2, one matrix instead of two.
 //   moe_down    : y[slot] = W_down act[slot], the same tiling, 32-bit output.
 //   moe_combine : out[token] = T( sum_k weight_k y[slot(token, k)] + id_weight h[token] + shared_w[token] shared[token] ),
-//                 the last term for a shared expert that every token uses (may be absent).
+//                 the last term for a shared expert that every token uses (may be absent; without shared_w its weight
+//                 is 1).
 //
 // The products accumulate in 32-bit in ascending order of k whatever the tile a pair falls into, so a token's
 // result does not depend on what else is in the step.  Float tiles run on fmaf; bfloat16 tiles on the tensor cores
@@ -96,7 +98,7 @@ moe_route_kernel(const T* __restrict__ h, const T* __restrict__ w_router, const 
     if (by_logit == 2) {                         // every output's score by itself: sigmoid(z)
         for (int e = 0; e < n_out; ++e) {
             z[e] = 1.0f / (1.0f + expf(-z[e]));
-            choice[e] = z[e] + correction[e];
+            choice[e] = z[e] + (correction != nullptr ? correction[e] : 0.0f);
         }
     } else {
         float m = -INFINITY, sum = 0.0f;
@@ -108,7 +110,7 @@ moe_route_kernel(const T* __restrict__ h, const T* __restrict__ w_router, const 
         const float inv = 1.0f / sum;
         for (int e = 0; e < n_out; ++e) {
             z[e] *= inv;
-            choice[e] = z[e] + correction[e];
+            choice[e] = z[e] + (correction != nullptr ? correction[e] : 0.0f);
         }
     }
     if (group_count > 1) {
@@ -262,7 +264,7 @@ __device__ __forceinline__ void tile_product(const T* __restrict__ X, int64_t x_
     }
 }
 
-template <typename T, int TM>
+template <typename T, int TM, bool GATE>
 __global__ void __launch_bounds__(256)
 moe_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gate_up, const int* __restrict__ offsets,
               const int* __restrict__ pair_of_slot, T* __restrict__ act, int n_real, int top, int hidden, int ff, float limit,
@@ -275,9 +277,9 @@ moe_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gate_up, const in
     if (!find_tile<TM>(offsets, n_real, blockIdx.y, expert, row0, rows)) return;
     if (threadIdx.x < TM) src_row[threadIdx.x] = threadIdx.x < rows ? pair_of_slot[row0 + threadIdx.x] / top : 0;
     const int col0 = blockIdx.x * TN;
-    const T* wg = w_gate_up + (int64_t)expert * 2 * ff * hidden;      // [gate rows; up rows] of the expert
+    const T* wg = w_gate_up + (int64_t)expert * (GATE ? 2 : 1) * ff * hidden;      // [gate rows; up rows] of the expert (or up rows alone)
     float g[(TM + 15) / 16][4], u[(TM + 15) / 16][4];
-    tile_product<T, TM, true>(h, hidden, src_row, rows, wg, wg + (int64_t)ff * hidden, ff, col0, hidden, g, u, xs, ws0, ws1);
+    tile_product<T, TM, GATE>(h, hidden, src_row, rows, wg, GATE ? wg + (int64_t)ff * hidden : nullptr, ff, col0, hidden, g, u, xs, ws0, ws1);
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
 #pragma unroll
     for (int a = 0; a < (TM + 15) / 16; ++a) {
@@ -287,6 +289,11 @@ moe_up_kernel(const T* __restrict__ h, const T* __restrict__ w_gate_up, const in
         for (int b = 0; b < 4; ++b) {
             const int c = col0 + tx * 4 + b;
             if (c >= ff) continue;
+            if constexpr (!GATE) {
+                const float v = fmaxf(g[a][b], 0.0f);
+                act[(int64_t)(row0 + rr) * ff + c] = from_f32<T>(v * v);
+                continue;
+            }
             const float gv = fminf(g[a][b], limit), uv = fminf(fmaxf(u[a][b], -limit), limit);
             act[(int64_t)(row0 + rr) * ff + c] = from_f32<T>(gv / (1.0f + expf(-alpha * gv)) * (uv + up_offset));
         }
@@ -335,7 +342,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const T* __restr
             const int slot = slot_of_pair[t * top + k];
             if (slot >= 0) v = fmaf(top_w[t * top + k], y[(int64_t)slot * hidden + c], v);
         }
-        if (shared != nullptr) v = fmaf(shared_w[t], to_f32<T>(shared[t * hidden + c]), v);
+        if (shared != nullptr) v = fmaf(shared_w != nullptr ? shared_w[t] : 1.0f, to_f32<T>(shared[t * hidden + c]), v);
         out[t * hidden + c] = from_f32<T>(v);
     }
 }
@@ -427,6 +434,7 @@ __device__ __forceinline__ void tile_product(const bf16* __restrict__ X, int64_t
     cp_async_wait<0>();
 }
 
+template <bool GATE>
 __global__ void __launch_bounds__(256)
 moe_up_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w_gate_up, const int* __restrict__ offsets,
               const int* __restrict__ pair_of_slot, bf16* __restrict__ act, int n_real, int top, int hidden, int ff, float limit,
@@ -440,9 +448,9 @@ moe_up_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w_gate_up, co
     if (threadIdx.x < BM) src_row[threadIdx.x] = pair_of_slot[row0 + min((int)threadIdx.x, rows - 1)] / top;
     __syncthreads();
     const int col0 = blockIdx.x * BN;
-    const bf16* wg = w_gate_up + (int64_t)expert * 2 * ff * hidden;
+    const bf16* wg = w_gate_up + (int64_t)expert * (GATE ? 2 : 1) * ff * hidden;
     float g[4][4], u[4][4];
-    tile_product<true>(h, hidden, src_row, wg, wg + (int64_t)ff * hidden, ff, col0, hidden, smem, g, u);
+    tile_product<GATE>(h, hidden, src_row, wg, GATE ? wg + (int64_t)ff * hidden : nullptr, ff, col0, hidden, smem, g, u);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad = lane >> 2, tq = lane & 3;
 #pragma unroll
     for (int n = 0; n < 4; ++n)
@@ -450,6 +458,11 @@ moe_up_kernel(const bf16* __restrict__ h, const bf16* __restrict__ w_gate_up, co
         for (int e = 0; e < 4; ++e) {
             const int rr = (warp & 3) * 16 + quad + (e >> 1) * 8, c = col0 + (warp >> 2) * 32 + n * 8 + tq * 2 + (e & 1);
             if (rr < rows && c < ff) {
+                if constexpr (!GATE) {
+                    const float v = fmaxf(g[n][e], 0.0f);
+                    act[(int64_t)(row0 + rr) * ff + c] = __float2bfloat16_rn(v * v);
+                    continue;
+                }
                 const float gv = fminf(g[n][e], limit), uv = fminf(fmaxf(u[n][e], -limit), limit);
                 act[(int64_t)(row0 + rr) * ff + c] = __float2bfloat16_rn(gv / (1.0f + expf(-alpha * gv)) * (uv + up_offset));
             }
@@ -481,15 +494,16 @@ moe_down_kernel(const bf16* __restrict__ act, const bf16* __restrict__ w_down, c
 }
 
 int experts_launch(const bf16* h, const bf16* w_gate_up, const bf16* w_down, const int* offsets, const int* pair_of_slot, bf16* act,
-                   float* y, int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha, float up_offset, cudaStream_t stream) {
+                   float* y, int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha, float up_offset, int gated, cudaStream_t stream) {
     const int tiles = (n_pairs + BM - 1) / BM + n_real;          // an upper bound on the row tiles of all experts together
     if (tiles > 65535) return Q3_ERR_TOO_LARGE;
-    static Q3PerDevice up_ok, down_ok;
-    cudaError_t e = q3_allow_shared_memory(moe_up_kernel, STAGES * 3 * TILE, up_ok);
+    static Q3PerDevice up_ok, plain_ok, down_ok;
+    const int up_smem = STAGES * (gated ? 3 : 2) * TILE;
+    cudaError_t e = gated ? q3_allow_shared_memory(moe_up_kernel<true>, up_smem, up_ok) : q3_allow_shared_memory(moe_up_kernel<false>, up_smem, plain_ok);
     if (e == cudaSuccess) e = q3_allow_shared_memory(moe_down_kernel, STAGES * 2 * TILE, down_ok);
     if (e != cudaSuccess) return (int)e;
-    int code = (int)q3_launch(moe_up_kernel, dim3((ff + BN - 1) / BN, tiles), dim3(256), STAGES * 3 * TILE, stream, h, w_gate_up,
-                              offsets, pair_of_slot, act, n_real, top, hidden, ff, limit, alpha, up_offset);
+    int code = (int)q3_launch(gated ? moe_up_kernel<true> : moe_up_kernel<false>, dim3((ff + BN - 1) / BN, tiles), dim3(256), up_smem, stream, h,
+                              w_gate_up, offsets, pair_of_slot, act, n_real, top, hidden, ff, limit, alpha, up_offset);
     if (code != 0) return code;
     return (int)q3_launch(moe_down_kernel, dim3((hidden + BN - 1) / BN, tiles), dim3(256), STAGES * 2 * TILE, stream, act, w_down,
                           offsets, y, n_real, hidden, ff);
@@ -498,10 +512,10 @@ int experts_launch(const bf16* h, const bf16* w_gate_up, const bf16* w_down, con
 
 template <typename T, int TM>
 int moe_experts_launch(const T* h, const T* w_gate_up, const T* w_down, const int* offsets, const int* pair_of_slot, T* act, float* y,
-                       int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha, float up_offset, cudaStream_t stream) {
+                       int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha, float up_offset, int gated, cudaStream_t stream) {
     const int tiles = (n_pairs + TM - 1) / TM + n_real;         // an upper bound on the row tiles of all experts together
     if (tiles > 65535) return Q3_ERR_TOO_LARGE;
-    int code = (int)q3_launch(moe_up_kernel<T, TM>, dim3((ff + TN - 1) / TN, tiles), dim3(256), 0, stream, h, w_gate_up, offsets,
+    int code = (int)q3_launch(gated ? moe_up_kernel<T, TM, true> : moe_up_kernel<T, TM, false>, dim3((ff + TN - 1) / TN, tiles), dim3(256), 0, stream, h, w_gate_up, offsets,
                               pair_of_slot, act, n_real, top, hidden, ff, limit, alpha, up_offset);
     if (code != 0) return code;
     return (int)q3_launch(moe_down_kernel<T, TM>, dim3((hidden + TN - 1) / TN, tiles), dim3(256), 0, stream, act, w_down, offsets, y,
@@ -526,14 +540,14 @@ int moe_experts_launch(const T* h, const T* w_gate_up, const T* w_down, const in
     }                                                                                                                     \
     Q3_EXPORT int q3_moe_experts_##SUFFIX(const void* h, const void* w_gate_up, const void* w_down, const int* offsets,   \
                                           const int* pair_of_slot, void* act, float* y, int n_pairs, int n_real, int top, \
-                                          int hidden, int ff, float limit, float alpha, float up_offset, void* stream) {                   \
+                                          int hidden, int ff, float limit, float alpha, float up_offset, int gated, void* stream) {                   \
         if (n_pairs <= 0 || n_real <= 0) return 0;                                                                        \
         if (n_pairs <= 64)                                                                                                \
             return moe_experts_launch<T, 8>((const T*)h, (const T*)w_gate_up, (const T*)w_down, offsets, pair_of_slot,    \
-                                            (T*)act, y, n_pairs, n_real, top, hidden, ff, limit, alpha, up_offset,                   \
+                                            (T*)act, y, n_pairs, n_real, top, hidden, ff, limit, alpha, up_offset, gated,            \
                                             (cudaStream_t)stream);                                                        \
         return moe_experts_launch<T, 32>((const T*)h, (const T*)w_gate_up, (const T*)w_down, offsets, pair_of_slot,       \
-                                         (T*)act, y, n_pairs, n_real, top, hidden, ff, limit, alpha, up_offset, (cudaStream_t)stream); \
+                                         (T*)act, y, n_pairs, n_real, top, hidden, ff, limit, alpha, up_offset, gated, (cudaStream_t)stream); \
     }                                                                                                                     \
     Q3_EXPORT int q3_moe_combine_##SUFFIX(const float* y, const void* h, const int* slot_of_pair, const float* top_w,     \
                                           const float* id_weight, void* out, int64_t n_tokens, int top, int hidden,       \
@@ -556,12 +570,12 @@ Q3_EXPORT int q3_moe_sort(const int* top_ids, int n_pairs, int n_real, int* offs
 // bfloat16 with both widths in steps of 32 (and 16-byte aligned rows): the tensor-core tiles; else the fmaf tiles.
 Q3_EXPORT int q3_moe_experts_tc_bf16(const void* h, const void* w_gate_up, const void* w_down, const int* offsets,
                                      const int* pair_of_slot, void* act, float* y, int n_pairs, int n_real, int top, int hidden, int ff,
-                                     float limit, float alpha, float up_offset, void* stream) {
+                                     float limit, float alpha, float up_offset, int gated, void* stream) {
     if (n_pairs <= 0 || n_real <= 0) return 0;
     if (hidden % 32 != 0 || ff % 32 != 0 || hidden <= 0 || ff <= 0) return Q3_ERR_BAD_SIZE;
     if (!aligned16(h) || !aligned16(w_gate_up) || !aligned16(w_down) || !aligned16(act)) return Q3_ERR_MISALIGNED;
     return mma::experts_launch((const bf16*)h, (const bf16*)w_gate_up, (const bf16*)w_down, offsets, pair_of_slot, (bf16*)act, y, n_pairs,
-                               n_real, top, hidden, ff, limit, alpha, up_offset, (cudaStream_t)stream);
+                               n_real, top, hidden, ff, limit, alpha, up_offset, gated, (cudaStream_t)stream);
 }
 
 Q3_MOE_EXPORTS(f32, float)

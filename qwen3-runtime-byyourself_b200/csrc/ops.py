@@ -9,6 +9,7 @@ from __future__ import annotations
 
 import ctypes
 import os
+from dataclasses import dataclass
 from ctypes import c_float, c_int, c_int64, c_uint64, c_void_p
 from typing import Optional
 
@@ -320,9 +321,11 @@ def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, 
 
 
 def sandwich_norm(stream: torch.Tensor, branch: Optional[torch.Tensor], w_post: Optional[torch.Tensor], eps_post: float,
-                  w_pre: Optional[torch.Tensor], eps_pre: float, out: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
+                  w_pre: Optional[torch.Tensor], eps_pre: float, out: Optional[torch.Tensor], groups_post: int = 1,
+                  groups_pre: int = 1) -> Optional[torch.Tensor]:
     """In one pass over the rows of the float32 `stream`: with `branch` (compute type), stream += RMSNorm(branch) *
-    w_post; with `out` (compute type), out = RMSNorm(stream) * w_pre of the sum.  Statistics and sums are 32-bit."""
+    w_post; with `out` (compute type), out = RMSNorm(stream) * w_pre of the sum.  Statistics and sums are 32-bit.
+    `groups_post`, `groups_pre`: the norm splits a row into so many equal consecutive parts with an rms of their own."""
     rows, size = stream.shape
     if stream.dtype != torch.float32 or (branch is None) != (w_post is None) or (out is None) != (w_pre is None):
         raise KernelError("sandwich_norm: a float32 stream, a branch with its weights, an output with its weights")
@@ -336,10 +339,10 @@ def sandwich_norm(stream: torch.Tensor, branch: Optional[torch.Tensor], w_post: 
         if w is not None and w.numel() != size:
             raise KernelError("sandwich_norm: weights do not fit the rows")
     fn = _fn("stream_f32.cu", f"q3_sandwich_norm_{_suffix(ref)}",
-             [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_float, c_float, c_void_p])
+             [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_float, c_float, c_int, c_int, c_void_p])
     _check(fn(_dev(stream, "stream"), _ptr(branch, "branch"), _ptr(w_post, "w_post", torch.float32),
-              _ptr(w_pre, "w_pre", torch.float32), _ptr(out, "out"), rows, size, float(eps_post), float(eps_pre), _stream()),
-           "sandwich_norm")
+              _ptr(w_pre, "w_pre", torch.float32), _ptr(out, "out"), rows, size, float(eps_post), float(eps_pre),
+              int(groups_post), int(groups_pre), _stream()), "sandwich_norm")
     return out
 
 
@@ -353,15 +356,30 @@ def concat_cast(a: torch.Tensor, b: torch.Tensor, out: torch.Tensor) -> torch.Te
     return out
 
 
-def gather_rows_norm(stream: torch.Tensor, idx: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
-    """out[r] = RMSNorm(stream[idx[r]]) * weight, from a float32 stream into out's type."""
+def normed_sum(a: torch.Tensor, b: torch.Tensor, w_a: torch.Tensor, w_b: torch.Tensor, scale_a: float, scale_b: float, eps: float,
+               out: torch.Tensor) -> torch.Tensor:
+    """out = scale_a * RMSNorm(a) * w_a + scale_b * RMSNorm(b) * w_b, row by row, in 32-bit; a, b, out in the compute type, the
+    weights float32."""
+    rows, size = a.shape
+    if b.shape != a.shape or out.shape != a.shape or b.dtype != a.dtype or out.dtype != a.dtype or w_a.numel() != size or w_b.numel() != size:
+        raise KernelError("normed_sum: shapes do not fit")
+    fn = _fn("stream_f32.cu", f"q3_normed_sum_{_suffix(a)}",
+             [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_float, c_void_p, c_int64, c_int, c_void_p])
+    _check(fn(_dev(a, "a"), _dev(b, "b"), _dev(w_a, "w_a", torch.float32), _dev(w_b, "w_b", torch.float32), float(scale_a), float(scale_b),
+              float(eps), _dev(out, "out"), rows, size, _stream()), "normed_sum")
+    return out
+
+
+def gather_rows_norm(stream: torch.Tensor, idx: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                     groups: int = 1) -> torch.Tensor:
+    """out[r] = RMSNorm(stream[idx[r]]) * weight, from a float32 stream into out's type; `groups` as for `sandwich_norm`."""
     rows, size = idx.numel(), stream.shape[-1]
     if stream.dtype != torch.float32 or out.shape[0] < rows or out.shape[-1] != size or weight.numel() != size:
         raise KernelError("gather_rows_norm: shapes do not fit")
     fn = _fn("stream_f32.cu", f"q3_gather_rows_norm_{_suffix(out)}",
-             [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_float, c_void_p])
+             [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_float, c_int, c_void_p])
     _check(fn(_dev(stream, "stream"), _dev(idx, "idx", torch.int32), _dev(weight, "weight", torch.float32), _dev(out, "out"),
-              rows, size, float(eps), _stream()), "gather_rows_norm")
+              rows, size, float(eps), int(groups), _stream()), "gather_rows_norm")
     return out
 
 
@@ -412,28 +430,89 @@ def _rotary_dim(cos, sin, d: int) -> int:
 
 def qkv_prepare(qkv, q_out, k_pages, v_pages, q_norm_w, k_norm_w, cos, sin, token_seq, token_pos, page_table,
                 n_tokens: int, nq: int, nkv: int, d: int, eps: float, write_kv: bool = True, bias=None,
-                value_dim: Optional[int] = None, value_heads: Optional[int] = None):
+                value_dim: Optional[int] = None, value_heads: Optional[int] = None, tied_values: bool = False,
+                norm_once: bool = False, value_cos: Optional[torch.Tensor] = None, value_sin: Optional[torch.Tensor] = None):
     """Per-head norm of q and k, rotation, and the write of k and v into the cache pages
     (`write_kv=False`: only q is prepared, for a layer that reads another layer's cache).  `bias` (float32, one
     value per column of the projection) is added first; `value_dim` is the size of a value head if not `d`,
-    `value_heads` their number if not `nkv` (values that several key heads share)."""
+    `value_heads` their number if not `nkv` (values that several key heads share).  A row of `qkv` may go on beyond the
+    values.  `tied_values`: the values are the projected keys as they are, and `qkv` has no columns for them; `norm_once`: a
+    normed and rotated value is rounded once, when it is stored; `value_cos`, `value_sin` [positions, value_dim / 2]: the
+    values are rotated by their position too, over the whole head."""
     s = _suffix(qkv)
     vd, nv = int(value_dim or d), int(value_heads or nkv)
     if not 0 < d <= 256 or not 0 < vd <= 256 or (d % 2 != 0 and cos is not None and 2 * cos.shape[-1] == d):
         raise KernelError(f"head_dim {d} / value_dim {vd} is not supported: sizes up to 256, an even number of rotated values")
-    if qkv.shape[-1] != (nq + nkv) * d + nv * vd or k_pages.dtype != qkv.dtype or k_pages.shape[1:] != (nkv, PAGE_TOKENS, d) \
-            or v_pages.shape[1:] != (nv, PAGE_TOKENS, vd) or nkv % nv or (bias is not None and bias.numel() != qkv.shape[-1]):
+    columns = (nq + nkv) * d + (0 if tied_values else nv * vd)
+    if qkv.shape[-1] < columns or k_pages.dtype != qkv.dtype or k_pages.shape[1:] != (nkv, PAGE_TOKENS, d) \
+            or v_pages.shape[1:] != (nv, PAGE_TOKENS, vd) or nkv % nv or (bias is not None and bias.numel() != columns) \
+            or (tied_values and (vd != d or nv != nkv)) or (value_cos is None) != (value_sin is None) \
+            or (value_cos is not None and (2 * value_cos.shape[-1] != vd or value_sin.shape != value_cos.shape)):
         raise KernelError("qkv_prepare: shapes do not fit")
     rot = _rotary_dim(cos, sin, d)
     fn = _fn("attention.cu", f"q3_qkv_prepare_{s}",
-             [c_void_p] * 11 + [c_int, c_int64, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+             [c_void_p] * 11 + [c_int, c_int64, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_int64, c_int, c_int,
+                                c_void_p, c_void_p, c_void_p])
     _check(fn(_dev(qkv, "qkv"), _dev(q_out, "q_out", qkv.dtype), _dev(k_pages, "k_pages"), _dev(v_pages, "v_pages"),
               _ptr(q_norm_w, "q_norm_w", torch.float32), _ptr(k_norm_w, "k_norm_w", torch.float32),
               _ptr(cos, "cos", torch.float32), _ptr(sin, "sin", torch.float32),
               _dev(token_seq, "token_seq", torch.int32), _dev(token_pos, "token_pos", torch.int32),
               _dev(page_table, "page_table", torch.int32), page_table.shape[-1], n_tokens, nq, nkv, d, float(eps),
-              int(bool(write_kv)), rot, _ptr(bias, "bias", torch.float32), vd, nv, _stream()), "qkv_prepare")
+              int(bool(write_kv)), rot, _ptr(bias, "bias", torch.float32), vd, nv, qkv.shape[-1], int(bool(tied_values)),
+              int(bool(norm_once)), _ptr(value_cos, "value_cos", torch.float32), _ptr(value_sin, "value_sin", torch.float32), _stream()),
+           "qkv_prepare")
     return q_out
+
+
+@dataclass
+class Pool:
+    """Pooled blocks beside a window: their pages [pages, kv heads, PAGE_TOKENS, size of a key or value], the step's page
+    table of them, and the tokens of a block."""
+    keys: torch.Tensor
+    values: torch.Tensor
+    table: torch.Tensor
+    size: int
+
+
+def _pool_args(pool: Optional[Pool], k_pages, v_pages, page_table, window, name: str):
+    """(keys, values, table, tokens of a block) for a launch; all zero without pooled blocks."""
+    if pool is None:
+        return None, None, None, 0
+    if not window or pool.size <= 0 or pool.keys.shape[1:] != k_pages.shape[1:] or pool.values.shape[1:] != v_pages.shape[1:] \
+            or pool.table.shape != page_table.shape:
+        raise KernelError(f"{name}: the pooled blocks do not fit the pages")
+    return (_dev(pool.keys, "pool keys", k_pages.dtype), _dev(pool.values, "pool values", v_pages.dtype),
+            _dev(pool.table, "pool table", torch.int32), int(pool.size))
+
+
+def pool_blocks(k_pages, v_pages, page_table, pool: Pool, seq_start, seq_pos0, n_seqs: int, max_new: int) -> None:
+    """Writes the pooled key and value (the means over a block's cached keys and values) of every block of `pool.size` tokens
+    that the step completes; the step's own keys and values are in their pages already."""
+    nkv, _, d = k_pages.shape[1:]
+    vd = v_pages.shape[-1]
+    keys, values, table, size = _pool_args(pool, k_pages, v_pages, page_table, 1, "pool_blocks")
+    if v_pages.shape[1] != nkv:
+        raise KernelError("pool_blocks: as many value heads as key heads")
+    fn = _fn("attention.cu", f"q3_pool_blocks_{_suffix(k_pages)}", [c_void_p] * 8 + [c_int] * 7 + [c_void_p])
+    _check(fn(_dev(k_pages, "k_pages"), _dev(v_pages, "v_pages", k_pages.dtype), _dev(page_table, "page_table", torch.int32), keys, values,
+              table, _dev(seq_start, "seq_start", torch.int32), _dev(seq_pos0, "seq_pos0", torch.int32), page_table.shape[-1], int(n_seqs),
+              int(max_new), nkv, d, vd, size, _stream()), "pool_blocks")
+
+
+def turn_back_gate(x: torch.Tensor, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], token_pos, gate: Optional[torch.Tensor],
+                   heads: int, vd: int) -> torch.Tensor:
+    """In place on x [N, heads * vd]: every head turned back by its token's position (pairs (i, i + vd/2), tables
+    [positions, vd / 2]; None: not turned), then multiplied value by value by sigmoid(gate) (a view of [N, heads * vd]
+    columns; None: no gate)."""
+    N = x.shape[0]
+    if x.shape[1] != heads * vd or vd % 2 or (cos is None) != (sin is None) or (cos is not None and (2 * cos.shape[-1] != vd or sin.shape != cos.shape)) \
+            or (gate is not None and (gate.shape != x.shape or gate.stride(1) != 1 or gate.dtype != x.dtype)):
+        raise KernelError("turn_back_gate: shapes do not fit")
+    fn = _fn("attention.cu", f"q3_turn_back_gate_{_suffix(x)}", [c_void_p] * 5 + [c_int64, c_int, c_int, c_int64, c_void_p])
+    _check(fn(_dev(x, "x"), _ptr(cos, "cos", torch.float32), _ptr(sin, "sin", torch.float32), _dev(token_pos, "token_pos", torch.int32),
+              gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0, int(heads), int(vd), N, _stream()),
+           "turn_back_gate")
+    return x
 
 
 def _sink_ptr(sink, sink_values, nq: int):
@@ -447,7 +526,7 @@ def _sink_ptr(sink, sink_values, nq: int):
 def attention_generic(q, k_pages, v_pages, out, token_seq, token_pos, page_table, n_tokens: int, nq: int, nkv: int,
                       d: int, scale: float, window: Optional[int] = None, value_dim: Optional[int] = None,
                       softcap: float = 0.0, chunk: Optional[int] = None, sink: bool = False, value_heads: Optional[int] = None,
-                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0):
+                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None):
     """Causal grouped-query attention of every token of the step over its sequence's pages.  `keep_first` (with `window`):
     the first so many keys of the sequence are seen beside the window's.  `softcap` > 0 caps the
     scores smoothly (s <- softcap * tanh(s / softcap)); `chunk`: a query reads only the keys of its own chunk of that
@@ -465,14 +544,14 @@ def attention_generic(q, k_pages, v_pages, out, token_seq, token_pos, page_table
         raise KernelError("attention: a window or chunks, not both")
     fn = _fn("attention.cu", f"q3_attention_generic_{s}",
              [c_void_p] * 7 + [c_int, c_int64, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int, c_int, c_int,
-                               c_void_p, c_int, c_void_p])
+                               c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", q.dtype), _dev(v_pages, "v_pages", q.dtype),
               _dev(out, "out"), _dev(token_seq, "token_seq", torch.int32),
               _dev(token_pos, "token_pos", torch.int32), _dev(page_table, "page_table", torch.int32),
               page_table.shape[-1], n_tokens, nq, nkv, d, float(scale), int(window or 0), vd, float(softcap or 0.0),
               int(chunk or 0), int(bool(sink)), nv, int(out.dtype == torch.float32 and q.dtype != torch.float32),
-              _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0, _stream()),
-           "attention_generic")
+              _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
+              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_generic"), _stream()), "attention_generic")
     return out
 
 
@@ -566,20 +645,27 @@ def hyper_norm(streams: torch.Tensor, n_streams: int, branch: Optional[torch.Ten
 # ------------------------------------------------------------------ linear attention with a decay and a state per sequence
 def lightning_attention(proj: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, seq_start: torch.Tensor,
                         seq_slots: torch.Tensor, out: torch.Tensor, n_seqs: int, heads: int, d: int, vd: int,
-                        chunked: bool = False) -> torch.Tensor:
+                        chunked: bool = False, silu: bool = True, k_scale: float = 1.0, cos: Optional[torch.Tensor] = None,
+                        sin: Optional[torch.Tensor] = None, token_pos: Optional[torch.Tensor] = None) -> torch.Tensor:
     """S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t over the new tokens of every sequence, from and to the state rows
     [slot, heads, d, vd] (float32).  `proj` [N, 2 heads d + 2 heads vd] holds q, k, v (SiLU is applied here) and a gate
-    that is not read; `out` [N, heads * vd] float32.  `chunked`: the form for prompts (32 tokens at a time)."""
-    if proj.shape[1] != 2 * heads * (d + vd) or tuple(state.shape[1:]) != (heads, d, vd) or out.shape[1] != heads * vd \
-            or out.dtype != torch.float32 or decay.numel() != heads:
+    that is not read; `out` [N, heads * vd] float32.  `chunked`: the form for prompts (32 tokens at a time).
+    Retention: `silu=False` (q, k, v as projected), the first 2 * tables' width values of every head of q and k rotated by
+    `token_pos` in pairs (i, i + width) with the tables `cos`, `sin` [positions, width], k multiplied by `k_scale`; `state` may
+    also be a view [slots, heads * d * vd] of wider rows."""
+    if proj.shape[1] != 2 * heads * (d + vd) or tuple(state.shape[1:]) not in ((heads, d, vd), (heads * d * vd,)) or out.shape[1] != heads * vd \
+            or out.dtype != torch.float32 or decay.numel() != heads or state.dtype != torch.float32 or not state[0].is_contiguous() \
+            or (cos is not None and token_pos is None):
         raise KernelError("lightning_attention: shapes do not fit")
+    rot = _rotary_dim(cos, sin, d) if cos is not None else 0
     name = "chunks" if chunked else "scan"
     if chunked and proj.dtype == torch.bfloat16 and lightning_tensor_cores and lightning_chunks_tc_fit(d, vd):
         name = "chunks_tc"                                   # the chunks' products on the tensor cores (TF32 hi + lo operands)
-    fn = _fn("lightning.cu", f"q3_lightning_{name}_{_suffix(proj)}", [c_void_p] * 6 + [c_int, c_int, c_int, c_int, c_void_p])
-    _check(fn(_dev(proj, "proj"), _dev(state, "state", torch.float32), _dev(decay, "decay", torch.float32),
+    fn = _fn("lightning.cu", f"q3_lightning_{name}_{_suffix(proj)}", [c_void_p] * 6 + [c_int] * 5 + [c_float, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p])
+    _check(fn(_dev(proj, "proj"), state.data_ptr(), _dev(decay, "decay", torch.float32),
               _dev(seq_start, "seq_start", torch.int32), _dev(seq_slots, "seq_slots", torch.int32), _dev(out, "out"),
-              int(n_seqs), heads, d, vd, _stream()), f"lightning_{name}")
+              int(n_seqs), heads, d, vd, int(bool(silu)), float(k_scale), _ptr(cos, "cos", torch.float32), _ptr(sin, "sin", torch.float32),
+              rot, _ptr(token_pos, "token_pos", torch.int32), state.stride(0), _stream()), f"lightning_{name}")
     return out
 
 
@@ -674,21 +760,21 @@ def memory_gates(z: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, ca
               _dev(low, "low", torch.float32), heads, 2 * heads, int(n_seqs), _stream()), "memory_gates")
 
 
-def head_gated_norm(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, eps: float, out: torch.Tensor, heads: int, vd: int,
+def head_gated_norm(o: torch.Tensor, weight: Optional[torch.Tensor], gate: torch.Tensor, eps: float, out: torch.Tensor, heads: int, vd: int,
                     act: str = "sigmoid", low: Optional[torch.Tensor] = None, floor: float = 0.0) -> torch.Tensor:
     """Per (token, head): x = o[t, h, :vd] (with `low` [N, heads]: divided by max(|o[t, h, vd]|, low) + floor, the row then
     holding vd + 1 values), out = x / sqrt(mean(x^2) + eps) * weight * act(gate), act 'sigmoid' or 'silu'; `weight` float32
-    [vd] (one for all heads) or [heads * vd]; `gate` a view of [N, heads * vd] columns; out in the gate's type."""
+    [vd] (one for all heads), [heads * vd], or None (no weight); `gate` a view of [N, heads * vd] columns; out in the gate's type."""
     N = o.shape[0]
     vdx = vd + (1 if low is not None else 0)
-    if o.shape[1] != heads * vdx or o.dtype != torch.float32 or not o.is_contiguous() or weight.numel() not in (vd, heads * vd) \
+    if o.shape[1] != heads * vdx or o.dtype != torch.float32 or not o.is_contiguous() or (weight is not None and weight.numel() not in (vd, heads * vd)) \
             or gate.shape != (N, heads * vd) or gate.stride(1) != 1 or out.shape != (N, heads * vd) or out.dtype != gate.dtype \
             or not out.is_contiguous() or act not in ("sigmoid", "silu") or (low is not None and low.numel() < N * heads):
         raise KernelError("head_gated_norm: shapes do not fit")
     fn = _fn("linear_scan.cu", f"q3_head_gated_norm_{_suffix(out)}",
              [c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_float, c_int, c_void_p])
-    _check(fn(o.data_ptr(), _ptr(low, "low", torch.float32), float(floor), _dev(weight, "weight", torch.float32),
-              int(weight.numel() == heads * vd and heads > 1), gate.data_ptr(), gate.stride(0), out.data_ptr(), N, heads, vd, vdx, float(eps),
+    _check(fn(o.data_ptr(), _ptr(low, "low", torch.float32), float(floor), _ptr(weight, "weight", torch.float32),
+              int(weight is not None and weight.numel() == heads * vd and heads > 1), gate.data_ptr(), gate.stride(0), out.data_ptr(), N, heads, vd, vdx, float(eps),
               int(act == "silu"), _stream()), "head_gated_norm")
     return out
 
@@ -707,11 +793,12 @@ def diff_combine(a: torch.Tensor, out: torch.Tensor, n_tokens: int, heads: int, 
 
 
 # ------------------------------------------------------------------ feed-forwards: a plain activation; routed experts
-PLAIN_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu": 2}
+PLAIN_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu": 2, "relu2": 3}
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tensor:
-    """out = act(x) elementwise (`out` may be `x`); kinds: silu, gelu_tanh, gelu (with the error function)."""
+    """out = act(x) elementwise (`out` may be `x`); kinds: silu, gelu_tanh, gelu (with the error function),
+    relu2 (max(x, 0)^2)."""
     if out.shape != x.shape or out.dtype != x.dtype:
         raise KernelError("activation: output does not fit")
     fn = _fn("elementwise.cu", f"q3_activation_{_suffix(x)}", [c_void_p, c_void_p, c_int64, c_int, c_void_p])
@@ -719,19 +806,19 @@ def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> torch.Tensor:
     return out
 
 
-def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor, top_ids: torch.Tensor, top_w: torch.Tensor,
+def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], top_ids: torch.Tensor, top_w: torch.Tensor,
               id_weight: torch.Tensor, n_real: int, top: int, group_count: int = 1, group_keep: int = 1, by_logit: bool = False,
               gate_out: Optional[torch.Tensor] = None, sigmoid: bool = False, group_pair: bool = False,
               weight_scale: float = 1.0) -> None:
     """Router of a mixture of experts for every token of h [N, hidden]: float32 logits, softmax over all outputs
-    (`sigmoid`: each output's sigmoid by itself), choice by score + correction within the kept groups (a group's mark:
+    (`sigmoid`: each output's sigmoid by itself), choice by score + correction (None: by the score alone) within the kept groups (a group's mark:
     its best choice score, or with `group_pair` the sum of its two best), weights = plain scores times `weight_scale`;
     `by_logit`: the largest logits are chosen and weighted by the softmax over the chosen logits alone (the correction is
     not read).  With `gate_out` [N] the router matrix has one more row, and gate_out = sigmoid of its logit; see csrc/moe.cu."""
     N, hidden = h.shape
     n_out = w_router.shape[0] - (1 if gate_out is not None else 0)
     if w_router.shape[1] != hidden or w_router.dtype != h.dtype or (correction is not None and correction.numel() != n_out) \
-            or (correction is None and not by_logit) or top_ids.numel() < N * top or top_w.numel() < N * top or id_weight.numel() < N \
+            or top_ids.numel() < N * top or top_w.numel() < N * top or id_weight.numel() < N \
             or (gate_out is not None and gate_out.numel() < N) or (by_logit and sigmoid):
         raise KernelError("moe_route: shapes do not fit")
     fn = _fn("moe.cu", f"q3_moe_route_{_suffix(h)}",
@@ -758,29 +845,30 @@ moe_tensor_cores = True      # tests switch it off to run the fmaf tiles in bflo
 
 def moe_experts(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, offsets: torch.Tensor, pair_of_slot: torch.Tensor,
                 act: torch.Tensor, y: torch.Tensor, n_pairs: int, n_real: int, top: int, ff: int, limit: float, alpha: float,
-                up_offset: float = 1.0) -> None:
+                up_offset: float = 1.0, gated: bool = True) -> None:
     """The experts' two products for the sorted pairs: act[slot] = g sigmoid(alpha g) (u + up_offset) with g = min(W_gate x, limit),
     u = clamp(W_up x, -limit, limit) (limit infinity, alpha 1, up_offset 0: SiLU(gate) * up), then y[slot] = W_down act[slot] (float32).  w_gate_up [n_real, 2 ff, hidden] (an
-    expert's gate rows, then its up rows), w_down [n_real, hidden, ff]."""
+    expert's gate rows, then its up rows), w_down [n_real, hidden, ff].  `gated=False`: act[slot] = max(W_up x, 0)^2 with
+    w_gate_up [n_real, ff, hidden]."""
     hidden = h.shape[1]
-    if w_gate_up.numel() != n_real * 2 * ff * hidden or w_down.numel() != n_real * hidden * ff or act.numel() < n_pairs * ff \
+    if w_gate_up.numel() != n_real * (2 if gated else 1) * ff * hidden or w_down.numel() != n_real * hidden * ff or act.numel() < n_pairs * ff \
             or y.numel() < n_pairs * hidden or y.dtype != torch.float32 or act.dtype != h.dtype or w_gate_up.dtype != h.dtype:
         raise KernelError("moe_experts: shapes do not fit")
     tensor_cores = h.dtype == torch.bfloat16 and hidden % 32 == 0 and ff % 32 == 0 and moe_tensor_cores
     name = "q3_moe_experts_tc_bf16" if tensor_cores else f"q3_moe_experts_{_suffix(h)}"
-    fn = _fn("moe.cu", name, [c_void_p] * 7 + [c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p])
+    fn = _fn("moe.cu", name, [c_void_p] * 7 + [c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p])
     _check(fn(_dev(h, "h"), _dev(w_gate_up, "w_gate_up"), _dev(w_down, "w_down"), _dev(offsets, "offsets", torch.int32),
               _dev(pair_of_slot, "pair_of_slot", torch.int32), _dev(act, "act"), _dev(y, "y"), int(n_pairs), int(n_real), int(top),
-              hidden, int(ff), float(limit), float(alpha), float(up_offset), _stream()), "moe_experts")
+              hidden, int(ff), float(limit), float(alpha), float(up_offset), int(bool(gated)), _stream()), "moe_experts")
     _count_extra(1)
 
 
 def moe_combine(y: torch.Tensor, h: torch.Tensor, slot_of_pair: torch.Tensor, top_w: torch.Tensor, id_weight: torch.Tensor,
                 out: torch.Tensor, top: int, shared: Optional[torch.Tensor] = None, shared_w: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """out[t] = sum_k top_w[t, k] y[slot_of_pair[t, k]] + id_weight[t] h[t] (+ shared_w[t] shared[t])."""
+    """out[t] = sum_k top_w[t, k] y[slot_of_pair[t, k]] + id_weight[t] h[t] (+ shared_w[t] shared[t]; shared_w None: + shared[t])."""
     N, hidden = h.shape
-    if out.shape != h.shape or out.dtype != h.dtype or (shared is None) != (shared_w is None) \
-            or (shared is not None and (shared.shape != h.shape or shared.dtype != h.dtype or shared_w.numel() < N)):
+    if out.shape != h.shape or out.dtype != h.dtype or (shared is None and shared_w is not None) \
+            or (shared is not None and (shared.shape != h.shape or shared.dtype != h.dtype)) or (shared_w is not None and shared_w.numel() < N):
         raise KernelError("moe_combine: shapes do not fit")
     fn = _fn("moe.cu", f"q3_moe_combine_{_suffix(h)}", [c_void_p] * 6 + [c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p])
     _check(fn(_dev(y, "y", torch.float32), _dev(h, "h"), _dev(slot_of_pair, "slot_of_pair", torch.int32),
@@ -803,9 +891,10 @@ def _capped_defines(d: int, vd: int):
 def attention_capped_prefill(q, k_pages, v_pages, out, seq_start, seq_pos0, page_table, n_seqs: int, max_new: int, nq: int,
                              nkv: int, d: int, vd: int, scale: float, softcap: float = 0.0, chunk: Optional[int] = None,
                              sink: bool = False, window: Optional[int] = None, value_heads: Optional[int] = None,
-                             sink_values: Optional[torch.Tensor] = None, keep_first: int = 0):
+                             sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None):
     """Attention of every new token of every sequence over its pages (bfloat16, tiled, tensor cores) with capped scores,
-    chunked visibility or a sliding window (beside which the first `keep_first` keys of the sequence stay visible), and a sink (its score per query head in `sink_values`, else 0); q [tokens, nq * d], out [tokens, nq * vd] in bfloat16 or float32;
+    chunked visibility or a sliding window (beside which the first `keep_first` keys of the sequence stay visible, or the pooled
+    blocks of `pool`), and a sink (its score per query head in `sink_values`, else 0); q [tokens, nq * d], out [tokens, nq * vd] in bfloat16 or float32;
     `value_heads`: the number of value heads if not `nkv` (each serves nkv / value_heads key heads)."""
     nv = int(value_heads or nkv)
     if q.dtype != torch.bfloat16 or not attention_capped_fits(d, vd, None, 1) or out.dtype not in (torch.bfloat16, torch.float32):
@@ -814,14 +903,14 @@ def attention_capped_prefill(q, k_pages, v_pages, out, seq_start, seq_pos0, page
         raise KernelError("attention_capped_prefill: shapes do not fit")
     fn = _fn("attention_capped.cu", "q3_attention_capped_prefill_bf16",
              [c_void_p] * 7 + [c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                               c_int, c_void_p],
+                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
              defines=_capped_defines(d, vd))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out"), _dev(seq_start, "seq_start", torch.int32),
               _dev(seq_pos0, "seq_pos0", torch.int32), _dev(page_table, "page_table", torch.int32), page_table.shape[-1],
               n_seqs, max_new, nq, nkv, float(scale), float(softcap or 0.0), int(chunk or 0), int(bool(sink)), int(window or 0), nv,
-              int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0, _stream()),
-           "attention_capped_prefill")
+              int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
+              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_prefill"), _stream()), "attention_capped_prefill")
     return out
 
 
@@ -834,7 +923,7 @@ def attention_capped_splits(n_tokens: int, nkv: int, sm_count: int, max_keys: in
 def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_pos, page_table, n_tokens: int, nq: int,
                             nkv: int, d: int, vd: int, scale: float, softcap: float, chunk: Optional[int], sink: bool,
                             n_splits: int, window: Optional[int] = None, value_heads: Optional[int] = None,
-                            sink_values: Optional[torch.Tensor] = None, keep_first: int = 0):
+                            sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None):
     """The same for one new token per sequence, the keys split over `n_splits` blocks per (token, kv head); `scratch`
     holds n_tokens * nq * n_splits * (vd + 2) float32."""
     nv = int(value_heads or nkv)
@@ -845,15 +934,15 @@ def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_
         raise KernelError("attention_capped_decode: shapes do not fit")
     fn = _fn("attention_capped.cu", "q3_attention_capped_decode_bf16",
              [c_void_p] * 8 + [c_int, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                               c_int, c_void_p],
+                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
              defines=_capped_defines(d, vd))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out"), _dev(scratch, "scratch", torch.float32),
               _dev(token_seq, "token_seq", torch.int32), _dev(token_pos, "token_pos", torch.int32),
               _dev(page_table, "page_table", torch.int32), page_table.shape[-1], n_tokens, nq, nkv, float(scale),
               float(softcap or 0.0), int(chunk or 0), int(bool(sink)), int(n_splits), int(window or 0), nv,
-              int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0, _stream()),
-           "attention_capped_decode")
+              int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
+              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_decode"), _stream()), "attention_capped_decode")
     _count_extra(1)                                              # the split kernel and the merge kernel
     return out
 
@@ -889,19 +978,19 @@ def attention_capped_prefill_tc_fits(d: int, vd: int, window: Optional[int]) -> 
 
 def attention_capped_prefill_tc(q, k_pages, v_pages, out, seq_start, seq_pos0, page_table, n_seqs: int, max_new: int,
                                 n_tokens: int, nq: int, nkv: int, d: int, scale: float, softcap: float = 0.0,
-                                chunk: Optional[int] = None, sink: bool = False):
+                                chunk: Optional[int] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None):
     """`attention_capped_prefill` with both products on tcgen05 (TMA-fed, scores and output in tensor memory): head
     sizes 64 and 128, values as wide as keys."""
     if q.dtype != torch.bfloat16 or not attention_capped_prefill_tc_fits(d, d, None) or not scale > 0:
         raise KernelError("attention_capped_prefill_tc: bfloat16, head size 64 or 128, a positive scale")
     fn = _fn("attention_prefill_tc.cu", "q3_attention_capped_prefill_tc_bf16",
-             [c_void_p] * 7 + [c_int, c_int, c_int, c_int64, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p],
+             [c_void_p] * 7 + [c_int, c_int, c_int, c_int64, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
              defines=(f"Q3_HEAD_DIM={d}", "Q3_CAPPED=1"))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out", torch.bfloat16), _dev(seq_start, "seq_start", torch.int32),
               _dev(seq_pos0, "seq_pos0", torch.int32), _dev(page_table, "page_table", torch.int32),
               page_table.shape[-1], n_seqs, max_new, n_tokens, k_pages.shape[0], nq, nkv, float(scale), float(softcap or 0.0),
-              int(chunk or 0), int(bool(sink)), _status_word(q.device).data_ptr(), _stream()), "attention_capped_prefill_tc")
+              int(chunk or 0), int(bool(sink)), _sink_ptr(sink, sink_values, nq), _status_word(q.device).data_ptr(), _stream()), "attention_capped_prefill_tc")
     return out
 
 

@@ -8,8 +8,11 @@
 //                      sublayer, the residual sum and the norm before the next sublayer in one
 //                      pass over the row.  Either half may be left out (no branch: a plain norm
 //                      of the stream; no output: the sum alone).  rms(x) = sqrt(mean(x^2) + eps).
+//                      Each norm may be in groups: the row is split into that many equal consecutive parts
+//                      and every part is divided by its own rms.
 //   concat_cast      : out[t] = T([a[t]; b[t]])  (the input of a product over two streams)
 //   gather_rows_norm : rows of the stream picked by index and normalised    (float -> T)
+//   normed_sum       : out = T( s_a a / rms(a) * w_a + s_b b / rms(b) * w_b ), two branches of one layer (T)
 //   scale_softcap    : x <- cap * tanh(x * scale / cap), or x * scale without a cap (float, in place)
 //
 // Statistics, weights and sums are 32-bit; only `out` is rounded to T.
@@ -54,19 +57,57 @@ __global__ void embedding_scaled_kernel(const int* __restrict__ ids, const T* __
 
 // ---------------------------------------------------------------- norm after a branch + sum + norm before the next
 // One block per row; a thread keeps PER groups of four values of the row in registers, so the stream is read and
-// written once.  PER = 0: any size, the row walked three times through the cache.
-template <typename T, int PER>
+// written once.  PER = 0: any size, the row walked three times through the cache.  GROUPS: norms over equal parts of
+// the row (the statistics of a part are summed by one warp in a fixed order); else over the row as a whole.
+struct SandwichArgs {
+    int size;
+    int parts_post, parts_pre;
+    float eps_post, eps_pre;
+};
+
+// inv[p] = 1 / rms of part p from the sums of squares of the row's quads (dynamic shared memory: quads, then parts).
+__device__ __forceinline__ void part_scales(const float* quad_sq, float* inv, int size, int parts, float eps) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5, per = size / 4 / parts;
+    __syncthreads();
+    for (int p = warp; p < parts; p += n_warps) {
+        float sum = 0.0f;
+        for (int i = lane; i < per; i += 32) sum += quad_sq[p * per + i];
+        sum = warp_sum(sum);
+        if (lane == 0) inv[p] = rsqrtf(sum / (float)(size / parts) + eps);
+    }
+    __syncthreads();
+}
+// The same from the row itself, `at(c)` its value at column c.
+template <typename F> __device__ __forceinline__ void part_scales_of(F&& at, float* inv, int size, int parts, float eps) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5, per = size / parts;
+    __syncthreads();
+    for (int p = warp; p < parts; p += n_warps) {
+        float sum = 0.0f;
+        for (int i = lane; i < per; i += 32) {
+            const float v = at(p * per + i);
+            sum += v * v;
+        }
+        sum = warp_sum(sum);
+        if (lane == 0) inv[p] = rsqrtf(sum / (float)per + eps);
+    }
+    __syncthreads();
+}
+
+template <typename T, int PER, bool GROUPS>
 __global__ void sandwich_norm_kernel(float* __restrict__ stream, const T* __restrict__ branch, const float* __restrict__ w_post,
-                                     const float* __restrict__ w_pre, T* __restrict__ out, int size, float eps_post,
-                                     float eps_pre) {
+                                     const float* __restrict__ w_pre, T* __restrict__ out, const SandwichArgs args) {
     __shared__ float scratch[33];
+    extern __shared__ float parts_s[];
     pdl_launch_dependents();
     pdl_wait();
+    const int size = args.size;
     const int64_t row = blockIdx.x;
     float* xr = stream + row * size;
     const T* yr = branch ? branch + row * size : nullptr;
     T* outr = out ? out + row * size : nullptr;
     if constexpr (PER > 0) {
+        float* quad_sq = parts_s;                          // [size / 4]
+        float* inv_s = parts_s + size / 4;                 // [parts]
         float x[PER][4], y[PER][4];
         float sq = 0.0f;
 #pragma unroll
@@ -76,17 +117,21 @@ __global__ void sandwich_norm_kernel(float* __restrict__ stream, const T* __rest
                 load4<float>(xr + c, x[p]);
                 if (yr) {
                     load4<T>(yr + c, y[p]);
+                    if constexpr (GROUPS) quad_sq[c >> 2] = (y[p][0] * y[p][0] + y[p][1] * y[p][1]) + (y[p][2] * y[p][2] + y[p][3] * y[p][3]);
 #pragma unroll
                     for (int i = 0; i < 4; ++i) sq += y[p][i] * y[p][i];
                 }
             }
         }
         if (yr) {
-            const float inv = rsqrtf(block_sum(sq, scratch) / (float)size + eps_post);
+            float inv = 0.0f;
+            if constexpr (GROUPS) part_scales(quad_sq, inv_s, size, args.parts_post, args.eps_post);
+            else inv = rsqrtf(block_sum(sq, scratch) / (float)size + args.eps_post);
 #pragma unroll
             for (int p = 0; p < PER; ++p) {
                 const int c = (p * blockDim.x + threadIdx.x) * 4;
                 if (c < size) {
+                    if constexpr (GROUPS) inv = inv_s[c / (size / args.parts_post)];
                     float w[4];
                     load4<float>(w_post + c, w);
 #pragma unroll
@@ -101,15 +146,19 @@ __global__ void sandwich_norm_kernel(float* __restrict__ stream, const T* __rest
         for (int p = 0; p < PER; ++p) {
             const int c = (p * blockDim.x + threadIdx.x) * 4;
             if (c < size) {
+                if constexpr (GROUPS) quad_sq[c >> 2] = (x[p][0] * x[p][0] + x[p][1] * x[p][1]) + (x[p][2] * x[p][2] + x[p][3] * x[p][3]);
 #pragma unroll
                 for (int i = 0; i < 4; ++i) sq += x[p][i] * x[p][i];
             }
         }
-        const float inv = rsqrtf(block_sum(sq, scratch) / (float)size + eps_pre);
+        float inv = 0.0f;
+        if constexpr (GROUPS) part_scales(quad_sq, inv_s, size, args.parts_pre, args.eps_pre);
+        else inv = rsqrtf(block_sum(sq, scratch) / (float)size + args.eps_pre);
 #pragma unroll
         for (int p = 0; p < PER; ++p) {
             const int c = (p * blockDim.x + threadIdx.x) * 4;
             if (c < size) {
+                if constexpr (GROUPS) inv = inv_s[c / (size / args.parts_pre)];
                 float w[4], v[4];
                 load4<float>(w_pre + c, w);
 #pragma unroll
@@ -118,44 +167,121 @@ __global__ void sandwich_norm_kernel(float* __restrict__ stream, const T* __rest
             }
         }
     } else {
+        float* inv_s = parts_s;                            // [parts]
         if (yr) {
-            float sq = 0.0f;
-            for (int c = threadIdx.x; c < size; c += blockDim.x) {
-                const float v = to_f32<T>(yr[c]);
-                sq += v * v;
-            }
-            const float inv = rsqrtf(block_sum(sq, scratch) / (float)size + eps_post);
-            for (int c = threadIdx.x; c < size; c += blockDim.x) xr[c] += to_f32<T>(yr[c]) * inv * w_post[c];
+            const int per = size / args.parts_post;
+            part_scales_of([&](int c) { return to_f32<T>(yr[c]); }, inv_s, size, args.parts_post, args.eps_post);
+            for (int c = threadIdx.x; c < size; c += blockDim.x) xr[c] += to_f32<T>(yr[c]) * inv_s[c / per] * w_post[c];
         }
         if (outr == nullptr) return;
-        float sq = 0.0f;
-        for (int c = threadIdx.x; c < size; c += blockDim.x) sq += xr[c] * xr[c];       // the thread's own writes
-        const float inv = rsqrtf(block_sum(sq, scratch) / (float)size + eps_pre);
-        for (int c = threadIdx.x; c < size; c += blockDim.x) outr[c] = from_f32<T>(xr[c] * inv * w_pre[c]);
+        const int per = size / args.parts_pre;
+        part_scales_of([&](int c) { return xr[c]; }, inv_s, size, args.parts_pre, args.eps_pre);
+        for (int c = threadIdx.x; c < size; c += blockDim.x) outr[c] = from_f32<T>(xr[c] * inv_s[c / per] * w_pre[c]);
     }
 }
 
 template <typename T>
 int sandwich_norm_launch(float* stream, const T* branch, const float* w_post, const float* w_pre, T* out, int64_t rows, int size,
-                         float eps_post, float eps_pre, cudaStream_t s) {
+                         float eps_post, float eps_pre, int parts_post, int parts_pre, cudaStream_t s) {
     if (rows <= 0) return 0;
     if (size <= 0 || (branch != nullptr) != (w_post != nullptr) || (out != nullptr) != (w_pre != nullptr)) return Q3_ERR_BAD_SIZE;
+    if (parts_post <= 0 || parts_pre <= 0 || size % parts_post != 0 || size % parts_pre != 0) return Q3_ERR_BAD_SIZE;
     if (rows > 0x7fffffffLL) return Q3_ERR_TOO_LARGE;
-    const bool vec = size % 4 == 0 && aligned16(stream) && (branch == nullptr || aligned16(branch)) && (out == nullptr || aligned16(out)) &&
+    const bool grouped = parts_post > 1 || parts_pre > 1;
+    const bool vec = size % 4 == 0 && (!grouped || ((size / parts_post) % 4 == 0 && (size / parts_pre) % 4 == 0)) && aligned16(stream) &&
+                     (branch == nullptr || aligned16(branch)) && (out == nullptr || aligned16(out)) &&
                      (w_post == nullptr || aligned16(w_post)) && (w_pre == nullptr || aligned16(w_pre));
-    const int groups = size / 4;
-    auto launch = [&](auto kernel, int threads) {
-        return (int)q3_launch(kernel, dim3((unsigned)rows), dim3(threads), 0, s, stream, branch, w_post, w_pre, out, size, eps_post, eps_pre);
+    const int groups = size / 4, parts = parts_post > parts_pre ? parts_post : parts_pre;
+    const SandwichArgs args = {size, parts_post, parts_pre, eps_post, eps_pre};
+    auto launch = [&](auto kernel, int threads, size_t smem) {
+        return (int)q3_launch(kernel, dim3((unsigned)rows), dim3(threads), smem, s, stream, branch, w_post, w_pre, out, args);
     };
     if (vec && groups <= 2048) {
         const int per = groups <= 256 ? 1 : (groups <= 512 ? 2 : (groups <= 1024 ? 4 : 8));
         const int threads = ((groups + per - 1) / per + 31) / 32 * 32;
-        if (per == 1) return launch(sandwich_norm_kernel<T, 1>, threads);
-        if (per == 2) return launch(sandwich_norm_kernel<T, 2>, threads);
-        if (per == 4) return launch(sandwich_norm_kernel<T, 4>, threads);
-        return launch(sandwich_norm_kernel<T, 8>, threads);
+        const size_t smem = grouped ? (size_t)(groups + parts) * sizeof(float) : 0;
+#define Q3_SANDWICH(PER) return grouped ? launch(sandwich_norm_kernel<T, PER, true>, threads, smem) : launch(sandwich_norm_kernel<T, PER, false>, threads, 0)
+        if (per == 1) Q3_SANDWICH(1);
+        if (per == 2) Q3_SANDWICH(2);
+        if (per == 4) Q3_SANDWICH(4);
+        Q3_SANDWICH(8);
+#undef Q3_SANDWICH
     }
-    return launch(sandwich_norm_kernel<T, 0>, size >= 1024 ? 512 : 128);
+    if (parts > 8192) return Q3_ERR_TOO_LARGE;
+    return launch(sandwich_norm_kernel<T, 0, true>, size >= 1024 ? 512 : 128, (size_t)parts * sizeof(float));
+}
+
+// ---------------------------------------------------------------- two normed branches in one sum
+// One block per row.  PER > 0: a thread keeps PER groups of four values of both rows in registers.
+template <typename T, int PER>
+__global__ void normed_sum_kernel(const T* __restrict__ a, const T* __restrict__ b, const float* __restrict__ w_a,
+                                  const float* __restrict__ w_b, float s_a, float s_b, float eps, T* __restrict__ out, int size) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const T* ar = a + (int64_t)blockIdx.x * size;
+    const T* br = b + (int64_t)blockIdx.x * size;
+    T* outr = out + (int64_t)blockIdx.x * size;
+    float sq_a = 0.0f, sq_b = 0.0f;
+    if constexpr (PER > 0) {
+        float x[PER][4], y[PER][4];
+#pragma unroll
+        for (int p = 0; p < PER; ++p) {
+            const int c = (p * blockDim.x + threadIdx.x) * 4;
+            if (c < size) {
+                load4<T>(ar + c, x[p]);
+                load4<T>(br + c, y[p]);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    sq_a += x[p][i] * x[p][i];
+                    sq_b += y[p][i] * y[p][i];
+                }
+            }
+        }
+        const float inv_a = s_a * rsqrtf(block_sum(sq_a, scratch) / (float)size + eps), inv_b = s_b * rsqrtf(block_sum(sq_b, scratch) / (float)size + eps);
+#pragma unroll
+        for (int p = 0; p < PER; ++p) {
+            const int c = (p * blockDim.x + threadIdx.x) * 4;
+            if (c < size) {
+                float wa[4], wb[4], v[4];
+                load4<float>(w_a + c, wa);
+                load4<float>(w_b + c, wb);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) v[i] = x[p][i] * inv_a * wa[i] + y[p][i] * inv_b * wb[i];
+                store4<T>(outr + c, v);
+            }
+        }
+    } else {
+        for (int c = threadIdx.x; c < size; c += blockDim.x) {
+            const float x = to_f32<T>(ar[c]), y = to_f32<T>(br[c]);
+            sq_a += x * x;
+            sq_b += y * y;
+        }
+        const float inv_a = s_a * rsqrtf(block_sum(sq_a, scratch) / (float)size + eps), inv_b = s_b * rsqrtf(block_sum(sq_b, scratch) / (float)size + eps);
+        for (int c = threadIdx.x; c < size; c += blockDim.x)
+            outr[c] = from_f32<T>(to_f32<T>(ar[c]) * inv_a * w_a[c] + to_f32<T>(br[c]) * inv_b * w_b[c]);
+    }
+}
+
+template <typename T>
+int normed_sum_launch(const T* a, const T* b, const float* w_a, const float* w_b, float s_a, float s_b, float eps, T* out, int64_t rows,
+                      int size, cudaStream_t s) {
+    if (rows <= 0) return 0;
+    if (size <= 0 || w_a == nullptr || w_b == nullptr) return Q3_ERR_BAD_SIZE;
+    if (rows > 0x7fffffffLL) return Q3_ERR_TOO_LARGE;
+    auto launch = [&](auto kernel, int threads) {
+        return (int)q3_launch(kernel, dim3((unsigned)rows), dim3(threads), 0, s, a, b, w_a, w_b, s_a, s_b, eps, out, size);
+    };
+    const int groups = size / 4;
+    if (size % 4 == 0 && groups <= 2048 && aligned16(a) && aligned16(b) && aligned16(w_a) && aligned16(w_b) && aligned16(out)) {
+        const int per = groups <= 256 ? 1 : (groups <= 512 ? 2 : (groups <= 1024 ? 4 : 8));
+        const int threads = ((groups + per - 1) / per + 31) / 32 * 32;
+        if (per == 1) return launch(normed_sum_kernel<T, 1>, threads);
+        if (per == 2) return launch(normed_sum_kernel<T, 2>, threads);
+        if (per == 4) return launch(normed_sum_kernel<T, 4>, threads);
+        return launch(normed_sum_kernel<T, 8>, threads);
+    }
+    return launch(normed_sum_kernel<T, 0>, size >= 1024 ? 512 : 128);
 }
 
 // ---------------------------------------------------------------- [a; b] in the compute type
@@ -192,15 +318,23 @@ __global__ void concat_cast_kernel(const float* __restrict__ a, const float* __r
 // ---------------------------------------------------------------- picked rows, normalised
 template <typename T>
 __global__ void gather_rows_norm_kernel(const float* __restrict__ stream, const int* __restrict__ idx, const float* __restrict__ w,
-                                        T* __restrict__ out, int size, float eps) {
+                                        T* __restrict__ out, int size, float eps, int parts) {
     __shared__ float scratch[33];
+    extern __shared__ float inv_s[];                       // [parts] if there are several
     pdl_launch_dependents();
     pdl_wait();
     const float* xr = stream + (int64_t)idx[blockIdx.x] * size;
-    float sq = 0.0f;
-    for (int c = threadIdx.x; c < size; c += blockDim.x) sq += xr[c] * xr[c];
-    const float inv = rsqrtf(block_sum(sq, scratch) / (float)size + eps);
-    for (int c = threadIdx.x; c < size; c += blockDim.x) out[(int64_t)blockIdx.x * size + c] = from_f32<T>(xr[c] * inv * w[c]);
+    float inv = 0.0f;
+    const int per = size / parts;
+    if (parts == 1) {
+        float sq = 0.0f;
+        for (int c = threadIdx.x; c < size; c += blockDim.x) sq += xr[c] * xr[c];
+        inv = rsqrtf(block_sum(sq, scratch) / (float)size + eps);
+    } else {
+        part_scales_of([&](int c) { return xr[c]; }, inv_s, size, parts, eps);
+    }
+    for (int c = threadIdx.x; c < size; c += blockDim.x)
+        out[(int64_t)blockIdx.x * size + c] = from_f32<T>(xr[c] * (parts == 1 ? inv : inv_s[c / per]) * w[c]);
 }
 
 // ---------------------------------------------------------------- scale and smooth cap, in place
@@ -232,9 +366,14 @@ static unsigned grid_for(int64_t work, int threads) {
     }                                                                                                                    \
     Q3_EXPORT int q3_sandwich_norm_##SUFFIX(float* stream_rows, const void* branch, const float* w_post, const float* w_pre, \
                                             void* out, int64_t rows, int size, float eps_post, float eps_pre,           \
-                                            void* stream) {                                                              \
+                                            int parts_post, int parts_pre, void* stream) {                               \
         return sandwich_norm_launch<T>(stream_rows, (const T*)branch, w_post, w_pre, (T*)out, rows, size, eps_post,      \
-                                       eps_pre, (cudaStream_t)stream);                                                   \
+                                       eps_pre, parts_post, parts_pre, (cudaStream_t)stream);                            \
+    }                                                                                                                    \
+    Q3_EXPORT int q3_normed_sum_##SUFFIX(const void* a, const void* b, const float* w_a, const float* w_b, float s_a,    \
+                                         float s_b, float eps, void* out, int64_t rows, int size, void* stream) {        \
+        return normed_sum_launch<T>((const T*)a, (const T*)b, w_a, w_b, s_a, s_b, eps, (T*)out, rows, size,              \
+                                    (cudaStream_t)stream);                                                               \
     }                                                                                                                    \
     Q3_EXPORT int q3_concat_cast_##SUFFIX(const float* a, const float* b, void* out, int64_t rows, int size, void* stream) { \
         if (rows <= 0) return 0;                                                                                         \
@@ -246,11 +385,12 @@ static unsigned grid_for(int64_t work, int threads) {
                               (cudaStream_t)stream, a, b, (T*)out, rows, size);                                          \
     }                                                                                                                    \
     Q3_EXPORT int q3_gather_rows_norm_##SUFFIX(const float* stream_rows, const int* idx, const float* w, void* out,      \
-                                               int64_t rows, int size, float eps, void* stream) {                        \
+                                               int64_t rows, int size, float eps, int parts, void* stream) {             \
         if (rows <= 0) return 0;                                                                                         \
-        if (size <= 0 || rows > 0x7fffffffLL) return Q3_ERR_BAD_SIZE;                                                    \
-        return (int)q3_launch(gather_rows_norm_kernel<T>, dim3((unsigned)rows), dim3(size >= 1024 ? 256 : 128), 0,       \
-                              (cudaStream_t)stream, stream_rows, idx, w, (T*)out, size, eps);                            \
+        if (size <= 0 || rows > 0x7fffffffLL || parts <= 0 || size % parts != 0 || parts > 8192) return Q3_ERR_BAD_SIZE; \
+        return (int)q3_launch(gather_rows_norm_kernel<T>, dim3((unsigned)rows), dim3(size >= 1024 ? 256 : 128),          \
+                              parts > 1 ? (size_t)parts * sizeof(float) : 0, (cudaStream_t)stream, stream_rows, idx, w,  \
+                              (T*)out, size, eps, parts);                                                                \
     }
 
 Q3_STREAM_EXPORTS(f32, float)

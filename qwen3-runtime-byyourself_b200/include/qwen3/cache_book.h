@@ -7,7 +7,9 @@
 // pages that covers its length.  Layers whose mixers ask the same of the cache form a *group* with
 // a page pool of its own; a group that needs only a window of keys returns the pages that fell out
 // of the window after each step (but for the pages of the first keys, if its queries keep reading those), and a group whose queries read only the keys of their own chunk of
-// positions (chunks of a fixed size, counted from position 0) returns the pages of finished chunks.
+// positions (chunks of a fixed size, counted from position 0) returns the pages of finished chunks.  A group of
+// pooled blocks keeps one entry for every whole block of a fixed number of tokens, `page_tokens` entries a page, for
+// as long as the sequence lives.
 //
 // A step is three calls: reserve (all or nothing: a step that does not fit changes nothing), the
 // launch, then commit (lengths advance once) or cancel (the launch failed: the pages go back).
@@ -35,7 +37,7 @@ struct CacheFull : CacheError {
     using CacheError::CacheError;
 };
 
-enum class GroupKind : int { Full = 0, Window = 1, Chunk = 2 };
+enum class GroupKind : int { Full = 0, Window = 1, Chunk = 2, Pooled = 3 };
 
 // The pages of the layers that share one need.
 class PageGroup {
@@ -78,7 +80,7 @@ public:
     }
     // Give back the pages that no later query of this sequence can read (window and chunk groups).
     void trim_window(int slot, int64_t length) {
-        if (kind_ == GroupKind::Full) return;
+        if (kind_ == GroupKind::Full || kind_ == GroupKind::Pooled) return;
         int64_t dead;
         if (kind_ == GroupKind::Window) {
             // a query at position >= length reads keys > length - window
@@ -90,7 +92,7 @@ public:
         }
         int32_t* r = table_.data() + (size_t)slot * pages_per_slot_;
         // the pages that hold one of the first `keep_first` keys stay: every later query of a window group reads them
-        const int64_t kept = kind_ == GroupKind::Window ? pages_for(keep_first_) : 0;
+        const int64_t kept = kind_ == GroupKind::Window ? (keep_first_ + page_tokens_ - 1) / page_tokens_ : 0;
         for (int64_t i = std::max(first_live_[slot], kept); i < dead; ++i)
             if (r[i] >= 0) {
                 free_.push_back(r[i]);
@@ -109,7 +111,11 @@ public:
     }
 
 private:
-    int64_t pages_for(int64_t tokens) const { return (tokens + page_tokens_ - 1) / page_tokens_; }
+    // the pages that a sequence of `tokens` tokens needs: one entry a token, or one a whole block of `window_` tokens
+    int64_t pages_for(int64_t tokens) const {
+        const int64_t entries = kind_ == GroupKind::Pooled ? tokens / window_ : tokens;
+        return (entries + page_tokens_ - 1) / page_tokens_;
+    }
 
     GroupKind kind_;
     int window_, keep_first_, n_pages_, pages_per_slot_, page_tokens_;
@@ -120,7 +126,8 @@ private:
 // What one layer group asks of the cache.
 struct GroupNeed {
     GroupKind kind = GroupKind::Full;
-    int window = 0;        // Window groups: the number of keys a query reads; Chunk groups: the size of a chunk
+    int window = 0;        // Window groups: the number of keys a query reads; Chunk groups: the size of a chunk;
+                           // Pooled groups: the tokens of a block
     int keep_first = 0;    // Window groups: so many keys at the start of a sequence stay readable beside the window
 };
 
@@ -139,9 +146,11 @@ public:
         held_.assign(n_slots_, 0);
         for (int s = n_slots_ - 1; s >= 0; --s) free_slots_.push_back(s);
         for (const GroupNeed& g : groups) {
-            if (g.kind != GroupKind::Full && g.window <= 0) throw std::invalid_argument("a window or chunk group needs a positive size");
+            if (g.kind != GroupKind::Full && g.window <= 0) throw std::invalid_argument("a window, chunk or pooled group needs a positive size");
             if (g.keep_first < 0) throw std::invalid_argument("keep_first must not be negative");
-            groups_.emplace_back(g.kind, g.window, n_pages_, n_slots_, pages_per_slot_, page_tokens, g.keep_first);
+            // a pooled group never needs more than a page for every `window` pages of tokens and one more per sequence
+            const int pages = g.kind == GroupKind::Pooled ? (int)std::min<int64_t>(n_pages_, (int64_t)n_pages_ / g.window + n_slots_) : n_pages_;
+            groups_.emplace_back(g.kind, g.window, pages, n_slots_, pages_per_slot_, page_tokens, g.keep_first);
         }
     }
 

@@ -46,7 +46,7 @@ int q3_silu_mul_bf16(const void* gate_up, void* out, int64_t rows, int inter, in
 /* the same with the activation as a parameter: act 0 = SiLU, 1 = the tanh form of GELU */
 int q3_act_mul_f32(const void* gate_up, void* out, int64_t rows, int inter, int interleaved, int act, void* stream);
 int q3_act_mul_bf16(const void* gate_up, void* out, int64_t rows, int inter, int interleaved, int act, void* stream);
-/* out = act(x) elementwise: act 0 = SiLU, 1 = the tanh form of GELU, 2 = GELU with the error function */
+/* out = act(x) elementwise: act 0 = SiLU, 1 = the tanh form of GELU, 2 = GELU with the error function, 3 = max(x, 0)^2 */
 int q3_activation_f32(const void* x, void* out, int64_t n, int act, void* stream);
 int q3_activation_bf16(const void* x, void* out, int64_t n, int act, void* stream);
 /* out[r] = x[idx[r]] (+ delta[idx[r]]) */
@@ -62,17 +62,23 @@ int q3_place_rows(const void* src, int src_kind, void* dst, int dst_kind, int64_
 int q3_embedding_scaled_f32(const int* ids, const void* table, float* out, int64_t n_tokens, int hidden, int vocab, float scale, void* stream);
 int q3_embedding_scaled_bf16(const int* ids, const void* table, float* out, int64_t n_tokens, int hidden, int vocab, float scale, void* stream);
 /* stream += RMSNorm(branch) * w_post (branch and w_post may both be null), then out = RMSNorm(stream) * w_pre (out and
-   w_pre may both be null), one pass over a row */
+   w_pre may both be null), one pass over a row; parts_post, parts_pre: a norm splits the row into that many equal
+   consecutive parts, each with an rms of its own (1: the row as a whole) */
 int q3_sandwich_norm_f32(float* stream_rows, const void* branch, const float* w_post, const float* w_pre, void* out, int64_t rows,
-                         int size, float eps_post, float eps_pre, void* stream);
+                         int size, float eps_post, float eps_pre, int parts_post, int parts_pre, void* stream);
 int q3_sandwich_norm_bf16(float* stream_rows, const void* branch, const float* w_post, const float* w_pre, void* out, int64_t rows,
-                          int size, float eps_post, float eps_pre, void* stream);
+                          int size, float eps_post, float eps_pre, int parts_post, int parts_pre, void* stream);
 /* out[t] = [a[t]; b[t]] in the compute type */
 int q3_concat_cast_f32(const float* a, const float* b, void* out, int64_t rows, int size, void* stream);
 int q3_concat_cast_bf16(const float* a, const float* b, void* out, int64_t rows, int size, void* stream);
-/* out[r] = RMSNorm(stream_rows[idx[r]]) * w */
-int q3_gather_rows_norm_f32(const float* stream_rows, const int* idx, const float* w, void* out, int64_t rows, int size, float eps, void* stream);
-int q3_gather_rows_norm_bf16(const float* stream_rows, const int* idx, const float* w, void* out, int64_t rows, int size, float eps, void* stream);
+/* out = s_a * RMSNorm(a) * w_a + s_b * RMSNorm(b) * w_b, row by row */
+int q3_normed_sum_f32(const void* a, const void* b, const float* w_a, const float* w_b, float s_a, float s_b, float eps, void* out,
+                      int64_t rows, int size, void* stream);
+int q3_normed_sum_bf16(const void* a, const void* b, const float* w_a, const float* w_b, float s_a, float s_b, float eps, void* out,
+                       int64_t rows, int size, void* stream);
+/* out[r] = RMSNorm(stream_rows[idx[r]]) * w (parts as above) */
+int q3_gather_rows_norm_f32(const float* stream_rows, const int* idx, const float* w, void* out, int64_t rows, int size, float eps, int parts, void* stream);
+int q3_gather_rows_norm_bf16(const float* stream_rows, const int* idx, const float* w, void* out, int64_t rows, int size, float eps, int parts, void* stream);
 /* x <- cap * tanh(x * scale / cap) in place, x * scale for cap = 0 */
 int q3_scale_softcap_f32(float* x, int64_t n, float scale, float cap, void* stream);
 
@@ -83,25 +89,49 @@ int q3_scale_softcap_f32(float* x, int64_t n, float scale, float cap, void* stre
 int q3_qkv_prepare_f32(const void* qkv, void* q_out, void* k_pages, void* v_pages, const float* q_norm_w, const float* k_norm_w,
                        const float* cos_tab, const float* sin_tab, const int* token_seq, const int* token_pos, const int* page_table,
                        int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d, float eps, int write_kv, int rotary_dim,
-                       const float* bias, int value_dim, int value_heads, void* stream);
+                       const float* bias, int value_dim, int value_heads, int64_t row, int tied_values, int norm_once,
+                       const float* v_cos, const float* v_sin, void* stream);
 int q3_qkv_prepare_bf16(const void* qkv, void* q_out, void* k_pages, void* v_pages, const float* q_norm_w, const float* k_norm_w,
                         const float* cos_tab, const float* sin_tab, const int* token_seq, const int* token_pos, const int* page_table,
                         int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d, float eps, int write_kv, int rotary_dim,
-                       const float* bias, int value_dim, int value_heads, void* stream);
-/* (q3_qkv_prepare: value_heads 0 = nkv; fewer value heads than key heads: values that several key heads share)
+                       const float* bias, int value_dim, int value_heads, int64_t row, int tied_values, int norm_once,
+                       const float* v_cos, const float* v_sin, void* stream);
+/* (q3_qkv_prepare: value_heads 0 = nkv; fewer value heads than key heads: values that several key heads share; row 0 = the
+   columns read, else values from one row of the projection to the next; tied_values: the values are the projected keys and
+   have no columns; norm_once: a normed value is rounded once, when it is stored; v_cos, v_sin [positions, value_dim / 2], may
+   be null: the values are rotated by their position, over the whole head) */
+/* the pooled blocks that the step completes: block b of a sequence, its tokens b size .. b size + size - 1, gets the means of
+   their cached keys and values as entry b of the sequence's pool pages (pool_table: as page_table) */
+int q3_pool_blocks_f32(const void* k_pages, const void* v_pages, const int* page_table, void* pool_k, void* pool_v,
+                       const int* pool_table, const int* seq_start, const int* seq_pos0, int pages_per_seq, int n_seqs, int max_new,
+                       int nkv, int d, int value_dim, int size, void* stream);
+int q3_pool_blocks_bf16(const void* k_pages, const void* v_pages, const int* page_table, void* pool_k, void* pool_v,
+                        const int* pool_table, const int* seq_start, const int* seq_pos0, int pages_per_seq, int n_seqs, int max_new,
+                        int nkv, int d, int value_dim, int size, void* stream);
+/* in place on x [N, heads * vd]: heads turned back by their token's position (tables [positions, vd / 2], may be null), then
+   multiplied by sigmoid(gate) value by value (gate rows are gate_row apart; may be null) */
+int q3_turn_back_gate_f32(void* x, const float* cos_tab, const float* sin_tab, const int* token_pos, const void* gate, int64_t gate_row,
+                          int heads, int vd, int64_t n_tokens, void* stream);
+int q3_turn_back_gate_bf16(void* x, const float* cos_tab, const float* sin_tab, const int* token_pos, const void* gate, int64_t gate_row,
+                           int heads, int vd, int64_t n_tokens, void* stream);
+/*
    causal grouped-query attention of every token over its sequence's pages; window 0 = every key; value_dim 0 = d;
    value_heads 0 = nkv, else each value head serves nkv / value_heads key heads; out_f32: `out` is float whatever q is;
    softcap > 0: scores s <- softcap * tanh(s / softcap); chunk > 0: a query reads the keys of its own chunk of that many
    positions only; sink != 0: one more term exp(0) in the softmax's denominator, or exp(sink_values[head]) where sink_values
-   (one float per query head) is given; keep_first (with window): the first so many keys of the sequence are seen too */
+   (one float per query head) is given; keep_first (with window): the first so many keys of the sequence are seen too; pool_size
+   (with window, without keep_first): every block of so many tokens that ends before the window is seen as the entry of the pool
+   pages that q3_pool_blocks wrote */
 int q3_attention_generic_f32(const void* q, const void* k_pages, const void* v_pages, void* out, const int* token_seq,
                              const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d,
                              float scale, int window, int value_dim, float softcap, int chunk, int sink, int value_heads, int out_f32,
-                             const float* sink_values, int keep_first, void* stream);
+                             const float* sink_values, int keep_first,
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
 int q3_attention_generic_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, const int* token_seq,
                               const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d,
                               float scale, int window, int value_dim, float softcap, int chunk, int sink, int value_heads, int out_f32,
-                              const float* sink_values, int keep_first, void* stream);
+                              const float* sink_values, int keep_first,
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
 
 /* the same from the q/k/v projection's output as it is: bias (may be null), rotation of the first rotary_dim values of q and k
    (tables may be null) and the write of the new key and value into their pages in the attention's own kernel */
@@ -110,11 +140,12 @@ int q3_attention_capped_decode_fused_bf16(const void* qkv, void* k_pages, void* 
                                           const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq,
                                           int nkv, float scale, float softcap, int chunk, int sink, int n_splits, void* stream);
 /* attention_prefill_tc.cu compiled with -DQ3_CAPPED=1: the tcgen05 prompt attention with capped scores, chunks and a sink
-   (head sizes 64 and 128, values as wide as keys); arguments as q3_attention_prefill_tc_bf16 plus softcap, chunk, sink */
+   (head sizes 64 and 128, values as wide as keys); arguments as q3_attention_prefill_tc_bf16 plus softcap, chunk, sink and
+   sink_values (one score per query head; may be null) */
 int q3_attention_capped_prefill_tc_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, const int* seq_start,
                                         const int* seq_pos0, const int* page_table, int pages_per_seq, int n_seqs, int max_new,
                                         int64_t n_tokens, int64_t n_cache_pages, int nq, int nkv, float scale, float softcap, int chunk,
-                                        int sink, int* status, void* stream);
+                                        int sink, const float* sink_values, int* status, void* stream);
 
 /* ---- attention_capped.cu (-DQ3_HEAD_DIM, -DQ3_VALUE_DIM): bfloat16 attention with scores capped by softcap * tanh(s / softcap)
    (0: none), chunked visibility (chunk 0: causal only), a sink term in the softmax's denominator, values of their own size */
@@ -123,15 +154,17 @@ int q3_attention_capped_value_dim(void);
 int q3_attention_capped_prefill_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, const int* seq_start,
                                      const int* seq_pos0, const int* page_table, int pages_per_seq, int n_seqs, int max_new, int nq,
                                      int nkv, float scale, float softcap, int chunk, int sink, int window, int value_heads,
-                                     int out_f32, const float* sink_values, int keep_first, void* stream);
+                                     int out_f32, const float* sink_values, int keep_first,
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
 /* (window > 0: a sliding window of that many keys instead of chunks, beside which the first keep_first keys of the sequence
    stay visible; value_heads 0 = nkv, else each value head serves nkv / value_heads key heads; out_f32: `out` is float;
-   sink_values (may be null): the sink's score per query head) */
+   sink_values (may be null): the sink's score per query head; pool_*: as for q3_attention_generic) */
 /* one new token per sequence; scratch: n_tokens * nq * n_splits * (value_dim + 2) float32 */
 int q3_attention_capped_decode_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, float* scratch,
                                     const int* token_seq, const int* token_pos, const int* page_table, int pages_per_seq,
                                     int64_t n_tokens, int nq, int nkv, float scale, float softcap, int chunk, int sink, int n_splits,
-                                    int window, int value_heads, int out_f32, const float* sink_values, int keep_first, void* stream);
+                                    int window, int value_heads, int out_f32, const float* sink_values, int keep_first,
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
 
 /* ---- attention_decode.cu (-DQ3_HEAD_DIM): one new token per sequence, bfloat16 ---------------------------- */
 int q3_attention_decode_head_dim(void);
@@ -207,19 +240,26 @@ int q3_hyper_norm_bf16(float* streams, const void* branch, const float* mix, con
                        int hidden, int normalize, void* stream);
 
 /* ---- lightning.cu: linear attention with a per-head decay and a float32 state [slot, heads, d, vd] ------------- */
-/* proj [N, 2 heads d + 2 heads vd] = q, k, v (SiLU applied here), gate; S <- decay S + k v^T, out = S^T q, token by token */
+/* proj [N, 2 heads d + 2 heads vd] = q, k, v, gate; S <- decay S + k v^T, out = S^T q, token by token.  silu: q, k and v go
+   through SiLU first; the first `rot` values of every head of q and k are rotated by token_pos (tables [positions, rot / 2], may
+   be null), k is multiplied by k_scale; slot_stride: values from one slot's state to the next */
 int q3_lightning_scan_f32(const void* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
-                          float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                          float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale, const float* cos_tab,
+                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, void* stream);
 int q3_lightning_scan_bf16(const void* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
-                           float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                           float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale, const float* cos_tab,
+                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, void* stream);
 /* the same for prompts, 32 tokens at a time */
 int q3_lightning_chunks_f32(const void* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
-                            float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                            float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale, const float* cos_tab,
+                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, void* stream);
 int q3_lightning_chunks_bf16(const void* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
-                             float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                             float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale, const float* cos_tab,
+                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, void* stream);
 /* the chunks' products on the tensor cores (operands as TF32 hi + lo terms): head sizes in steps of 8 */
 int q3_lightning_chunks_tc_bf16(const void* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
-                                float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                                float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale, const float* cos_tab,
+                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, void* stream);
 /* out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate), row by row; gate rows are gate_stride apart */
 int q3_gated_norm_f32(const float* o, const void* gate, int64_t gate_stride, const float* w, float eps, void* out,
                       int64_t n_tokens, int size, void* stream);
@@ -238,7 +278,7 @@ int q3_diff_combine_bf16(const float* a, void* out, int64_t n_tokens, int heads,
    the outputs from n_real on are identity experts (their weights are summed into id_weight); by_logit: the largest logits
    are chosen, weighted by the softmax over the chosen logits alone; gate_out (may be null): the router matrix has one more
    row and gate_out[t] = sigmoid of its logit; by_logit 2: scores sigmoid(z) instead of the softmax; group_pair: a group's mark
-   is the sum of its two best choice scores; the weights are multiplied by weight_scale */
+   is the sum of its two best choice scores; the weights are multiplied by weight_scale; correction may be null */
 int q3_moe_route_f32(const void* h, const void* w_router, const float* correction, int* top_ids, float* top_w, float* id_weight,
                      int64_t n_tokens, int hidden, int n_out, int n_real, int top, int group_count, int group_keep, int by_logit,
                      float* gate_out, int group_pair, float weight_scale, void* stream);
@@ -247,18 +287,20 @@ int q3_moe_route_bf16(const void* h, const void* w_router, const float* correcti
                       float* gate_out, int group_pair, float weight_scale, void* stream);
 /* offsets [n_real + 1], slot_of_pair (-1: identity) and pair_of_slot of the (token, choice) pairs laid out by expert */
 int q3_moe_sort(const int* top_ids, int n_pairs, int n_real, int* offsets, int* slot_of_pair, int* pair_of_slot, void* stream);
-/* act[slot] = g sigmoid(alpha g) (u + up_offset), g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit); y[slot] = W_down act */
+/* act[slot] = g sigmoid(alpha g) (u + up_offset), g = min(W_gate x, limit), u = clamp(W_up x, -limit, limit);
+   gated 0: act[slot] = max(W_up x, 0)^2, one matrix of up rows per expert; y[slot] = W_down act */
 int q3_moe_experts_f32(const void* h, const void* w_gate_up, const void* w_down, const int* offsets, const int* pair_of_slot,
                        void* act, float* y, int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha,
-                       float up_offset, void* stream);
+                       float up_offset, int gated, void* stream);
 int q3_moe_experts_bf16(const void* h, const void* w_gate_up, const void* w_down, const int* offsets, const int* pair_of_slot,
                         void* act, float* y, int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha,
-                        float up_offset, void* stream);
+                        float up_offset, int gated, void* stream);
 /* the same on the tensor cores: bfloat16, hidden and ff multiples of 32 */
 int q3_moe_experts_tc_bf16(const void* h, const void* w_gate_up, const void* w_down, const int* offsets, const int* pair_of_slot,
                            void* act, float* y, int n_pairs, int n_real, int top, int hidden, int ff, float limit, float alpha,
-                           float up_offset, void* stream);
-/* out[t] = sum_k top_w[t, k] y[slot_of_pair[t, k]] + id_weight[t] h[t] + shared_w[t] shared[t] (the last may be null) */
+                           float up_offset, int gated, void* stream);
+/* out[t] = sum_k top_w[t, k] y[slot_of_pair[t, k]] + id_weight[t] h[t] + shared_w[t] shared[t] (shared may be null; shared_w
+   null: weight 1) */
 int q3_moe_combine_f32(const float* y, const void* h, const int* slot_of_pair, const float* top_w, const float* id_weight,
                        void* out, int64_t n_tokens, int top, int hidden, const void* shared, const float* shared_w, void* stream);
 int q3_moe_combine_bf16(const float* y, const void* h, const int* slot_of_pair, const float* top_w, const float* id_weight,
@@ -366,7 +408,8 @@ int q3_decay_scan_bf16(const void* q, const void* k, const void* v, int64_t row,
 int q3_memory_gates(const float* zi, const float* zf, const float* bias_i, const float* bias_f, float cap, float* m_state,
                     int64_t slot_stride, const int* seq_start, const int* seq_slots, float* keep, float* write, float* low, int heads,
                     int64_t z_row, int n_seqs, void* stream);
-/* per (token, head): x = o[:vd] (/ (max(|o[vd]|, low) + floor_add) if vdx > vd); out = x / sqrt(mean(x^2) + eps) * w * act(gate) */
+/* per (token, head): x = o[:vd] (/ (max(|o[vd]|, low) + floor_add) if vdx > vd); out = x / sqrt(mean(x^2) + eps) * w * act(gate)
+   (w null: no weight) */
 int q3_head_gated_norm_f32(const float* o, const float* low, float floor_add, const float* w, int w_per_head, const void* gate,
                            int64_t gate_row, void* out, int64_t n_tokens, int heads, int vd, int vdx, float eps, int act, void* stream);
 int q3_head_gated_norm_bf16(const float* o, const float* low, float floor_add, const float* w, int w_per_head, const void* gate,

@@ -71,7 +71,7 @@ inline void pack_step(const CacheBook& book, const StepLayout& lay, const int* s
 
 // A decode step of a fixed number of `rows`, of which the first `n_live` belong to sequences (one token
 // each) and the rest are padding: token 0 at position 0 of the spare slot (number n_slots) and the spare
-// page (number n_pages), which belong to no sequence.  Every row's logits are wanted.
+// page of every group (number n_pages of the group), which belong to no sequence.  Every row's logits are wanted.
 inline void pack_decode_step(const CacheBook& book, const StepLayout& lay, int rows, const int* slots, int n_live,
                              const int32_t* token_ids, int32_t* out) {
     const int P = book.pages_per_slot();
@@ -94,7 +94,7 @@ inline void pack_decode_step(const CacheBook& book, const StepLayout& lay, int r
                 const int32_t* row = book.group(g).row(slots[i]);
                 for (int p = 0; p < P; ++p) to[p] = row[p];
             } else {
-                for (int p = 0; p < P; ++p) to[p] = book.n_pages();
+                for (int p = 0; p < P; ++p) to[p] = book.group(g).n_pages();
             }
         }
 }

@@ -24,6 +24,15 @@ over time on every channel of q, k and v right after the projection, before the 
 [heads, hidden]); `value_mix`: values blended across layers: the layer that says "first" keeps the step's values
 (after the bias) for the others, a layer that says "blend" goes on with v <- (1 - lambda) v + lambda v_first, lambda
 its scalar tensor `value_mix`, and caches the blend (a "first" layer may store the scalar too; it is not read).
+
+And: `pool` (with `window`): beside the window's tokens, every block of so many tokens that lies wholly before the window is
+seen as one key and one value, the means of the block's cached keys and values, kept in pages of their own; `tied_values`:
+the values are the keys as projected, before norm and rotation, and there is no value projection; `value_position`: a
+rotary encoding of the values over their whole head, by which every head's output is turned back at its own position;
+`out_gate`: the heads side by side are multiplied value by value by sigmoid(W_g x) (tensor `out_gate`, its product is
+part of the projection's); `learned_sink`: the sink's score is a number per head (tensor `sink`) instead of 0; `norm_once`:
+a normed query or key is rounded to the compute type once, after the rotation (else also after the division by its rms and
+after the weight, as Qwen3 is).
 """
 from __future__ import annotations
 
@@ -53,7 +62,7 @@ FUSED_PROJECTION_KERNELS = []
 TENSOR_NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                 "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
                 "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "o_bias": "o_proj.bias", "value_mix": "value_mix",
-                "head_gate": "gate.weight", "conv_suffix": ".conv"}
+                "head_gate": "gate.weight", "conv_suffix": ".conv", "out_gate": "out_gate.weight", "sink": "sink"}
 
 
 class GQAAttention(Part):
@@ -62,6 +71,7 @@ class GQAAttention(Part):
     keep_first, out_bias, value_mix, conv_taps, head_gate = 0, False, None, 0, False
     o_bias = bias_v = conv_weight = w_gate = None
     mix_lambda = 0.0
+    pool, tied_values, out_gate, learned_sink, norm_once, value_position = 0, False, False, False, False, None
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                  qk_norm: Optional[PartSpec] = None, position: Optional[PartSpec] = None,
@@ -69,7 +79,8 @@ class GQAAttention(Part):
                  softcap: Optional[float] = None, chunk: Optional[int] = None, sink: bool = False,
                  names: Optional[dict] = None, value_heads: Optional[int] = None, out_float32: bool = False,
                  keep_first: int = 0, out_bias: bool = False, value_mix: Optional[str] = None, conv_taps: int = 0,
-                 head_gate: bool = False):
+                 head_gate: bool = False, pool: int = 0, tied_values: bool = False, value_position: Optional[PartSpec] = None,
+                 out_gate: bool = False, learned_sink: bool = False, norm_once: bool = False):
         self.sink_values = None      # float32 [num_heads]: the sink's score per head, for a part that has learned ones (else 0)
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
@@ -81,6 +92,16 @@ class GQAAttention(Part):
             raise ValueError("attention takes a window or chunks, not both")
         if value_mix not in (None, "first", "blend") or keep_first < 0 or conv_taps < 0 or (keep_first and not window):
             raise ValueError("attention: value_mix is 'first' or 'blend'; keep_first goes with a window")
+        if pool < 0 or (pool and (not window or keep_first)):
+            raise ValueError("attention: pooled blocks go with a window that keeps no first keys")
+        if tied_values and (value_dim != head_dim or bias or value_mix or conv_taps or (value_heads or num_kv_heads) != num_kv_heads):
+            raise ValueError("attention: values that are the keys have their size and heads, and no bias, blend or convolution of their own")
+        if (out_gate or value_position or pool) and (conv_taps or value_mix or out_float32 or (value_heads or num_kv_heads) != num_kv_heads):
+            raise ValueError("attention: an output gate, rotated values and pooled blocks do not go with convolutions, blends or shared values")
+        self.pool, self.tied_values, self.out_gate = int(pool), bool(tied_values), bool(out_gate)
+        self.learned_sink, self.norm_once = bool(learned_sink), bool(norm_once)
+        self.value_position = build_part("position", value_position) if value_position else None
+        sink = sink or learned_sink
         self.keep_first, self.out_bias, self.value_mix = int(keep_first), bool(out_bias), value_mix
         self.conv_taps, self.head_gate = int(conv_taps), bool(head_gate)
         self.out_name = "mixer.out"  # the scratch buffer of the result; a part that runs several mixers side by side renames it
@@ -106,14 +127,25 @@ class GQAAttention(Part):
         self.reordered = False       # the rows of the q and k projections follow the position encoding's kernel order
         # what the kernels written for Qwen3's attention take
         self.plain = not (self.has_bias or self.softcap or self.chunk or self.sink or value_dim != head_dim or head_dim % 16
-                          or self.shared_values or self.keep_first or self.value_mix)
+                          or self.shared_values or self.keep_first or self.value_mix or self.special())
+
+    def special(self) -> bool:
+        """Options that change what a query, a key or a value is made from, or what becomes of the output: the kernels that
+        prepare a step's rows themselves do not take them."""
+        return bool(self.pool or self.tied_values or self.value_position or self.out_gate or (self.norm_once and self.q_norm is not None))
 
     # -- weights
     def weight_specs(self, prefix: str) -> dict:
         p, n = prefix + self.prefix, self.names
         nq, nkv, d, vd, H, nv = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.hidden_size, self.value_heads
         specs = {p + n["q"]: WeightSpec((nq * d, H)), p + n["k"]: WeightSpec((nkv * d, H)),
-                 p + n["v"]: WeightSpec((nv * vd, H)), p + n["o"]: WeightSpec((H, self.output_width()))}
+                 p + n["o"]: WeightSpec((H, self.output_width()))}
+        if not self.tied_values:
+            specs[p + n["v"]] = WeightSpec((nv * vd, H))
+        if self.out_gate:
+            specs[p + n["out_gate"]] = WeightSpec((nq * vd, H))
+        if self.learned_sink:
+            specs[p + n["sink"]] = WeightSpec((nq,), "bias")
         if self.has_bias:
             specs.update({p + n["q_bias"]: WeightSpec((nq * d,), "bias"), p + n["k_bias"]: WeightSpec((nkv * d,), "bias"),
                           p + n["v_bias"]: WeightSpec((nv * vd,), "bias")})
@@ -138,13 +170,16 @@ class GQAAttention(Part):
     def bind(self, weights: dict, prefix: str, dtype, device) -> None:
         p, n = prefix + self.prefix, self.names
         nq, nkv, d = self.num_heads, self.num_kv_heads, self.head_dim
-        self.w_qkv = fuse_rows(weights, [p + n["q"], p + n["k"], p + n["v"]])
+        parts = ["q", "k"] + ([] if self.tied_values else ["v"]) + (["out_gate"] if self.out_gate else [])
+        self.w_qkv = fuse_rows(weights, [p + n[k] for k in parts])
         self.w_o = weights.pop(p + n["o"]).contiguous()
         if self.has_bias:
             tensors = [weights[p + n[k]] for k in ("q_bias", "k_bias", "v_bias")]
             getattr(weights, "wait", lambda: None)()          # a streamed checkpoint: the tensors are in place now
             self.bias = torch.cat([t.to(device=device, dtype=torch.float32).reshape(-1) for t in tensors]).contiguous()
         f32 = dict(device=device, dtype=torch.float32)
+        if self.learned_sink:
+            self.sink_values = weights[p + n["sink"]].to(**f32).reshape(-1).contiguous()
         if self.out_bias:
             self.o_bias = weights[p + n["o_bias"]].to(**f32).contiguous()
         if self.head_gate:
@@ -167,6 +202,8 @@ class GQAAttention(Part):
             # of the rotation where the kernels expect them, once
             if self.q_norm is not None:
                 raise ValueError("an interleaved rotation with per-head norm weights is not supported")
+            if self.tied_values:
+                raise ValueError("an interleaved rotation of keys that are the values too is not supported")
             getattr(weights, "wait", lambda: None)()
             rows = (torch.arange(nq + nkv, device=self.w_qkv.device)[:, None] * d
                     + torch.tensor(order, device=self.w_qkv.device)[None, :]).reshape(-1)
@@ -186,14 +223,17 @@ class GQAAttention(Part):
     def cache_need(self) -> CacheNeed:
         kind = "window" if self.window else ("chunk" if self.chunk else "full")
         state = ((self.conv_taps - 1) * self.projection_width(),) if self.conv_taps > 1 else ()
-        return CacheNeed(kind, self.num_kv_heads, self.head_dim, self.window or self.chunk,
+        # with pooled blocks the tokens of an unfinished block stay until its means are taken
+        return CacheNeed(kind, self.num_kv_heads, self.head_dim, max(self.window, self.pool) if self.pool else self.window or self.chunk,
+                         pool=self.pool,
                          value_dim=self.value_dim if self.value_dim != self.head_dim else None,
                          value_heads=self.value_heads if self.value_heads != self.num_kv_heads else None,
                          keep_first=self.keep_first if self.window else 0, state_shape=state)
 
     def projection_width(self) -> int:
-        """Columns of the q/k/v projection."""
-        return (self.num_heads + self.num_kv_heads) * self.head_dim + self.value_heads * self.value_dim
+        """Columns of the q/k/v projection (and of the output gate's, if there is one)."""
+        return (self.num_heads + self.num_kv_heads) * self.head_dim + (0 if self.tied_values else self.value_heads * self.value_dim) \
+            + (self.num_heads * self.value_dim if self.out_gate else 0)
 
     # -- step
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
@@ -247,14 +287,38 @@ class GQAAttention(Part):
                 if kernel(self, qkv, cache, attn, ctx, table, qw, kw, norm_eps, cos, sin):
                     return attn
         q = ctx.scratch.get("attn.q", (N, nq * d), ctx.dtype)
+        v_cos = v_sin = None
+        if self.value_position is not None:
+            self.value_position.prepare(ctx.max_positions, ctx.device)
+            v_cos, v_sin = self.value_position.cos, self.value_position.sin
         if tables:
             ops.qkv_prepare(qkv, q, cache.keys, cache.values, qw, kw, cos, sin, ctx.token_seq, ctx.token_pos, table,
                             N, nq, nkv, d, norm_eps, write_kv=not cache.shared, bias=self.bias, value_dim=vd,
-                            value_heads=self.value_heads)
+                            value_heads=self.value_heads, tied_values=self.tied_values, norm_once=self.norm_once,
+                            value_cos=v_cos, value_sin=v_sin)
+        elif self.special():
+            raise ops.KernelError("this attention takes a position encoding with tables, or none")
         else:
             self._prepare_unfused(qkv, q, cache, ctx, table, qw, kw, norm_eps)
+        if self.pool and not cache.shared:
+            ops.pool_blocks(cache.keys, cache.values, table, self.pooled(ctx, cache), ctx.seq_start, ctx.seq_pos0, ctx.n_seqs, ctx.max_new)
         self.attend(q, cache, attn, ctx, table)
+        if self.out_gate or self.value_position is not None:
+            gate = qkv[:, self.projection_width() - nq * vd:] if self.out_gate else None
+            ops.turn_back_gate(attn, v_cos, v_sin, ctx.token_pos, gate, nq, vd)
         return attn
+
+    def pooled(self, ctx, cache):
+        """The pooled blocks of this layer as the kernels take them (None: there are none)."""
+        if not self.pool:
+            return None
+        return ops.Pool(cache.pool_keys, cache.pool_values, ctx.page_tables[cache.pool_group], self.pool)
+
+    def keys_seen(self, max_context: int) -> int:
+        """A bound on the keys (and pooled blocks) that one query reads in a context of `max_context` tokens."""
+        if not self.window:
+            return min(self.chunk or max_context, max_context)
+        return min(self.window + self.keep_first + (max_context // self.pool if self.pool else 0), max_context)
 
     def attend(self, q, cache, out, ctx, table) -> None:
         if ctx.dtype == torch.bfloat16:
@@ -264,7 +328,8 @@ class GQAAttention(Part):
         ops.attention_generic(q, cache.keys, cache.values, out, ctx.token_seq, ctx.token_pos, table, ctx.n_tokens,
                               self.num_heads, self.num_kv_heads, self.head_dim, self.scale, self.window,
                               value_dim=self.value_dim, softcap=self.softcap, chunk=self.chunk, sink=self.sink,
-                              value_heads=self.value_heads, sink_values=self.sink_values, keep_first=self.keep_first)
+                              value_heads=self.value_heads, sink_values=self.sink_values, keep_first=self.keep_first,
+                              pool=self.pooled(ctx, cache))
 
     def _prepare_unfused(self, qkv, q, cache, ctx, table, qw, kw, eps) -> None:
         """A position encoding without kernel tables: norm, then `apply_`, then the cache write."""
@@ -384,7 +449,7 @@ def _prefill_capped_kernel(part, q, cache, out, ctx, table) -> bool:
     ops.attention_capped_prefill(q, cache.keys, cache.values, out, ctx.seq_start, ctx.seq_pos0, table, ctx.n_seqs, ctx.max_new,
                                  part.num_heads, part.num_kv_heads, part.head_dim, part.value_dim, part.scale, part.softcap,
                                  part.chunk, part.sink, window=part.window, value_heads=part.value_heads,
-                                 sink_values=part.sink_values, keep_first=part.keep_first)
+                                 sink_values=part.sink_values, keep_first=part.keep_first, pool=part.pooled(ctx, cache))
     return True
 
 
@@ -392,11 +457,11 @@ def _prefill_capped_tcgen05_kernel(part, q, cache, out, ctx, table) -> bool:
     """The same on tcgen05 with TMA-fed tiles: head sizes 64 and 128, values as wide as keys, and enough new tokens
     for 128-row tiles to be worth it."""
     if part.plain or part.keep_first or part.shared_values or not ops.attention_capped_prefill_tc_fits(part.head_dim, part.value_dim, part.window) \
-            or ctx.max_new < tc_prefill_rows or part.scale <= 0 or part.sink_values is not None:
+            or ctx.max_new < tc_prefill_rows or part.scale <= 0:
         return False
     ops.attention_capped_prefill_tc(q[:ctx.n_tokens], cache.keys, cache.values, out, ctx.seq_start, ctx.seq_pos0, table,
                                     ctx.n_seqs, ctx.max_new, ctx.n_tokens, part.num_heads, part.num_kv_heads, part.head_dim,
-                                    part.scale, part.softcap, part.chunk, part.sink)
+                                    part.scale, part.softcap, part.chunk, part.sink, sink_values=part.sink_values)
     return True
 
 
@@ -405,20 +470,19 @@ def _decode_capped_kernel(part, q, cache, out, ctx, table) -> bool:
     nq, nkv = part.num_heads, part.num_kv_heads
     if part.plain or not ops.attention_capped_fits(part.head_dim, part.value_dim, part.window, nq // nkv):
         return False
-    splits = ops.attention_capped_splits(ctx.n_tokens, nkv, _sm_count(ctx.device),
-                                         min(part.chunk or (part.window or 0) + part.keep_first or ctx.max_context, ctx.max_context))
+    splits = ops.attention_capped_splits(ctx.n_tokens, nkv, _sm_count(ctx.device), part.keys_seen(ctx.max_context))
     scratch = ctx.scratch.get("attn.capped_scratch", (ctx.n_tokens * nq * splits * (part.value_dim + 2),), torch.float32)
     ops.attention_capped_decode(q, cache.keys, cache.values, out, scratch, ctx.token_seq, ctx.token_pos, table, ctx.n_tokens,
                                 nq, nkv, part.head_dim, part.value_dim, part.scale, part.softcap, part.chunk, part.sink, splits,
                                 window=part.window, value_heads=part.value_heads, sink_values=part.sink_values,
-                                keep_first=part.keep_first)
+                                keep_first=part.keep_first, pool=part.pooled(ctx, cache))
     return True
 
 
 def _decode_capped_fused_kernel(part, qkv, cache, out, ctx, table, q_norm_w, k_norm_w, eps, cos, sin) -> bool:
     """Bias, rotation, cache write and the split-key attention of a decode step in one kernel (and the small merge)."""
     nq, nkv = part.num_heads, part.num_kv_heads
-    if part.plain or part.shared_values or part.window or q_norm_w is not None or cache.shared or part.sink_values is not None \
+    if part.plain or part.shared_values or part.window or q_norm_w is not None or cache.shared or part.sink_values is not None or part.special() \
             or not ops.attention_capped_fits(part.head_dim, part.value_dim, part.window, nq // nkv):
         return False
     splits = ops.attention_capped_splits(ctx.n_tokens, nkv, _sm_count(ctx.device), part.chunk or ctx.max_context)

@@ -63,7 +63,8 @@ def settle(residual, pending, norm=None, out=None):
         return out
     return ops.sandwich_norm(residual, pending.branch if pending else None, pending.norm.weight if pending else None,
                              pending.norm.eps if pending else 0.0, norm.weight if norm else None,
-                             norm.eps if norm else 0.0, out)
+                             norm.eps if norm else 0.0, out, groups_post=pending.norm.groups if pending else 1,
+                             groups_pre=norm.groups if norm else 1)
 
 
 class SandwichNormBlock(Part):
@@ -82,6 +83,12 @@ class SandwichNormBlock(Part):
         if self.feed_forward is not None:
             specs.update(self.feed_forward.weight_specs(prefix))
         return specs
+
+    def ignorable(self, prefix: str):
+        """The norms of a feed-forward that the layer does not have may be stored all the same."""
+        if self.feed_forward is not None:
+            return []
+        return [n for name in self.names[2:] for n in self.norms[0].weight_specs(prefix + name)]
 
     def bind(self, weights: dict, prefix: str, dtype, device) -> None:
         for part, name in zip(self.norms, self.names):

@@ -72,10 +72,11 @@ class SwiGLU(Part):
 
 class DenseMLP(Part):
     """A feed-forward without a gate: down( act(up(x)) ); act one of `ops.PLAIN_ACTIVATIONS` (GELU with the error
-    function by default).  The checkpoint names of the two matrices are parameters."""
+    function by default; "relu2": the square of relu).  The checkpoint names of the two matrices are parameters."""
 
     def __init__(self, hidden_size: int, intermediate_size: int, prefix: str = "", activation: str = "gelu",
-                 names: Optional[dict] = None):
+                 names: Optional[dict] = None, out_name: str = "ff.out"):
+        self.out_name = out_name         # the scratch buffer of the result
         if activation not in ops.PLAIN_ACTIVATIONS:
             raise ValueError(f"activation {activation!r}: one of {sorted(ops.PLAIN_ACTIVATIONS)}")
         self.hidden_size, self.intermediate_size, self.prefix = int(hidden_size), int(intermediate_size), prefix
@@ -97,7 +98,7 @@ class DenseMLP(Part):
         act = ctx.scratch.get("ff.act", (N, self.intermediate_size), ctx.dtype)
         linear(x, self.w_up, act)
         ops.activation(act, act, self.activation)
-        out = ctx.scratch.get("ff.out", (N, self.hidden_size), ctx.dtype)
+        out = ctx.scratch.get(self.out_name, (N, self.hidden_size), ctx.dtype)
         return linear(act, self.w_down, out)
 
 

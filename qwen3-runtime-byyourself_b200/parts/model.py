@@ -139,7 +139,8 @@ class Model:
                 settle(residual, delta, self.final_norm, normed)
             else:
                 settle(residual, delta)
-                ops.gather_rows_norm(residual, ctx.want_rows[:R], self.final_norm.weight, self.final_norm.eps, normed)
+                ops.gather_rows_norm(residual, ctx.want_rows[:R], self.final_norm.weight, self.final_norm.eps, normed,
+                                     groups=self.final_norm.groups)
         elif ctx.want_all:                                 # a decode step: the last residual sum rides in the norm
             self.final_norm(residual, normed, delta)
         else:

@@ -16,9 +16,12 @@ from .base import Part, register_part
 class RMSNorm(Part):
     stream_kind = "rms"          # how the kernels of a float32 stream apply this part (ops.NORM_KINDS)
 
-    def __init__(self, size: int, eps: float, one_plus: bool = False):
-        """`one_plus`: the stored weight lies around zero and the norm multiplies by 1 + weight."""
-        self.size, self.eps, self.one_plus = int(size), float(eps), bool(one_plus)
+    def __init__(self, size: int, eps: float, one_plus: bool = False, groups: int = 1):
+        """`one_plus`: the stored weight lies around zero and the norm multiplies by 1 + weight.  `groups`: the row is split
+        into so many equal consecutive parts, each divided by its own rms (applied by the kernels of a float32 stream)."""
+        self.size, self.eps, self.one_plus, self.groups = int(size), float(eps), bool(one_plus), int(groups)
+        if self.groups <= 0 or self.size % self.groups:
+            raise ValueError("a norm in groups: the groups divide the row")
         self.weight = None
 
     def weight_specs(self, name: str) -> dict:
@@ -32,6 +35,8 @@ class RMSNorm(Part):
             self.weight = (self.weight + 1.0).contiguous()
 
     def __call__(self, x: torch.Tensor, out: torch.Tensor, delta=None) -> torch.Tensor:
+        if self.groups > 1:
+            raise ops.KernelError("a norm in groups is applied on a float32 stream by sandwich_norm")
         return ops.rms_norm(x, self.weight, self.eps, out, delta)
 
 
