@@ -6,6 +6,7 @@ model with random weights in bfloat16 on one B200, batch 8 at a context of 4,096
     python bench.py --designs lagulorn   (the same for a Lagulorn model)
     python bench.py --designs fagunex    (a Fagunex model beside the Lagulorn model of the same widths)
     python bench.py --designs fedinex    (a Fedinex model beside the Fagunex model of the same widths)
+    python bench.py --designs vogerax    (a Vogerax model beside the Fedinex model of the same widths)
 
 Prints ONE JSON line.  A "step" is one decode step of the whole batch.
   value     decoded tokens a second, timed on the device with CUDA events around K steps;
@@ -522,6 +523,45 @@ def fedinex_side_by_side(q, torch, Sampler, steps, warmup, batch=8, context=4096
     return out
 
 
+def vogerax_config(width, heads, kv, d, ff, layers, window=1024, pool=16, experts=16, top=2):
+    """A Vogerax model of the widths of the Fedinex model beside it: attention whose values are its keys, a window of `window`
+    tokens with pooled blocks of `pool` beside it, half of every head rotated, on three layers of four; on the third of every
+    four attention over every earlier key (normed queries and keys, YaRN, rotated values, a sink, an output gate) beside
+    retention of width / (2 d) heads of d x d.  Norms in two groups.  The first layer's feed-forward is dense, the others routed
+    (`experts` experts of ff / (2 top), `top` per token) with a shared expert of the same size; no feed-forward has a gate."""
+    windowed = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5,
+                                                "rot": {"base": 1000000.0, "dims": d // 2, "scaling": {"factor": 2.0}},
+                                                "mask": {"size": window, "pool": pool}}}
+    small = max(width // (2 * d), 1)
+    yarn = {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    both = {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5,
+                 "rot": {"base": 500000.0, "dims": d // 2, "scaling": yarn}},
+        "right": {"heads": small, "dim": d, "vdim": d, "rot": {"base": 10000.0, "dims": d},
+                  "decay": [1.0 - 2.0 ** -(5 + 3 * h / max(small - 1, 1)) for h in range(small)]}}}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top)}, "router": {"experts": experts, "top": top}, "shared": {"ff": ff // (2 * top)}}
+    order = [windowed, windowed, both, windowed]
+    return {"architecture": "Vogerax", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": width ** 0.5},
+            "norm": {"eps": 1e-6, "groups": 2},
+            "layers": [dict(order[i % 4], mlp={"kind": "dense", "ff": ff} if i == 0 else moe) for i in range(layers)]}
+
+
+def vogerax_side_by_side(q, torch, Sampler, steps, warmup, batch=8, context=4096):
+    """Vogerax beside Fedinex, the closest of the other designs (a 32-bit hidden state, attention with a window in turn with
+    attention beside a recurrence, routed experts), at equal widths (random weights, bfloat16): decode at `batch` x `context`, a
+    prompt step of 2,048 tokens, and the time of every kernel of one step of each kind."""
+    import numpy as np
+    out = {"batch": batch, "context": context, "prompt_tokens": PREFILL_TOKENS, "vocab": DESIGN_VOCAB, "sizes": {}}
+    for name, width, heads, kv, d, ff, layers in DESIGN_SIZES:
+        row = {"width": width, "heads": heads, "kv_heads": kv, "head_dim": d, "ff": ff, "layers": layers}
+        row["vogerax"] = design_point(q, torch, Sampler, vogerax_config(width, heads, kv, d, ff, layers), np.random.default_rng(0),
+                                      batch, context, steps, warmup)
+        row["fedinex"] = design_point(q, torch, Sampler, fedinex_config(width, heads, kv, d, ff, layers), np.random.default_rng(0),
+                                      batch, context, steps, warmup)
+        out["sizes"][name] = row
+    return out
+
+
 def designs_side_by_side(q, torch, Sampler, steps, warmup, batch=8, context=4096):
     """Dozazen beside Qwen3 at equal sizes (random weights, bfloat16): decode at `batch` x `context`, a prompt step of
     2,048 tokens; chunks longer than the context (every key is read, as in Qwen3) and chunks of 1,024."""
@@ -557,10 +597,11 @@ def main() -> int:
     ap.add_argument("--kernels", action="store_true",
                     help="instead of the benchmark: time every kernel of one decode step and of one 2,048-token prompt step "
                          "with CUDA events (steps launched afresh, not replayed) and print the sums per entry point")
-    ap.add_argument("--designs", nargs="?", const="dozazen", default=None, choices=["dozazen", "lagulorn", "fagunex", "fedinex"],
+    ap.add_argument("--designs", nargs="?", const="dozazen", default=None, choices=["dozazen", "lagulorn", "fagunex", "fedinex", "vogerax"],
                     help="instead of the benchmark: decode and prompt throughput of a Dozazen (default) or Lagulorn model beside "
-                         "the Qwen3 model of the same widths (or of a Fagunex model beside the Lagulorn one) at two sizes, with the "
-                         "time of every kernel of one step of each kind")
+                         "the Qwen3 model of the same widths (or of a Fagunex model beside the Lagulorn one, a Fedinex model beside "
+                         "the Fagunex one, a Vogerax model beside the Fedinex one) at two sizes, with the time "
+                         "of every kernel of one step of each kind")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -582,7 +623,7 @@ def main() -> int:
     if args.designs:
         torch.cuda.set_device(0)
         side_by_side = {"lagulorn": lagulorn_side_by_side, "fagunex": fagunex_side_by_side,
-                        "fedinex": fedinex_side_by_side}.get(args.designs, designs_side_by_side)
+                        "fedinex": fedinex_side_by_side, "vogerax": vogerax_side_by_side}.get(args.designs, designs_side_by_side)
         print(json.dumps(side_by_side(q, torch, Sampler, min(args.steps, 64), warmup, args.batch or 8, args.context or 4096)))
         return 0
     if args.products:
