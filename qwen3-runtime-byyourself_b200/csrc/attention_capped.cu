@@ -105,6 +105,16 @@ struct PoolArgs {
     const bf16* v;
     const int* table;           // [sequences, pages_per_seq]
     int size;
+    int write;                  // decode: the block that a token completes is pooled by the kernel that reads its query
+};
+
+// What becomes of a decode step's output where the splits are merged (all null: nothing).
+struct FinishArgs {
+    const float* cos_tab;       // [positions, VD / 2]: heads turned back by the token's position, pairs (i, i + VD/2)
+    const float* sin_tab;
+    const int* token_pos;
+    const bf16* gate;           // then multiplied by sigmoid(gate), value by value; rows gate_row apart
+    int64_t gate_row;
 };
 
 template <typename TO> __device__ __forceinline__ void store_pair(TO* p, float a, float b);
@@ -228,6 +238,8 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
                 }
             }
             const bool edge = blocks ? key_base + PAGE > warp_first_block : key_base + PAGE - 1 > warp_first_pos || key_base < warp_last_start;
+            // the entries of this page that each row sees: from .. to (and the kept keys)
+            const int from_lo = blocks ? 0 : c_lo, from_hi = blocks ? 0 : c_hi, to_lo = blocks ? b_lo - 1 : p_lo, to_hi = blocks ? b_hi - 1 : p_hi;
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int j = 0; j < 8; ++j)
@@ -236,7 +248,7 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
                     float v = score_log2(s[j][e], scale, cap, inv_cap);
                     if (edge) {
                         const int key = key_base + j * 8 + tq * 2 + (e & 1);
-                        const bool seen = blocks ? key < ((e >> 1) ? b_hi : b_lo) : (e >> 1) ? (key <= p_hi && (key >= c_hi || key < keep)) : (key <= p_lo && (key >= c_lo || key < keep));
+                        const bool seen = (e >> 1) ? (key <= to_hi && (key >= from_hi || (!POOL && key < keep))) : (key <= to_lo && (key >= from_lo || (!POOL && key < keep)));
                         v = seen ? v : -INFINITY;
                     }
                     s[j][e] = v;
@@ -396,6 +408,28 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
     };
 #pragma unroll
     for (int s = 0; s < STAGES - 1; ++s) issue(s);
+
+    if constexpr (POOL) {
+        // the token completes a block (its row is in its page by now): one thread block of the (token, kv head) takes the means.
+        // No query of this step sees that block.
+        if (pool.write && split == n_splits - 1 && (pos + 1) % pool.size == 0) {
+            const int b = pos / pool.size;
+            const int64_t to = ((int64_t)pool_list[b / PAGE] * nkv + kvh) * PAGE + b % PAGE;
+            const float inv = 1.0f / (float)pool.size;
+            for (int i = threadIdx.x; i < D + VD; i += WARPS * 32) {
+                const bool is_v = i >= D;
+                const int c = is_v ? i - D : i, width = is_v ? VD : D;
+                const bf16* from = (is_v ? v_pages : k_pages) + c;
+                float sum = 0.0f;
+#pragma unroll 4
+                for (int j = 0; j < pool.size; ++j) {
+                    const int p = b * pool.size + j;
+                    sum += __bfloat162float(from[(((int64_t)pages[p / PAGE] * nkv + kvh) * PAGE + p % PAGE) * width]);
+                }
+                const_cast<bf16*>(is_v ? pool.v : pool.k)[to * width + c] = __float2bfloat16_rn(sum * inv);
+            }
+        }
+    }
 
     // the block that holds the token's own page owns the new key and value
     const bool owner = FUSED && count > 0 && pg_end == n_pages;
@@ -576,10 +610,11 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
     }
 }
 
-// One block per (query head, token): the splits' partial results, the sink, the division.
-template <typename TO>
+// One block per (query head, token): the splits' partial results, the sink, the division; then (FINISH) the head is turned
+// back and gated.
+template <typename TO, bool FINISH>
 __global__ void decode_capped_merge_kernel(const float* __restrict__ part, TO* __restrict__ out, int nq, int n_splits, int sink,
-                                           const float* __restrict__ sink_values) {
+                                           const float* __restrict__ sink_values, const FinishArgs finish) {
     pdl_launch_dependents();
     pdl_wait();
     const int head = blockIdx.x;
@@ -594,14 +629,35 @@ __global__ void decode_capped_merge_kernel(const float* __restrict__ part, TO* _
         if (ms != -INFINITY) l += exp2f(ms - m) * p[s * (VD + 2) + VD + 1];
     }
     const float inv = 1.0f / l;
-    for (int c = threadIdx.x; c < VD; c += blockDim.x) {
+    auto value = [&](int c) {
         float acc = 0.0f;
         for (int s = 0; s < n_splits; ++s) {
             const float ms = p[s * (VD + 2) + VD];
             if (ms != -INFINITY) acc += exp2f(ms - m) * p[s * (VD + 2) + c];
         }
-        out[(t * nq + head) * VD + c] = from_f32<TO>(acc * inv);
+        return acc * inv;
+    };
+    if constexpr (FINISH) {
+        constexpr int HALF = VD / 2;
+        for (int c = threadIdx.x; c < HALF; c += blockDim.x) {
+            float a = value(c), b = value(c + HALF);
+            if (finish.cos_tab != nullptr) {
+                const int64_t at = (int64_t)finish.token_pos[t] * HALF + c;
+                const float cs = finish.cos_tab[at], sn = finish.sin_tab[at], u = a * cs + b * sn;
+                b = b * cs - a * sn;
+                a = u;
+            }
+            if (finish.gate != nullptr) {
+                const bf16* g = finish.gate + t * finish.gate_row + (int64_t)head * VD + c;
+                a *= 1.0f / (1.0f + expf(-__bfloat162float(g[0])));
+                b *= 1.0f / (1.0f + expf(-__bfloat162float(g[HALF])));
+            }
+            out[(t * nq + head) * VD + c] = from_f32<TO>(a);
+            out[(t * nq + head) * VD + c + HALF] = from_f32<TO>(b);
+        }
+        return;
     }
+    for (int c = threadIdx.x; c < VD; c += blockDim.x) out[(t * nq + head) * VD + c] = from_f32<TO>(value(c));
 }
 
 }  // namespace
@@ -624,7 +680,7 @@ Q3_EXPORT int q3_attention_capped_prefill_bf16(const void* q, const void* k_page
     if (n_seqs <= 0 || max_new <= 0) return 0;
     if (keep_first < 0 || (keep_first > 0 && window <= 0) || !pool_fits(pool_k, pool_v, pool_table, pool_size, window, keep_first))
         return Q3_ERR_BAD_SIZE;
-    const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size};
+    const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size, 0};
     if (value_heads <= 0) value_heads = nkv;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nkv % value_heads != 0 || softcap < 0.0f || chunk < 0 || window < 0 ||
         (chunk > 0 && window > 0))
@@ -653,11 +709,15 @@ Q3_EXPORT int q3_attention_capped_decode_bf16(const void* q, const void* k_pages
                                               int pages_per_seq, int64_t n_tokens, int nq, int nkv, float scale, float softcap,
                                               int chunk, int sink, int n_splits, int window, int value_heads, int out_f32,
                                               const float* sink_values, int keep_first, const void* pool_k, const void* pool_v,
-                                              const int* pool_table, int pool_size, void* stream) {
+                                              const int* pool_table, int pool_size, int pool_write, const float* back_cos,
+                                              const float* back_sin, const void* gate, int64_t gate_row, void* stream) {
     if (n_tokens <= 0) return 0;
     if (keep_first < 0 || (keep_first > 0 && window <= 0) || !pool_fits(pool_k, pool_v, pool_table, pool_size, window, keep_first))
         return Q3_ERR_BAD_SIZE;
-    const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size};
+    const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size, pool_write};
+    const FinishArgs finish = {back_cos, back_sin, token_pos, (const bf16*)gate, gate_row};
+    const bool finishing = back_cos != nullptr || gate != nullptr;
+    if ((back_cos == nullptr) != (back_sin == nullptr) || (finishing && out_f32)) return Q3_ERR_BAD_SIZE;
     if (value_heads <= 0) value_heads = nkv;
     if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || nq / nkv > 16 || nkv % value_heads != 0 || softcap < 0.0f || chunk < 0 ||
         window < 0 || (chunk > 0 && window > 0) || n_splits <= 0)
@@ -677,10 +737,10 @@ Q3_EXPORT int q3_attention_capped_decode_bf16(const void* q, const void* k_pages
                                         : launch(decode_capped_split_kernel<false, false>, configured[0]);
     if (e != cudaSuccess) return (int)e;
     if (out_f32)
-        return (int)q3_launch(decode_capped_merge_kernel<float>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
-                              (cudaStream_t)stream, (const float*)scratch, (float*)out, nq, n_splits, sink, sink_values);
-    return (int)q3_launch(decode_capped_merge_kernel<bf16>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
-                          (cudaStream_t)stream, (const float*)scratch, (bf16*)out, nq, n_splits, sink, sink_values);
+        return (int)q3_launch(decode_capped_merge_kernel<float, false>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
+                              (cudaStream_t)stream, (const float*)scratch, (float*)out, nq, n_splits, sink, sink_values, finish);
+    return (int)q3_launch(finishing ? decode_capped_merge_kernel<bf16, true> : decode_capped_merge_kernel<bf16, false>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
+                          (cudaStream_t)stream, (const float*)scratch, (bf16*)out, nq, n_splits, sink, sink_values, finish);
 }
 
 // The same from the output of the q/k/v projection as it is, qkv [tokens, (nq + nkv) * D + nkv * VD]: the bias (may be null),
@@ -707,6 +767,6 @@ Q3_EXPORT int q3_attention_capped_decode_fused_bf16(const void* qkv, void* k_pag
                               DECODE_SMEM_FUSED, (cudaStream_t)stream, (const bf16*)nullptr, (const bf16*)k_pages, (const bf16*)v_pages,
                               scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, scale, softcap, chunk, fused, nkv, 0, PoolArgs{});
     if (e != cudaSuccess) return (int)e;
-    return (int)q3_launch(decode_capped_merge_kernel<bf16>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
-                          (cudaStream_t)stream, (const float*)scratch, (bf16*)out, nq, n_splits, sink, (const float*)nullptr);
+    return (int)q3_launch(decode_capped_merge_kernel<bf16, false>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
+                          (cudaStream_t)stream, (const float*)scratch, (bf16*)out, nq, n_splits, sink, (const float*)nullptr, FinishArgs{});
 }

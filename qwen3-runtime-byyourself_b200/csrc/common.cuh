@@ -120,6 +120,17 @@ template <int GATED> __device__ __forceinline__ float gate_activation(float z) {
     return z / (1.0f + expf(-z));
 }
 
+// What a product's epilogue does, beside 0 (nothing): 1 and 2 take pairs of gate and up columns (see above), 3 is the
+// square of relu on every value.
+template <int GATED> constexpr bool q3_paired = GATED == 1 || GATED == 2;
+template <int GATED> __device__ __forceinline__ float q3_plain_epilogue(float v) {
+    if constexpr (GATED == 3) {
+        const float z = fmaxf(v, 0.0f);
+        return z * z;
+    }
+    return v;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -39,7 +39,8 @@ template <> __device__ __forceinline__ bf16 to_out<bf16>(float v) { return __flo
 // over them.  PF: k-blocks (of 32) a warp keeps in flight in registers.  MINB: blocks per SM the
 // register budget is held to, so that the whole grid is resident at once for the layer sizes.
 // GATED: W holds gate and up rows interleaved in blocks of eight (rows 16t..16t+7 gate, 16t+8..
-// 16t+15 up, both for features 8t..8t+7); the kernel then writes round(silu(g)) * u, [M, N/2].
+// 16t+15 up, both for features 8t..8t+7); the kernel then writes round(silu(g)) * u, [M, N/2].  GATED 3: every value of
+// the product becomes the square of its relu.
 template <int MT, int R, int WARPS, int PF, int MINB, int GATED, typename OutT>
 __global__ void __launch_bounds__(WARPS * 32, MINB)
 gemm_skinny_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, OutT* __restrict__ Y, int M, int N, int K) {
@@ -130,14 +131,14 @@ gemm_skinny_kernel(const bf16* __restrict__ X, const bf16* __restrict__ W, OutT*
             mine[(c + 1) * LD + n + 8] = acc[r][m][3];
         }
     __syncthreads();
-    if constexpr (GATED == 0) {
+    if constexpr (!q3_paired<GATED>) {
         for (int idx = threadIdx.x; idx < ROWS * COLS; idx += WARPS * 32) {
             const int n = idx % ROWS, m = idx / ROWS;
             if (m >= M || n0 + n >= N) continue;
             float sum = 0.0f;
 #pragma unroll
             for (int w2 = 0; w2 < WARPS; ++w2) sum += red[w2 * COLS * LD + m * LD + n];
-            Y[(int64_t)m * N + n0 + n] = to_out<OutT>(sum);
+            Y[(int64_t)m * N + n0 + n] = to_out<OutT>(q3_plain_epilogue<GATED>(sum));
         }
     } else {
         // feature f = (row tile) * 8 + j has its gate in row 16t + j and its up in row 16t + 8 + j; both
@@ -182,7 +183,7 @@ int launch(const bf16* X, const bf16* W, OutT* Y, int M, int N, int K, cudaStrea
 template <int GATED, typename OutT>
 int dispatch(const bf16* X, const bf16* W, OutT* Y, int M, int N, int K, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 != 0 || M > 64 || (GATED && N % 16 != 0)) return Q3_ERR_BAD_SIZE;
+    if (K <= 0 || K % 8 != 0 || M > 64 || (q3_paired<GATED> && N % 16 != 0)) return Q3_ERR_BAD_SIZE;
     if (!aligned16(X) || !aligned16(W)) return Q3_ERR_MISALIGNED;
     const bool few_rows = (N + 15) / 16 <= 296;
     if (M <= 8) {
@@ -217,8 +218,10 @@ Q3_EXPORT int q3_gemm_skinny_gated_bf16(const void* X, const void* W, void* Y, i
     return dispatch<1, bf16>((const bf16*)X, (const bf16*)W, (bf16*)Y, M, N, K, (cudaStream_t)stream);
 }
 
-// The same with the activation as an argument: act 1 = SiLU, 2 = the tanh form of GELU.
+// The same with the activation as an argument: act 1 = SiLU, 2 = the tanh form of GELU; act 3: no gate, Y [M, N] = max(x, 0)^2 of
+// the product's values.
 Q3_EXPORT int q3_gemm_skinny_act_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int act, void* stream) {
+    if (act == 3) return dispatch<3, bf16>((const bf16*)X, (const bf16*)W, (bf16*)Y, M, N, K, (cudaStream_t)stream);
     if (act == 2) return dispatch<2, bf16>((const bf16*)X, (const bf16*)W, (bf16*)Y, M, N, K, (cudaStream_t)stream);
     if (act == 1) return dispatch<1, bf16>((const bf16*)X, (const bf16*)W, (bf16*)Y, M, N, K, (cudaStream_t)stream);
     return Q3_ERR_BAD_SIZE;

@@ -214,21 +214,23 @@ gemm_tcgen05_mid_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_
     // ---------------- reduce over the cluster: this block finishes the tokens m with m % ranks == rank
     pdl_wait();                                                               // no global write before this
     {
-        const int out_n = GATED ? (N >> 1) : N;
+        const int out_n = q3_paired<GATED> ? (N >> 1) : N;
         const bool vec = (out_n % 4 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
-        constexpr int GROUPS = GATED ? 16 : 32;                               // groups of four outputs per token and tile
+        constexpr int GROUPS = q3_paired<GATED> ? 16 : 32;                               // groups of four outputs per token and tile
         const int my_tokens = (MT - (int)rank + (int)ranks - 1) / (int)ranks;
         for (int idx = threadIdx.x; idx < my_tokens * GROUPS; idx += THREADS) {
             const int local = (idx / GROUPS) * (int)ranks + (int)rank, g = idx % GROUPS;
             const int m = m0 + local;
             if (m >= M) continue;
-            if constexpr (GATED == 0) {
+            if constexpr (!q3_paired<GATED>) {
                 const uint32_t addr = base + (uint32_t)(local * PART_LD + 4 * g) * 4u;
                 float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
                 for (uint32_t s = 0; s < ranks; ++s) {
                     const float4 v = ld_cluster_f4(map_to_rank(addr, s));
                     sum.x += v.x; sum.y += v.y; sum.z += v.z; sum.w += v.w;
                 }
+                sum = make_float4(q3_plain_epilogue<GATED>(sum.x), q3_plain_epilogue<GATED>(sum.y), q3_plain_epilogue<GATED>(sum.z),
+                                  q3_plain_epilogue<GATED>(sum.w));
                 const int n = n0 + 4 * g;
                 if (n < N) store4<OutT>(Y + (int64_t)m * N + n, sum, vec, N - n);
             } else {
@@ -303,12 +305,13 @@ template <> __device__ __forceinline__ void store_run8<bf16>(bf16* p, const uint
 // the epilogue then writes round(silu(g)) * u, [M, N/2], instead of the raw product.
 // 32 consecutive columns (rows of W n0 + c ..) of one token's accumulator row, converted and stored; `row` points at
 // the token's first output of this tile.  GATED: the columns are gate[8] up[8] gate[8] up[8] of 16 features and
-// the output is round(silu(g)) * u with both rounded to bfloat16 first (src/ops/elementwise.cu:47-65).
+// the output is round(silu(g)) * u with both rounded to bfloat16 first (src/ops/elementwise.cu:47-65).  GATED 3: the square of
+// relu of every value.
 template <int GATED, typename OutT>
 __device__ __forceinline__ void store_chunk32(const uint32_t (&r)[32], OutT* row, int c, int n0, bool token_valid, int N,
                                               bool vec_ok) {
     if (!token_valid) return;
-    if constexpr (GATED != 0) {
+    if constexpr (q3_paired<GATED>) {
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
             const int n = n0 + c + h * 16;           // first gate column of this block
@@ -332,12 +335,15 @@ __device__ __forceinline__ void store_chunk32(const uint32_t (&r)[32], OutT* row
 #pragma unroll
         for (int j = 0; j < 32; j += 8) {
             const int n = n0 + c + j;
+            uint32_t v[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = __float_as_uint(q3_plain_epilogue<GATED>(__uint_as_float(r[j + e])));
             if (vec_ok && n + 8 <= N) {
-                store_run8<OutT>(row + c + j, r + j);
+                store_run8<OutT>(row + c + j, v);
             } else {
 #pragma unroll
                 for (int e = 0; e < 8; ++e)
-                    if (n + e < N) row[c + j + e] = to_out<OutT>(__uint_as_float(r[j + e]));
+                    if (n + e < N) row[c + j + e] = to_out<OutT>(__uint_as_float(v[e]));
             }
         }
     }
@@ -427,7 +433,7 @@ gemm_tcgen05_prompt_kernel(const __grid_constant__ CUtensorMap map_x, const __gr
     } else {
         pdl_wait();
         const int lane_base = (warp & 3) * 32;
-        const bool vec_ok = ((GATED ? (N >> 1) : N) % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
+        const bool vec_ok = ((q3_paired<GATED> ? (N >> 1) : N) % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
         uint32_t local = 0;
         for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x, ++local) {
             const uint32_t buf = local & 1u;
@@ -438,7 +444,7 @@ gemm_tcgen05_prompt_kernel(const __grid_constant__ CUtensorMap map_x, const __gr
             }
             tc_fence_after();
             const int m = m0 + lane_base + lane;
-            OutT* row = Y + (int64_t)m * (GATED ? (N >> 1) : N) + (GATED ? (n0 >> 1) : n0);
+            OutT* row = Y + (int64_t)m * (q3_paired<GATED> ? (N >> 1) : N) + (q3_paired<GATED> ? (n0 >> 1) : n0);
 #pragma unroll 1
             for (int c = 0; c < BN; c += 32) {
                 uint32_t r[32];
@@ -778,7 +784,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
     } else {
         pdl_wait();
         const int lane_base = (warp & 3) * 32;
-        const bool vec_ok = ((GATED ? (N >> 1) : N) % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
+        const bool vec_ok = ((q3_paired<GATED> ? (N >> 1) : N) % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
         uint32_t local = 0;
         for (int tile = first; tile < tiles; tile += stride, ++local) {
             const uint32_t buf = local & 1u;
@@ -792,7 +798,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
             if constexpr (QKV) {
                 qkv_tile_epilogue(tmem_base + ((uint32_t)lane_base << 16) + buf * BN, m, m < M, n0, N, qkv);
             } else {
-                OutT* row = Y + (int64_t)m * (GATED ? (N >> 1) : N) + (GATED ? (n0 >> 1) : n0);
+                OutT* row = Y + (int64_t)m * (q3_paired<GATED> ? (N >> 1) : N) + (q3_paired<GATED> ? (n0 >> 1) : n0);
 #pragma unroll 1
                 for (int c = 0; c < BN; c += 32) {
                     uint32_t r[32];
@@ -941,9 +947,9 @@ gemm_tcgen05_pair_splitk_kernel(const __grid_constant__ CUtensorMap map_x, const
 
     if (warp >= 2 && acc_ok) {
         pdl_wait();                                           // no global write before this
-        const bool vec_ok = ((GATED ? (N >> 1) : N) % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
+        const bool vec_ok = ((q3_paired<GATED> ? (N >> 1) : N) % 8 == 0) && ((reinterpret_cast<uintptr_t>(Y) & 15u) == 0);
         const int m = m0 + row;
-        OutT* out_row = Y + (int64_t)m * (GATED ? (N >> 1) : N) + (GATED ? (n0 >> 1) : n0);
+        OutT* out_row = Y + (int64_t)m * (q3_paired<GATED> ? (N >> 1) : N) + (q3_paired<GATED> ? (n0 >> 1) : n0);
 #pragma unroll 1
         for (int c = split; c < CHUNKS; c += splits) {
             uint32_t own[32], r[32];
@@ -1132,23 +1138,26 @@ Q3_EXPORT int q3_gemm_tcgen05_prompt_bf16(const void* X, const void* W, void* Y,
 }
 
 // The prompt form on pairs of SMs: tiles of 256 tokens x 256 rows of W, each block of a pair loading half of
-// the W tile.  `gated` as below (bfloat16 output only; 1 = SiLU, 2 = the tanh form of GELU).  `splits` (1..4) > 1: K split over that many pairs of a
+// the W tile.  `gated` as below (bfloat16 output only; 1 = SiLU, 2 = the tanh form of GELU; 3: no gate, Y [M, N] = the square of
+// relu of the product).  `splits` (1..4) > 1: K split over that many pairs of a
 // cluster, one tile per cluster.
 Q3_EXPORT int q3_gemm_tcgen05_pair_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int out_is_f32, int gated,
                                         int splits, int* status, void* stream_) {
     if (M <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 != 0 || (gated && (N % 16 != 0 || out_is_f32)) || splits < 1 || splits > 4) return Q3_ERR_BAD_SIZE;
+    if (K <= 0 || K % 8 != 0 || (gated && ((gated != 3 && N % 16 != 0) || out_is_f32)) || gated < 0 || gated > 3 || splits < 1 || splits > 4) return Q3_ERR_BAD_SIZE;
     if (!aligned16(X) || !aligned16(W)) return Q3_ERR_MISALIGNED;
     cudaStream_t stream = (cudaStream_t)stream_;
     const bf16* x = (const bf16*)X;
     const bf16* w = (const bf16*)W;
     if (splits > (K + BK - 1) / BK) splits = (K + BK - 1) / BK;
     if (splits > 1) {
+        if (gated == 3) return launch_pair_splitk<6, 3, bf16>(x, w, (bf16*)Y, M, N, K, splits, status, stream);
         if (gated == 2) return launch_pair_splitk<6, 2, bf16>(x, w, (bf16*)Y, M, N, K, splits, status, stream);
         if (gated) return launch_pair_splitk<6, 1, bf16>(x, w, (bf16*)Y, M, N, K, splits, status, stream);
         return out_is_f32 ? launch_pair_splitk<6, 0, float>(x, w, (float*)Y, M, N, K, splits, status, stream)
                           : launch_pair_splitk<6, 0, bf16>(x, w, (bf16*)Y, M, N, K, splits, status, stream);
     }
+    if (gated == 3) return launch_pair<6, 3, bf16>(x, w, (bf16*)Y, M, N, K, status, stream);
     if (gated == 2) return launch_pair<6, 2, bf16>(x, w, (bf16*)Y, M, N, K, status, stream);
     if (gated) return launch_pair<6, 1, bf16>(x, w, (bf16*)Y, M, N, K, status, stream);
     return out_is_f32 ? launch_pair<6, 0, float>(x, w, (float*)Y, M, N, K, status, stream)
@@ -1194,18 +1203,21 @@ Q3_EXPORT int q3_gemm_tcgen05_prompt_gated_bf16(const void* X, const void* W, vo
 
 // The weights-first form for a few hundred rows of X at most (W is read once per 256 rows).  `splits` K ranges per tile of 128 rows of W (one cluster;
 // 0 = chosen from N and K).  `gated`: W [N, K] holds gate and up rows interleaved in blocks of eight and
-// Y is [M, N/2] = round(act(g)) * u, act = SiLU (gated 1) or the tanh form of GELU (gated 2).  `status` is a device int that a kernel sets to 1/2/3 if a bounded
+// Y is [M, N/2] = round(act(g)) * u, act = SiLU (gated 1) or the tanh form of GELU (gated 2); gated 3: no gate, Y [M, N] = the square of relu of the product.  `status` is a device int that a kernel sets to 1/2/3 if a bounded
 // wait ran out (0 otherwise).
 Q3_EXPORT int q3_gemm_tcgen05_mid_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int out_is_f32, int gated,
                                        int splits, int* status, void* stream_) {
     if (M <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 != 0 || M > 256 * 1024 || splits < 0 || splits > 8 || (gated && N % 16 != 0)) return Q3_ERR_BAD_SIZE;
+    if (K <= 0 || K % 8 != 0 || M > 256 * 1024 || splits < 0 || splits > 8 || ((gated == 1 || gated == 2) && N % 16 != 0) || gated < 0 ||
+        gated > 3 || (gated == 3 && out_is_f32))
+        return Q3_ERR_BAD_SIZE;
     if (!aligned16(X) || !aligned16(W)) return Q3_ERR_MISALIGNED;
     cudaStream_t stream = (cudaStream_t)stream_;
     const bf16* x = (const bf16*)X;
     const bf16* w = (const bf16*)W;
     if (splits == 0) splits = mid_splits(N, K, M <= 128 ? 0 : (M + 255) / 256);
     if (splits > (K + BK - 1) / BK) splits = (K + BK - 1) / BK;
+    if (gated == 3) return dispatch_mid<3, bf16>(x, w, (bf16*)Y, M, N, K, splits, status, stream);
     if (gated == 2)
         return out_is_f32 ? dispatch_mid<2, float>(x, w, (float*)Y, M, N, K, splits, status, stream)
                           : dispatch_mid<2, bf16>(x, w, (bf16*)Y, M, N, K, splits, status, stream);

@@ -923,10 +923,17 @@ def attention_capped_splits(n_tokens: int, nkv: int, sm_count: int, max_keys: in
 def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_pos, page_table, n_tokens: int, nq: int,
                             nkv: int, d: int, vd: int, scale: float, softcap: float, chunk: Optional[int], sink: bool,
                             n_splits: int, window: Optional[int] = None, value_heads: Optional[int] = None,
-                            sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None):
+                            sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None,
+                            pool_write: bool = False, back_cos: Optional[torch.Tensor] = None, back_sin: Optional[torch.Tensor] = None,
+                            gate: Optional[torch.Tensor] = None):
     """The same for one new token per sequence, the keys split over `n_splits` blocks per (token, kv head); `scratch`
-    holds n_tokens * nq * n_splits * (vd + 2) float32."""
+    holds n_tokens * nq * n_splits * (vd + 2) float32.  `pool_write`: a block of tokens that a token completes is pooled by this
+    kernel (as `pool_blocks` does); `back_cos`, `back_sin`, `gate`: what `turn_back_gate` does to the output, done where the
+    splits are merged."""
     nv = int(value_heads or nkv)
+    if (back_cos is None) != (back_sin is None) or (back_cos is not None and (2 * back_cos.shape[-1] != vd or back_sin.shape != back_cos.shape)) \
+            or (gate is not None and (gate.shape != (n_tokens, nq * vd) or gate.stride(1) != 1 or gate.dtype != q.dtype)):
+        raise KernelError("attention_capped_decode: the output's rotation or gate does not fit")
     if q.dtype != torch.bfloat16 or not attention_capped_fits(d, vd, None, nq // nkv) or out.dtype not in (torch.bfloat16, torch.float32):
         raise KernelError("attention_capped_decode: bfloat16, head sizes in steps of 16 up to 256, groups of up to 16 heads")
     if k_pages.shape[1:] != (nkv, PAGE_TOKENS, d) or v_pages.shape[1:] != (nv, PAGE_TOKENS, vd) or out.shape[-1] != nq * vd \
@@ -934,7 +941,7 @@ def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_
         raise KernelError("attention_capped_decode: shapes do not fit")
     fn = _fn("attention_capped.cu", "q3_attention_capped_decode_bf16",
              [c_void_p] * 8 + [c_int, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int64, c_void_p],
              defines=_capped_defines(d, vd))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out"), _dev(scratch, "scratch", torch.float32),
@@ -942,7 +949,10 @@ def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_
               _dev(page_table, "page_table", torch.int32), page_table.shape[-1], n_tokens, nq, nkv, float(scale),
               float(softcap or 0.0), int(chunk or 0), int(bool(sink)), int(n_splits), int(window or 0), nv,
               int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
-              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_decode"), _stream()), "attention_capped_decode")
+              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_decode"), int(bool(pool_write)),
+              _ptr(back_cos, "back_cos", torch.float32), _ptr(back_sin, "back_sin", torch.float32),
+              gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0, _stream()),
+           "attention_capped_decode")
     _count_extra(1)                                              # the split kernel and the merge kernel
     return out
 
@@ -1207,6 +1217,27 @@ def gemm_skinny_gated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activ
     fn = _fn("gemm_skinny_bf16.cu", "q3_gemm_skinny_act_bf16", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     _check(fn(_dev(x, "x", torch.bfloat16), _dev(w, "w", torch.bfloat16), _dev(out, "out", torch.bfloat16), M, N, K,
               ACTIVATIONS[activation] + 1, _stream()), "gemm_skinny_gated")
+    return out
+
+
+def gemm_relu2(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, form: str, splits: int = 0) -> torch.Tensor:
+    """out[M, N] = max(x . w^T, 0)^2 with the square in the product's epilogue, bfloat16; `form`: "skinny" (M <= 64), "mid" (weights
+    first) or "pair" (pairs of SMs; `splits` K ranges), as the products of these names above and below."""
+    M, K = x.shape
+    N = w.shape[0]
+    if w.shape[1] != K or out.shape != (M, N) or K % 8 != 0 or (form == "skinny" and not gemm_skinny_fits(M, K)):
+        raise KernelError(f"gemm_relu2: shapes {tuple(x.shape)} x {tuple(w.shape)}^T -> {tuple(out.shape)}")
+    pointers = (_dev(x, "x", torch.bfloat16), _dev(w, "w", torch.bfloat16), _dev(out, "out", torch.bfloat16))
+    if form == "skinny":
+        fn = _fn("gemm_skinny_bf16.cu", "q3_gemm_skinny_act_bf16", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+        _check(fn(*pointers, M, N, K, 3, _stream()), "gemm_skinny_relu2")
+        return out
+    if form not in ("mid", "pair"):
+        raise KernelError(f"gemm_relu2: form {form!r}")
+    fn = _fn("gemm_tcgen05.cu", f"q3_gemm_tcgen05_{form}_bf16",
+             [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p])
+    _check(fn(*pointers, M, N, K, 0, 3, int(splits) if form == "mid" else max(int(splits), 1), _status_word(x.device).data_ptr(), _stream()),
+           f"gemm_tcgen05_{form}_relu2")
     return out
 
 

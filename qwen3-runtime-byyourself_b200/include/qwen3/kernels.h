@@ -159,12 +159,16 @@ int q3_attention_capped_prefill_bf16(const void* q, const void* k_pages, const v
 /* (window > 0: a sliding window of that many keys instead of chunks, beside which the first keep_first keys of the sequence
    stay visible; value_heads 0 = nkv, else each value head serves nkv / value_heads key heads; out_f32: `out` is float;
    sink_values (may be null): the sink's score per query head; pool_*: as for q3_attention_generic) */
-/* one new token per sequence; scratch: n_tokens * nq * n_splits * (value_dim + 2) float32 */
+/* one new token per sequence; scratch: n_tokens * nq * n_splits * (value_dim + 2) float32.  pool_write: the block that this token
+   completes, if it does, is pooled here.  back_cos, back_sin [positions, value_dim / 2], may be null: every head of the output is
+   turned back by the token's position; gate (may be null; rows gate_row apart): then multiplied by sigmoid(gate) (both for a
+   bfloat16 output) */
 int q3_attention_capped_decode_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, float* scratch,
                                     const int* token_seq, const int* token_pos, const int* page_table, int pages_per_seq,
                                     int64_t n_tokens, int nq, int nkv, float scale, float softcap, int chunk, int sink, int n_splits,
                                     int window, int value_heads, int out_f32, const float* sink_values, int keep_first,
-                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, int pool_write,
+                                    const float* back_cos, const float* back_sin, const void* gate, int64_t gate_row, void* stream);
 
 /* ---- attention_decode.cu (-DQ3_HEAD_DIM): one new token per sequence, bfloat16 ---------------------------- */
 int q3_attention_decode_head_dim(void);
@@ -202,10 +206,12 @@ int q3_gemm_tn_bf16(const void* X, const void* W, void* Y, int M, int N, int K, 
 int q3_gemm_skinny_bf16(const void* X, const void* W, void* Y, int M, int N, int K, void* stream);
 int q3_gemm_skinny_bf16_f32out(const void* X, const void* W, void* Y, int M, int N, int K, void* stream);
 int q3_gemm_skinny_gated_bf16(const void* X, const void* W, void* Y, int M, int N, int K, void* stream);
-/* the same with the activation as an argument: act 1 = SiLU, 2 = the tanh form of GELU */
+/* the same with the activation as an argument: act 1 = SiLU, 2 = the tanh form of GELU; 3: no gate, Y [M, N] = max(x, 0)^2 of the
+   product */
 int q3_gemm_skinny_act_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int act, void* stream);
 /* gemm_tcgen05.cu: TMA + tcgen05; weights first with K split over a cluster (`mid`), tokens first on single SMs
-   (`prompt`, tile_n 128 or 256) and on pairs of SMs (`pair`) */
+   (`prompt`, tile_n 128 or 256) and on pairs of SMs (`pair`).  gated: 0 the product, 1 and 2 gated pairs of columns as above,
+   3 max(x, 0)^2 of every value (bfloat16 output) */
 int q3_gemm_tcgen05_mid_bf16(const void* X, const void* W, void* Y, int M, int N, int K, int out_is_f32, int gated, int splits,
                              int* status, void* stream);
 int q3_gemm_tcgen05_mid_splits(int N, int K, int M);

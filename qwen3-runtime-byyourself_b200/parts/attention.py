@@ -300,6 +300,10 @@ class GQAAttention(Part):
             raise ops.KernelError("this attention takes a position encoding with tables, or none")
         else:
             self._prepare_unfused(qkv, q, cache, ctx, table, qw, kw, norm_eps)
+        if self.decodes_split(ctx):                 # that kernel pools a finished block, turns back and gates itself
+            gate = qkv[:, self.projection_width() - nq * vd:] if self.out_gate else None
+            self.decode_split(q, cache, attn, ctx, table, v_cos, v_sin, gate)
+            return attn
         if self.pool and not cache.shared:
             ops.pool_blocks(cache.keys, cache.values, table, self.pooled(ctx, cache), ctx.seq_start, ctx.seq_pos0, ctx.n_seqs, ctx.max_new)
         self.attend(q, cache, attn, ctx, table)
@@ -307,6 +311,21 @@ class GQAAttention(Part):
             gate = qkv[:, self.projection_width() - nq * vd:] if self.out_gate else None
             ops.turn_back_gate(attn, v_cos, v_sin, ctx.token_pos, gate, nq, vd)
         return attn
+
+    def decodes_split(self, ctx) -> bool:
+        """Whether a step goes to the split-key decode kernel for attention beyond the plain form."""
+        return (ctx.is_decode and ctx.dtype == torch.bfloat16 and not self.plain
+                and ops.attention_capped_fits(self.head_dim, self.value_dim, self.window, self.num_heads // self.num_kv_heads))
+
+    def decode_split(self, q, cache, out, ctx, table, back_cos=None, back_sin=None, gate=None) -> None:
+        nq, nkv, vd = self.num_heads, self.num_kv_heads, self.value_dim
+        splits = ops.attention_capped_splits(ctx.n_tokens, nkv, _sm_count(ctx.device), self.keys_seen(ctx.max_context))
+        scratch = ctx.scratch.get("attn.capped_scratch", (ctx.n_tokens * nq * splits * (vd + 2),), torch.float32)
+        ops.attention_capped_decode(q, cache.keys, cache.values, out, scratch, ctx.token_seq, ctx.token_pos, table, ctx.n_tokens,
+                                    nq, nkv, self.head_dim, vd, self.scale, self.softcap, self.chunk, self.sink, splits,
+                                    window=self.window, value_heads=self.value_heads, sink_values=self.sink_values,
+                                    keep_first=self.keep_first, pool=self.pooled(ctx, cache), pool_write=not cache.shared,
+                                    back_cos=back_cos, back_sin=back_sin, gate=gate)
 
     def pooled(self, ctx, cache):
         """The pooled blocks of this layer as the kernels take them (None: there are none)."""
@@ -467,15 +486,9 @@ def _prefill_capped_tcgen05_kernel(part, q, cache, out, ctx, table) -> bool:
 
 def _decode_capped_kernel(part, q, cache, out, ctx, table) -> bool:
     """The same for decode steps: split over the keys of the chunk (or of the whole context), merged with the sink."""
-    nq, nkv = part.num_heads, part.num_kv_heads
-    if part.plain or not ops.attention_capped_fits(part.head_dim, part.value_dim, part.window, nq // nkv):
+    if not part.decodes_split(ctx):
         return False
-    splits = ops.attention_capped_splits(ctx.n_tokens, nkv, _sm_count(ctx.device), part.keys_seen(ctx.max_context))
-    scratch = ctx.scratch.get("attn.capped_scratch", (ctx.n_tokens * nq * splits * (part.value_dim + 2),), torch.float32)
-    ops.attention_capped_decode(q, cache.keys, cache.values, out, scratch, ctx.token_seq, ctx.token_pos, table, ctx.n_tokens,
-                                nq, nkv, part.head_dim, part.value_dim, part.scale, part.softcap, part.chunk, part.sink, splits,
-                                window=part.window, value_heads=part.value_heads, sink_values=part.sink_values,
-                                keep_first=part.keep_first, pool=part.pooled(ctx, cache))
+    part.decode_split(q, cache, out, ctx, table)
     return True
 
 

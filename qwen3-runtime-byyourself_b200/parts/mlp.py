@@ -96,8 +96,17 @@ class DenseMLP(Part):
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         N = ctx.n_tokens
         act = ctx.scratch.get("ff.act", (N, self.intermediate_size), ctx.dtype)
-        linear(x, self.w_up, act)
-        ops.activation(act, act, self.activation)
+        if self.activation == "relu2" and ctx.dtype == torch.bfloat16 and self.hidden_size % 8 == 0 and not linear_module.set_bf16_kernel_active():
+            M, I, K = N, self.intermediate_size, self.hidden_size          # the square in the product's epilogue
+            if M <= linear_module.skinny_rows:
+                ops.gemm_relu2(x, self.w_up, act, "skinny")
+            elif linear_module.tcgen05_form(M, I, K, gated=True) == "weights_first":
+                ops.gemm_relu2(x, self.w_up, act, "mid")
+            else:
+                ops.gemm_relu2(x, self.w_up, act, "pair", splits=linear_module.pair_plan(M, I, K)[1])
+        else:
+            linear(x, self.w_up, act)
+            ops.activation(act, act, self.activation)
         out = ctx.scratch.get(self.out_name, (N, self.hidden_size), ctx.dtype)
         return linear(act, self.w_down, out)
 

@@ -303,6 +303,22 @@ def test_dense_squared_relu_feed_forward(dtype, rows, hidden, ff):
     assert Ctx.scratch.violations() == []
 
 
+@pytest.mark.parametrize("form,M,N,K,splits", [("skinny", 1, 48, 64, 0), ("skinny", 8, 4800, 256, 0), ("skinny", 40, 130, 72, 0), ("mid", 9, 100, 256, 0),
+                                               ("mid", 100, 520, 2048, 4), ("mid", 300, 257, 128, 1), ("pair", 300, 512, 256, 1), ("pair", 513, 264, 512, 2),
+                                               ("pair", 129, 77, 192, 3)])
+def test_products_with_the_square_of_relu_in_their_epilogue(form, M, N, K, splits):
+    import torch
+    from qwen3_b200.csrc import ops
+    rng = np.random.default_rng(M + N)
+    x, w = dev(rng.standard_normal((M, K)), torch.bfloat16), dev(rng.standard_normal((N, K)) / np.sqrt(K), torch.bfloat16)
+    out = ops.gemm_relu2(x, w, torch.full((M, N), -1.0, dtype=torch.bfloat16, device="cuda"), form, splits=splits)
+    want = plain.relu_squared(f64(x) @ f64(w).T)
+    assert np.allclose(f64(out), want, rtol=2 ** -7, atol=1e-4) and (want == 0.0).any()
+    assert ops.tcgen05_status(torch.device("cuda")) == 0
+    with pytest.raises(ops.KernelError):
+        ops.gemm_relu2(x, w, out, "other")
+
+
 # ---------------------------------------------------------------- pooled blocks
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("G,d,vd,size", [(2, 16, 16, 5), (1, 64, 64, 16), (3, 11, 7, 3), (1, 128, 128, 1), (2, 8, 8, 64), (1, 8, 24, 100)])
@@ -482,6 +498,69 @@ def test_tiled_attention_walks_the_blocks_before_the_window_s_pages(H, G, d, win
             got = f64(out).reshape(4, H, d)
             for s, p in enumerate(last):
                 assert np.allclose(got[s], want[s][p], atol=3e-2), (where, s, p, splits)
+
+
+@pytest.mark.parametrize("H,G,d,size,window", [(4, 2, 16, 5, 9), (2, 1, 64, 16, 20), (2, 2, 128, 1, 3), (1, 1, 32, 70, 70)])
+def test_the_split_decode_pools_a_block_that_its_token_completes(H, G, d, size, window):
+    """Token by token over a page's worth of blocks: after every step the pool holds exactly the whole blocks, and the output is
+    that of the kernel which leaves the pooling to `pool_blocks`."""
+    import torch
+    from qwen3_b200.csrc import ops
+    rng = np.random.default_rng(d)
+    T, totals = torch.bfloat16, [150, 7]
+    table, k_pages = scattered_pages(rng, totals, G, d, T)
+    v_pages = torch.zeros_like(k_pages)
+    for s, n in enumerate(totals):
+        for j in range(n):
+            k_pages[table[s, j // PAGE], :, j % PAGE] = dev(rng.standard_normal((G, d)), T)
+            v_pages[table[s, j // PAGE], :, j % PAGE] = dev(rng.standard_normal((G, d)), T)
+    pool_table, pool_k = scattered_pages(rng, totals, G, d, T)
+    pool_v, own_k, own_v = (torch.zeros_like(pool_k) for _ in range(3))
+    by_kernel, by_itself = ops.Pool(pool_k, pool_v, dev(pool_table, torch.int32), size), ops.Pool(own_k, own_v, dev(pool_table, torch.int32), size)
+    seq, start, dev_table = dev([0, 1], torch.int32), dev([0, 1, 2], torch.int32), dev(table, torch.int32)
+    for p in range(140):
+        at = [p, min(p, 6)]
+        pos, q = dev(at, torch.int32), dev(rng.standard_normal((2, H * d)), T)
+        outs = []
+        for pool, write in ((by_itself, True), (by_kernel, False)):
+            if not write:
+                ops.pool_blocks(k_pages, v_pages, dev_table, pool, start, pos, 2, 1)
+            scratch, out = torch.empty(2 * H * 3 * (d + 2), dtype=torch.float32, device="cuda"), torch.empty((2, H * d), dtype=T, device="cuda")
+            ops.attention_capped_decode(q, k_pages, v_pages, out, scratch, seq, pos, dev_table, 2, H, G, d, d, 0.3, 0.0, None, False, 3,
+                                        window=window, pool=pool, pool_write=write)
+            outs.append(out)
+        assert torch.equal(outs[0], outs[1]), p
+        if p % 13 == 0 or p > 130:
+            for a, b in ((pool_k, own_k), (pool_v, own_v)):
+                assert np.allclose(f64(a), f64(b), rtol=2 ** -8, atol=1e-6), p
+            n = (p + 1) // size
+            assert np.allclose(read_pages(own_k, pool_table, 0, n), plain.pooled_blocks(read_pages(k_pages, table, 0, p + 1), size), rtol=2 ** -8, atol=1e-6)
+
+
+@pytest.mark.parametrize("H,G,d,vd,turn,gate", [(4, 2, 16, 24, True, True), (2, 1, 128, 128, True, False), (2, 2, 64, 32, False, True), (6, 2, 32, 256, True, True)])
+def test_the_split_decode_turns_its_output_back_and_gates_it(H, G, d, vd, turn, gate):
+    """vd 24 is no size the tiled kernel takes: 32 stands in for it there."""
+    import torch
+    from qwen3_b200.csrc import ops
+    vd = 32 if vd == 24 else vd
+    rng = np.random.default_rng(vd)
+    T, totals = torch.bfloat16, [100, 1, 65]
+    table, k_pages = scattered_pages(rng, totals, G, d, T)
+    k_pages.copy_(dev(rng.standard_normal(k_pages.shape), T))
+    v_pages = dev(rng.standard_normal(k_pages.shape[:-1] + (vd,)), T)
+    pos, seq = dev([n - 1 for n in totals], torch.int32), dev([0, 1, 2], torch.int32)
+    q, both = dev(rng.standard_normal((3, H * d)), T), dev(rng.standard_normal((3, 16 + H * vd)), T)
+    a = np.arange(128)[:, None] * plain.plain_frequencies(200.0, vd)[None, :]
+    cos, sin = (dev(np.cos(a), torch.float32), dev(np.sin(a), torch.float32)) if turn else (None, None)
+    sinks = dev(rng.standard_normal(H), torch.float32)
+    outs = []
+    for fused in (True, False):
+        scratch, out = torch.empty(3 * H * 2 * (vd + 2), dtype=torch.float32, device="cuda"), torch.empty((3, H * vd), dtype=T, device="cuda")
+        kw = dict(back_cos=cos, back_sin=sin, gate=both[:, 16:] if gate else None) if fused else {}
+        ops.attention_capped_decode(q, k_pages, v_pages, out, scratch, seq, pos, dev(table, torch.int32), 3, H, G, d, vd, 0.3, 0.0, None, True, 2,
+                                    sink_values=sinks, **kw)
+        outs.append(out if fused else ops.turn_back_gate(out, cos, sin, pos, both[:, 16:] if gate else None, H, vd))
+    assert np.allclose(f64(outs[0]), f64(outs[1]), rtol=2e-2, atol=1e-2)
 
 
 def test_pooled_blocks_that_do_not_fit_are_refused():
