@@ -19,7 +19,8 @@
 //                     o_i = decay^(i+1) S_0^T q_i + sum_(j<=i) decay^(i-j) (q_i . k_j) v_j  and
 //                     S_C = decay^C S_0 + sum_j decay^(C-1-j) k_j v_j^T, all in 32-bit; the powers are
 //                     formed as exp2(n log2 decay), never as quotients, so a small decay cannot overflow.
-//   lightning_chunks_tc : the chunked form with its four products per chunk on the tensor cores (namespace tc below).
+//   lightning_chunks_tc : the chunked form with its four products per chunk on the tensor cores, long prompts in segments that run
+//                     side by side (namespace tc below).
 //   gated_norm      : out = T( o / sqrt(mean(o^2) + eps) * w * sigmoid(g) ) over a token's H*vd values.
 #include "common.cuh"
 
@@ -281,8 +282,18 @@ int lightning_chunks_launch(const T* proj, float* state, const float* decay, con
 // factor - well beyond what a compute type of bfloat16 asks of a 32-bit recurrence, and it is used for that compute type only
 // (the float32 path stays on fmaf).  A block of 8 warps per (head, sequence, tile of `vt` state columns) keeps q, k (C x d), its
 // columns of v, the C x C scores and its share of the state, d x vt, in shared memory; head sizes in steps of 8.
+//
+// Long prompts of few sequences are cut into segments that run side by side, since the decay is a number: STATES gives every
+// segment's own contribution to the state (from zero), `segment_starts_kernel` joins them, S before segment s + 1 =
+// decay^length S before segment s + contribution of s, and OUTPUTS walks every segment from its start; the last one
+// leaves the sequence's state.  WHOLE walks a sequence's new tokens from and to its state in one go.
 namespace tc {
 constexpr int C = 32;
+enum Walk { WHOLE, STATES, OUTPUTS };
+struct Segments {
+    float* states;             // [sequences, count, H, d, vd]
+    int length, count;
+};
 
 __device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
     asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
@@ -330,11 +341,11 @@ __device__ __forceinline__ void tile(float (&c)[4], const float* A, int lda, con
     }
 }
 
-template <typename T>
+template <typename T, Walk WALK>
 __global__ void __launch_bounds__(256)
 lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state, const float* __restrict__ decay,
                            const int* __restrict__ seq_start, const int* __restrict__ seq_slots, float* __restrict__ out, int H, int d,
-                           int vd, int vt, const Input in) {
+                           int vd, int vt, const Input in, const Segments segments) {
     extern __shared__ float smem[];
     const int dp = (d + 15) & ~15;                      // rows of the state in whole 16-row tiles; the padding stays zero
     const int ldq = dp + 4, ldv = vt + 8, lda = C + 4;  // row lengths that spread the fragments' rows over the banks
@@ -346,21 +357,27 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
     __shared__ float pw[C + 1], pw_rev[C];
     pdl_launch_dependents();
     pdl_wait();
-    const int head = blockIdx.x, seq = blockIdx.y, col0 = blockIdx.z * vt;
+    const int col_tiles = (vd + vt - 1) / vt, segment = WALK == WHOLE ? 0 : (int)blockIdx.z / col_tiles;
+    const int head = blockIdx.x, seq = blockIdx.y, col0 = ((int)blockIdx.z - segment * col_tiles) * vt;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    const int seq_end = seq_start[seq + 1], t_begin = seq_start[seq] + (WALK == WHOLE ? 0 : segment * segments.length);
+    const int t_end = WALK == WHOLE ? seq_end : min(seq_end, t_begin + segments.length);
+    if (WALK != WHOLE && t_begin >= seq_end) return;
+    if (WALK == STATES && t_end == seq_end) return;      // the last segment's walk leaves the state itself
     const float lam = decay[head];
     const float l2 = lam > 0.0f ? log2f(lam) : 0.0f;
     for (int n = tid; n <= C; n += 256) pw[n] = n == 0 ? 1.0f : (lam > 0.0f ? exp2f((float)n * l2) : 0.0f);
     const int64_t cols = 2 * (int64_t)H * d + 2 * (int64_t)H * vd;
     float* S_g = state + (int64_t)seq_slots[seq] * in.slot_stride + (int64_t)head * d * vd;
+    float* S_seg = WALK == WHOLE ? nullptr : segments.states + (((int64_t)seq * segments.count + segment) * H + head) * d * vd;
+    const float* S_from = WALK == WHOLE ? S_g : S_seg;
     for (int x = tid; x < dp * ldv; x += 256) {
         const int i = x / ldv, c = x % ldv;
-        S_s[x] = (i < d && c < vt && col0 + c < vd) ? S_g[(int64_t)i * vd + col0 + c] : 0.0f;
+        S_s[x] = (WALK != STATES && i < d && c < vt && col0 + c < vd) ? S_from[(int64_t)i * vd + col0 + c] : 0.0f;
     }
     for (int x = tid; x < 2 * C * ldq + C * ldv; x += 256) smem[x] = 0.0f;     // the padding of q, k and v stays zero
     const int n_tiles = vt / 8;                          // 8-column tiles of this block's state columns
-    const int t_end = seq_start[seq + 1];
-    for (int t0 = seq_start[seq]; t0 < t_end; t0 += C) {
+    for (int t0 = t_begin; t0 < t_end; t0 += C) {
         const int Cn = min(C, t_end - t0);
         __syncthreads();                                 // the chunk before is done with the buffers; S_s holds its state
         // 16-byte packets of the projection's rows (head sizes are multiples of 8); rows beyond the chunk are zero
@@ -403,7 +420,7 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
             }
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
-                q_s[i * ldq + c + e] = qv[e];
+                if constexpr (WALK != STATES) q_s[i * ldq + c + e] = qv[e];
                 k_s[i * ldq + c + e] = kv[e];
             }
         }
@@ -422,6 +439,7 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
         }
         if (tid < C) pw_rev[tid] = tid < Cn ? pw[Cn - 1 - tid] : 0.0f;
         __syncthreads();
+        if constexpr (WALK != STATES) {
         // the scores of the chunk: 2 x 4 tiles of 16 x 8, one per warp
         {
             const int mi = warp & 1, ni = warp >> 1;
@@ -456,6 +474,7 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
                 }
             }
         }
+        }
         // the state after the chunk: 16-row tiles of the state dealt to the warps
         for (int mt = warp; mt < dp / 16; mt += 8) {
             for (int ni = 0; ni < n_tiles; ++ni) {
@@ -469,10 +488,31 @@ lightning_chunks_tc_kernel(const T* __restrict__ proj, float* __restrict__ state
             }
         }
     }
+    if (WALK == OUTPUTS && t_end < seq_end) return;
+    float* S_to = WALK == STATES ? S_seg : S_g;
     __syncthreads();
     for (int x = tid; x < d * vt; x += 256) {
         const int i = x / vt, c = x % vt;
-        if (col0 + c < vd) S_g[(int64_t)i * vd + col0 + c] = S_s[i * ldv + c];
+        if (col0 + c < vd) S_to[(int64_t)i * vd + col0 + c] = S_s[i * ldv + c];
+    }
+}
+
+// A thread per value of a sequence's state: the contributions of its segments become the states before them.
+__global__ void segment_starts_kernel(const float* __restrict__ state, const float* __restrict__ decay, const int* __restrict__ seq_start,
+                                      const int* __restrict__ seq_slots, int64_t slot_stride, int H, int per_head, const Segments segments) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int seq = blockIdx.y;
+    const int64_t x = (int64_t)blockIdx.x * blockDim.x + threadIdx.x, all = (int64_t)H * per_head;
+    if (x >= all) return;
+    const int live = (seq_start[seq + 1] - seq_start[seq] + segments.length - 1) / segments.length;
+    const float lam = decay[x / per_head], power = lam > 0.0f ? exp2f((float)segments.length * log2f(lam)) : 0.0f;
+    float S = state[(int64_t)seq_slots[seq] * slot_stride + x];
+    float* at = segments.states + (int64_t)seq * segments.count * all + x;
+    for (int s = 0; s < live; ++s, at += all) {
+        const float own = s + 1 < live ? *at : 0.0f;
+        *at = S;
+        S = fmaf(power, S, own);
     }
 }
 
@@ -481,23 +521,49 @@ static inline size_t smem_bytes(int d, int vt) {
     return (size_t)(2 * C * (dp + 4) + C * (vt + 8) + C * (C + 4) + dp * (vt + 8)) * sizeof(float);
 }
 
+// The number of segments (1: none) for prompts of at most `max_new` tokens: enough blocks of 64 columns for two per
+// multiprocessor, segments of at least 128 tokens, at most 64 MB of states.
+static inline int segment_count(int n_seqs, int max_new, int H, int d, int vd) {
+    const int64_t blocks = (int64_t)H * n_seqs * ((vd + 63) / 64), bytes = (int64_t)n_seqs * H * d * vd * 4;
+    const int64_t want = (2 * (int64_t)q3_device_sm_count() + blocks - 1) / blocks;
+    int64_t count = want < max_new / 128 ? want : max_new / 128;
+    if (count > (64ll << 20) / bytes) count = (64ll << 20) / bytes;
+    return count < 2 ? 1 : (int)count;
+}
+
 template <typename T>
 int launch(const T* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots, float* out, int n_seqs, int H,
-           int d, int vd, const Input& in, cudaStream_t stream) {
+           int d, int vd, const Input& in, float* scratch, int max_new, int count, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     if (H <= 0 || d <= 0 || vd <= 0 || d > 256 || vd > 256 || d % 8 != 0 || vd % 8 != 0 || n_seqs > 65535) return Q3_ERR_BAD_SIZE;
     if (!aligned16(proj)) return Q3_ERR_MISALIGNED;
+    if (scratch == nullptr || count < 1) count = 1;
     // as many state columns a block as keep the multiprocessors busy: 64, or 32 / 16 while the blocks are too few (measured on
-    // one prompt of 2,048 tokens with 16 heads of 128 x 128: 1.03 ms with 64 columns, 0.77 with 32, 0.63 with 16, 0.76 with 8)
+    // one prompt of 2,048 tokens with 16 heads of 128 x 128 in one walk: 1.03 ms with 64 columns, 0.77 with 32, 0.63 with 16,
+    // 0.76 with 8)
     int vt = min(vd, 64);
-    while (vt > 16 && vt % 16 == 0 && (int64_t)H * n_seqs * ((vd + vt - 1) / vt) < q3_device_sm_count()) vt /= 2;
+    while (vt > 16 && vt % 16 == 0 && (int64_t)H * n_seqs * count * ((vd + vt - 1) / vt) < q3_device_sm_count()) vt /= 2;
     const size_t smem = smem_bytes(d, vt);
     if (smem > 200 * 1024) return Q3_ERR_BAD_SIZE;
-    static Q3PerDevice allowed;
-    const cudaError_t e = q3_allow_shared_memory(lightning_chunks_tc_kernel<T>, 200 * 1024, allowed);
-    if (e != cudaSuccess) return (int)e;
-    return (int)q3_launch(lightning_chunks_tc_kernel<T>, dim3(H, n_seqs, (vd + vt - 1) / vt), dim3(256), smem, stream, proj, state, decay,
-                          seq_start, seq_slots, out, H, d, vd, vt, in);
+    const int tiles = (vd + vt - 1) / vt;
+    static Q3PerDevice allowed[3];
+    auto walk = [&](auto kernel, Q3PerDevice& done, int segs, const Segments& segments) {
+        const cudaError_t e = q3_allow_shared_memory(kernel, 200 * 1024, done);
+        if (e != cudaSuccess) return (int)e;
+        return (int)q3_launch(kernel, dim3(H, n_seqs, tiles * segs), dim3(256), smem, stream, proj, state, decay, seq_start, seq_slots, out, H,
+                              d, vd, vt, in, segments);
+    };
+    if (count == 1) return walk(lightning_chunks_tc_kernel<T, WHOLE>, allowed[0], 1, Segments{nullptr, 0, 1});
+    const int length = ((max_new + count - 1) / count + C - 1) / C * C;
+    const Segments segments = {scratch, length, count};
+    if ((int64_t)length * count < max_new || tiles * count > 65535) return Q3_ERR_BAD_SIZE;
+    int code = walk(lightning_chunks_tc_kernel<T, STATES>, allowed[1], count - 1, segments);
+    if (code != 0) return code;
+    const int64_t all = (int64_t)H * d * vd;
+    code = (int)q3_launch(segment_starts_kernel, dim3((unsigned)((all + 255) / 256), n_seqs), dim3(256), 0, stream, (const float*)state, decay,
+                          seq_start, seq_slots, in.slot_stride, H, d * vd, segments);
+    if (code != 0) return code;
+    return walk(lightning_chunks_tc_kernel<T, OUTPUTS>, allowed[2], count, segments);
 }
 }  // namespace tc
 
@@ -558,10 +624,16 @@ static inline bool input_fits(const Input& in, int d) {
 Q3_EXPORT int q3_lightning_chunks_tc_bf16(const void* proj, float* state, const float* decay, const int* seq_start,
                                           const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale,
                                           const float* cos_tab, const float* sin_tab, int rot, const int* token_pos,
-                                          int64_t slot_stride, void* stream) {
+                                          int64_t slot_stride, float* scratch, int max_new, int segments, void* stream) {
     const Input in = {silu, k_scale, cos_tab, sin_tab, rot, token_pos, slot_stride};
     if (!input_fits(in, d)) return Q3_ERR_BAD_SIZE;
-    return tc::launch<bf16>((const bf16*)proj, state, decay, seq_start, seq_slots, out, n_seqs, heads, d, vd, in, (cudaStream_t)stream);
+    return tc::launch<bf16>((const bf16*)proj, state, decay, seq_start, seq_slots, out, n_seqs, heads, d, vd, in, scratch, max_new, segments,
+                            (cudaStream_t)stream);
+}
+// How many segments a step of prompts is cut into (1: none); `scratch` holds n_seqs * segments * heads * d * vd float32.
+Q3_EXPORT int q3_lightning_segments(int n_seqs, int max_new, int heads, int d, int vd) {
+    if (n_seqs <= 0 || max_new <= 0 || heads <= 0 || d <= 0 || vd <= 0) return 1;
+    return tc::segment_count(n_seqs, max_new, heads, d, vd);
 }
 
 Q3_LIGHTNING_EXPORTS(f32, float)

@@ -646,13 +646,16 @@ def hyper_norm(streams: torch.Tensor, n_streams: int, branch: Optional[torch.Ten
 def lightning_attention(proj: torch.Tensor, state: torch.Tensor, decay: torch.Tensor, seq_start: torch.Tensor,
                         seq_slots: torch.Tensor, out: torch.Tensor, n_seqs: int, heads: int, d: int, vd: int,
                         chunked: bool = False, silu: bool = True, k_scale: float = 1.0, cos: Optional[torch.Tensor] = None,
-                        sin: Optional[torch.Tensor] = None, token_pos: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        sin: Optional[torch.Tensor] = None, token_pos: Optional[torch.Tensor] = None,
+                        scratch: Optional[torch.Tensor] = None, max_new: int = 0, segments: int = 1) -> torch.Tensor:
     """S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t over the new tokens of every sequence, from and to the state rows
     [slot, heads, d, vd] (float32).  `proj` [N, 2 heads d + 2 heads vd] holds q, k, v (SiLU is applied here) and a gate
     that is not read; `out` [N, heads * vd] float32.  `chunked`: the form for prompts (32 tokens at a time).
     Retention: `silu=False` (q, k, v as projected), the first 2 * tables' width values of every head of q and k rotated by
     `token_pos` in pairs (i, i + width) with the tables `cos`, `sin` [positions, width], k multiplied by `k_scale`; `state` may
-    also be a view [slots, heads * d * vd] of wider rows."""
+    also be a view [slots, heads * d * vd] of wider rows.  `segments` > 1 (see `lightning_segments`; `chunked`, bfloat16): prompts
+    of up to `max_new` tokens are cut into so many stretches that run side by side, with `scratch` (float32,
+    n_seqs * segments * heads * d * vd) for the states between them."""
     if proj.shape[1] != 2 * heads * (d + vd) or tuple(state.shape[1:]) not in ((heads, d, vd), (heads * d * vd,)) or out.shape[1] != heads * vd \
             or out.dtype != torch.float32 or decay.numel() != heads or state.dtype != torch.float32 or not state[0].is_contiguous() \
             or (cos is not None and token_pos is None):
@@ -661,15 +664,30 @@ def lightning_attention(proj: torch.Tensor, state: torch.Tensor, decay: torch.Te
     name = "chunks" if chunked else "scan"
     if chunked and proj.dtype == torch.bfloat16 and lightning_tensor_cores and lightning_chunks_tc_fit(d, vd):
         name = "chunks_tc"                                   # the chunks' products on the tensor cores (TF32 hi + lo operands)
-    fn = _fn("lightning.cu", f"q3_lightning_{name}_{_suffix(proj)}", [c_void_p] * 6 + [c_int] * 5 + [c_float, c_void_p, c_void_p, c_int, c_void_p, c_int64, c_void_p])
+    tail, more = [], []
+    if name == "chunks_tc":
+        if segments > 1 and (scratch is None or scratch.numel() < n_seqs * segments * heads * d * vd or max_new <= 0):
+            raise KernelError("lightning_attention: segments need a scratch for the states between them")
+        tail, more = [c_void_p, c_int, c_int], [_ptr(scratch, "scratch", torch.float32) if segments > 1 else None, int(max_new), int(segments)]
+    fn = _fn("lightning.cu", f"q3_lightning_{name}_{_suffix(proj)}",
+             [c_void_p] * 6 + [c_int] * 5 + [c_float, c_void_p, c_void_p, c_int, c_void_p, c_int64] + tail + [c_void_p])
     _check(fn(_dev(proj, "proj"), state.data_ptr(), _dev(decay, "decay", torch.float32),
               _dev(seq_start, "seq_start", torch.int32), _dev(seq_slots, "seq_slots", torch.int32), _dev(out, "out"),
               int(n_seqs), heads, d, vd, int(bool(silu)), float(k_scale), _ptr(cos, "cos", torch.float32), _ptr(sin, "sin", torch.float32),
-              rot, _ptr(token_pos, "token_pos", torch.int32), state.stride(0), _stream()), f"lightning_{name}")
+              rot, _ptr(token_pos, "token_pos", torch.int32), state.stride(0), *more, _stream()), f"lightning_{name}")
+    if name == "chunks_tc" and segments > 1:
+        _count_extra(2)
     return out
 
 
 lightning_tensor_cores = True      # tests switch it off to run the fmaf form of the chunks in bfloat16
+
+
+def lightning_segments(dtype, n_seqs: int, max_new: int, heads: int, d: int, vd: int) -> int:
+    """Into how many segments `lightning_attention` best cuts a step of prompts (1: none; the tensor-core form only)."""
+    if dtype != torch.bfloat16 or not lightning_tensor_cores or not lightning_chunks_tc_fit(d, vd):
+        return 1
+    return int(_fn_untimed("lightning.cu", "q3_lightning_segments", [c_int] * 5)(int(n_seqs), int(max_new), heads, d, vd))
 
 
 def lightning_chunks_tc_fit(d: int, vd: int) -> bool:

@@ -265,7 +265,11 @@ int q3_lightning_chunks_bf16(const void* proj, float* state, const float* decay,
 /* the chunks' products on the tensor cores (operands as TF32 hi + lo terms): head sizes in steps of 8 */
 int q3_lightning_chunks_tc_bf16(const void* proj, float* state, const float* decay, const int* seq_start, const int* seq_slots,
                                 float* out, int n_seqs, int heads, int d, int vd, int silu, float k_scale, const float* cos_tab,
-                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, void* stream);
+                          const float* sin_tab, int rot, const int* token_pos, int64_t slot_stride, float* scratch, int max_new,
+                          int segments, void* stream);
+/* how many segments long prompts of few sequences are cut into, which run side by side (1: none); scratch (may be null: one
+   walk) then holds n_seqs * segments * heads * d * vd float32, max_new is the most new tokens of a sequence */
+int q3_lightning_segments(int n_seqs, int max_new, int heads, int d, int vd);
 /* out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate), row by row; gate rows are gate_stride apart */
 int q3_gated_norm_f32(const float* o, const void* gate, int64_t gate_stride, const float* w, float eps, void* out,
                       int64_t n_tokens, int size, void* stream);

@@ -27,6 +27,15 @@ TENSOR_NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "norm": "norm"
 chunk_rows = 16      # from this many new tokens of the longest sequence on, the chunked form runs
 
 
+def segment_scratch(ctx, heads: int, d: int, vd: int, chunked: bool) -> dict:
+    """The arguments with which `ops.lightning_attention` walks long prompts in segments side by side, where that pays."""
+    segments = ops.lightning_segments(ctx.dtype, ctx.n_seqs, ctx.max_new, heads, d, vd) if chunked else 1
+    if segments == 1:
+        return {}
+    return {"scratch": ctx.scratch.get("lightning.segments", (ctx.n_seqs * segments * heads * d * vd,), torch.float32),
+            "max_new": ctx.max_new, "segments": segments}
+
+
 class LightningAttention(Part):
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, value_dim: int, decay: Sequence[float], eps: float,
                  prefix: str = "", names: Optional[dict] = None):
@@ -61,7 +70,8 @@ class LightningAttention(Part):
         linear(x, self.w_in, proj)
         o = ctx.scratch.get("lightning.o", (N, h * vd), torch.float32)
         chunked = not ctx.is_decode and ctx.max_new >= chunk_rows and ops.lightning_chunks_fit(d, vd)
-        ops.lightning_attention(proj, cache.state, self.decay, ctx.seq_start, ctx.seq_slots, o, ctx.n_seqs, h, d, vd, chunked)
+        ops.lightning_attention(proj, cache.state, self.decay, ctx.seq_start, ctx.seq_slots, o, ctx.n_seqs, h, d, vd, chunked,
+                                **segment_scratch(ctx, h, d, vd, chunked))
         gated = ctx.scratch.get("lightning.gated", (N, h * vd), ctx.dtype)
         ops.gated_norm(o, proj[:, 2 * h * d + h * vd:], self.norm_weight, self.eps, gated)
         out = ctx.scratch.get("mixer.out", (N, self.hidden_size), ctx.dtype)

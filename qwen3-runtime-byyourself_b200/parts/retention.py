@@ -71,7 +71,8 @@ class Retention(Part):
         o = ctx.scratch.get("retention.o", (N, h * vd), torch.float32)
         chunked = not ctx.is_decode and ctx.max_new >= lightning.chunk_rows and ops.lightning_chunks_fit(d, vd)
         ops.lightning_attention(proj, cache.state, self.decay, ctx.seq_start, ctx.seq_slots, o, ctx.n_seqs, h, d, vd, chunked,
-                                silu=False, k_scale=self.k_scale, cos=cos, sin=sin, token_pos=ctx.token_pos)
+                                silu=False, k_scale=self.k_scale, cos=cos, sin=sin, token_pos=ctx.token_pos,
+                                **lightning.segment_scratch(ctx, h, d, vd, chunked))
         gated = ctx.scratch.get("retention.gated", (N, h * vd), ctx.dtype)
         ops.head_gated_norm(o, None, proj[:, 2 * h * d + h * vd:], self.eps, gated, h, vd, act="silu")
         out = ctx.scratch.get(self.out_name, (N, self.hidden_size), ctx.dtype)

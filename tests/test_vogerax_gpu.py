@@ -226,6 +226,46 @@ def test_retention_over_unequal_sequences_and_from_its_state(dtype, heads, d, vd
     assert np.all(final[:, :before] == 7.0) and np.all(final[:, -after:] == -7.0) and np.all(final[[1, 3, 6, 7], before:-after] == 0.0)
 
 
+@pytest.mark.parametrize("heads,d,vd,dims,silu", [(2, 16, 24, 8, False), (1, 64, 128, 64, False), (3, 128, 64, 0, True)])
+@pytest.mark.parametrize("segments", [None, 2, 3, 7])
+def test_long_prompts_walked_in_segments_side_by_side(heads, d, vd, dims, silu, segments):
+    """The same numbers as one walk, whatever the number of segments: prompts that fill every segment, that end inside one and
+    that lie in the first alone; from states that are not zero, twice in a row."""
+    import torch
+    from qwen3_b200.csrc import ops
+    rng = np.random.default_rng(d + vd)
+    T, decay = torch.bfloat16, dev(np.array([0.999, 0.9, 0.0])[:heads], torch.float32)
+    angle = np.arange(2000)[:, None] * plain.plain_frequencies(90.0, dims)[None, :] if dims else None
+    kw = dict(silu=silu, k_scale=d ** -0.5)
+    if dims:
+        kw.update(cos=dev(np.cos(angle), torch.float32), sin=dev(np.sin(angle), torch.float32))
+    first = dev(rng.standard_normal((6, heads * d * vd)), torch.float32)
+    states, outs = [first.clone(), first.clone()], []
+    at = {s: 0 for s in (4, 0, 2)}
+    for lengths in ([700, 1, 200], [131, 640, 32]):
+        start, _ = packed(lengths)
+        N = int(start[-1])
+        pos = np.concatenate([np.arange(at[s], at[s] + n) for s, n in zip((4, 0, 2), lengths)])
+        proj = dev(rng.standard_normal((N, 2 * heads * (d + vd))) * 0.7, T)
+        count = segments or ops.lightning_segments(T, 3, max(lengths), heads, d, vd)
+        assert segments or count > 1
+        scratch = torch.full((3 * count * heads * d * vd,), 9.0, dtype=torch.float32, device="cuda")
+        got = []
+        for state, more in zip(states, (dict(), dict(scratch=scratch, max_new=max(lengths), segments=count))):
+            out = torch.full((N, heads * vd), 9.0, dtype=torch.float32, device="cuda")
+            ops.lightning_attention(proj, state, decay, dev(start, torch.int32), dev([4, 0, 2], torch.int32), out, 3, heads, d, vd, True,
+                                    token_pos=dev(pos, torch.int32), **kw, **more)
+            got.append(f64(out))
+        assert np.allclose(got[0], got[1], rtol=1e-4, atol=1e-4)
+        assert np.allclose(f64(states[0]), f64(states[1]), rtol=1e-4, atol=1e-4)
+        for s, n in zip((4, 0, 2), lengths):
+            at[s] += n
+    assert np.array_equal(f64(states[1])[[1, 3, 5]], f64(first)[[1, 3, 5]])
+    with pytest.raises(ops.KernelError, match="segments"):
+        ops.lightning_attention(proj, states[0], decay, dev(start, torch.int32), dev([4, 0, 2], torch.int32), out, 3, heads, d, vd, True,
+                                token_pos=dev(pos, torch.int32), segments=2, **kw)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_retention_s_heads_are_normed_without_a_weight_and_gated(dtype):
     import torch
