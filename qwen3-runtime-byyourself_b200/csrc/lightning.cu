@@ -509,10 +509,15 @@ __global__ void segment_starts_kernel(const float* __restrict__ state, const flo
     const float lam = decay[x / per_head], power = lam > 0.0f ? exp2f((float)segments.length * log2f(lam)) : 0.0f;
     float S = state[(int64_t)seq_slots[seq] * slot_stride + x];
     float* at = segments.states + (int64_t)seq * segments.count * all + x;
-    for (int s = 0; s < live; ++s, at += all) {
-        const float own = s + 1 < live ? *at : 0.0f;
-        *at = S;
-        S = fmaf(power, S, own);
+    for (int s0 = 0; s0 < live; s0 += 8, at += 8 * all) {
+        float own[8];                                    // eight loads on their way together
+#pragma unroll
+        for (int i = 0; i < 8; ++i) own[i] = s0 + i + 1 < live ? at[i * all] : 0.0f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            if (s0 + i < live) at[i * all] = S;
+            S = fmaf(power, S, own[i]);
+        }
     }
 }
 

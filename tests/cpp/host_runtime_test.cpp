@@ -39,6 +39,26 @@ static std::vector<int> held_pages(const qwen3::CacheBook& book, int group, int 
 
 int main() {
     using namespace qwen3;
+    {   // pooled blocks: one entry a whole block, kept for as long as the sequence lives; a spare page of each group's own
+        CacheBook book({GroupNeed{GroupKind::Window, 9, 0}, GroupNeed{GroupKind::Pooled, 3, 0}}, 9 * 64, 9 * 64, 2);
+        CHECK(book.group(0).n_pages() == 9 && book.group(1).n_pages() == 5);
+        const int a = book.alloc_slot();
+        int slots[1] = {a};
+        for (int64_t n : {2, 1, 190, 1, 200}) {
+            int64_t n_new[1] = {n};
+            book.reserve(slots, n_new, 1);
+            book.commit(slots, n_new, 1);
+            CHECK((int64_t)held_pages(book, 1, a).size() == (book.length(a) / 3 + 63) / 64);
+        }
+        CHECK(held_pages(book, 0, a).size() == 2 && held_pages(book, 1, a).size() == 3);
+        const StepLayout lay(2, 2, 2, 2, book.pages_per_slot());
+        std::vector<int32_t> meta(lay.total, -7);
+        const int32_t ids[1] = {5};
+        pack_decode_step(book, lay, 2, slots, 1, ids, meta.data());
+        CHECK(meta[lay.tables[0] + book.pages_per_slot()] == 9 && meta[lay.tables[1] + book.pages_per_slot()] == 5);
+        book.free_slot(a);
+        CHECK(book.group(0).n_free() == 9 && book.group(1).n_free() == 5);
+    }
     {   // lengths, pages, reuse, all-or-nothing reservation, cancel
         CacheBook book({GroupNeed{}}, 5 * 64, 4 * 64);
         CHECK(book.n_pages() == 5 && book.pages_per_slot() == 4 && book.n_slots() == 5);
