@@ -50,7 +50,7 @@ int main() {
             book.commit(slots, n_new, 1);
             CHECK((int64_t)held_pages(book, 1, a).size() == (book.length(a) / 3 + 63) / 64);
         }
-        CHECK(held_pages(book, 0, a).size() == 2 && held_pages(book, 1, a).size() == 3);
+        CHECK(held_pages(book, 0, a).size() == 1 && held_pages(book, 1, a).size() == 3);
         const StepLayout lay(2, 2, 2, 2, book.pages_per_slot());
         std::vector<int32_t> meta(lay.total, -7);
         const int32_t ids[1] = {5};
