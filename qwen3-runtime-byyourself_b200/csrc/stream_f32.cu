@@ -212,11 +212,26 @@ int sandwich_norm_launch(float* stream, const T* branch, const float* w_post, co
 }
 
 // ---------------------------------------------------------------- two normed branches in one sum
+// Two sums over a block at once; `scratch` holds 66 floats.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = (blockDim.x + 31) >> 5;
+    a = warp_sum(a);
+    b = warp_sum(b);
+    if (lane == 0) {
+        scratch[warp] = a;
+        scratch[33 + warp] = b;
+    }
+    __syncthreads();
+    a = warp_sum(lane < n_warps ? scratch[lane] : 0.0f);        // every warp adds them up for itself
+    b = warp_sum(lane < n_warps ? scratch[33 + lane] : 0.0f);
+    return make_float2(a, b);
+}
+
 // One block per row.  PER > 0: a thread keeps PER groups of four values of both rows in registers.
 template <typename T, int PER>
 __global__ void normed_sum_kernel(const T* __restrict__ a, const T* __restrict__ b, const float* __restrict__ w_a,
                                   const float* __restrict__ w_b, float s_a, float s_b, float eps, T* __restrict__ out, int size) {
-    __shared__ float scratch[33];
+    __shared__ float scratch[66];
     pdl_launch_dependents();
     pdl_wait();
     const T* ar = a + (int64_t)blockIdx.x * size;
@@ -238,7 +253,8 @@ __global__ void normed_sum_kernel(const T* __restrict__ a, const T* __restrict__
                 }
             }
         }
-        const float inv_a = s_a * rsqrtf(block_sum(sq_a, scratch) / (float)size + eps), inv_b = s_b * rsqrtf(block_sum(sq_b, scratch) / (float)size + eps);
+        const float2 sums = block_sum2(sq_a, sq_b, scratch);
+        const float inv_a = s_a * rsqrtf(sums.x / (float)size + eps), inv_b = s_b * rsqrtf(sums.y / (float)size + eps);
 #pragma unroll
         for (int p = 0; p < PER; ++p) {
             const int c = (p * blockDim.x + threadIdx.x) * 4;
@@ -257,7 +273,8 @@ __global__ void normed_sum_kernel(const T* __restrict__ a, const T* __restrict__
             sq_a += x * x;
             sq_b += y * y;
         }
-        const float inv_a = s_a * rsqrtf(block_sum(sq_a, scratch) / (float)size + eps), inv_b = s_b * rsqrtf(block_sum(sq_b, scratch) / (float)size + eps);
+        const float2 sums = block_sum2(sq_a, sq_b, scratch);
+        const float inv_a = s_a * rsqrtf(sums.x / (float)size + eps), inv_b = s_b * rsqrtf(sums.y / (float)size + eps);
         for (int c = threadIdx.x; c < size; c += blockDim.x)
             outr[c] = from_f32<T>(to_f32<T>(ar[c]) * inv_a * w_a[c] + to_f32<T>(br[c]) * inv_b * w_b[c]);
     }
