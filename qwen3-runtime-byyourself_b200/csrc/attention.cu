@@ -21,6 +21,10 @@
 // blocks beside a window: every block of `size` tokens that lies wholly before a query's window is seen as one key and
 // one value, the means of the block's cached keys and values, which `pool_blocks` makes when a block is complete.
 //
+// Further still: queries multiplied by a temperature of their position, 1 + coef ln(floor((p + 1) / every) + 1), after
+// their norm; and a bias added to every scaled score by the distance between query and key, one number per head and
+// distance up to a last one that stands for all that are further.
+//
 // Cache layout: pages [page, kv head, PAGE tokens, head_dim]; `page_table[seq]` lists
 // the pages of a sequence in order.  Keys are visited page by page in ascending
 // position, so the result for one (position, head) does not depend on how the tokens
@@ -55,6 +59,18 @@ struct PrepareOptions {
     int norm_once;          // a normed value is rounded once, when it is stored (else after the division and the weight too)
     const float* v_cos;     // [positions, vd / 2] or null: values are rotated by their position, over the whole head
     const float* v_sin;
+    float temp_coef;        // queries are multiplied by 1 + temp_coef ln((pos + 1) / temp_every + 1), a whole quotient (0: by nothing)
+    int temp_every;
+};
+
+__device__ __forceinline__ float query_temperature(const PrepareOptions& opt, int pos) {
+    return 1.0f + opt.temp_coef * logf((float)((pos + 1) / opt.temp_every + 1));
+}
+
+// Biases by distance: table [query heads][count], the last column for every distance from count - 1 on (null: none).
+struct DistanceBias {
+    const float* table;
+    int count;
 };
 
 template <typename T>
@@ -149,6 +165,18 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ qkv, T* __restrict__ q_
             }
         }
     }
+    if (opt.temp_coef != 0.0f && head < nq) {
+        const float temp = query_temperature(opt, pos);
+#pragma unroll
+        for (int n = 0; n < MAX_HEAD_DIM / 64; ++n) {
+            a[n] *= temp;
+            b[n] *= temp;
+        }
+        if (rot < d) {
+#pragma unroll
+            for (int n = 0; n < MAX_HEAD_DIM / 32; ++n) c[n] *= temp;
+        }
+    }
 #pragma unroll
     for (int n = 0; n < MAX_HEAD_DIM / 64; ++n) {
         const int i = lane + 32 * n;
@@ -189,7 +217,7 @@ __global__ void qkv_prepare_vec_kernel(const T* __restrict__ qkv, T* __restrict_
     pdl_wait();
     const int lph = (d >> 1) / VEC, hpw = 32 / lph;                   // lanes per head, heads per warp
     const int lane = threadIdx.x & 31, sub = lane % lph, grp = lane / lph;
-    const int heads = nq + 2 * nkv;
+    const int heads = write_kv ? nq + 2 * nkv : nq;
     const int64_t warp = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int64_t pair = warp * hpw + grp;                             // flat (token, head) index
     const bool active = grp < hpw && pair < n_tokens * heads;
@@ -238,6 +266,14 @@ __global__ void qkv_prepare_vec_kernel(const T* __restrict__ qkv, T* __restrict_
         }
     }
     if (!live) return;
+    if (opt.temp_coef != 0.0f && is_q) {
+        const float temp = query_temperature(opt, pos);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            a[i] *= temp;
+            b[i] *= temp;
+        }
+    }
     if (rotate) {
         const float* c = cs_tab + (int64_t)pos * rhalf + a_at;
         const float* sn = sn_tab + (int64_t)pos * rhalf + a_at;
@@ -309,7 +345,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
                          T* __restrict__ out, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                          const int* __restrict__ page_table, int pages_per_seq, int nq, int nkv, int d, float scale,
                          int window, int vd, float softcap, int chunk, int sink, int nv, int out_f32,
-                         const float* __restrict__ sink_values, int keep_first, const PoolView<T> pool) {
+                         const float* __restrict__ sink_values, int keep_first, const PoolView<T> pool, const DistanceBias bias) {
     __shared__ float q_s[GENERIC_KEY_DIM];
     __shared__ float score[PAGE];
     __shared__ float prob[PAGE];
@@ -353,6 +389,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
             }
             dot = warp_sum(dot) * scale;
             if (softcap > 0.0f) dot = softcap * tanhf(dot * inv_cap);
+            if (bias.table != nullptr) dot += bias.table[(int64_t)head * bias.count + min(max(pos - pg * PAGE - j, 0), bias.count - 1)];
             if (lane == 0) score[j] = (j >= j_lo && j <= j_hi && !(j >= gap_lo && j < gap_hi)) ? dot : -INFINITY;
         }
         __syncthreads();
@@ -401,16 +438,18 @@ int qkv_prepare_launch(const T* qkv, T* q_out, T* k_pages, T* v_pages, const flo
     if (rot % 2 != 0) rot = 0;                   // an odd head without tables: every value passes through
     if (vd <= 0) vd = d;                         // values as wide as keys
     if (vd > MAX_HEAD_DIM) return Q3_ERR_BAD_SIZE;
-    const int64_t columns = (int64_t)(nq + nkv) * d + (opt.tied ? 0 : (int64_t)nv * vd);
+    // a projection of the queries alone is enough when no key is written
+    const int64_t columns = write_kv ? (int64_t)(nq + nkv) * d + (opt.tied ? 0 : (int64_t)nv * vd) : (int64_t)nq * d;
+    if (opt.temp_coef != 0.0f && opt.temp_every <= 0) return Q3_ERR_BAD_SIZE;
     if (opt.row <= 0) opt.row = columns;
     if (opt.row < columns || (opt.tied && (vd != d || nv != nkv)) || (opt.v_cos == nullptr) != (opt.v_sin == nullptr) ||
         (opt.v_cos != nullptr && vd % 2 != 0))
         return Q3_ERR_BAD_SIZE;
     constexpr int VEC = Pack<T>::N;
-    if ((rot / 2) % VEC == 0 && (d - rot) % (2 * VEC) == 0 && rot % 2 == 0 && vd == d && nv == nkv && n_tokens >= 64 && (d / 2) % VEC == 0 &&
+    if ((rot / 2) % VEC == 0 && (d - rot) % (2 * VEC) == 0 && rot % 2 == 0 && ((vd == d && nv == nkv) || !write_kv) && n_tokens >= 64 && (d / 2) % VEC == 0 &&
         (d / 2) / VEC <= 32 && opt.row % VEC == 0 && aligned16(qkv) && aligned16(q_out) && aligned16(k_pages) && aligned16(v_pages)) {
         const int hpw = 32 / ((d / 2) / VEC);
-        const int64_t n_warps = (n_tokens * (nq + 2 * nkv) + hpw - 1) / hpw;
+        const int64_t n_warps = (n_tokens * (write_kv ? nq + 2 * nkv : nq) + hpw - 1) / hpw;
         const int64_t blocks = (n_warps + 7) / 8;
         if (blocks > 0x7fffffffLL) return Q3_ERR_TOO_LARGE;
         return (int)q3_launch(qkv_prepare_vec_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, qkv, q_out, k_pages,
@@ -419,7 +458,7 @@ int qkv_prepare_launch(const T* qkv, T* q_out, T* k_pages, T* v_pages, const flo
     }
     if (n_tokens > 65535) return Q3_ERR_TOO_LARGE;
     const int warps = 4;
-    const dim3 grid((nq + nkv + nv + warps - 1) / warps, (unsigned)n_tokens);
+    const dim3 grid(((write_kv ? nq + nkv + nv : nq) + warps - 1) / warps, (unsigned)n_tokens);
     return (int)q3_launch(qkv_prepare_kernel<T>, grid, dim3(warps * 32), 0, stream, qkv, q_out, k_pages, v_pages, q_norm_w,
                           k_norm_w, cos_tab, sin_tab, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, d, eps, write_kv, rot,
                           bias, vd, nv, opt);
@@ -429,8 +468,9 @@ template <typename T>
 int attention_generic_launch(const T* q, const T* k_pages, const T* v_pages, T* out, const int* token_seq,
                              const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq,
                              int nkv, int d, float scale, int window, int vd, float softcap, int chunk, int sink, int nv,
-                             int out_f32, const float* sink_values, int keep_first, PoolView<T> pool, cudaStream_t stream) {
+                             int out_f32, const float* sink_values, int keep_first, PoolView<T> pool, DistanceBias bias, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (bias.table != nullptr && (bias.count <= 0 || pool.size > 0)) return Q3_ERR_BAD_SIZE;
     if (pool.size < 0 || (pool.size > 0 && (window <= 0 || keep_first > 0 || pool.k == nullptr || pool.v == nullptr || pool.table == nullptr)))
         return Q3_ERR_BAD_SIZE;
     if (vd <= 0) vd = d;
@@ -442,7 +482,7 @@ int attention_generic_launch(const T* q, const T* k_pages, const T* v_pages, T* 
     const dim3 grid(nq, (unsigned)n_tokens);
     return (int)q3_launch(attention_generic_kernel<T>, grid, dim3(128), 0, stream, q, k_pages, v_pages, out, token_seq,
                           token_pos, page_table, pages_per_seq, nq, nkv, d, scale, window, vd, softcap, chunk, sink, nv, out_f32, sink_values,
-                          keep_first, pool);
+                          keep_first, pool, bias);
 }
 
 template <typename T>
@@ -586,8 +626,9 @@ int launch_flat(Kernel kernel, int64_t work, cudaStream_t stream, Args... args) 
                                           int nkv, int d, float eps, int write_kv, int rotary_dim,           \
                                           const float* bias, int value_dim, int value_heads, int64_t row,             \
                                           int tied_values, int norm_once, const float* v_cos, const float* v_sin,     \
-                                          void* stream) {                                                             \
+                                          float temp_coef, int temp_every, void* stream) {                            \
         PrepareOptions opt;                                                                                           \
+        opt.temp_coef = temp_coef; opt.temp_every = temp_every;                                                       \
         opt.row = row; opt.tied = tied_values; opt.norm_once = norm_once; opt.v_cos = v_cos; opt.v_sin = v_sin;       \
         return qkv_prepare_launch<T>((const T*)qkv, (T*)q_out, (T*)k_pages, (T*)v_pages, q_norm_w, k_norm_w, cos_tab, \
                                      sin_tab, token_seq, token_pos, page_table, pages_per_seq, n_tokens, nq, nkv, d,  \
@@ -621,12 +662,12 @@ int launch_flat(Kernel kernel, int64_t work, cudaStream_t stream, Args... args) 
                                                 int chunk, int sink, int value_heads, int out_f32,                   \
                                                 const float* sink_values, int keep_first, const void* pool_k,         \
                                                 const void* pool_v, const int* pool_table, int pool_size,             \
-                                                void* stream) {                                                       \
+                                                const float* bias, int bias_count, void* stream) {                    \
         const PoolView<T> pool = {(const T*)pool_k, (const T*)pool_v, pool_table, pool_size};                         \
         return attention_generic_launch<T>((const T*)q, (const T*)k_pages, (const T*)v_pages, (T*)out, token_seq,     \
                                            token_pos, page_table, pages_per_seq, n_tokens, nq, nkv, d, scale, window, \
                                            value_dim, softcap, chunk, sink, value_heads, out_f32, sink_values,        \
-                                           keep_first, pool, (cudaStream_t)stream);                                   \
+                                           keep_first, pool, DistanceBias{bias, bias_count}, (cudaStream_t)stream);                                   \
     }                                                                                                                 \
     Q3_EXPORT int q3_value_mix_##SUFFIX(void* rows, int64_t row, int64_t v_off, int width, const float* bias,         \
                                         void* first, int save, float lambda, int64_t n_tokens, void* stream) {        \

@@ -10,6 +10,8 @@
 //                        ends before the window: block b = the tokens bP .. bP + P - 1 is seen from i if b < lo / P with
 //                        lo the window's first key; its key and value, the means of its tokens', lie in pages of
 //                        their own, which are walked before the window's
+//     and, with biases by distance, s_j = q.k_j * scale + table[head][min(i - j, count - 1)], one number per head and
+//                        distance, the last one for all that are further
 //     p_j = exp(s_j) / (sink + sum_visible exp(s_j)),  sink = 1 or 0
 //     o   = sum_j p_j v_j
 //
@@ -117,6 +119,13 @@ struct FinishArgs {
     int64_t gate_row;
 };
 
+// Biases by distance (null: none): table [query heads][count], natural units.  A page whose keys all lie count - 1 or more
+// before a row gets one number.
+struct BiasArgs {
+    const float* table;
+    int count;
+};
+
 template <typename TO> __device__ __forceinline__ void store_pair(TO* p, float a, float b);
 template <> __device__ __forceinline__ void store_pair<bf16>(bf16* p, float a, float b) {
     *reinterpret_cast<uint32_t*>(p) = pack_bf16(a, b);
@@ -140,12 +149,12 @@ constexpr int BM = 64;
 constexpr int K_TILE = PAGE * K_ROW, V_TILE = PAGE * V_ROW;
 constexpr int PREFILL_SMEM = 2 * (K_TILE + V_TILE);
 
-template <typename TO, bool POOL>
+template <typename TO, bool POOL, bool BIAS>
 __global__ void __launch_bounds__(WARPS * 32)
 prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                       TO* __restrict__ out, const int* __restrict__ seq_start, const int* __restrict__ seq_pos0,
                       const int* __restrict__ page_table, int pages_per_seq, int nq, int nkv, float scale, float cap, int chunk,
-                      int sink, int nv, const float* __restrict__ sink_values, int keep, const PoolArgs pool) {
+                      int sink, int nv, const float* __restrict__ sink_values, int keep, const PoolArgs pool, const BiasArgs bias) {
     extern __shared__ __align__(16) unsigned char smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -197,6 +206,8 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
     const int warp_last_start = chunk_start(warp_first_pos + 15, chunk);       // from here on every row of the warp may see
     const int warp_first_block = pooling ? warp_first_key / pool.size : 0, warp_last_block = pooling ? warp_last_start / pool.size : 0;
     const uint32_t base = smem_u32(smem);
+    const float* __restrict__ bias_row = BIAS ? bias.table + (int64_t)head * bias.count : nullptr;
+    const float bias_far = BIAS ? bias_row[bias.count - 1] * LOG2E : 0.0f;
 
     auto issue = [&](int i) {
         if (i < n_walk) {
@@ -241,11 +252,20 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
             // the entries of this page that each row sees: from .. to (and the kept keys)
             const int from_lo = blocks ? 0 : c_lo, from_hi = blocks ? 0 : c_hi, to_lo = blocks ? b_lo - 1 : p_lo, to_hi = blocks ? b_hi - 1 : p_hi;
             float mx[2] = {-INFINITY, -INFINITY};
+            const bool far = BIAS && warp_first_pos - (key_base + PAGE - 1) >= bias.count - 1;   // one bias for the whole page
 #pragma unroll
             for (int j = 0; j < 8; ++j)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     float v = score_log2(s[j][e], scale, cap, inv_cap);
+                    if constexpr (BIAS) {
+                        if (far) {
+                            v += bias_far;
+                        } else {
+                            const int back = ((e >> 1) ? p_hi : p_lo) - (key_base + j * 8 + tq * 2 + (e & 1));
+                            v = fmaf(__ldg(bias_row + min(max(back, 0), bias.count - 1)), LOG2E, v);
+                        }
+                    }
                     if (edge) {
                         const int key = key_base + j * 8 + tq * 2 + (e & 1);
                         const bool seen = (e >> 1) ? (key <= to_hi && (key >= from_hi || (!POOL && key < keep))) : (key <= to_lo && (key >= from_lo || (!POOL && key < keep)));
@@ -363,12 +383,12 @@ __device__ __forceinline__ void prepare_head(const bf16* __restrict__ src, const
 
 // part: [tokens, nq, splits, VD + 2] float32: the unnormalised sums, then the maximum (base-2 scale) and the denominator.
 // FUSED: `q` is unused; the pages are written by the block that holds the token's own page.
-template <bool FUSED, bool POOL>
+template <bool FUSED, bool POOL, bool BIAS>
 __global__ void __launch_bounds__(WARPS * 32)
 decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, const bf16* v_pages,
                            float* __restrict__ part, const int* __restrict__ token_seq, const int* __restrict__ token_pos,
                            const int* __restrict__ page_table, int pages_per_seq, int nq, int nkv, float scale, float cap,
-                           int chunk, const FusedArgs fused, int nv, int keep, const PoolArgs pool) {
+                           int chunk, const FusedArgs fused, int nv, int keep, const PoolArgs pool, const BiasArgs bias) {
     extern __shared__ __align__(16) unsigned char smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -489,6 +509,15 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
 #pragma unroll
     for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};   // rows quad and quad + 8
+    const float* bias_row[2] = {nullptr, nullptr};
+    float bias_far[2] = {0.0f, 0.0f};
+    if constexpr (BIAS) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            bias_row[r] = bias.table + (int64_t)(kvh * G + min(quad + 8 * r, G - 1)) * bias.count;
+            bias_far[r] = bias_row[r][bias.count - 1] * LOG2E;
+        }
+    }
 
     for (int i = 0; i < count; ++i) {
         cp_async_wait<STAGES - 2>();
@@ -514,7 +543,11 @@ decode_capped_split_kernel(const bf16* __restrict__ q, const bf16* k_pages, cons
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = key0 + j * 8 + (e & 1);
-                const float v = ((key >= seen_from || key < keep) && key <= seen_to) ? score_log2(s[j][e], scale, cap, inv_cap) : -INFINITY;
+                float v = ((key >= seen_from || key < keep) && key <= seen_to) ? score_log2(s[j][e], scale, cap, inv_cap) : -INFINITY;
+                if constexpr (BIAS) {
+                    const int back = pos - key;
+                    v += back >= bias.count - 1 ? bias_far[e >> 1] : __ldg(bias_row[e >> 1] + max(back, 0)) * LOG2E;
+                }
                 s[j][e] = v;
                 mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }
@@ -676,8 +709,11 @@ Q3_EXPORT int q3_attention_capped_prefill_bf16(const void* q, const void* k_page
                                                int pages_per_seq, int n_seqs, int max_new, int nq, int nkv, float scale,
                                                float softcap, int chunk, int sink, int window, int value_heads, int out_f32,
                                                const float* sink_values, int keep_first, const void* pool_k, const void* pool_v,
-                                               const int* pool_table, int pool_size, void* stream) {
+                                               const int* pool_table, int pool_size, const float* bias_table, int bias_count,
+                                               void* stream) {
     if (n_seqs <= 0 || max_new <= 0) return 0;
+    if (bias_table != nullptr && (bias_count <= 0 || pool_size > 0 || out_f32)) return Q3_ERR_BAD_SIZE;
+    const BiasArgs bias = {bias_table, bias_count};
     if (keep_first < 0 || (keep_first > 0 && window <= 0) || !pool_fits(pool_k, pool_v, pool_table, pool_size, window, keep_first))
         return Q3_ERR_BAD_SIZE;
     const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size, 0};
@@ -687,20 +723,21 @@ Q3_EXPORT int q3_attention_capped_prefill_bf16(const void* q, const void* k_page
         return Q3_ERR_BAD_SIZE;
     if (n_seqs > 65535 || nq > 65535) return Q3_ERR_TOO_LARGE;
     const int span = window > 0 ? -window : chunk;             // see chunk_start
-    static Q3PerDevice configured[4];
+    static Q3PerDevice configured[5];
     const dim3 grid((max_new + BM - 1) / BM, nq, n_seqs);
     auto launch = [&](auto kernel, auto* to, Q3PerDevice& state) {
         const cudaError_t e = q3_allow_shared_memory(kernel, PREFILL_SMEM, state);
         if (e != cudaSuccess) return (int)e;
         return (int)q3_launch(kernel, grid, dim3(WARPS * 32), PREFILL_SMEM, (cudaStream_t)stream, (const bf16*)q, (const bf16*)k_pages,
                               (const bf16*)v_pages, to, seq_start, seq_pos0, page_table, pages_per_seq, nq, nkv, scale, softcap, span,
-                              sink, value_heads, sink_values, keep_first, pool);
+                              sink, value_heads, sink_values, keep_first, pool, bias);
     };
+    if (bias_table != nullptr) return launch(prefill_capped_kernel<bf16, false, true>, (bf16*)out, configured[4]);
     if (pool_size > 0)
-        return out_f32 ? launch(prefill_capped_kernel<float, true>, (float*)out, configured[3])
-                       : launch(prefill_capped_kernel<bf16, true>, (bf16*)out, configured[2]);
-    return out_f32 ? launch(prefill_capped_kernel<float, false>, (float*)out, configured[1])
-                   : launch(prefill_capped_kernel<bf16, false>, (bf16*)out, configured[0]);
+        return out_f32 ? launch(prefill_capped_kernel<float, true, false>, (float*)out, configured[3])
+                       : launch(prefill_capped_kernel<bf16, true, false>, (bf16*)out, configured[2]);
+    return out_f32 ? launch(prefill_capped_kernel<float, false, false>, (float*)out, configured[1])
+                   : launch(prefill_capped_kernel<bf16, false, false>, (bf16*)out, configured[0]);
 }
 
 // One new token per sequence: scratch holds n_tokens * nq * n_splits * (VD + 2) float32.
@@ -710,8 +747,11 @@ Q3_EXPORT int q3_attention_capped_decode_bf16(const void* q, const void* k_pages
                                               int chunk, int sink, int n_splits, int window, int value_heads, int out_f32,
                                               const float* sink_values, int keep_first, const void* pool_k, const void* pool_v,
                                               const int* pool_table, int pool_size, int pool_write, const float* back_cos,
-                                              const float* back_sin, const void* gate, int64_t gate_row, void* stream) {
+                                              const float* back_sin, const void* gate, int64_t gate_row, const float* bias_table,
+                                              int bias_count, void* stream) {
     if (n_tokens <= 0) return 0;
+    if (bias_table != nullptr && (bias_count <= 0 || pool_size > 0)) return Q3_ERR_BAD_SIZE;
+    const BiasArgs bias = {bias_table, bias_count};
     if (keep_first < 0 || (keep_first > 0 && window <= 0) || !pool_fits(pool_k, pool_v, pool_table, pool_size, window, keep_first))
         return Q3_ERR_BAD_SIZE;
     const PoolArgs pool = {(const bf16*)pool_k, (const bf16*)pool_v, pool_table, pool_size, pool_write};
@@ -724,17 +764,18 @@ Q3_EXPORT int q3_attention_capped_decode_bf16(const void* q, const void* k_pages
         return Q3_ERR_BAD_SIZE;
     const int span = window > 0 ? -window : chunk;             // see chunk_start
     if (n_tokens > 65535 || nkv > 65535 || nq > 0x7fffffff / 2) return Q3_ERR_TOO_LARGE;
-    static Q3PerDevice configured[2];
+    static Q3PerDevice configured[3];
     const FusedArgs none = {};
     auto launch = [&](auto kernel, Q3PerDevice& state) {
         const cudaError_t e = q3_allow_shared_memory(kernel, DECODE_SMEM, state);
         if (e != cudaSuccess) return e;
         return q3_launch(kernel, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32), DECODE_SMEM, (cudaStream_t)stream, (const bf16*)q,
                          (const bf16*)k_pages, (const bf16*)v_pages, scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv,
-                         scale, softcap, span, none, value_heads, keep_first, pool);
+                         scale, softcap, span, none, value_heads, keep_first, pool, bias);
     };
-    const cudaError_t e = pool_size > 0 ? launch(decode_capped_split_kernel<false, true>, configured[1])
-                                        : launch(decode_capped_split_kernel<false, false>, configured[0]);
+    const cudaError_t e = bias_table != nullptr ? launch(decode_capped_split_kernel<false, false, true>, configured[2])
+                          : pool_size > 0       ? launch(decode_capped_split_kernel<false, true, false>, configured[1])
+                                                : launch(decode_capped_split_kernel<false, false, false>, configured[0]);
     if (e != cudaSuccess) return (int)e;
     if (out_f32)
         return (int)q3_launch(decode_capped_merge_kernel<float, false>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
@@ -757,15 +798,15 @@ Q3_EXPORT int q3_attention_capped_decode_fused_bf16(const void* qkv, void* k_pag
     if (n_tokens > 65535 || nkv > 65535 || nq > 0x7fffffff / 2) return Q3_ERR_TOO_LARGE;
     static Q3PerDevice configured;
     {
-        cudaError_t e = q3_allow_shared_memory(decode_capped_split_kernel<true, false>, DECODE_SMEM_FUSED, configured);
+        cudaError_t e = q3_allow_shared_memory(decode_capped_split_kernel<true, false, false>, DECODE_SMEM_FUSED, configured);
         if (e != cudaSuccess) return (int)e;
     }
     FusedArgs fused;
     fused.qkv = (const bf16*)qkv; fused.bias = bias; fused.cos_tab = cos_tab; fused.sin_tab = sin_tab;
     fused.rot = rotary_dim > 0 ? rotary_dim : D;
-    cudaError_t e = q3_launch(decode_capped_split_kernel<true, false>, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32),
+    cudaError_t e = q3_launch(decode_capped_split_kernel<true, false, false>, dim3(n_splits, nkv, (unsigned)n_tokens), dim3(WARPS * 32),
                               DECODE_SMEM_FUSED, (cudaStream_t)stream, (const bf16*)nullptr, (const bf16*)k_pages, (const bf16*)v_pages,
-                              scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, scale, softcap, chunk, fused, nkv, 0, PoolArgs{});
+                              scratch, token_seq, token_pos, page_table, pages_per_seq, nq, nkv, scale, softcap, chunk, fused, nkv, 0, PoolArgs{}, BiasArgs{});
     if (e != cudaSuccess) return (int)e;
     return (int)q3_launch(decode_capped_merge_kernel<bf16, false>, dim3(nq, (unsigned)n_tokens), dim3(VD >= 128 ? 128 : 64), 0,
                           (cudaStream_t)stream, (const float*)scratch, (bf16*)out, nq, n_splits, sink, (const float*)nullptr, FinishArgs{});

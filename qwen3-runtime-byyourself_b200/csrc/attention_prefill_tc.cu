@@ -28,6 +28,7 @@
 //   starts at 0 and the running sum at the sink's weight.  The softmax and its weights are computed in 32-bit and
 //   enter the second product as two bfloat16 terms, p = hi + lo with hi = bf16(p) and lo = bf16(p - hi) (TMEM
 //   columns [64,96) and [96,128), two sets of tcgen05.mma per page), so the product sees them to 16 bits of mantissa.
+//   -DQ3_CAPPED=2: with a sink and biases by distance instead of a cap or chunks; the biases are added to the scaled scores: one number a page for pages far enough back, else one a score.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -44,7 +45,7 @@
 
 namespace {
 
-constexpr bool CAPPED = Q3_CAPPED != 0;
+constexpr bool CAPPED = Q3_CAPPED != 0, BIAS = Q3_CAPPED == 2;
 // What the capped form needs beyond the plain one's arguments (all zero in the plain form).
 struct CapArgs {
     float scale;       // of the raw dot
@@ -52,6 +53,8 @@ struct CapArgs {
     int chunk;         // 0: every earlier key is seen
     int sink;          // 1: one more term exp(0) in the denominator
     const float* sink_values;   // one score per query head instead of that 0 (may be null)
+    const float* bias;          // biases by distance, [query heads][bias_count], the last one for all that is further (may be null;
+    int bias_count;             // not together with a cap)
 };
 
 constexpr int D = Q3_HEAD_DIM;
@@ -161,7 +164,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int rows = min(BM, n_new - tile * BM);
     // pages first_page .. the one of the last row (first_page: where the chunk of the tile's first row starts)
-    const int first_page = (CAPPED && capped.chunk > 0) ? ((pos0 + tile * BM) / capped.chunk * capped.chunk) / PAGE : 0;
+    const int first_page = (CAPPED && !BIAS && capped.chunk > 0) ? ((pos0 + tile * BM) / capped.chunk * capped.chunk) / PAGE : 0;
     const int n_pages = (pos0 + tile * BM + rows - 1) / PAGE + 1 - first_page;
 
     const uint32_t base = smem_u32(smem_raw);
@@ -287,11 +290,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         float m_run = -INFINITY, l_run = 0.0f;
         bool ok = true;
         // the capped form: the first key this row sees, and the constants of s -> cap * tanh(s * scale / cap) in log2 units
-        const int c_row = (CAPPED && capped.chunk > 0) ? p_row / capped.chunk * capped.chunk : 0;
-        const int c_last = (CAPPED && capped.chunk > 0) ? (pos0 + tile * BM + BM - 1) / capped.chunk * capped.chunk : 0;
+        const int c_row = (CAPPED && !BIAS && capped.chunk > 0) ? p_row / capped.chunk * capped.chunk : 0;
+        const int c_last = (CAPPED && !BIAS && capped.chunk > 0) ? (pos0 + tile * BM + BM - 1) / capped.chunk * capped.chunk : 0;
         const float cap_l2 = capped.cap * 1.4426950408889634f;                       // the cap in log2 units
         const float tanh_k = capped.cap > 0.0f ? 2.0f * capped.scale * 1.4426950408889634f / capped.cap : 0.0f;
         const float sink_score = CAPPED && capped.sink_values != nullptr ? capped.sink_values[head] * 1.4426950408889634f : 0.0f;
+        const float* __restrict__ bias_row = BIAS ? capped.bias + (int64_t)head * capped.bias_count : nullptr;
+        const float bias_last = BIAS ? bias_row[capped.bias_count - 1] * 1.4426950408889634f : 0.0f;
+        const float inv_scale = BIAS ? 1.0f / capped.scale : 0.0f;
         for (int j = 0; j < n_pages && ok; ++j) {
             ok = mbar_wait(bar_s_full, (uint32_t)j & 1u);
             if (!ok) { if (lane == 0) atomicExch(status, 15); break; }
@@ -311,6 +317,20 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 for (int c = 0; c < 64; ++c)
                     if (key0 + c > p_row || (CAPPED && key0 + c < c_row)) s[c] = 0xff800000u;                // -inf
             }
+            // biases by distance: far pages take one number after the scale; near ones a number per score, put into the
+            // raw dots in units of 1 / scale so that what follows does not change
+            float bias_far = 0.0f;
+            if constexpr (BIAS) {
+                if (pos0 + tile * BM - (key0 + PAGE - 1) >= capped.bias_count - 1) {
+                    bias_far = bias_last;
+                } else {
+#pragma unroll
+                    for (int c = 0; c < 64; ++c) {
+                        const float b = __ldg(bias_row + min(max(p_row - key0 - c, 0), capped.bias_count - 1));
+                        s[c] = __float_as_uint(fmaf(b, inv_scale, __uint_as_float(s[c])));
+                    }
+                }
+            }
             // the page's maximum on the raw dots (the scale is positive), four chains side by side
             float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -319,10 +339,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 for (int e = 0; e < 4; ++e) mx[e] = max3(mx[e], __uint_as_float(s[c + e]), __uint_as_float(s[c + 4 + e]));
             }
             float m_page = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-            if (CAPPED && capped.cap > 0.0f) {          // the cap is monotonic: the maximum of the capped scores is the capped maximum
+            if (CAPPED && !BIAS && capped.cap > 0.0f) {          // the cap is monotonic: the maximum of the capped scores is the capped maximum
                 if (m_page != -INFINITY) m_page = cap_l2 * (1.0f - 2.0f * rcp_approx(ex2_approx(m_page * tanh_k) + 1.0f));
             } else {
-                m_page *= scale_log2;
+                m_page = BIAS ? fmaf(m_page, scale_log2, bias_far) : m_page * scale_log2;
             }
             float alpha = 1.0f;
             bool raise = false;
@@ -341,7 +361,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
                 raise = true;
             }
             // p = 2^(dot * scale - m): one multiply-add and one ex2 per score, four sums side by side
-            const float neg_m = -m_run;
+            const float neg_m = BIAS ? bias_far - m_run : -m_run;
             // (the multiply-adds and the sums take two scores an instruction: fma.rn.f32x2, add.f32x2)
             const uint64_t scale2 = pack_f32x2(scale_log2, scale_log2), neg_m2 = pack_f32x2(neg_m, neg_m);
             uint64_t part2[2] = {pack_f32x2(0.0f, 0.0f), pack_f32x2(0.0f, 0.0f)};
@@ -350,7 +370,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             // the capped form: x = cap_l2 * (1 - 2 / (2^(dot * tanh_k) + 1)) - m = -2 cap_l2 / (...) + (cap_l2 - m)
             const uint64_t tanh_k2 = pack_f32x2(tanh_k, tanh_k), one2 = pack_f32x2(1.0f, 1.0f);
             const uint64_t slope2 = pack_f32x2(-2.0f * cap_l2, -2.0f * cap_l2), shift2 = pack_f32x2(cap_l2 + neg_m, cap_l2 + neg_m);
-            const bool use_cap = CAPPED && capped.cap > 0.0f;
+            const bool use_cap = CAPPED && !BIAS && capped.cap > 0.0f;
 #pragma unroll
             for (int c = 0; c < 64; c += 4) {
                 float x0, x1, x2, x3;
@@ -491,9 +511,11 @@ Q3_EXPORT int q3_attention_capped_prefill_tc_bf16(const void* q, const void* k_p
                                                   const int* seq_start, const int* seq_pos0, const int* page_table,
                                                   int pages_per_seq, int n_seqs, int max_new, int64_t n_tokens,
                                                   int64_t n_cache_pages, int nq, int nkv, float scale, float softcap, int chunk,
-                                                  int sink, const float* sink_values, int* status, void* stream) {
-    if (softcap < 0.0f || chunk < 0) return Q3_ERR_BAD_SIZE;
+                                                  int sink, const float* sink_values, const float* bias, int bias_count, int* status,
+                                                  void* stream) {
+    if (softcap < 0.0f || chunk < 0 || BIAS != (bias != nullptr) || (BIAS && (bias_count <= 0 || softcap > 0.0f || chunk > 0))) return Q3_ERR_BAD_SIZE;
     CapArgs capped;
+    capped.bias = bias; capped.bias_count = bias_count;
     capped.scale = scale; capped.cap = softcap; capped.chunk = chunk; capped.sink = sink ? 1 : 0; capped.sink_values = sink_values;
     return launch_prefill_tc(q, k_pages, v_pages, out, seq_start, seq_pos0, page_table, pages_per_seq, n_seqs, max_new, n_tokens,
                              n_cache_pages, nq, nkv, scale, status, stream, capped);

@@ -12,6 +12,10 @@
 //                  the values, vdx = vd + 1, whose value is 1 for every token: that column is the normaliser
 //                  n_t = a_t n_(t-1) + b_t k_t, and its output n_t . q_t.
 //
+//   state space  : the per-head form with a_t = exp(-exp(A_log[h]) dt), b_t = dt = softplus(z[t, h] + dt_bias[h]) made from a
+//                  32-bit logit per token and head by the blocks that need them; D_h v_t is added to the output, and
+//                  `share` neighbouring heads read the same q and k (Mamba-2: q = C, k = B, v = x).
+//
 //   decay_scan   : one block per (head, sequence, tile of up to 16 columns of the state: columns do not depend on
 //                  one another) walks the sequence's new tokens in order with its share of the state in registers:
 //                  thread (j, r) owns column j of the tile and the rows r * ROWS .. r * ROWS + ROWS - 1; the threads of
@@ -29,6 +33,7 @@
 //   head_gated_norm : per (token, head): x = o (divided by max(|n . q|, low) + floor if the state has the normaliser
 //                  column), y = x / sqrt(mean(x^2) + eps) * w * act(gate), act = sigmoid or SiLU; w one vector per
 //                  head, one for all heads, or none.
+//   gate_group_norm : x = o * SiLU(gate), then every one of `groups` equal parts of the row to unit rms by itself, times w.
 //
 // Decays, gates, state and outputs are 32-bit whatever T; T is the type of q, k, v, the output gate and the result.
 #include "common.cuh"
@@ -44,6 +49,7 @@ constexpr int PRE_V = 2;          // values of v
 // Asks for a line to be brought into L2; nothing waits for it.
 __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
 
+__device__ __forceinline__ float softplus_f32(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 
 struct ScanArgs {
@@ -62,6 +68,10 @@ struct ScanArgs {
     const int* seq_slots;
     float* out;                    // [N, H, vdx]
     int H, d, vd, vdx;
+    int share;                     // neighbouring heads that read the same q and k
+    const float* dt_bias;          // state space (else null): `keep` holds the logits z, one per token and head
+    const float* a_log;
+    const float* skip;
 };
 
 // MAXT: the most threads a block has (256 for keys up to 128 wide, which leaves a thread room for the values it holds for
@@ -82,8 +92,8 @@ decay_scan_kernel(const ScanArgs p, int R, int vt, int stage) {
     const int tid = threadIdx.x, nthreads = blockDim.x, jt = tid % vt, j = col0 + jt, r = tid / vt;
     const bool live = r < R && j < vdx;
     // nothing this kernel writes is read by it again: the inputs go through the read-only path
-    const T* __restrict__ q_g = reinterpret_cast<const T*>(p.q) + (int64_t)head * d;
-    const T* __restrict__ k_g = reinterpret_cast<const T*>(p.k) + (int64_t)head * d;
+    const T* __restrict__ q_g = reinterpret_cast<const T*>(p.q) + (int64_t)(head / p.share) * d;
+    const T* __restrict__ k_g = reinterpret_cast<const T*>(p.k) + (int64_t)(head / p.share) * d;
     const T* __restrict__ v_g = reinterpret_cast<const T*>(p.v) + (int64_t)head * vd;
     const float* __restrict__ z_g = p.z, * __restrict__ keep_g = p.keep, * __restrict__ write_g = p.write;
     float* __restrict__ out_g = p.out;
@@ -148,7 +158,7 @@ decay_scan_kernel(const ScanArgs p, int R, int vt, int stage) {
         if constexpr (!PER_CHANNEL) {
             if (tid < n_stage) {
                 keep_raw = __ldg(keep_g + (int64_t)(t0 + tid) * H + head);
-                write_raw = __ldg(write_g + (int64_t)(t0 + tid) * H + head);
+                if (p.dt_bias == nullptr) write_raw = __ldg(write_g + (int64_t)(t0 + tid) * H + head);
             }
         }
         // the stage after that one: its lines are asked into L2 now (one request per 32 bytes), so that its loads, a stage
@@ -188,6 +198,10 @@ decay_scan_kernel(const ScanArgs p, int R, int vt, int stage) {
         }
         if constexpr (!PER_CHANNEL) {
             if (tid < n_stage) {
+                if (p.dt_bias != nullptr) {
+                    write_raw = softplus_f32(keep_raw + p.dt_bias[head]);
+                    keep_raw = expf(-expf(p.a_log[head]) * write_raw);
+                }
                 a_s[tid] = keep_raw;
                 a_s[MAX_STAGE + tid] = write_raw;
             }
@@ -243,6 +257,7 @@ decay_scan_kernel(const ScanArgs p, int R, int vt, int stage) {
             if (col0 + c < vdx) {
                 float o = 0.0f;
                 for (int rr = 0; rr < R; ++rr) o += red[(tt * R + rr) * vt + c];
+                if (!PER_CHANNEL && p.skip != nullptr) o = fmaf(p.skip[head], v_s[tt * vt + c], o);
                 out_g[((int64_t)(t0 + tt) * H + head) * vdx + col0 + c] = o;
             }
         }
@@ -262,6 +277,7 @@ template <typename T, bool PER_CHANNEL>
 int decay_scan_launch(const ScanArgs& p, int n_seqs, cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     const int d = p.d, vdx = p.vdx;
+    if (p.share <= 0 || p.H % p.share != 0 || (PER_CHANNEL && p.share != 1)) return Q3_ERR_BAD_SIZE;
     if (p.H <= 0 || d <= 0 || p.vd <= 0 || d > 256 || vdx > 256 || vdx < p.vd || vdx > p.vd + 1 || n_seqs > 65535 || p.H > 65535)
         return Q3_ERR_BAD_SIZE;
     const int vt = min(vdx, COL_TILE);
@@ -376,6 +392,64 @@ __global__ void head_gated_norm_kernel(const float* __restrict__ o, const float*
     }
 }
 
+// One block per (part, token); a thread keeps up to PER values of the part in registers (PER = 0: any size, walked twice).
+template <typename T, int PER>
+__global__ void gate_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t gate_row, const float* __restrict__ w,
+                                       T* __restrict__ out, int part, int size, float eps) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t t = blockIdx.y;
+    const int col0 = blockIdx.x * part;
+    const float* x = o + t * size + col0;
+    const T* g = gate + t * gate_row + col0;
+    auto gated = [&](int c) {
+        const float z = to_f32<T>(g[c]);
+        return x[c] * (z / (1.0f + expf(-z)));
+    };
+    float v[PER > 0 ? PER : 1], sq = 0.0f;
+    if constexpr (PER > 0) {
+#pragma unroll
+        for (int n = 0; n < PER; ++n) {
+            const int c = n * blockDim.x + threadIdx.x;
+            v[n] = c < part ? gated(c) : 0.0f;
+            sq += v[n] * v[n];
+        }
+    } else {
+        for (int c = threadIdx.x; c < part; c += blockDim.x) {
+            const float y = gated(c);
+            sq += y * y;
+        }
+    }
+    const float inv = rsqrtf(block_sum(sq, scratch) / (float)part + eps);
+    T* to = out + t * size + col0;
+    if constexpr (PER > 0) {
+#pragma unroll
+        for (int n = 0; n < PER; ++n) {
+            const int c = n * blockDim.x + threadIdx.x;
+            if (c < part) to[c] = from_f32<T>(v[n] * inv * w[col0 + c]);
+        }
+    } else {
+        for (int c = threadIdx.x; c < part; c += blockDim.x) to[c] = from_f32<T>(gated(c) * inv * w[col0 + c]);
+    }
+}
+
+template <typename T>
+int gate_group_norm_launch(const float* o, const T* gate, int64_t gate_row, const float* w, T* out, int64_t n_tokens, int size, int groups,
+                           float eps, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (size <= 0 || groups <= 0 || size % groups != 0 || groups > 65535 || gate_row < size) return Q3_ERR_BAD_SIZE;
+    if (n_tokens > 65535) return Q3_ERR_TOO_LARGE;
+    const int part = size / groups;
+    const dim3 grid(groups, (unsigned)n_tokens);
+    auto launch = [&](auto kernel, int threads) {
+        return (int)q3_launch(kernel, grid, dim3(threads), 0, stream, o, gate, gate_row, w, out, part, size, eps);
+    };
+    if (part <= 512) return launch(gate_group_norm_kernel<T, 4>, (part + 127) / 128 * 32);
+    if (part <= 4096) return launch(gate_group_norm_kernel<T, 8>, (part + 255) / 256 * 32);
+    return launch(gate_group_norm_kernel<T, 0>, 512);
+}
+
 }  // namespace
 
 #define Q3_SCAN_EXPORTS(SUFFIX, T)                                                                                           \
@@ -383,15 +457,25 @@ __global__ void head_gated_norm_kernel(const float* __restrict__ o, const float*
                                          const float* keep, const float* write,                                             \
                                          float q_scale, int ones, float* state, int64_t slot_stride, const int* seq_start,  \
                                          const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd,           \
+                                         int share, const float* dt_bias, const float* a_log, const float* skip,           \
                                          void* stream) {                                                                   \
         ScanArgs p;                                                                                                         \
+        p.share = share; p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip;                                               \
+        if ((dt_bias == nullptr) != (a_log == nullptr) || (dt_bias != nullptr && (keep == nullptr || ones)) ||              \
+            (skip != nullptr && keep == nullptr))                                                                           \
+            return Q3_ERR_BAD_SIZE;                                                                                         \
         p.q = q; p.k = k; p.v = v; p.row = row; p.z = z; p.keep = keep;                                                     \
         p.write = write; p.q_scale = q_scale; p.ones = ones; p.state = state; p.slot_stride = slot_stride;                  \
         p.seq_start = seq_start; p.seq_slots = seq_slots; p.out = out; p.H = heads; p.d = d; p.vd = vd;                     \
         p.vdx = vd + (ones ? 1 : 0);                                                                                        \
-        if ((z == nullptr) == (keep == nullptr) || (keep != nullptr && write == nullptr)) return Q3_ERR_BAD_SIZE;           \
+        if ((z == nullptr) == (keep == nullptr) || (keep != nullptr && write == nullptr && dt_bias == nullptr)) return Q3_ERR_BAD_SIZE;           \
         if (z != nullptr) return decay_scan_launch<T, true>(p, n_seqs, (cudaStream_t)stream);                               \
         return decay_scan_launch<T, false>(p, n_seqs, (cudaStream_t)stream);                                                \
+    }                                                                                                                       \
+    Q3_EXPORT int q3_gate_group_norm_##SUFFIX(const float* o, const void* gate, int64_t gate_row, const float* w, void* out, \
+                                              int64_t n_tokens, int size, int groups, float eps, void* stream) {            \
+        return gate_group_norm_launch<T>(o, (const T*)gate, gate_row, w, (T*)out, n_tokens, size, groups, eps,              \
+                                         (cudaStream_t)stream);                                                             \
     }                                                                                                                       \
     Q3_EXPORT int q3_head_gated_norm_##SUFFIX(const float* o, const float* low, float floor_add, const float* w,            \
                                               int w_per_head, const void* gate, int64_t gate_row, void* out,               \

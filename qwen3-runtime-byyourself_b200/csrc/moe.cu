@@ -8,7 +8,7 @@
 //                 scores s.  The last `identity` outputs are experts without tensors whose output is the
 //                 token itself: their weights are summed into id_weight[token].
 //                 `by_logit` 1: the `top` largest logits win instead and the weights are the softmax over the chosen
-//                 logits only; 2: the scores are sigmoid(z), each output by itself.  `group_pair`: a group's score is
+//                 logits only (the correction, if there is one, is a bias on the logits); 2: the scores are sigmoid(z), each output by itself.  `group_pair`: a group's score is
 //                 the sum of its two largest choice scores.  The weights are multiplied by `weight_scale`.  With `gate_out`, the router matrix has one more row after the outputs whose logit
 //                 is no expert's: gate_out[token] = sigmoid(that logit), the weight of a shared expert.
 //   moe_sort    : one block.  Counts the (token, choice) pairs of every real expert, lays the experts out one
@@ -73,7 +73,10 @@ moe_route_kernel(const T* __restrict__ h, const T* __restrict__ w_router, const 
     if (by_logit == 1) {
         // the largest logits (ties: the lower index), weighted by the softmax over the chosen logits alone
         float best_z = 0.0f, sum = 0.0f;
-        for (int e = 0; e < n_out; ++e) choice[e] = z[e];
+        for (int e = 0; e < n_out; ++e) {
+            if (correction != nullptr) z[e] += correction[e];
+            choice[e] = z[e];
+        }
         for (int k = 0; k < top; ++k) {
             int best = -1;
             for (int e = 0; e < n_out; ++e)

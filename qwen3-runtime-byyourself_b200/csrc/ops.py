@@ -320,6 +320,21 @@ def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, 
     return out
 
 
+def embedding_sinusoid(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, freq: torch.Tensor, out: torch.Tensor,
+                       scale: float) -> torch.Tensor:
+    """out[t] = table[ids[t]] * scale as float32, plus sin(p f_i) in column 2i and cos(p f_i) in column 2i + 1 with p the
+    token's position; `freq` float32 [2, (hidden + 1) // 2]: frequencies as a leading term and what its rounding dropped."""
+    n, hidden = ids.numel(), table.shape[1]
+    if out.shape[0] < n or out.shape[1] != hidden or out.dtype != torch.float32 or positions.numel() < n \
+            or tuple(freq.shape) != (2, (hidden + 1) // 2):
+        raise KernelError("embedding_sinusoid: output or frequencies do not fit")
+    fn = _fn("stream_f32.cu", f"q3_embedding_sinusoid_{_suffix(table)}",
+             [c_void_p] * 5 + [c_int64, c_int, c_int, c_float, c_void_p])
+    _check(fn(_dev(ids, "ids", torch.int32), _dev(positions, "positions", torch.int32), _dev(table, "table"),
+              _dev(freq, "freq", torch.float32), _dev(out, "out"), n, hidden, table.shape[0], float(scale), _stream()), "embedding_sinusoid")
+    return out
+
+
 def sandwich_norm(stream: torch.Tensor, branch: Optional[torch.Tensor], w_post: Optional[torch.Tensor], eps_post: float,
                   w_pre: Optional[torch.Tensor], eps_pre: float, out: Optional[torch.Tensor], groups_post: int = 1,
                   groups_pre: int = 1) -> Optional[torch.Tensor]:
@@ -431,19 +446,23 @@ def _rotary_dim(cos, sin, d: int) -> int:
 def qkv_prepare(qkv, q_out, k_pages, v_pages, q_norm_w, k_norm_w, cos, sin, token_seq, token_pos, page_table,
                 n_tokens: int, nq: int, nkv: int, d: int, eps: float, write_kv: bool = True, bias=None,
                 value_dim: Optional[int] = None, value_heads: Optional[int] = None, tied_values: bool = False,
-                norm_once: bool = False, value_cos: Optional[torch.Tensor] = None, value_sin: Optional[torch.Tensor] = None):
+                norm_once: bool = False, value_cos: Optional[torch.Tensor] = None, value_sin: Optional[torch.Tensor] = None,
+                temperature: Optional[tuple] = None):
     """Per-head norm of q and k, rotation, and the write of k and v into the cache pages
-    (`write_kv=False`: only q is prepared, for a layer that reads another layer's cache).  `bias` (float32, one
+    (`write_kv=False`: only q is prepared, for a layer that reads another layer's cache; `qkv` may then hold the query
+    columns alone).  `bias` (float32, one
     value per column of the projection) is added first; `value_dim` is the size of a value head if not `d`,
     `value_heads` their number if not `nkv` (values that several key heads share).  A row of `qkv` may go on beyond the
     values.  `tied_values`: the values are the projected keys as they are, and `qkv` has no columns for them; `norm_once`: a
     normed and rotated value is rounded once, when it is stored; `value_cos`, `value_sin` [positions, value_dim / 2]: the
-    values are rotated by their position too, over the whole head."""
+    values are rotated by their position too, over the whole head.  `temperature` = (coef, every): a normed query is
+    multiplied by 1 + coef ln((p + 1) // every + 1), p its position."""
     s = _suffix(qkv)
+    temp_coef, temp_every = (float(temperature[0]), int(temperature[1])) if temperature else (0.0, 1)
     vd, nv = int(value_dim or d), int(value_heads or nkv)
     if not 0 < d <= 256 or not 0 < vd <= 256 or (d % 2 != 0 and cos is not None and 2 * cos.shape[-1] == d):
         raise KernelError(f"head_dim {d} / value_dim {vd} is not supported: sizes up to 256, an even number of rotated values")
-    columns = (nq + nkv) * d + (0 if tied_values else nv * vd)
+    columns = (nq + nkv) * d + (0 if tied_values else nv * vd) if write_kv else nq * d
     if qkv.shape[-1] < columns or k_pages.dtype != qkv.dtype or k_pages.shape[1:] != (nkv, PAGE_TOKENS, d) \
             or v_pages.shape[1:] != (nv, PAGE_TOKENS, vd) or nkv % nv or (bias is not None and bias.numel() != columns) \
             or (tied_values and (vd != d or nv != nkv)) or (value_cos is None) != (value_sin is None) \
@@ -452,15 +471,15 @@ def qkv_prepare(qkv, q_out, k_pages, v_pages, q_norm_w, k_norm_w, cos, sin, toke
     rot = _rotary_dim(cos, sin, d)
     fn = _fn("attention.cu", f"q3_qkv_prepare_{s}",
              [c_void_p] * 11 + [c_int, c_int64, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_int64, c_int, c_int,
-                                c_void_p, c_void_p, c_void_p])
+                                c_void_p, c_void_p, c_float, c_int, c_void_p])
     _check(fn(_dev(qkv, "qkv"), _dev(q_out, "q_out", qkv.dtype), _dev(k_pages, "k_pages"), _dev(v_pages, "v_pages"),
               _ptr(q_norm_w, "q_norm_w", torch.float32), _ptr(k_norm_w, "k_norm_w", torch.float32),
               _ptr(cos, "cos", torch.float32), _ptr(sin, "sin", torch.float32),
               _dev(token_seq, "token_seq", torch.int32), _dev(token_pos, "token_pos", torch.int32),
               _dev(page_table, "page_table", torch.int32), page_table.shape[-1], n_tokens, nq, nkv, d, float(eps),
               int(bool(write_kv)), rot, _ptr(bias, "bias", torch.float32), vd, nv, qkv.shape[-1], int(bool(tied_values)),
-              int(bool(norm_once)), _ptr(value_cos, "value_cos", torch.float32), _ptr(value_sin, "value_sin", torch.float32), _stream()),
-           "qkv_prepare")
+              int(bool(norm_once)), _ptr(value_cos, "value_cos", torch.float32), _ptr(value_sin, "value_sin", torch.float32), temp_coef,
+              temp_every, _stream()), "qkv_prepare")
     return q_out
 
 
@@ -523,17 +542,27 @@ def _sink_ptr(sink, sink_values, nq: int):
     return _dev(sink_values, "sink_values", torch.float32)
 
 
+def _bias_args(bias: Optional[torch.Tensor], nq: int):
+    """(table, numbers per head) of biases by distance, float32 [nq, count]; none: (None, 0)."""
+    if bias is None:
+        return None, 0
+    if bias.dim() != 2 or bias.shape[0] != nq or bias.shape[1] == 0:
+        raise KernelError("attention: biases by distance are [query heads, distances]")
+    return _dev(bias, "bias", torch.float32), bias.shape[1]
+
+
 def attention_generic(q, k_pages, v_pages, out, token_seq, token_pos, page_table, n_tokens: int, nq: int, nkv: int,
                       d: int, scale: float, window: Optional[int] = None, value_dim: Optional[int] = None,
                       softcap: float = 0.0, chunk: Optional[int] = None, sink: bool = False, value_heads: Optional[int] = None,
-                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None):
+                      sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None, bias: Optional[torch.Tensor] = None):
     """Causal grouped-query attention of every token of the step over its sequence's pages.  `keep_first` (with `window`):
     the first so many keys of the sequence are seen beside the window's.  `softcap` > 0 caps the
     scores smoothly (s <- softcap * tanh(s / softcap)); `chunk`: a query reads only the keys of its own chunk of that
     many positions; `sink`: one more term exp(0), without a value, in the softmax's denominator (exp(sink_values[head])
     with `sink_values`, float32 [nq]); `value_dim`: the
     size of a value head (and of an output head) if not `d`; `value_heads`: the number of value heads if not `nkv`
-    (each serves nkv / value_heads key heads).  `out` has q's type, or is float32 for a caller that goes on in 32-bit."""
+    (each serves nkv / value_heads key heads).  `bias` (float32 [nq, count]): added to the scaled score by the distance between query and
+    key, the last column for every distance from count - 1 on.  `out` has q's type, or is float32 for a caller that goes on in 32-bit."""
     s = _suffix(q)
     vd, nv = int(value_dim or d), int(value_heads or nkv)
     if out.dtype not in (q.dtype, torch.float32) or nkv % nv:
@@ -544,14 +573,14 @@ def attention_generic(q, k_pages, v_pages, out, token_seq, token_pos, page_table
         raise KernelError("attention: a window or chunks, not both")
     fn = _fn("attention.cu", f"q3_attention_generic_{s}",
              [c_void_p] * 7 + [c_int, c_int64, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int, c_int, c_int,
-                               c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+                               c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p])
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", q.dtype), _dev(v_pages, "v_pages", q.dtype),
               _dev(out, "out"), _dev(token_seq, "token_seq", torch.int32),
               _dev(token_pos, "token_pos", torch.int32), _dev(page_table, "page_table", torch.int32),
               page_table.shape[-1], n_tokens, nq, nkv, d, float(scale), int(window or 0), vd, float(softcap or 0.0),
               int(chunk or 0), int(bool(sink)), nv, int(out.dtype == torch.float32 and q.dtype != torch.float32),
               _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
-              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_generic"), _stream()), "attention_generic")
+              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_generic"), *_bias_args(bias, nq), _stream()), "attention_generic")
     return out
 
 
@@ -581,20 +610,24 @@ def head_gate(x: torch.Tensor, gate: torch.Tensor, heads: int, vd: int) -> torch
 
 
 def short_conv(u: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, token_seq, seq_start, seq_slots, out: torch.Tensor,
-               n_seqs: int) -> torch.Tensor:
+               n_seqs: int, bias: Optional[torch.Tensor] = None, silu: bool = False) -> torch.Tensor:
     """Causal convolution over time on the first C columns of u [N, >= C]: out[t, c] = sum_j weight[j, c] u[t - taps + 1 + j, c]
     within every sequence, the rows before the step from `state` (a view [slots, (taps - 1) * C] of float32 rows, the
     oldest row first), which is moved on afterwards.  weight float32 [taps, C] (a checkpoint's [C, taps] transposed);
-    out [N, C] in u's type."""
+    out [N, C] in u's type.  `bias` (float32 [C]) is added to the sum; `silu`: the result goes through SiLU, both before the
+    rounding."""
     N, (taps, C) = u.shape[0], weight.shape
     if out.shape != (N, C) or out.dtype != u.dtype or u.shape[1] < C or u.stride(1) != 1 or state.shape[1] != (taps - 1) * C \
-            or state.dtype != torch.float32 or (taps > 1 and state.stride(1) != 1) or not out.is_contiguous() or out.data_ptr() == u.data_ptr():
+            or state.dtype != torch.float32 or (taps > 1 and state.stride(1) != 1) or not out.is_contiguous() or out.data_ptr() == u.data_ptr() \
+            or (bias is not None and bias.numel() != C):
         raise KernelError("short_conv: shapes do not fit")
     fn = _fn("short_conv.cu", f"q3_short_conv_{_suffix(u)}",
-             [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int64, c_int, c_void_p])
+             [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int64, c_int, c_void_p, c_int,
+              c_void_p])
     _check(fn(u.data_ptr(), u.stride(0), _dev(weight, "weight", torch.float32), state.data_ptr(), state.stride(0),
               _dev(token_seq, "token_seq", torch.int32), _dev(seq_start, "seq_start", torch.int32),
-              _dev(seq_slots, "seq_slots", torch.int32), out.data_ptr(), C, taps, N, int(n_seqs), _stream()), "short_conv")
+              _dev(seq_slots, "seq_slots", torch.int32), out.data_ptr(), C, taps, N, int(n_seqs), _ptr(bias, "bias", torch.float32), int(bool(silu)),
+              _stream()), "short_conv")
     if taps > 1:
         _count_extra(1)
     return out
@@ -716,37 +749,54 @@ def gated_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: f
 
 
 # ------------------------------------------------------------------ linear attention with keys: a decay per channel, or gates per head
-def _scan_views(q, k, v, state, out, heads, d, vd, vdx):
+def _scan_views(q, k, v, state, out, heads, d, vd, vdx, share=1):
     row = q.stride(0)
     if q.dtype != k.dtype or q.dtype != v.dtype or k.stride(0) != row or v.stride(0) != row or q.stride(1) != 1 or k.stride(1) != 1 \
-            or v.stride(1) != 1 or q.shape[1] != heads * d or k.shape[1] != heads * d or v.shape[1] != heads * vd \
+            or v.stride(1) != 1 or heads % share or q.shape[1] != heads // share * d or k.shape[1] != heads // share * d or v.shape[1] != heads * vd \
             or state.dtype != torch.float32 or state.shape[1] != heads * d * vdx or state.stride(1) != 1 \
             or out.dtype != torch.float32 or out.shape[1] != heads * vdx or not out.is_contiguous():
         raise KernelError("decay_scan: shapes do not fit")
     return row
 
 
+def _check_dt(N, heads, dt_logits, dt_bias, a_log, skip):
+    if (dt_logits is None) != (dt_bias is None) or (dt_bias is None) != (a_log is None) \
+            or (dt_logits is not None and (dt_logits.numel() < N * heads or dt_bias.numel() != heads or a_log.numel() != heads)) \
+            or (skip is not None and skip.numel() != heads):
+        raise KernelError("step sizes: logits [N, heads] with a bias and a log decay rate per head")
+
+
 def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, seq_slots: torch.Tensor,
                out: torch.Tensor, n_seqs: int, heads: int, d: int, vd: int, q_scale: float = 1.0, decay: Optional[torch.Tensor] = None,
-               keep: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None, ones: bool = False) -> torch.Tensor:
+               keep: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None, ones: bool = False, share: int = 1,
+               dt_logits: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None, a_log: Optional[torch.Tensor] = None,
+               skip: Optional[torch.Tensor] = None) -> torch.Tensor:
     """S_t = diag(a_t) S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T (q_t * q_scale) over the new tokens of every sequence, from and to
     the state rows (`state`: a view [slots, heads * d * vdx] of float32 rows).  q, k, v: column views of one projection
     output (same row stride).  With `decay` [N, heads * d] (float32, see `channel_decay`): a per channel, b = 1.  With
     `keep`, `write` [N, heads] (float32): a and b per head.  `ones`: vdx = vd + 1, the state's last column takes
-    the value 1 (a normaliser); else vdx = vd.  out [N, heads * vdx] float32."""
+    the value 1 (a normaliser); else vdx = vd.  `dt_logits` [N, heads] with `dt_bias`, `a_log` [heads] (float32) instead of
+    `keep` and `write`: b = softplus(logit + dt_bias), a = exp(-exp(a_log) b).  `skip` [heads]: skip_h v_t is added to the output.
+    `share`: so many neighbouring heads read the same q and k.  out [N, heads * vdx] float32."""
     vdx = vd + (1 if ones else 0)
-    row = _scan_views(q, k, v, state, out, heads, d, vd, vdx)
+    row = _scan_views(q, k, v, state, out, heads, d, vd, vdx, share)
     N = q.shape[0]
     z = decay
+    _check_dt(N, heads, dt_logits, dt_bias, a_log, skip)
+    if dt_logits is not None:
+        if keep is not None or write is not None or ones:
+            raise KernelError("decay_scan: step sizes come as logits or as gates per head, without a normaliser")
+        keep = write = dt_logits
     if (z is None) == (keep is None) or (z is not None and (tuple(z.shape) != (N, heads * d) or not z.is_contiguous())) \
             or (keep is not None and (write is None or keep.numel() < N * heads or write.numel() < N * heads)):
         raise KernelError("decay_scan: a decay per channel or gates per head (keep, write)")
     fn = _fn("linear_scan.cu", f"q3_decay_scan_{_suffix(q)}",
              [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int64,
-              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
     _check(fn(q.data_ptr(), k.data_ptr(), v.data_ptr(), row, _ptr(z, "decay", torch.float32), _ptr(keep, "keep", torch.float32), _ptr(write, "write", torch.float32), float(q_scale), int(bool(ones)),
               state.data_ptr(), state.stride(0), _dev(seq_start, "seq_start", torch.int32), _dev(seq_slots, "seq_slots", torch.int32),
-              _dev(out, "out"), int(n_seqs), heads, d, vd, _stream()), "decay_scan")
+              _dev(out, "out"), int(n_seqs), heads, d, vd, int(share), _ptr(dt_bias, "dt_bias", torch.float32),
+              _ptr(a_log, "a_log", torch.float32), _ptr(skip, "skip", torch.float32), _stream()), "decay_scan")
     return out
 
 
@@ -797,6 +847,20 @@ def head_gated_norm(o: torch.Tensor, weight: Optional[torch.Tensor], gate: torch
     return out
 
 
+def gate_group_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, groups: int) -> torch.Tensor:
+    """x = o * silu(gate), every one of `groups` equal parts of a row divided by its own rms, times weight; o float32 [N, size],
+    `gate` a view of [N, size] columns, weight float32 [size], out in the gate's type."""
+    N, size = o.shape
+    if gate.shape != o.shape or gate.stride(1) != 1 or out.shape != o.shape or gate.dtype != out.dtype or not out.is_contiguous() \
+            or weight.numel() != size or groups <= 0 or size % groups:
+        raise KernelError("gate_group_norm: shapes do not fit")
+    fn = _fn("linear_scan.cu", f"q3_gate_group_norm_{_suffix(out)}",
+             [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_float, c_void_p])
+    _check(fn(_dev(o, "o", torch.float32), gate.data_ptr(), gate.stride(0), _dev(weight, "weight", torch.float32), out.data_ptr(), N, size,
+              int(groups), float(eps), _stream()), "gate_group_norm")
+    return out
+
+
 # ------------------------------------------------------------------ differential attention
 def diff_combine(a: torch.Tensor, out: torch.Tensor, n_tokens: int, heads: int, per_group: int, vd: int, lam: float, eps: float,
                  gain: float) -> torch.Tensor:
@@ -832,7 +896,7 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torc
     (`sigmoid`: each output's sigmoid by itself), choice by score + correction (None: by the score alone) within the kept groups (a group's mark:
     its best choice score, or with `group_pair` the sum of its two best), weights = plain scores times `weight_scale`;
     `by_logit`: the largest logits are chosen and weighted by the softmax over the chosen logits alone (the correction is
-    not read).  With `gate_out` [N] the router matrix has one more row, and gate_out = sigmoid of its logit; see csrc/moe.cu."""
+    then a bias on the logits).  With `gate_out` [N] the router matrix has one more row, and gate_out = sigmoid of its logit; see csrc/moe.cu."""
     N, hidden = h.shape
     n_out = w_router.shape[0] - (1 if gate_out is not None else 0)
     if w_router.shape[1] != hidden or w_router.dtype != h.dtype or (correction is not None and correction.numel() != n_out) \
@@ -909,11 +973,12 @@ def _capped_defines(d: int, vd: int):
 def attention_capped_prefill(q, k_pages, v_pages, out, seq_start, seq_pos0, page_table, n_seqs: int, max_new: int, nq: int,
                              nkv: int, d: int, vd: int, scale: float, softcap: float = 0.0, chunk: Optional[int] = None,
                              sink: bool = False, window: Optional[int] = None, value_heads: Optional[int] = None,
-                             sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None):
+                             sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None,
+                             bias: Optional[torch.Tensor] = None):
     """Attention of every new token of every sequence over its pages (bfloat16, tiled, tensor cores) with capped scores,
     chunked visibility or a sliding window (beside which the first `keep_first` keys of the sequence stay visible, or the pooled
     blocks of `pool`), and a sink (its score per query head in `sink_values`, else 0); q [tokens, nq * d], out [tokens, nq * vd] in bfloat16 or float32;
-    `value_heads`: the number of value heads if not `nkv` (each serves nkv / value_heads key heads)."""
+    `value_heads`: the number of value heads if not `nkv` (each serves nkv / value_heads key heads); `bias`: see `attention_generic`."""
     nv = int(value_heads or nkv)
     if q.dtype != torch.bfloat16 or not attention_capped_fits(d, vd, None, 1) or out.dtype not in (torch.bfloat16, torch.float32):
         raise KernelError("attention_capped_prefill: bfloat16, head sizes in steps of 16 up to 256")
@@ -921,14 +986,14 @@ def attention_capped_prefill(q, k_pages, v_pages, out, seq_start, seq_pos0, page
         raise KernelError("attention_capped_prefill: shapes do not fit")
     fn = _fn("attention_capped.cu", "q3_attention_capped_prefill_bf16",
              [c_void_p] * 7 + [c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
              defines=_capped_defines(d, vd))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out"), _dev(seq_start, "seq_start", torch.int32),
               _dev(seq_pos0, "seq_pos0", torch.int32), _dev(page_table, "page_table", torch.int32), page_table.shape[-1],
               n_seqs, max_new, nq, nkv, float(scale), float(softcap or 0.0), int(chunk or 0), int(bool(sink)), int(window or 0), nv,
               int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
-              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_prefill"), _stream()), "attention_capped_prefill")
+              *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_prefill"), *_bias_args(bias, nq), _stream()), "attention_capped_prefill")
     return out
 
 
@@ -943,7 +1008,7 @@ def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_
                             n_splits: int, window: Optional[int] = None, value_heads: Optional[int] = None,
                             sink_values: Optional[torch.Tensor] = None, keep_first: int = 0, pool: Optional[Pool] = None,
                             pool_write: bool = False, back_cos: Optional[torch.Tensor] = None, back_sin: Optional[torch.Tensor] = None,
-                            gate: Optional[torch.Tensor] = None):
+                            gate: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None):
     """The same for one new token per sequence, the keys split over `n_splits` blocks per (token, kv head); `scratch`
     holds n_tokens * nq * n_splits * (vd + 2) float32.  `pool_write`: a block of tokens that a token completes is pooled by this
     kernel (as `pool_blocks` does); `back_cos`, `back_sin`, `gate`: what `turn_back_gate` does to the output, done where the
@@ -959,7 +1024,7 @@ def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_
         raise KernelError("attention_capped_decode: shapes do not fit")
     fn = _fn("attention_capped.cu", "q3_attention_capped_decode_bf16",
              [c_void_p] * 8 + [c_int, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int64, c_void_p],
+                               c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_void_p],
              defines=_capped_defines(d, vd))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out"), _dev(scratch, "scratch", torch.float32),
@@ -969,7 +1034,7 @@ def attention_capped_decode(q, k_pages, v_pages, out, scratch, token_seq, token_
               int(out.dtype == torch.float32), _sink_ptr(sink, sink_values, nq), int(keep_first or 0) if window else 0,
               *_pool_args(pool, k_pages, v_pages, page_table, window, "attention_capped_decode"), int(bool(pool_write)),
               _ptr(back_cos, "back_cos", torch.float32), _ptr(back_sin, "back_sin", torch.float32),
-              gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0, _stream()),
+              gate.data_ptr() if gate is not None else None, gate.stride(0) if gate is not None else 0, *_bias_args(bias, nq), _stream()),
            "attention_capped_decode")
     _count_extra(1)                                              # the split kernel and the merge kernel
     return out
@@ -1006,19 +1071,20 @@ def attention_capped_prefill_tc_fits(d: int, vd: int, window: Optional[int]) -> 
 
 def attention_capped_prefill_tc(q, k_pages, v_pages, out, seq_start, seq_pos0, page_table, n_seqs: int, max_new: int,
                                 n_tokens: int, nq: int, nkv: int, d: int, scale: float, softcap: float = 0.0,
-                                chunk: Optional[int] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None):
+                                chunk: Optional[int] = None, sink: bool = False, sink_values: Optional[torch.Tensor] = None,
+                                bias: Optional[torch.Tensor] = None):
     """`attention_capped_prefill` with both products on tcgen05 (TMA-fed, scores and output in tensor memory): head
     sizes 64 and 128, values as wide as keys."""
     if q.dtype != torch.bfloat16 or not attention_capped_prefill_tc_fits(d, d, None) or not scale > 0:
         raise KernelError("attention_capped_prefill_tc: bfloat16, head size 64 or 128, a positive scale")
     fn = _fn("attention_prefill_tc.cu", "q3_attention_capped_prefill_tc_bf16",
-             [c_void_p] * 7 + [c_int, c_int, c_int, c_int64, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
-             defines=(f"Q3_HEAD_DIM={d}", "Q3_CAPPED=1"))
+             [c_void_p] * 7 + [c_int, c_int, c_int, c_int64, c_int64, c_int, c_int, c_float, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
+             defines=(f"Q3_HEAD_DIM={d}", "Q3_CAPPED=1" if bias is None else "Q3_CAPPED=2"))
     _check(fn(_dev(q, "q"), _dev(k_pages, "k_pages", torch.bfloat16), _dev(v_pages, "v_pages", torch.bfloat16),
               _dev(out, "out", torch.bfloat16), _dev(seq_start, "seq_start", torch.int32),
               _dev(seq_pos0, "seq_pos0", torch.int32), _dev(page_table, "page_table", torch.int32),
               page_table.shape[-1], n_seqs, max_new, n_tokens, k_pages.shape[0], nq, nkv, float(scale), float(softcap or 0.0),
-              int(chunk or 0), int(bool(sink)), _sink_ptr(sink, sink_values, nq), _status_word(q.device).data_ptr(), _stream()), "attention_capped_prefill_tc")
+              int(chunk or 0), int(bool(sink)), _sink_ptr(sink, sink_values, nq), *_bias_args(bias, nq), _status_word(q.device).data_ptr(), _stream()), "attention_capped_prefill_tc")
     return out
 
 
@@ -1384,7 +1450,7 @@ def attention_prefill_tc(q, k_pages, v_pages, out, seq_start, seq_pos0, page_tab
 
 
 # ------------------------------------------------------------------ a float32 stream with norms of several kinds, a token shift, a side input
-NORM_KINDS = {"none": 0, "rms": 1, "dynamic_tanh": 2, "round": 3}
+NORM_KINDS = {"none": 0, "rms": 1, "dynamic_tanh": 2, "round": 3, "layer": 4}
 
 
 def _norm_args(norm, size: int, what: str):
@@ -1406,8 +1472,8 @@ def settle_norm(stream: torch.Tensor, branch: Optional[torch.Tensor], post, pre,
                 compute_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
     """One pass over the rows of the float32 `stream`: with `branch` (compute type) and the norm part `post`,
     stream += post(branch); with `out` and `pre` (a norm part, or "round"), out = pre(stream) of the sum.  `out` is of the
-    compute type or float32.  The norm parts are RMS norms (unit rms times a weight) or dynamic-tanh norms
-    (tanh(alpha x) * weight + b).  With `rows` (int32) only those rows are read, nothing is written to the stream
+    compute type or float32.  The norm parts are RMS norms (unit rms times a weight), layer norms (centred, no
+    bias) or dynamic-tanh norms (tanh(alpha x) * weight + b).  With `rows` (int32) only those rows are read, nothing is written to the stream
     and out[r] belongs to rows[r]."""
     total, size = stream.shape
     if stream.dtype != torch.float32 or (branch is None) != (post is None) or (out is None) != (pre is None):

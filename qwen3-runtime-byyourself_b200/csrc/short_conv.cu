@@ -3,6 +3,8 @@
 //
 //     y[t, c] = sum_j w[c, j] * u[t - taps + 1 + j, c],   j = 0 .. taps - 1,   u = 0 before the sequence's start
 //
+// With `bias` a number per channel is added to the sum, with `silu` the result goes through SiLU, all before the rounding.
+//
 //   short_conv       : one thread per (token, channel) - or, for 2 to 4 taps and rows of 16-byte packets, per run of up to 16
 //                      tokens and packet of channels, the last rows kept in registers; an input row before the step's first
 //                      token comes from the state [slot][taps - 1][C] (float32; the oldest row first), zeros for a new sequence.
@@ -17,11 +19,17 @@
 
 namespace {
 
+__device__ __forceinline__ float finish(float acc, const float* __restrict__ bias, int c, int silu) {
+    if (bias != nullptr) acc += bias[c];
+    return silu ? acc / (1.0f + expf(-acc)) : acc;
+}
+
 // VEC channels a thread (16 bytes of a row where the sizes allow it, else one).
 template <typename T, int VEC>
 __global__ void short_conv_kernel(const T* __restrict__ u, int64_t row_in, const float* __restrict__ w, const float* __restrict__ state,
                                   int64_t slot_stride, const int* __restrict__ token_seq, const int* __restrict__ seq_start,
-                                  const int* __restrict__ seq_slots, T* __restrict__ y, int C, int taps, int64_t n_tokens) {
+                                  const int* __restrict__ seq_slots, T* __restrict__ y, int C, int taps, int64_t n_tokens,
+                                  const float* __restrict__ bias, int silu) {
     pdl_launch_dependents();
     pdl_wait();
     const int per_row = C / VEC;
@@ -54,11 +62,11 @@ __global__ void short_conv_kernel(const T* __restrict__ u, int64_t row_in, const
             for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w[(int64_t)j * C + c + k], x[k], acc[k]);
         }
         if constexpr (VEC == 1) {
-            y[t * C + c] = from_f32<T>(acc[0]);
+            y[t * C + c] = from_f32<T>(finish(acc[0], bias, c, silu));
         } else {
             Pack<T> pk;
 #pragma unroll
-            for (int k = 0; k < VEC; ++k) pk.set(k, acc[k]);
+            for (int k = 0; k < VEC; ++k) pk.set(k, finish(acc[k], bias, c + k, silu));
             store_pack<T>(y + t * C + c, pk);
         }
     }
@@ -70,7 +78,8 @@ __global__ void short_conv_kernel(const T* __restrict__ u, int64_t row_in, const
 template <typename T, int VEC, int TAPS>
 __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, const float* __restrict__ w, const float* __restrict__ state,
                                        int64_t slot_stride, const int* __restrict__ token_seq, const int* __restrict__ seq_start,
-                                       const int* __restrict__ seq_slots, T* __restrict__ y, int C, int64_t n_tokens, int run) {
+                                       const int* __restrict__ seq_slots, T* __restrict__ y, int C, int64_t n_tokens, int run,
+                                       const float* __restrict__ bias, int silu) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
@@ -116,7 +125,7 @@ __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, 
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
             acc[k] = fmaf(wt[TAPS - 1][k], x[k], acc[k]);
-            out.set(k, acc[k]);
+            out.set(k, finish(acc[k], bias, c + k, silu));
         }
         store_pack<T>(y + t * C + c, out);
 #pragma unroll
@@ -132,14 +141,15 @@ __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, 
 
 template <typename T, int TAPS>
 int short_conv_walk_launch(const T* u, int64_t row_in, const float* w, const float* state, int64_t slot_stride, const int* token_seq,
-                           const int* seq_start, const int* seq_slots, T* y, int C, int64_t n_tokens, cudaStream_t stream) {
+                           const int* seq_start, const int* seq_slots, T* y, int C, int64_t n_tokens, const float* bias, int silu,
+                           cudaStream_t stream) {
     constexpr int V = Pack<T>::N;
     const int run = n_tokens >= 1024 ? 16 : (n_tokens >= 128 ? 4 : 1);
     const int64_t runs = (n_tokens + run - 1) / run;
     if (runs > 65535) return Q3_ERR_TOO_LARGE;
     const dim3 grid((unsigned)((C / V + 127) / 128), (unsigned)runs);
     return (int)q3_launch(short_conv_walk_kernel<T, V, TAPS>, grid, dim3(128), 0, stream, u, row_in, w, state, slot_stride, token_seq,
-                          seq_start, seq_slots, y, C, n_tokens, run);
+                          seq_start, seq_slots, y, C, n_tokens, run, bias, silu);
 }
 
 template <typename T>
@@ -162,39 +172,41 @@ __global__ void short_conv_state_kernel(const T* __restrict__ u, int64_t row_in,
     }
 }
 
+template <typename T>
+int short_conv_launch(const T* u, int64_t row_in, const float* w, float* state, int64_t slot_stride, const int* token_seq, const int* seq_start,
+                      const int* seq_slots, T* y, int C, int taps, int64_t n_tokens, int n_seqs, const float* bias, int silu,
+                      cudaStream_t stream) {
+    if (n_tokens <= 0 || n_seqs <= 0) return 0;
+    if (C <= 0 || taps <= 0 || taps > 64 || row_in < C) return Q3_ERR_BAD_SIZE;
+    constexpr int V = Pack<T>::N;
+    const bool vec = C % V == 0 && row_in % V == 0 && aligned16(u) && aligned16(y);
+    int code;
+    if (vec && taps >= 2 && taps <= 4 && (n_tokens + 15) / 16 <= 65535) {
+        auto walk = [&](auto launch) {
+            return launch(u, row_in, w, state, slot_stride, token_seq, seq_start, seq_slots, y, C, n_tokens, bias, silu, stream);
+        };
+        code = taps == 2 ? walk(short_conv_walk_launch<T, 2>) : (taps == 3 ? walk(short_conv_walk_launch<T, 3>) : walk(short_conv_walk_launch<T, 4>));
+    } else {
+        const int64_t blocks = (n_tokens * (C / (vec ? V : 1)) + 255) / 256;
+        code = (int)q3_launch(vec ? short_conv_kernel<T, V> : short_conv_kernel<T, 1>, dim3((unsigned)(blocks < 65536 ? blocks : 65536)),
+                              dim3(256), 0, stream, u, row_in, w, (const float*)state, slot_stride, token_seq, seq_start, seq_slots, y, C,
+                              taps, n_tokens, bias, silu);
+    }
+    if (code != 0 || taps == 1) return code;
+    const int64_t blocks = ((int64_t)n_seqs * C + 255) / 256;
+    return (int)q3_launch(short_conv_state_kernel<T>, dim3((unsigned)(blocks < 65536 ? blocks : 65536)), dim3(256), 0, stream, u, row_in,
+                          state, slot_stride, seq_start, seq_slots, C, taps, n_seqs);
+}
+
 }  // namespace
 
 #define Q3_CONV_EXPORTS(SUFFIX, T)                                                                                        \
     Q3_EXPORT int q3_short_conv_##SUFFIX(const void* u, int64_t row_in, const float* w, float* state, int64_t slot_stride, \
                                          const int* token_seq, const int* seq_start, const int* seq_slots, void* y,      \
-                                         int channels, int taps, int64_t n_tokens, int n_seqs, void* stream) {           \
-        if (n_tokens <= 0 || n_seqs <= 0) return 0;                                                                       \
-        if (channels <= 0 || taps <= 0 || taps > 64 || row_in < channels) return Q3_ERR_BAD_SIZE;                         \
-        constexpr int V = Pack<T>::N;                                                                                     \
-        const bool vec = channels % V == 0 && row_in % V == 0 && aligned16(u) && aligned16(y);                            \
-        const int64_t blocks = (n_tokens * (channels / (vec ? V : 1)) + 255) / 256;                                       \
-        const dim3 grid((unsigned)(blocks < 65536 ? blocks : 65536));                                                     \
-        const bool walk = vec && taps >= 2 && taps <= 4 && (n_tokens + 15) / 16 <= 65535;                                 \
-        int code = walk ? (taps == 2 ? short_conv_walk_launch<T, 2>((const T*)u, row_in, w, state, slot_stride, token_seq, \
-                                                                    seq_start, seq_slots, (T*)y, channels, n_tokens,      \
-                                                                    (cudaStream_t)stream)                                 \
-                           : taps == 3 ? short_conv_walk_launch<T, 3>((const T*)u, row_in, w, state, slot_stride,         \
-                                                                      token_seq, seq_start, seq_slots, (T*)y, channels,   \
-                                                                      n_tokens, (cudaStream_t)stream)                     \
-                                       : short_conv_walk_launch<T, 4>((const T*)u, row_in, w, state, slot_stride,         \
-                                                                      token_seq, seq_start, seq_slots, (T*)y, channels,   \
-                                                                      n_tokens, (cudaStream_t)stream))                    \
-                   : vec ? (int)q3_launch(short_conv_kernel<T, V>, grid, dim3(256), 0, (cudaStream_t)stream, (const T*)u,   \
-                                        row_in, w, (const float*)state, slot_stride, token_seq, seq_start, seq_slots,    \
-                                        (T*)y, channels, taps, n_tokens)                                                  \
-                       : (int)q3_launch(short_conv_kernel<T, 1>, grid, dim3(256), 0, (cudaStream_t)stream, (const T*)u,   \
-                                        row_in, w, (const float*)state, slot_stride, token_seq, seq_start, seq_slots,    \
-                                        (T*)y, channels, taps, n_tokens);                                                 \
-        if (code != 0 || taps == 1) return code;                                                                          \
-        const int64_t sblocks = ((int64_t)n_seqs * channels + 255) / 256;                                                 \
-        return (int)q3_launch(short_conv_state_kernel<T>, dim3((unsigned)(sblocks < 65536 ? sblocks : 65536)), dim3(256), \
-                              0, (cudaStream_t)stream, (const T*)u, row_in, state, slot_stride, seq_start, seq_slots,     \
-                              channels, taps, n_seqs);                                                                    \
+                                         int channels, int taps, int64_t n_tokens, int n_seqs, const float* bias,        \
+                                         int silu, void* stream) {                                                        \
+        return short_conv_launch<T>((const T*)u, row_in, w, state, slot_stride, token_seq, seq_start, seq_slots, (T*)y,   \
+                                    channels, taps, n_tokens, n_seqs, bias, silu, (cudaStream_t)stream);                  \
     }
 
 Q3_CONV_EXPORTS(f32, float)

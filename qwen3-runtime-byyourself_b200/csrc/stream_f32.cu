@@ -2,6 +2,9 @@
 // compute type T of the matrix products (float for the 32-bit path, bf16 for serving):
 //
 //   embedding_scaled : stream[t] = table[ids[t]] * scale                        (T -> float)
+//   embedding_sinusoid : the same plus a vector of the token's position p: stream[t, 2i] += sin(p f_i), stream[t, 2i + 1] +=
+//                      cos(p f_i).  A frequency is the sum of two floats, so that the angle is right to 32-bit rounding
+//                      whatever the position.
 //   sandwich_norm    : a branch output y (T) is normalised with weights of its own and added to
 //                      the stream, stream += y / rms(y) * w_post, and the sum is normalised for
 //                      the next part, out = T(stream / rms(stream) * w_pre): the norm after a
@@ -53,6 +56,29 @@ __global__ void embedding_scaled_kernel(const int* __restrict__ ids, const T* __
     const bool ok = id >= 0 && id < vocab;                 // an id outside the table gives a zero row
     const T* src = table + (int64_t)(ok ? id : 0) * hidden;
     for (int c = threadIdx.x; c < hidden; c += blockDim.x) out[t * hidden + c] = ok ? to_f32<T>(src[c]) * scale : 0.0f;
+}
+
+// freq: [(hidden + 1) / 2] leading terms, then as many second terms.
+template <typename T>
+__global__ void embedding_sinusoid_kernel(const int* __restrict__ ids, const int* __restrict__ positions, const T* __restrict__ table,
+                                          const float* __restrict__ freq, float* __restrict__ out, int hidden, int vocab, float scale) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t t = blockIdx.x;
+    const int id = ids[t], pairs = (hidden + 1) / 2;
+    const float p = (float)positions[t];
+    const bool ok = id >= 0 && id < vocab;                 // an id outside the table adds nothing to the position's vector
+    const T* src = table + (int64_t)(ok ? id : 0) * hidden;
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+        // angle = a + rest, a the rounded leading product and rest what it dropped with the second term's part
+        const float f = freq[i], a = p * f, rest = fmaf(p, f, -a) + p * freq[pairs + i];
+        float s, c;
+        sincosf(a, &s, &c);
+        const float sine = fmaf(rest, c, s), cosine = fmaf(-rest, s, c);
+        float* dst = out + t * hidden + 2 * i;
+        dst[0] = (ok ? to_f32<T>(src[2 * i]) * scale : 0.0f) + sine;
+        if (2 * i + 1 < hidden) dst[1] = (ok ? to_f32<T>(src[2 * i + 1]) * scale : 0.0f) + cosine;
+    }
 }
 
 // ---------------------------------------------------------------- norm after a branch + sum + norm before the next
@@ -374,6 +400,15 @@ static unsigned grid_for(int64_t work, int threads) {
 }  // namespace
 
 #define Q3_STREAM_EXPORTS(SUFFIX, T)                                                                                     \
+    Q3_EXPORT int q3_embedding_sinusoid_##SUFFIX(const int* ids, const int* positions, const void* table, const float* freq, \
+                                                 float* out, int64_t n_tokens, int hidden, int vocab, float scale,        \
+                                                 void* stream) {                                                          \
+        if (n_tokens <= 0) return 0;                                                                                      \
+        if (hidden <= 0 || vocab <= 0) return Q3_ERR_BAD_SIZE;                                                            \
+        if (n_tokens > 0x7fffffffLL) return Q3_ERR_TOO_LARGE;                                                             \
+        return (int)q3_launch(embedding_sinusoid_kernel<T>, dim3((unsigned)n_tokens), dim3(hidden >= 512 ? 256 : 64), 0,  \
+                              (cudaStream_t)stream, ids, positions, (const T*)table, freq, out, hidden, vocab, scale);    \
+    }                                                                                                                     \
     Q3_EXPORT int q3_embedding_scaled_##SUFFIX(const int* ids, const void* table, float* out, int64_t n_tokens, int hidden, \
                                                int vocab, float scale, void* stream) {                                  \
         if (n_tokens <= 0) return 0;                                                                                     \

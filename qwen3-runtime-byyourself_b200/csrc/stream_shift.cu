@@ -7,6 +7,7 @@
 //                     1  unit rms with a weight:   x / sqrt(mean(x^2) + eps) * w
 //                     2  dynamic tanh:             tanh(alpha x) * w + b      (no statistics)
 //                     3  nothing but the rounding: x                          (the output only)
+//                     4  layer norm with a weight: (x - mean) / sqrt(mean((x - mean)^2) + eps) * w
 //                 `out` is T, or float for a reader that goes on in 32-bit (a token shift).  With a list of rows
 //                 only those rows are read, nothing is written to the stream and out[r] belongs to rows[r] (the
 //                 model's tail).
@@ -68,6 +69,12 @@ template <typename T, int V> __device__ __forceinline__ void st_t(T* p, const fl
     }
 }
 
+// What a norm with statistics subtracts and multiplies by: mean and 1 / (rms or standard deviation).
+struct RowStats {
+    float mean, inv;
+};
+
+// The general form: any size, the row walked through the cache once per statistic.
 template <typename T, int V>
 __global__ void settle_norm_kernel(float* __restrict__ stream, const T* __restrict__ branch, NormSpec post, NormSpec pre,
                                    void* __restrict__ out, int out_f32, const int* __restrict__ rows, int size) {
@@ -78,27 +85,41 @@ __global__ void settle_norm_kernel(float* __restrict__ stream, const T* __restri
     float* xr = stream + row * size;
     const T* yr = post.kind != 0 ? branch + row * size : nullptr;
     const int first = threadIdx.x * V, stride = blockDim.x * V;
-    float inv_post = 0.0f;
-    if (post.kind == 1) {
-        float sq = 0.0f;
-        for (int c = first; c < size; c += stride) {
-            float y[V];
-            ld_t<T, V>(yr + c, y);
+    auto stats = [&](const NormSpec& spec, auto&& values) {
+        RowStats st = {0.0f, 0.0f};
+        if (spec.kind == 4) {
+            float sum = 0.0f;
+            for (int c = first; c < size; c += stride) {
+                float v[V];
+                values(c, v);
 #pragma unroll
-            for (int i = 0; i < V; ++i) sq += y[i] * y[i];
+                for (int i = 0; i < V; ++i) sum += v[i];
+            }
+            st.mean = block_sum(sum, scratch) / (float)size;
         }
-        inv_post = rsqrtf(block_sum(sq, scratch) / (float)size + post.eps);
-    }
-    // the sum of V elements: every thread forms the elements it owns the same way in both passes below
+        if (spec.kind == 1 || spec.kind == 4) {
+            float sq = 0.0f;
+            for (int c = first; c < size; c += stride) {
+                float v[V];
+                values(c, v);
+#pragma unroll
+                for (int i = 0; i < V; ++i) sq += (v[i] - st.mean) * (v[i] - st.mean);
+            }
+            st.inv = rsqrtf(block_sum(sq, scratch) / (float)size + spec.eps);
+        }
+        return st;
+    };
+    const RowStats sp = stats(post, [&](int c, float (&v)[V]) { ld_t<T, V>(yr + c, v); });
+    // the sum of V elements: every thread forms the elements it owns the same way in all passes below
     auto settled = [&](int c, float (&x)[V]) {
         ld_f32<V>(xr + c, x);
         if (post.kind == 0) return;
         float y[V], w[V];
         ld_t<T, V>(yr + c, y);
         ld_f32<V>(post.w + c, w);
-        if (post.kind == 1) {
+        if (post.kind != 2) {
 #pragma unroll
-            for (int i = 0; i < V; ++i) x[i] += y[i] * inv_post * w[i];
+            for (int i = 0; i < V; ++i) x[i] += (y[i] - sp.mean) * sp.inv * w[i];
         } else {
             float b[V];
             ld_f32<V>(post.b + c, b);
@@ -106,17 +127,7 @@ __global__ void settle_norm_kernel(float* __restrict__ stream, const T* __restri
             for (int i = 0; i < V; ++i) x[i] += tanhf(post.alpha * y[i]) * w[i] + b[i];
         }
     };
-    float inv_pre = 0.0f;
-    if (pre.kind == 1) {
-        float sq = 0.0f;
-        for (int c = first; c < size; c += stride) {
-            float x[V];
-            settled(c, x);
-#pragma unroll
-            for (int i = 0; i < V; ++i) sq += x[i] * x[i];
-        }
-        inv_pre = rsqrtf(block_sum(sq, scratch) / (float)size + pre.eps);
-    }
+    const RowStats sx = stats(pre, settled);
     T* out_t = reinterpret_cast<T*>(out) + (int64_t)blockIdx.x * size;
     float* out_f = reinterpret_cast<float*>(out) + (int64_t)blockIdx.x * size;
     for (int c = first; c < size; c += stride) {
@@ -125,11 +136,11 @@ __global__ void settle_norm_kernel(float* __restrict__ stream, const T* __restri
         if (post.kind != 0 && rows == nullptr) st_f32<V>(xr + c, x);
         if (pre.kind == 0) continue;
         float y[V];
-        if (pre.kind == 1) {
+        if (pre.kind == 1 || pre.kind == 4) {
             float w[V];
             ld_f32<V>(pre.w + c, w);
 #pragma unroll
-            for (int i = 0; i < V; ++i) y[i] = x[i] * inv_pre * w[i];
+            for (int i = 0; i < V; ++i) y[i] = (x[i] - sx.mean) * sx.inv * w[i];
         } else if (pre.kind == 2) {
             float w[V], b[V];
             ld_f32<V>(pre.w + c, w);
@@ -142,6 +153,89 @@ __global__ void settle_norm_kernel(float* __restrict__ stream, const T* __restri
         }
         if (out_f32) st_f32<V>(out_f + c, y);
         else st_t<T, V>(out_t + c, y);
+    }
+}
+
+// Rows of up to 8,192 values in packets of four: a thread keeps PER packets of stream and branch in registers, so both are
+// read once, and the loads are all on their way before the first statistic.
+template <typename T, int PER>
+__global__ void settle_norm_rows_kernel(float* __restrict__ stream, const T* __restrict__ branch, NormSpec post, NormSpec pre,
+                                        void* __restrict__ out, int out_f32, const int* __restrict__ rows, int size) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int64_t row = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
+    float* xr = stream + row * size;
+    const T* yr = post.kind != 0 ? branch + row * size : nullptr;
+    float x[PER][4], y[PER][4];
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int c = (p * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) x[p][i] = y[p][i] = 0.0f;
+        if (c < size) {
+            ld_f32<4>(xr + c, x[p]);
+            if (yr != nullptr) ld_t<T, 4>(yr + c, y[p]);
+        }
+    }
+    auto stats = [&](const NormSpec& spec, const float (&v)[PER][4]) {
+        RowStats st = {0.0f, 0.0f};
+        if (spec.kind == 4) {
+            float sum = 0.0f;
+#pragma unroll
+            for (int p = 0; p < PER; ++p) sum += (v[p][0] + v[p][1]) + (v[p][2] + v[p][3]);
+            st.mean = block_sum(sum, scratch) / (float)size;
+        }
+        if (spec.kind == 1 || spec.kind == 4) {
+            float sq = 0.0f;
+#pragma unroll
+            for (int p = 0; p < PER; ++p) {
+                if ((p * blockDim.x + threadIdx.x) * 4 >= size) continue;
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sq += (v[p][i] - st.mean) * (v[p][i] - st.mean);
+            }
+            st.inv = rsqrtf(block_sum(sq, scratch) / (float)size + spec.eps);
+        }
+        return st;
+    };
+    const RowStats sp = stats(post, y);
+    if (post.kind != 0) {
+#pragma unroll
+        for (int p = 0; p < PER; ++p) {
+            const int c = (p * blockDim.x + threadIdx.x) * 4;
+            if (c >= size) continue;
+            float w[4];
+            ld_f32<4>(post.w + c, w);
+            if (post.kind != 2) {
+#pragma unroll
+                for (int i = 0; i < 4; ++i) x[p][i] += (y[p][i] - sp.mean) * sp.inv * w[i];
+            } else {
+                float b[4];
+                ld_f32<4>(post.b + c, b);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) x[p][i] += tanhf(post.alpha * y[p][i]) * w[i] + b[i];
+            }
+            if (rows == nullptr) st_f32<4>(xr + c, x[p]);
+        }
+    }
+    if (pre.kind == 0) return;
+    const RowStats sx = stats(pre, x);
+    T* out_t = reinterpret_cast<T*>(out) + (int64_t)blockIdx.x * size;
+    float* out_f = reinterpret_cast<float*>(out) + (int64_t)blockIdx.x * size;
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int c = (p * blockDim.x + threadIdx.x) * 4;
+        if (c >= size) continue;
+        float w[4], b[4];
+        if (pre.kind != 3) ld_f32<4>(pre.w + c, w);
+        if (pre.kind == 2) ld_f32<4>(pre.b + c, b);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            if (pre.kind == 2) x[p][i] = tanhf(pre.alpha * x[p][i]) * w[i] + b[i];
+            else if (pre.kind != 3) x[p][i] = (x[p][i] - sx.mean) * sx.inv * w[i];
+        }
+        if (out_f32) st_f32<4>(out_f + c, x[p]);
+        else st_t<T, 4>(out_t + c, x[p]);
     }
 }
 
@@ -197,8 +291,8 @@ __global__ void side_gate_kernel(const T* __restrict__ a, const int* __restrict_
 }
 
 bool spec_ok(const NormSpec& s, bool is_output) {
-    if (s.kind < 0 || s.kind > 3 || (s.kind == 3 && !is_output)) return false;
-    if ((s.kind == 1 || s.kind == 2) && s.w == nullptr) return false;
+    if (s.kind < 0 || s.kind > 4 || (s.kind == 3 && !is_output)) return false;
+    if ((s.kind == 1 || s.kind == 2 || s.kind == 4) && s.w == nullptr) return false;
     return s.kind != 2 || s.b != nullptr;
 }
 
@@ -215,8 +309,16 @@ bool spec_ok(const NormSpec& s, bool is_output) {
             (pre.kind != 0 && out == nullptr) || n_rows > 0x7fffffffLL)                                                      \
             return Q3_ERR_BAD_SIZE;                                                                                          \
         if (packets4(size, {stream_rows, branch, post_w, post_b, pre_w, pre_b, out})) {                                       \
-            const int lanes = size >= 2048 ? 512 : (size >= 1024 ? 256 : 128);                                               \
-            return (int)q3_launch(settle_norm_kernel<T, 4>, dim3((unsigned)n_rows), dim3(lanes), 0, (cudaStream_t)stream,    \
+            const int packets = size / 4, per = packets <= 512 ? 1 : (packets <= 1024 ? 2 : 4);                              \
+            const int lanes = per == 1 ? (packets + 31) / 32 * 32 : ((packets + per - 1) / per + 31) / 32 * 32;              \
+            auto rows_of = [&](auto kernel) {                                                                                \
+                return (int)q3_launch(kernel, dim3((unsigned)n_rows), dim3(lanes), 0, (cudaStream_t)stream, stream_rows,     \
+                                      (const T*)branch, post, pre, out, out_f32, rows, size);                                \
+            };                                                                                                               \
+            if (packets <= 2048)                                                                                             \
+                return per == 1 ? rows_of(settle_norm_rows_kernel<T, 1>)                                                     \
+                                : (per == 2 ? rows_of(settle_norm_rows_kernel<T, 2>) : rows_of(settle_norm_rows_kernel<T, 4>)); \
+            return (int)q3_launch(settle_norm_kernel<T, 4>, dim3((unsigned)n_rows), dim3(512), 0, (cudaStream_t)stream,      \
                                   stream_rows, (const T*)branch, post, pre, out, out_f32, rows, size);                       \
         }                                                                                                                    \
         const int threads = size >= 2048 ? 512 : (size >= 512 ? 256 : 128);                                                  \

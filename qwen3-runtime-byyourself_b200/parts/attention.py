@@ -33,10 +33,17 @@ rotary encoding of the values over their whole head, by which every head's outpu
 part of the projection's); `learned_sink`: the sink's score is a number per head (tensor `sink`) instead of 0; `norm_once`:
 a normed query or key is rounded to the compute type once, after the rotation (else also after the division by its rms and
 after the weight, as Qwen3 is).
+
+And: `temperature` {coef, every}: a normed query is multiplied by 1 + coef ln((p + 1) // every + 1), p its position;
+`distance_bias` D: a number is added to every scaled score by the distance n between query and key, from a stored table
+(tensor `rel` [rows, heads]) whose first half of the rows stand for one distance each and whose others for stretches that grow
+by equal factors up to D, the last one for all that is further (`distance_buckets`); `shared_kv`: the layer has no keys and
+values of its own (no tensors of them) and reads another layer's cache.
 """
 from __future__ import annotations
 
-from typing import Optional
+from fractions import Fraction
+from typing import List, Optional
 
 import torch
 
@@ -62,7 +69,35 @@ FUSED_PROJECTION_KERNELS = []
 TENSOR_NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                 "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
                 "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "o_bias": "o_proj.bias", "value_mix": "value_mix",
-                "head_gate": "gate.weight", "conv_suffix": ".conv", "out_gate": "out_gate.weight", "sink": "sink"}
+                "head_gate": "gate.weight", "conv_suffix": ".conv", "out_gate": "out_gate.weight", "sink": "sink",
+                "rel": "rel"}
+
+
+def distance_buckets(rows: int, reach) -> List[int]:
+    """The row of a table of `rows` biases for every distance n = 0, 1, ... up to the first one that the last row stands for
+    (and so does every further one): n itself below half = rows // 2, then
+    min(rows - 1, half + floor(ln(n / half) / ln(reach / half) * (rows - half))).  The steps are found in whole numbers,
+    (n / half)^(rows - half) >= (reach / half)^k, so that a distance on a step falls on its right side."""
+    half, reach = rows // 2, Fraction(reach)
+    if rows < 2 or reach <= half:
+        raise ValueError(f"biases by distance: at least two rows ({rows}) and a reach ({float(reach)}) beyond half of them")
+    top, steps = rows - half, []
+    for k in range(1, top):                              # step k: the first distance of row half + k
+        lo, hi = half, int(reach) + 1
+        while lo < hi:
+            n = (lo + hi) // 2
+            if Fraction(n, half) ** top >= (reach / half) ** k:
+                hi = n
+            else:
+                lo = n + 1
+        steps.append(lo)
+    last = steps[-1] if steps else half
+    buckets, k = list(range(half)), 0
+    for n in range(half, last + 1):
+        while k < len(steps) and n >= steps[k]:
+            k += 1
+        buckets.append(half + k)
+    return buckets
 
 
 class GQAAttention(Part):
@@ -72,6 +107,7 @@ class GQAAttention(Part):
     o_bias = bias_v = conv_weight = w_gate = None
     mix_lambda = 0.0
     pool, tied_values, out_gate, learned_sink, norm_once, value_position = 0, False, False, False, False, None
+    temperature, distance_bias, shared_kv, bias_table = None, None, False, None
 
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, scale: float,
                  qk_norm: Optional[PartSpec] = None, position: Optional[PartSpec] = None,
@@ -80,7 +116,8 @@ class GQAAttention(Part):
                  names: Optional[dict] = None, value_heads: Optional[int] = None, out_float32: bool = False,
                  keep_first: int = 0, out_bias: bool = False, value_mix: Optional[str] = None, conv_taps: int = 0,
                  head_gate: bool = False, pool: int = 0, tied_values: bool = False, value_position: Optional[PartSpec] = None,
-                 out_gate: bool = False, learned_sink: bool = False, norm_once: bool = False):
+                 out_gate: bool = False, learned_sink: bool = False, norm_once: bool = False,
+                 temperature: Optional[dict] = None, distance_bias=None, bias_rows: Optional[int] = None, shared_kv: bool = False):
         self.sink_values = None      # float32 [num_heads]: the sink's score per head, for a part that has learned ones (else 0)
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
@@ -98,6 +135,16 @@ class GQAAttention(Part):
             raise ValueError("attention: values that are the keys have their size and heads, and no bias, blend or convolution of their own")
         if (out_gate or value_position or pool) and (conv_taps or value_mix or out_float32 or (value_heads or num_kv_heads) != num_kv_heads):
             raise ValueError("attention: an output gate, rotated values and pooled blocks do not go with convolutions, blends or shared values")
+        if shared_kv and (bias or value_mix or conv_taps or pool or out_gate or tied_values):
+            raise ValueError("attention on another layer's cache: no bias, blend, convolution, pooled blocks, gate or tied values")
+        if distance_bias is not None and (pool or out_float32):
+            raise ValueError("attention: biases by distance do not go with pooled blocks or a 32-bit output")
+        if temperature is not None and (not (norm_once or qk_norm is None) or int(temperature["every"]) <= 0):
+            raise ValueError("attention: a query temperature goes with norms that are rounded once, and a positive `every`")
+        self.temperature = (float(temperature["coef"]), int(temperature["every"])) if temperature else None
+        # `bias_rows`: the rows of the table; None: read from the tensor's shape when the weights arrive
+        self.distance_bias, self.bias_rows, self.shared_kv = distance_bias, bias_rows, bool(shared_kv)
+        self.bias_table = None       # float32 [num_heads, distances]: the biases spread out by distance
         self.pool, self.tied_values, self.out_gate = int(pool), bool(tied_values), bool(out_gate)
         self.learned_sink, self.norm_once = bool(learned_sink), bool(norm_once)
         self.value_position = build_part("position", value_position) if value_position else None
@@ -132,15 +179,19 @@ class GQAAttention(Part):
     def special(self) -> bool:
         """Options that change what a query, a key or a value is made from, or what becomes of the output: the kernels that
         prepare a step's rows themselves do not take them."""
-        return bool(self.pool or self.tied_values or self.value_position or self.out_gate or (self.norm_once and self.q_norm is not None))
+        return bool(self.pool or self.tied_values or self.value_position or self.out_gate or self.temperature or self.shared_kv
+                    or self.distance_bias is not None or (self.norm_once and self.q_norm is not None))
 
     # -- weights
     def weight_specs(self, prefix: str) -> dict:
         p, n = prefix + self.prefix, self.names
         nq, nkv, d, vd, H, nv = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.hidden_size, self.value_heads
-        specs = {p + n["q"]: WeightSpec((nq * d, H)), p + n["k"]: WeightSpec((nkv * d, H)),
-                 p + n["o"]: WeightSpec((H, self.output_width()))}
-        if not self.tied_values:
+        specs = {p + n["q"]: WeightSpec((nq * d, H)), p + n["o"]: WeightSpec((H, self.output_width()))}
+        if not self.shared_kv:
+            specs[p + n["k"]] = WeightSpec((nkv * d, H))
+        if self.distance_bias is not None:
+            specs[p + n["rel"]] = WeightSpec((self.bias_rows or -1, nq), "bias")
+        if not self.tied_values and not self.shared_kv:
             specs[p + n["v"]] = WeightSpec((nv * vd, H))
         if self.out_gate:
             specs[p + n["out_gate"]] = WeightSpec((nq * vd, H))
@@ -170,7 +221,7 @@ class GQAAttention(Part):
     def bind(self, weights: dict, prefix: str, dtype, device) -> None:
         p, n = prefix + self.prefix, self.names
         nq, nkv, d = self.num_heads, self.num_kv_heads, self.head_dim
-        parts = ["q", "k"] + ([] if self.tied_values else ["v"]) + (["out_gate"] if self.out_gate else [])
+        parts = ["q"] + ([] if self.shared_kv else ["k"] + ([] if self.tied_values else ["v"])) + (["out_gate"] if self.out_gate else [])
         self.w_qkv = fuse_rows(weights, [p + n[k] for k in parts])
         self.w_o = weights.pop(p + n["o"]).contiguous()
         if self.has_bias:
@@ -178,6 +229,11 @@ class GQAAttention(Part):
             getattr(weights, "wait", lambda: None)()          # a streamed checkpoint: the tensors are in place now
             self.bias = torch.cat([t.to(device=device, dtype=torch.float32).reshape(-1) for t in tensors]).contiguous()
         f32 = dict(device=device, dtype=torch.float32)
+        if self.distance_bias is not None:
+            rel = weights[p + n["rel"]]
+            getattr(weights, "wait", lambda: None)()
+            rows = torch.tensor(distance_buckets(rel.shape[0], self.distance_bias), device=rel.device)
+            self.bias_table = rel.to(**f32)[rows.to(device)].t().contiguous()
         if self.learned_sink:
             self.sink_values = weights[p + n["sink"]].to(**f32).reshape(-1).contiguous()
         if self.out_bias:
@@ -232,6 +288,8 @@ class GQAAttention(Part):
 
     def projection_width(self) -> int:
         """Columns of the q/k/v projection (and of the output gate's, if there is one)."""
+        if self.shared_kv:
+            return self.num_heads * self.head_dim
         return (self.num_heads + self.num_kv_heads) * self.head_dim + (0 if self.tied_values else self.value_heads * self.value_dim) \
             + (self.num_heads * self.value_dim if self.out_gate else 0)
 
@@ -252,6 +310,8 @@ class GQAAttention(Part):
         N = ctx.n_tokens
         table = ctx.page_tables[cache.group]
         attn = ctx.scratch.get("attn.ctx", (N, nq * vd), torch.float32 if self.out_float32 else ctx.dtype)
+        if self.shared_kv and not cache.shared:
+            raise ops.KernelError("attention without keys of its own needs another layer's cache")
         norm_eps = self.q_norm.eps if self.q_norm is not None else 0.0
         qw = self.q_norm.weight if self.q_norm is not None else None
         kw = self.k_norm.weight if self.k_norm is not None else None
@@ -295,7 +355,7 @@ class GQAAttention(Part):
             ops.qkv_prepare(qkv, q, cache.keys, cache.values, qw, kw, cos, sin, ctx.token_seq, ctx.token_pos, table,
                             N, nq, nkv, d, norm_eps, write_kv=not cache.shared, bias=self.bias, value_dim=vd,
                             value_heads=self.value_heads, tied_values=self.tied_values, norm_once=self.norm_once,
-                            value_cos=v_cos, value_sin=v_sin)
+                            value_cos=v_cos, value_sin=v_sin, temperature=self.temperature)
         elif self.special():
             raise ops.KernelError("this attention takes a position encoding with tables, or none")
         else:
@@ -325,7 +385,7 @@ class GQAAttention(Part):
                                     nq, nkv, self.head_dim, vd, self.scale, self.softcap, self.chunk, self.sink, splits,
                                     window=self.window, value_heads=self.value_heads, sink_values=self.sink_values,
                                     keep_first=self.keep_first, pool=self.pooled(ctx, cache), pool_write=not cache.shared,
-                                    back_cos=back_cos, back_sin=back_sin, gate=gate)
+                                    back_cos=back_cos, back_sin=back_sin, gate=gate, bias=self.bias_table)
 
     def pooled(self, ctx, cache):
         """The pooled blocks of this layer as the kernels take them (None: there are none)."""
@@ -348,7 +408,7 @@ class GQAAttention(Part):
                               self.num_heads, self.num_kv_heads, self.head_dim, self.scale, self.window,
                               value_dim=self.value_dim, softcap=self.softcap, chunk=self.chunk, sink=self.sink,
                               value_heads=self.value_heads, sink_values=self.sink_values, keep_first=self.keep_first,
-                              pool=self.pooled(ctx, cache))
+                              pool=self.pooled(ctx, cache), bias=self.bias_table)
 
     def _prepare_unfused(self, qkv, q, cache, ctx, table, qw, kw, eps) -> None:
         """A position encoding without kernel tables: norm, then `apply_`, then the cache write."""
@@ -468,7 +528,7 @@ def _prefill_capped_kernel(part, q, cache, out, ctx, table) -> bool:
     ops.attention_capped_prefill(q, cache.keys, cache.values, out, ctx.seq_start, ctx.seq_pos0, table, ctx.n_seqs, ctx.max_new,
                                  part.num_heads, part.num_kv_heads, part.head_dim, part.value_dim, part.scale, part.softcap,
                                  part.chunk, part.sink, window=part.window, value_heads=part.value_heads,
-                                 sink_values=part.sink_values, keep_first=part.keep_first, pool=part.pooled(ctx, cache))
+                                 sink_values=part.sink_values, keep_first=part.keep_first, pool=part.pooled(ctx, cache), bias=part.bias_table)
     return True
 
 
@@ -480,7 +540,7 @@ def _prefill_capped_tcgen05_kernel(part, q, cache, out, ctx, table) -> bool:
         return False
     ops.attention_capped_prefill_tc(q[:ctx.n_tokens], cache.keys, cache.values, out, ctx.seq_start, ctx.seq_pos0, table,
                                     ctx.n_seqs, ctx.max_new, ctx.n_tokens, part.num_heads, part.num_kv_heads, part.head_dim,
-                                    part.scale, part.softcap, part.chunk, part.sink, sink_values=part.sink_values)
+                                    part.scale, part.softcap, part.chunk, part.sink, sink_values=part.sink_values, bias=part.bias_table)
     return True
 
 

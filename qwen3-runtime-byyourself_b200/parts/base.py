@@ -21,7 +21,7 @@ Interfaces (duck-typed; `Part` gives the defaults):
   block           built from (spec params, mixer, feed_forward); weight_specs/bind cover
                   its own norms; forward(residual, delta, ctx, cache) -> (residual, delta):
                   the hidden state is residual + delta, the sum is left to the next norm.
-  embedding       forward(token_ids, out) -> [N, hidden]
+  embedding       forward(token_ids, out, token_pos) -> [N, hidden]
   head            forward(x, out) -> float32 logits [R, vocab]
   stream          a step between layers: weight_specs(name), bind(weights, name, dtype, device),
                   forward(residual, delta, x0, ctx) -> (residual, delta), x0 being the embedding's output

@@ -10,6 +10,8 @@ in float32 whatever the compute type.  Here `delta` is a `NormedBranch`: a subla
 that still has to be normalised and added.  Whoever comes next does it (the next block, a
 stream step or the model's tail), in the same kernel that normalises the sum for its own
 input, so a layer costs two passes over the hidden state.
+
+`post_norm`: a norm after every sublayer only, x += norm(mixer(x)), on such a stream; the sublayers read the stream itself.
 """
 from __future__ import annotations
 
@@ -107,6 +109,113 @@ class SandwichNormBlock(Part):
         return residual, NormedBranch(self.feed_forward.forward(normed, ctx), self.norms[3])
 
 
+def settle_any(residual, pending, norm, out):
+    """As `settle`, with norms of any kind that `ops.settle_norm` takes; `norm` "round": out is the rounded sum."""
+    from ..csrc import ops
+    if pending is not None and not isinstance(pending, NormedBranch):
+        raise TypeError("a float32 stream takes a NormedBranch as its pending sum")
+    return ops.settle_norm(residual, pending.branch if pending else None, pending.norm if pending else None, norm, out)
+
+
+def finish_any(residual, pending, final_norm, ctx, out, normalize: bool = True):
+    """out[r] = final_norm(stream + pending) of wanted row r (the pending sum is done in registers for those rows only:
+    nothing reads the stream after the tail)."""
+    from ..csrc import ops
+    norm = final_norm if normalize else "round"
+    if ctx.want_all:
+        return settle_any(residual, pending, norm, out)
+    return ops.settle_norm(residual, pending.branch if pending else None, pending.norm if pending else None, norm, out,
+                           rows=ctx.want_rows[:ctx.n_want], n_rows=ctx.n_want, compute_dtype=ctx.dtype)
+
+
+class TokenSideInput(Part):
+    """A gated slice of a second embedding of the token, added after a layer's last sublayer: with e the columns
+    [index * dim, (index + 1) * dim) of a table that all layers share, g = gelu_tanh(W_gate x) * e, y = W_proj g and
+    x += y / sqrt(mean(y^2) + eps) * w.  The names are relative to the layer's prefix but for `table`."""
+
+    def __init__(self, hidden_size: int, table: str, vocab: int, columns: int, dim: int, index: int, eps: float, gate: str,
+                 proj: str, norm: str):
+        self.hidden_size, self.dim, self.index = int(hidden_size), int(dim), int(index)
+        self.table_name, self.table_shape, self.names = table, (int(vocab), int(columns)), (gate, proj, norm)
+        self.norm = build_part("norm", PartSpec("rms_norm", {"size": hidden_size, "eps": eps}))
+        self.table = self.w_gate = self.w_proj = None
+
+    def weight_specs(self, prefix: str) -> dict:
+        from ..weights.loader import WeightSpec
+        gate, proj, norm = self.names
+        return {self.table_name: WeightSpec(self.table_shape), prefix + gate: WeightSpec((self.dim, self.hidden_size)),
+                prefix + proj: WeightSpec((self.hidden_size, self.dim)), **self.norm.weight_specs(prefix + norm)}
+
+    def bind(self, weights: dict, prefix: str, dtype, device) -> None:
+        gate, proj, norm = self.names
+        self.table = weights[self.table_name]            # one tensor for all layers: not taken out of `weights`
+        self.w_gate = weights.pop(prefix + gate).contiguous()
+        self.w_proj = weights.pop(prefix + proj).contiguous()
+        self.norm.bind(weights, prefix + norm, dtype, device)
+
+    def forward(self, residual, pending, ctx):
+        """Settles `pending` and returns the side input's own pending sum."""
+        from ..csrc import ops
+        from .linear import linear
+        N, H = ctx.n_tokens, self.hidden_size
+        rounded = ctx.scratch.get("block.normed", (N, H), ctx.dtype)
+        settle_any(residual, pending, "round", rounded)
+        a = ctx.scratch.get("side.a", (N, self.dim), ctx.dtype)
+        linear(rounded, self.w_gate, a)
+        g = ctx.scratch.get("side.g", (N, self.dim), ctx.dtype)
+        ops.side_gate(a, ctx.token_ids, self.table, g, self.index * self.dim)
+        y = ctx.scratch.get("side.out", (N, H), ctx.dtype)
+        return NormedBranch(linear(g, self.w_proj, y), self.norm)
+
+
+class PostNormBlock(Part):
+    """Sublayers that read the float32 stream itself and whose output alone is normed, x += norm_1(mixer(x)) and then
+    x += norm_2(ff(x)) (a layer may lack the feed-forward), with norms of any kind that `ops.settle_norm` takes, and
+    optionally a token side input after them (`side`: the parameters of `TokenSideInput` but for the width).
+
+    A sublayer's input is the stream rounded to the compute type.  Every sum is left pending and done by the next reader's
+    kernel, which rounds the sum for its own input in the same pass."""
+    stream_dtype = "float32"
+
+    def __init__(self, mixer, feed_forward, norm: PartSpec, hidden_size: int, names=("norm1", "norm2"), side=None):
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.hidden_size, self.names = int(hidden_size), tuple(names)
+        self.norms = [build_part("norm", norm) for _ in range(2 if feed_forward is not None else 1)]
+        self.side = TokenSideInput(hidden_size, **side) if side else None
+
+    def parts(self, prefix: str):
+        yield from ((norm, prefix + name) for norm, name in zip(self.norms, self.names))
+        yield from ((part, prefix) for part in (self.mixer, self.feed_forward, self.side) if part is not None)
+
+    def weight_specs(self, prefix: str) -> dict:
+        specs = {}
+        for part, name in self.parts(prefix):
+            specs.update(part.weight_specs(name))
+        return specs
+
+    def ignorable(self, prefix: str):
+        """The norm of a feed-forward that the layer does not have may be stored all the same."""
+        return [] if self.feed_forward is not None else list(self.norms[0].weight_specs(prefix + self.names[1]))
+
+    def bind(self, weights: dict, prefix: str, dtype, device) -> None:
+        for part, name in self.parts(prefix):
+            part.bind(weights, name, dtype, device)
+
+    def forward(self, residual, delta, ctx, cache):
+        x = ctx.scratch.get("block.normed", (ctx.n_tokens, self.hidden_size), ctx.dtype)
+        settle_any(residual, delta, "round", x)
+        pending = NormedBranch(self.mixer.forward(x, ctx, cache), self.norms[0])
+        if self.feed_forward is not None:
+            settle_any(residual, pending, "round", x)
+            pending = NormedBranch(self.feed_forward.forward(x, ctx), self.norms[1])
+        if self.side is not None:
+            pending = self.side.forward(residual, pending, ctx)
+        return residual, pending
+
+    def finish(self, residual, pending, final_norm, ctx, out, normalize: bool = True):
+        return finish_any(residual, pending, final_norm, ctx, out, normalize)
+
+
 class ShiftSandwichBlock(Part):
     """Sandwich-norm sublayers on a float32 stream, x += norm_b(mixer(shift(norm_a(x)))), then the same around the
     feed-forward without the shift (a layer may lack it), with norms of any kind that `ops.settle_norm` takes.
@@ -115,10 +224,8 @@ class ShiftSandwichBlock(Part):
     row before it in the sequence as it was before this step (zeros before the first token).  The last h of a sequence
     is part of its state: `state_size` float32 values per sequence in the layer's cache (`LayerCache.block_state`).
 
-    Token side input (`side`, optional), after the feed-forward: with e the columns [index * dim, (index + 1) * dim) of
-    a second embedding table that all layers share, g = gelu_tanh(W_gate x) * e, y = W_proj g and
-    x += y / sqrt(mean(y^2) + eps) * w.  `side` = {table, vocab, columns, dim, index, eps, gate, proj, norm}, the names
-    relative to the layer's prefix but for `table`.
+    Token side input (`side`, optional), after the feed-forward: see `TokenSideInput`, whose parameters but for the width
+    `side` holds.
 
     Every sum is left pending and done by the next reader's kernel, which normalises the sum for its own input."""
     stream_dtype = "float32"
@@ -130,10 +237,7 @@ class ShiftSandwichBlock(Part):
         self.norms = [build_part("norm", norm) for _ in range(4 if feed_forward is not None else 2)]
         self.state_size = self.hidden_size
         self.mu = None
-        self.side = dict(side) if side else None
-        self.side_norm = self.side_table = self.w_side_gate = self.w_side_proj = None
-        if self.side:
-            self.side_norm = build_part("norm", PartSpec("rms_norm", {"size": self.hidden_size, "eps": self.side["eps"]}))
+        self.side = TokenSideInput(hidden_size, **side) if side else None
 
     def weight_specs(self, prefix: str) -> dict:
         from ..weights.loader import WeightSpec
@@ -141,12 +245,8 @@ class ShiftSandwichBlock(Part):
         for part, name in zip(self.norms, self.names):
             specs.update(part.weight_specs(prefix + name))
         specs[prefix + self.shift_name] = WeightSpec((H,), "bias")
-        if self.side:
-            sd = self.side
-            specs[sd["table"]] = WeightSpec((sd["vocab"], sd["columns"]))
-            specs[prefix + sd["gate"]] = WeightSpec((sd["dim"], H))
-            specs[prefix + sd["proj"]] = WeightSpec((H, sd["dim"]))
-            specs.update(self.side_norm.weight_specs(prefix + sd["norm"]))
+        if self.side is not None:
+            specs.update(self.side.weight_specs(prefix))
         specs.update(self.mixer.weight_specs(prefix))
         if self.feed_forward is not None:
             specs.update(self.feed_forward.weight_specs(prefix))
@@ -163,60 +263,33 @@ class ShiftSandwichBlock(Part):
         for part, name in zip(self.norms, self.names):
             part.bind(weights, prefix + name, dtype, device)
         self.mu = weights[prefix + self.shift_name].to(device=device, dtype=torch.float32).contiguous()
-        if self.side:
-            sd = self.side
-            self.side_table = weights[sd["table"]]           # one tensor for all layers: not taken out of `weights`
-            self.w_side_gate = weights.pop(prefix + sd["gate"]).contiguous()
-            self.w_side_proj = weights.pop(prefix + sd["proj"]).contiguous()
-            self.side_norm.bind(weights, prefix + sd["norm"], dtype, device)
+        if self.side is not None:
+            self.side.bind(weights, prefix, dtype, device)
         self.mixer.bind(weights, prefix, dtype, device)
         if self.feed_forward is not None:
             self.feed_forward.bind(weights, prefix, dtype, device)
 
-    @staticmethod
-    def _settle(residual, pending, norm, out):
-        from ..csrc import ops
-        if pending is not None and not isinstance(pending, NormedBranch):
-            raise TypeError("a float32 stream takes a NormedBranch as its pending sum")
-        return ops.settle_norm(residual, pending.branch if pending else None, pending.norm if pending else None, norm, out)
-
     def forward(self, residual, delta, ctx, cache):
         import torch
         from ..csrc import ops
-        from .linear import linear
         N, H = ctx.n_tokens, self.hidden_size
         if cache.block_state is None:
             raise ops.KernelError("the token shift keeps a row per sequence: the cache was built without block_state")
         h = ctx.scratch.get("block.h32", (N, H), torch.float32)
-        self._settle(residual, delta, self.norms[0], h)
+        settle_any(residual, delta, self.norms[0], h)
         shifted = ctx.scratch.get("block.normed", (N, H), ctx.dtype)
         ops.token_shift(h, self.mu, cache.block_state, shifted, ctx.token_seq, ctx.seq_start, ctx.seq_slots, N)
         pending = NormedBranch(self.mixer.forward(shifted, ctx, cache), self.norms[1])
         if self.feed_forward is not None:
             normed = ctx.scratch.get("block.normed", (N, H), ctx.dtype)
-            self._settle(residual, pending, self.norms[2], normed)
+            settle_any(residual, pending, self.norms[2], normed)
             pending = NormedBranch(self.feed_forward.forward(normed, ctx), self.norms[3])
-        if self.side:
-            sd = self.side
-            rounded = ctx.scratch.get("block.normed", (N, H), ctx.dtype)
-            self._settle(residual, pending, "round", rounded)
-            a = ctx.scratch.get("side.a", (N, sd["dim"]), ctx.dtype)
-            linear(rounded, self.w_side_gate, a)
-            g = ctx.scratch.get("side.g", (N, sd["dim"]), ctx.dtype)
-            ops.side_gate(a, ctx.token_ids, self.side_table, g, sd["index"] * sd["dim"])
-            y = ctx.scratch.get("side.out", (N, H), ctx.dtype)
-            pending = NormedBranch(linear(g, self.w_side_proj, y), self.side_norm)
+        if self.side is not None:
+            pending = self.side.forward(residual, pending, ctx)
         return residual, pending
 
     def finish(self, residual, pending, final_norm, ctx, out, normalize: bool = True):
-        """out[r] = final_norm(stream + pending) of wanted row r (the pending sum is done in registers for those rows
-        only: nothing reads the stream after the tail)."""
-        from ..csrc import ops
-        if ctx.want_all:
-            return self._settle(residual, pending, final_norm if normalize else "round", out)
-        return ops.settle_norm(residual, pending.branch if pending else None, pending.norm if pending else None,
-                               final_norm if normalize else "round", out, rows=ctx.want_rows[:ctx.n_want], n_rows=ctx.n_want,
-                               compute_dtype=ctx.dtype)
+        return finish_any(residual, pending, final_norm, ctx, out, normalize)
 
 
 class HyperPending:
@@ -319,6 +392,7 @@ class HyperConnectionBlock(Part):
 
 
 register_part("block", "hyper_connections", HyperConnectionBlock)
+register_part("block", "post_norm", PostNormBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "shift_sandwich", ShiftSandwichBlock)

@@ -111,7 +111,7 @@ class Model:
         N, H = ctx.n_tokens, self.plan.hidden_size
         stream_dtype = self.residual_dtype or ctx.dtype
         residual = ctx.scratch.get("model.residual", (N, self.plan.streams * H), stream_dtype)
-        self.embedding.forward(ctx.token_ids[:N], residual)
+        self.embedding.forward(ctx.token_ids[:N], residual, ctx.token_pos[:N])
         x0 = None
         if self.stream_steps:                              # the embedding's output is read again later: keep it
             x0 = residual

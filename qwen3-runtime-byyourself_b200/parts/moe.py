@@ -13,6 +13,8 @@ without limit.  `shared_size`: one more expert of that inner size (`shared.gate 
 output is multiplied by sigmoid(w_sg . x), one number per token (`shared.sg`, computed with the router's logits), and added
 (`shared_gate=False`: added as it is).  `expert_activation="relu2"`: an expert, and the shared one, is W_down max(W_up x, 0)^2,
 without a gate.  `correction=False`: the choice is made on the scores alone and no vector is stored.
+`router_bias` (with "top_logits"): a stored vector is added to the logits.  A shared expert of clamped experts is clamped like
+them, with `shared_limit` of its own.
 
 Nothing on the host depends on how many tokens an expert gets: the pairs (token, choice) are laid out expert by
 expert on the device and the experts' products walk that layout, so a decode step with this part can be captured.
@@ -36,7 +38,7 @@ class RoutedExperts(Part):
                  group_count: int = 1, group_keep: int = 1, prefix: str = "", alpha: float = SIGMOID_ALPHA,
                  names: Optional[dict] = None, scoring: str = "softmax_all", expert_activation: str = "clamped",
                  shared_size: Optional[int] = None, group_mark: str = "best", weight_scale: float = 1.0, shared_gate: bool = True,
-                 correction: bool = True):
+                 correction: bool = True, router_bias: bool = False, shared_limit: Optional[float] = None):
         outputs = experts + identity
         if not 0 < top <= outputs or outputs % group_count or not 0 < group_keep <= group_count \
                 or group_keep * (outputs // group_count) < top:
@@ -45,12 +47,15 @@ class RoutedExperts(Part):
             raise ValueError("routed experts: scoring 'softmax_all', 'sigmoid' or 'top_logits', expert_activation 'clamped', 'silu' or 'relu2'")
         if scoring == "top_logits" and (group_count != 1 or weight_scale != 1.0):
             raise ValueError("routed experts: groups and a weight scale go with scoring 'softmax_all' or 'sigmoid'")
+        if router_bias and scoring != "top_logits":
+            raise ValueError("routed experts: a bias on the logits goes with scoring 'top_logits'")
         if group_mark not in ("best", "top2_sum"):
             raise ValueError("routed experts: group_mark 'best' or 'top2_sum'")
         self.group_mark, self.weight_scale = group_mark, float(weight_scale)
         self.scoring, self.expert_activation = scoring, expert_activation
         self.gated, self.shared_gate = expert_activation != "relu2", bool(shared_gate)
         self.corrected = bool(correction) and scoring != "top_logits"
+        self.router_bias = bool(router_bias)
         self.shared_size = int(shared_size) if shared_size else None
         self.hidden_size, self.intermediate_size, self.prefix = int(hidden_size), int(intermediate_size), prefix
         self.experts, self.identity, self.top = int(experts), int(identity), int(top)
@@ -58,7 +63,7 @@ class RoutedExperts(Part):
         if expert_activation == "silu":
             self.limit, self.alpha, self.up_offset = float("inf"), 1.0, 0.0
         self.group_count, self.group_keep = int(group_count), int(group_keep)
-        self.names = dict({"router": "router", "correction": "correction", "expert": "e{}.", "gate": "gate", "up": "up",
+        self.names = dict({"router": "router", "correction": "correction", "router_bias": "router.b", "expert": "e{}.", "gate": "gate", "up": "up",
                            "down": "down", "shared": "shared.", "shared_gate": "shared.sg"}, **(names or {}))
         self.w_router = self.correction = self.w_gate_up = self.w_down = None
         self.shared = None
@@ -69,7 +74,9 @@ class RoutedExperts(Part):
         elif self.shared_size:
             from .mlp import SwiGLU
             self.shared = SwiGLU(hidden_size, self.shared_size, prefix=prefix + self.names["shared"],
-                                 names={k: self.names[k] for k in ("gate", "up", "down")})
+                                 names={k: self.names[k] for k in ("gate", "up", "down")},
+                                 activation="clamped" if expert_activation == "clamped" else "silu",
+                                 limit=float("inf") if shared_limit is None else float(shared_limit), alpha=self.alpha)
 
     def _expert(self, p: str, e: int, which: str) -> str:
         return p + self.names["expert"].format(e) + self.names[which]
@@ -79,6 +86,8 @@ class RoutedExperts(Part):
         specs = {p + self.names["router"]: WeightSpec((self.experts + self.identity, H))}
         if self.corrected:
             specs[p + self.names["correction"]] = WeightSpec((self.experts + self.identity,), "bias")
+        if self.router_bias:
+            specs[p + self.names["router_bias"]] = WeightSpec((self.experts + self.identity,), "bias")
         if self.shared is not None:
             if self.shared_gate:
                 specs[p + self.names["shared_gate"]] = WeightSpec((1, H))
@@ -99,6 +108,8 @@ class RoutedExperts(Part):
             self.w_router = weights.pop(p + self.names["router"]).contiguous()
         if self.corrected:
             self.correction = weights[p + self.names["correction"]].to(device=device, dtype=torch.float32).contiguous()
+        if self.router_bias:
+            self.correction = weights[p + self.names["router_bias"]].to(device=device, dtype=torch.float32).contiguous()
         if self.experts:
             # [expert, gate rows then up rows, hidden] (or the up rows alone) and [expert, hidden, ff], each one matrix
             parts = ("gate", "up") if self.gated else ("up",)

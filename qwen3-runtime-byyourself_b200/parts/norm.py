@@ -16,18 +16,25 @@ from .base import Part, register_part
 class RMSNorm(Part):
     stream_kind = "rms"          # how the kernels of a float32 stream apply this part (ops.NORM_KINDS)
 
-    def __init__(self, size: int, eps: float, one_plus: bool = False, groups: int = 1):
+    def __init__(self, size: int, eps: float, one_plus: bool = False, groups: int = 1, weighted: bool = True):
         """`one_plus`: the stored weight lies around zero and the norm multiplies by 1 + weight.  `groups`: the row is split
-        into so many equal consecutive parts, each divided by its own rms (applied by the kernels of a float32 stream)."""
+        into so many equal consecutive parts, each divided by its own rms (applied by the kernels of a float32 stream).
+        `weighted=False`: no weight is stored, the row is brought to unit rms alone."""
+        self.weighted = bool(weighted)
         self.size, self.eps, self.one_plus, self.groups = int(size), float(eps), bool(one_plus), int(groups)
         if self.groups <= 0 or self.size % self.groups:
             raise ValueError("a norm in groups: the groups divide the row")
         self.weight = None
 
     def weight_specs(self, name: str) -> dict:
+        if not self.weighted:
+            return {}
         return {name: WeightSpec((self.size,), "bias" if self.one_plus else "norm")}
 
     def bind(self, weights: dict, name: str, dtype, device) -> None:
+        if not self.weighted:
+            self.weight = torch.ones(self.size, dtype=torch.float32, device=device)
+            return
         # a scale vector is used in 32-bit whatever it was stored in (exact for bfloat16)
         self.weight = weights[name].to(device=device, dtype=torch.float32).contiguous()
         if self.one_plus:
@@ -38,6 +45,27 @@ class RMSNorm(Part):
         if self.groups > 1:
             raise ops.KernelError("a norm in groups is applied on a float32 stream by sandwich_norm")
         return ops.rms_norm(x, self.weight, self.eps, out, delta)
+
+
+class LayerNorm(Part):
+    """y = (x - mean) / sqrt(variance + eps) * weight, without a bias, the variance being the mean of the squared deviations.
+    Applied by the kernels of a float32 stream (`ops.settle_norm`)."""
+    stream_kind = "layer"
+
+    def __init__(self, size: int, eps: float):
+        self.size, self.eps = int(size), float(eps)
+        self.weight = None
+
+    def weight_specs(self, name: str) -> dict:
+        return {name: WeightSpec((self.size,), "norm")}
+
+    def bind(self, weights: dict, name: str, dtype, device) -> None:
+        self.weight = weights[name].to(device=device, dtype=torch.float32).contiguous()
+
+    def __call__(self, x: torch.Tensor, out: torch.Tensor, delta=None) -> torch.Tensor:
+        if x.dtype != torch.float32 or delta is not None:
+            raise ops.KernelError("layer_norm is applied on a float32 stream by settle_norm")
+        return ops.settle_norm(x, None, None, self, out)
 
 
 class DynamicTanh(Part):
@@ -71,3 +99,4 @@ class DynamicTanh(Part):
 
 register_part("norm", "rms_norm", RMSNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)
+register_part("norm", "layer_norm", LayerNorm)
