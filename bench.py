@@ -7,6 +7,7 @@ model with random weights in bfloat16 on one B200, batch 8 at a context of 4,096
     python bench.py --designs fagunex    (a Fagunex model beside the Lagulorn model of the same widths)
     python bench.py --designs fedinex    (a Fedinex model beside the Fagunex model of the same widths)
     python bench.py --designs vogerax    (a Vogerax model beside the Fedinex model of the same widths)
+    python bench.py --designs vinozen    (a Vinozen model beside the Vogerax model of the same widths)
 
 Prints ONE JSON line.  A "step" is one decode step of the whole batch.
   value     decoded tokens a second, timed on the device with CUDA events around K steps;
@@ -562,6 +563,42 @@ def vogerax_side_by_side(q, torch, Sampler, steps, warmup, batch=8, context=4096
     return out
 
 
+def vinozen_config(width, heads, kv, d, ff, layers, experts=16, top=2):
+    """A Vinozen model of the widths of the Vogerax model beside it: a state space (2 width / 64 heads of 64, a state of 128 rows,
+    8 groups, four taps) and attention over every earlier key (unit-rms queries and keys, a temperature, 32 biases that reach
+    128 tokens, a sink) in turn, every other attention layer on the keys of the one before it; a token side input of 256
+    columns a layer.  The first layer's feed-forward is dense, the others routed (`experts` experts of ff / (2 top), `top` per
+    token) with a shared expert of the same size."""
+    space = {"type": "mamba2", "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}}
+    attention = {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5, "bias_max": 128,
+                                                 "bias_rows": 32, "q_temp": {"coef": 0.1, "every": 1024}}}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top), "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": ff // (2 * top), "limit": 7.0}}
+
+    def kind(i):
+        if i % 2 == 0:
+            return space
+        return attention if i % 4 == 1 else {"type": "attention", "mixer": dict(attention["mixer"], kv_from=i - 2)}
+    return {"architecture": "Vinozen", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": width ** 0.5}, "norm": {"eps": 1e-6},
+            "token_side": {"dim": 256}, "layers": [dict(kind(i), mlp={"kind": "dense", "ff": ff} if i == 0 else moe) for i in range(layers)]}
+
+
+def vinozen_side_by_side(q, torch, Sampler, steps, warmup, batch=8, context=4096):
+    """Vinozen beside Vogerax, the closest of the other designs (a 32-bit hidden state, attention over every earlier key with normed
+    queries and keys and a sink, a recurrence, routed experts with a shared one), at equal widths (random weights, bfloat16):
+    decode at `batch` x `context`, a prompt step of 2,048 tokens, and the time of every kernel of one step of each kind."""
+    import numpy as np
+    out = {"batch": batch, "context": context, "prompt_tokens": PREFILL_TOKENS, "vocab": DESIGN_VOCAB, "sizes": {}}
+    for name, width, heads, kv, d, ff, layers in DESIGN_SIZES:
+        row = {"width": width, "heads": heads, "kv_heads": kv, "head_dim": d, "ff": ff, "layers": layers}
+        row["vinozen"] = design_point(q, torch, Sampler, vinozen_config(width, heads, kv, d, ff, layers), np.random.default_rng(0),
+                                      batch, context, steps, warmup)
+        row["vogerax"] = design_point(q, torch, Sampler, vogerax_config(width, heads, kv, d, ff, layers), np.random.default_rng(0),
+                                      batch, context, steps, warmup)
+        out["sizes"][name] = row
+    return out
+
+
 def designs_side_by_side(q, torch, Sampler, steps, warmup, batch=8, context=4096):
     """Dozazen beside Qwen3 at equal sizes (random weights, bfloat16): decode at `batch` x `context`, a prompt step of
     2,048 tokens; chunks longer than the context (every key is read, as in Qwen3) and chunks of 1,024."""
@@ -597,11 +634,11 @@ def main() -> int:
     ap.add_argument("--kernels", action="store_true",
                     help="instead of the benchmark: time every kernel of one decode step and of one 2,048-token prompt step "
                          "with CUDA events (steps launched afresh, not replayed) and print the sums per entry point")
-    ap.add_argument("--designs", nargs="?", const="dozazen", default=None, choices=["dozazen", "lagulorn", "fagunex", "fedinex", "vogerax"],
+    ap.add_argument("--designs", nargs="?", const="dozazen", default=None, choices=["dozazen", "lagulorn", "fagunex", "fedinex", "vogerax", "vinozen"],
                     help="instead of the benchmark: decode and prompt throughput of a Dozazen (default) or Lagulorn model beside "
                          "the Qwen3 model of the same widths (or of a Fagunex model beside the Lagulorn one, a Fedinex model beside "
-                         "the Fagunex one, a Vogerax model beside the Fedinex one) at two sizes, with the time "
-                         "of every kernel of one step of each kind")
+                         "the Fagunex one, a Vogerax model beside the Fedinex one, a Vinozen model beside the Vogerax one) at two sizes, "
+                         "with the time of every kernel of one step of each kind")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -623,7 +660,7 @@ def main() -> int:
     if args.designs:
         torch.cuda.set_device(0)
         side_by_side = {"lagulorn": lagulorn_side_by_side, "fagunex": fagunex_side_by_side,
-                        "fedinex": fedinex_side_by_side, "vogerax": vogerax_side_by_side}.get(args.designs, designs_side_by_side)
+                        "fedinex": fedinex_side_by_side, "vogerax": vogerax_side_by_side, "vinozen": vinozen_side_by_side}.get(args.designs, designs_side_by_side)
         print(json.dumps(side_by_side(q, torch, Sampler, min(args.steps, 64), warmup, args.batch or 8, args.context or 4096)))
         return 0
     if args.products:

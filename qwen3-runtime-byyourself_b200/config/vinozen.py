@@ -13,7 +13,8 @@ rotated.  The output projection is the embedding table.  What the file gives, ke
   layers[i].type      "attention": mixer {heads, kv_heads, dim, vdim, scale, bias_max, q_temp {coef, every}, kv_from}:
                       grouped-query attention over every earlier key with queries and keys at unit rms per head, a query
                       temperature that grows with the position, a learned bias by distance (far distances in stretches that
-                      grow by equal factors up to bias_max; the rows of the table are the tensor's) and a learned sink;
+                      grow by equal factors up to bias_max; the rows of the table are the tensor's, `bias_rows` states
+                      them where no checkpoint does) and a learned sink;
                       kv_from j: the layer has no keys and values of its own and reads layer j's
                       "mamba2": mixer {heads, vdim, state, groups, conv, norm_groups}: a selective state space with a short
                       convolution of `conv` taps and a gate before a norm in groups
@@ -21,7 +22,7 @@ rotated.  The output projection is the embedding table.  What the file gives, ke
                       | {kind "moe", expert {ff, limit}, router {experts, top}, shared {ff, limit}}: clamped experts chosen by
                       biased logits, and a shared one | null
 
-Optional keys (`embedding`, `token_side`, `mlp`, `mlp.shared`, `q_temp`, `kv_from`) may be null or absent: the mechanism is then
+Optional keys (`embedding`, `token_side`, `mlp`, `mlp.shared`, `q_temp`, `kv_from`, `bias_rows`) may be null or absent: the mechanism is then
 not there.  The file has no bound on positions and no stop tokens.  `plan()` states the model as data for the parts, the
 cache and the step function.
 """
@@ -113,6 +114,9 @@ class VinozenConfig:
             raise ConfigError(f"{w}scale must be positive")
         if not _get(m, "bias_max", float, w) > 0:
             raise ConfigError(f"{w}bias_max must be positive")
+        rows = _opt(m, "bias_rows", int, w)
+        if rows is not None and (rows < 2 or m["bias_max"] <= rows // 2):
+            raise ConfigError(f"{w}bias_rows: at least two, and half of them below bias_max")
         temp = _opt(m, "q_temp", dict, w)
         if temp is not None:
             _get(temp, "coef", float, w + "q_temp.")
@@ -178,8 +182,8 @@ class VinozenConfig:
             "hidden_size": self.width, "num_heads": m["heads"], "num_kv_heads": m["kv_heads"], "head_dim": m["dim"],
             "value_dim": m["vdim"], "scale": float(m["scale"]), "norm_once": True,
             "qk_norm": PartSpec("rms_norm", {"size": m["dim"], "eps": self.norm_eps, "weighted": False}),
-            "temperature": dict(m["q_temp"]) if m.get("q_temp") else None, "distance_bias": m["bias_max"], "learned_sink": True,
-            "shared_kv": m.get("kv_from") is not None, "prefix": "mix.",
+            "temperature": dict(m["q_temp"]) if m.get("q_temp") else None, "distance_bias": m["bias_max"],
+            "bias_rows": m.get("bias_rows"), "learned_sink": True, "shared_kv": m.get("kv_from") is not None, "prefix": "mix.",
             "names": {"q": "q", "k": "k", "v": "v", "o": "o", "rel": "rel", "sink": "sink"}})
 
     def _state_space(self, m: dict) -> PartSpec:

@@ -800,6 +800,46 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
     return out
 
 
+def ssd_prompt_fits(u: torch.Tensor, state: int, vd: int) -> bool:
+    """Whether `ssd_prompt` takes these sizes and rows: bfloat16, both sizes in steps of 16 up to 256, rows of 16-byte packets."""
+    return u.dtype == torch.bfloat16 and state % 16 == 0 and vd % 16 == 0 and 0 < state <= 256 and 0 < vd <= 256 and u.stride(0) % 8 == 0
+
+
+def _ssd_defines(state: int, vd: int):
+    return (f"Q3_STATE={state}", f"Q3_VALUE_DIM={vd}")
+
+
+def ssd_segments(n_seqs: int, max_new: int, heads: int, state: int, vd: int) -> int:
+    """Into how many segments `ssd_prompt` best cuts a step of prompts (1: none)."""
+    return int(_fn_untimed("ssd.cu", "q3_ssd_segments", [c_int] * 3, defines=_ssd_defines(state, vd))(int(n_seqs), int(max_new), int(heads)))
+
+
+def ssd_prompt(C: torch.Tensor, B: torch.Tensor, x: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, seq_slots: torch.Tensor,
+               out: torch.Tensor, n_seqs: int, heads: int, n: int, vd: int, share: int, dt_logits: torch.Tensor, dt_bias: torch.Tensor,
+               a_log: torch.Tensor, skip: torch.Tensor, max_new: int, scratch: Optional[torch.Tensor] = None,
+               segments: int = 1) -> torch.Tensor:
+    """What `decay_scan` does with step logits (q = C, k = B, v = x; bfloat16), 64 tokens at a time on the tensor cores: for prompts of
+    up to `max_new` tokens.  `segments` > 1 (see `ssd_segments`): they are cut into so many stretches that run side by side, with
+    `scratch` (float32, n_seqs * segments * heads * (n * vd + 1)) for the states between them."""
+    row = _scan_views(C, B, x, state, out, heads, n, vd, vd, share)
+    _check_dt(C.shape[0], heads, dt_logits, dt_bias, a_log, skip)
+    if not ssd_prompt_fits(x, n, vd):
+        raise KernelError("ssd_prompt: bfloat16, sizes in steps of 16 up to 256, rows of 16-byte packets")
+    if segments > 1 and (scratch is None or scratch.numel() < n_seqs * segments * heads * (n * vd + 1)):
+        raise KernelError("ssd_prompt: segments need a scratch for the states between them")
+    fn = _fn("ssd.cu", "q3_ssd_prompt_bf16",
+             [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
+              c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p], defines=_ssd_defines(n, vd))
+    _check(fn(x.data_ptr(), B.data_ptr(), C.data_ptr(), row, _dev(dt_logits, "dt_logits", torch.float32),
+              _dev(dt_bias, "dt_bias", torch.float32), _dev(a_log, "a_log", torch.float32), _dev(skip, "skip", torch.float32),
+              state.data_ptr(), state.stride(0), _dev(seq_start, "seq_start", torch.int32), _dev(seq_slots, "seq_slots", torch.int32),
+              _dev(out, "out"), int(n_seqs), heads, int(share), _ptr(scratch, "scratch", torch.float32) if segments > 1 else None,
+              int(max_new), int(segments), _stream()), "ssd_prompt")
+    if segments > 1:
+        _count_extra(2)
+    return out
+
+
 def channel_decay(z: torch.Tensor, bias: Optional[torch.Tensor], tau: float) -> torch.Tensor:
     """In place: z <- sigmoid(z + bias)^(1 / tau); z [N, width] float32 logits, bias float32 [width] or None."""
     if z.dtype != torch.float32 or z.dim() != 2 or (bias is not None and bias.numel() != z.shape[1]) or not tau > 0:

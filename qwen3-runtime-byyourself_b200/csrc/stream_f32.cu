@@ -72,9 +72,10 @@ __global__ void embedding_sinusoid_kernel(const int* __restrict__ ids, const int
     for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
         // angle = a + rest, a the rounded leading product and rest what it dropped with the second term's part
         const float f = freq[i], a = p * f, rest = fmaf(p, f, -a) + p * freq[pairs + i];
-        float s, c;
+        float s, c, sr, cr;
         sincosf(a, &s, &c);
-        const float sine = fmaf(rest, c, s), cosine = fmaf(-rest, s, c);
+        sincosf(rest, &sr, &cr);
+        const float sine = fmaf(c, sr, s * cr), cosine = fmaf(-s, sr, c * cr);
         float* dst = out + t * hidden + 2 * i;
         dst[0] = (ok ? to_f32<T>(src[2 * i]) * scale : 0.0f) + sine;
         if (2 * i + 1 < hidden) dst[1] = (ok ? to_f32<T>(src[2 * i + 1]) * scale : 0.0f) + cosine;

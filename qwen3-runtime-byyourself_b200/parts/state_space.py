@@ -10,7 +10,8 @@ carried from step to step):
 y is multiplied by SiLU(z), brought to unit rms in `norm_groups` equal parts of the row, multiplied by a weight and projected
 by W_o.  The step logits leave their product in 32-bit; step sizes, decays, state, outputs and norm are 32-bit whatever the
 compute type.  A sequence's state row holds heads x state x vdim values and, behind them, the convolution's last taps - 1
-input rows.  No keys in the cache.
+input rows.  No keys in the cache.  Decode steps and the 32-bit path walk token by token (`ops.decay_scan`); bfloat16 prompts
+run in chunks on the tensor cores (`ops.ssd_prompt`).
 """
 from __future__ import annotations
 
@@ -26,6 +27,8 @@ from .linear import linear
 
 TENSOR_NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "a_log": "A_log", "skip": "D", "norm": "norm",
                 "o": "o"}
+
+chunk_rows = 32      # from this many new tokens of the longest sequence on, bfloat16 steps run the chunked form
 
 
 class StateSpace(Part):
@@ -81,8 +84,14 @@ class StateSpace(Part):
                        bias=self.conv_bias, silu=True)
         B, C = u[:, inner:inner + G * n], u[:, inner + G * n:]
         y = s.get("ssm.y", (N, inner), torch.float32)
-        ops.decay_scan(C, B, u[:, :inner], rows[:, :self.cells()], ctx.seq_start, ctx.seq_slots, y, ctx.n_seqs, h, n, vd, share=h // G,
-                       dt_logits=dt, dt_bias=self.dt_bias, a_log=self.a_log, skip=self.skip)
+        steps = dict(share=h // G, dt_logits=dt, dt_bias=self.dt_bias, a_log=self.a_log, skip=self.skip)
+        args = (C, B, u[:, :inner], rows[:, :self.cells()], ctx.seq_start, ctx.seq_slots, y, ctx.n_seqs, h, n, vd)
+        if not ctx.is_decode and ctx.max_new >= chunk_rows and ops.ssd_prompt_fits(u, n, vd):
+            segments = ops.ssd_segments(ctx.n_seqs, ctx.max_new, h, n, vd)
+            between = s.get("ssm.segments", (ctx.n_seqs * segments * h * (n * vd + 1),), torch.float32) if segments > 1 else None
+            ops.ssd_prompt(*args, max_new=ctx.max_new, scratch=between, segments=segments, **steps)
+        else:
+            ops.decay_scan(*args, **steps)
         gated = s.get("ssm.gated", (N, inner), ctx.dtype)
         ops.gate_group_norm(y, proj[:, :inner], self.norm_weight, self.eps, gated, self.norm_groups)
         return linear(gated, self.w_o, s.get(self.out_name, (N, self.hidden_size), ctx.dtype))
