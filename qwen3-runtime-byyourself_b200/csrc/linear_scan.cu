@@ -26,6 +26,8 @@
 //                  16 tokens is about as long as a trip to DRAM and hides no more than that).  The launch
 //                  depends on the sizes only, never on the step: a token's output is the same bits however the
 //                  sequence was cut.  A decode step is the same kernel with one token.
+//   state_step   : the state-space form for steps of one token per sequence: a block per (head, sequence) passes over the state
+//                  once in 16-byte packets, every thread four columns of every so many rows.
 //   memory_gates : for every (sequence, head) one warp turns the gate logits zi, zf [N, H] (float32, biases added here)
 //                  into i = cap tanh(zi / cap), f = logsigmoid(cap tanh(zf / cap)), finds the running maximum
 //                  m_t = max(f_t + m_(t-1), i_t) from the slot's stored m (0 for a new sequence), 32 tokens at a time by a
@@ -392,45 +394,159 @@ __global__ void head_gated_norm_kernel(const float* __restrict__ o, const float*
     }
 }
 
-// One block per (part, token); a thread keeps up to PER values of the part in registers (PER = 0: any size, walked twice).
-template <typename T, int PER>
+// Thread (x, r) of TX x R owns the columns 4 x .. + 3 of the rows r, r + R, ..; the R partial outputs of a column meet in
+// shared memory.
+template <typename T>
+__global__ void __launch_bounds__(256)
+state_step_kernel(const ScanArgs p, int TX, int R) {
+    extern __shared__ __align__(16) float smem[];
+    float* q_s = smem;                                   // [d]
+    float* k_s = q_s + p.d;                              // [d]
+    float4* red = reinterpret_cast<float4*>(k_s + p.d + (2 * p.d) % 4);   // [R][TX]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, x = tid % TX, r = tid / TX, d = p.d, vd = p.vd;
+    const int64_t t = p.seq_start[seq];
+    if (t >= p.seq_start[seq + 1]) return;
+    const T* q_g = reinterpret_cast<const T*>(p.q) + t * p.row + (int64_t)(head / p.share) * d;
+    const T* k_g = reinterpret_cast<const T*>(p.k) + t * p.row + (int64_t)(head / p.share) * d;
+    const T* v_g = reinterpret_cast<const T*>(p.v) + t * p.row + (int64_t)head * vd;
+    float4* S_g = reinterpret_cast<float4*>(p.state + (int64_t)p.seq_slots[seq] * p.slot_stride + (int64_t)head * d * vd);
+    for (int i = tid; i < d; i += blockDim.x) {
+        q_s[i] = to_f32<T>(q_g[i]) * p.q_scale;
+        k_s[i] = to_f32<T>(k_g[i]);
+    }
+    const float dt = softplus_f32(p.keep[t * p.H + head] + p.dt_bias[head]), keep = expf(-expf(p.a_log[head]) * dt);
+    const bool live = r < R;
+    float v[4], acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+    for (int c = 0; c < 4; ++c) v[c] = live ? to_f32<T>(v_g[4 * x + c]) : 0.0f;
+    __syncthreads();
+    if (live) {
+        constexpr int BATCH = 8;                         // packets on their way together
+        for (int i0 = r; i0 < d; i0 += BATCH * R) {
+            float4 S[BATCH];
+#pragma unroll
+            for (int n = 0; n < BATCH; ++n)
+                if (i0 + n * R < d) S[n] = S_g[(int64_t)(i0 + n * R) * TX + x];
+#pragma unroll
+            for (int n = 0; n < BATCH; ++n) {
+                const int i = i0 + n * R;
+                if (i < d) {
+                    const float k = k_s[i], q = q_s[i];
+                    S[n].x = fmaf(keep, S[n].x, k * (v[0] * dt));
+                    S[n].y = fmaf(keep, S[n].y, k * (v[1] * dt));
+                    S[n].z = fmaf(keep, S[n].z, k * (v[2] * dt));
+                    S[n].w = fmaf(keep, S[n].w, k * (v[3] * dt));
+                    acc[0] = fmaf(S[n].x, q, acc[0]);
+                    acc[1] = fmaf(S[n].y, q, acc[1]);
+                    acc[2] = fmaf(S[n].z, q, acc[2]);
+                    acc[3] = fmaf(S[n].w, q, acc[3]);
+                    S_g[(int64_t)i * TX + x] = S[n];
+                }
+            }
+        }
+        red[r * TX + x] = make_float4(acc[0], acc[1], acc[2], acc[3]);
+    }
+    __syncthreads();
+    const float* red_f = reinterpret_cast<const float*>(red);
+    for (int c = tid; c < vd; c += blockDim.x) {
+        float o = 0.0f;
+        for (int rr = 0; rr < R; ++rr) o += red_f[rr * vd + c];
+        if (p.skip != nullptr) o = fmaf(p.skip[head], to_f32<T>(v_g[c]), o);
+        p.out[(t * p.H + head) * vd + c] = o;
+    }
+}
+
+template <typename T>
+int state_step_launch(const ScanArgs& p, int n_seqs, cudaStream_t stream) {
+    if (n_seqs <= 0) return 0;
+    if (p.H <= 0 || p.d <= 0 || p.vd <= 0 || p.d > 256 || p.vd > 256 || p.vd % 4 != 0 || p.share <= 0 || p.H % p.share != 0 || n_seqs > 65535 ||
+        p.dt_bias == nullptr || p.a_log == nullptr || p.slot_stride % 4 != 0)
+        return Q3_ERR_BAD_SIZE;
+    if (!aligned16(p.state)) return Q3_ERR_MISALIGNED;
+    const int TX = p.vd / 4, R = min(256 / TX, p.d), threads = (TX * R + 31) / 32 * 32;
+    const size_t smem = (size_t)(2 * p.d + (2 * p.d) % 4 + R * p.vd) * sizeof(float);
+    return (int)q3_launch(state_step_kernel<T>, dim3(p.H, n_seqs), dim3(threads), smem, stream, p, TX, R);
+}
+
+// One block per (part, token); a thread keeps up to PER packets of V values of the part in registers (PER = 0: any size, walked
+// twice).
+template <typename T, int V, int PER>
 __global__ void gate_group_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t gate_row, const float* __restrict__ w,
                                        T* __restrict__ out, int part, int size, float eps) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
     const int64_t t = blockIdx.y;
-    const int col0 = blockIdx.x * part;
+    const int col0 = blockIdx.x * part, stride = blockDim.x * V, first = threadIdx.x * V;
     const float* x = o + t * size + col0;
     const T* g = gate + t * gate_row + col0;
-    auto gated = [&](int c) {
-        const float z = to_f32<T>(g[c]);
-        return x[c] * (z / (1.0f + expf(-z)));
+    T* to = out + t * size + col0;
+    auto gated = [&](int c, float (&v)[V]) {
+        float z[V];
+        if constexpr (V == 4) {
+            const float4 a = *reinterpret_cast<const float4*>(x + c);
+            v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+            if constexpr (sizeof(T) == 4) {
+                const float4 b = *reinterpret_cast<const float4*>(g + c);
+                z[0] = b.x; z[1] = b.y; z[2] = b.z; z[3] = b.w;
+            } else {
+                const uint2 b = *reinterpret_cast<const uint2*>(g + c);
+                const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&b.x));
+                const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&b.y));
+                z[0] = lo.x; z[1] = lo.y; z[2] = hi.x; z[3] = hi.y;
+            }
+        } else {
+            v[0] = x[c];
+            z[0] = to_f32<T>(g[c]);
+        }
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] *= z[i] / (1.0f + expf(-z[i]));
     };
-    float v[PER > 0 ? PER : 1], sq = 0.0f;
+    auto store = [&](int c, const float (&v)[V], float inv) {
+        float y[V];
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[i] = v[i] * inv * w[col0 + c + i];
+        if constexpr (V == 4 && sizeof(T) == 2) {
+            uint2 raw;
+            *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(y[0], y[1]);
+            *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(y[2], y[3]);
+            *reinterpret_cast<uint2*>(to + c) = raw;
+        } else if constexpr (V == 4) {
+            *reinterpret_cast<float4*>(to + c) = make_float4(y[0], y[1], y[2], y[3]);
+        } else {
+            to[c] = from_f32<T>(y[0]);
+        }
+    };
+    float v[PER > 0 ? PER : 1][V], sq = 0.0f;
     if constexpr (PER > 0) {
 #pragma unroll
         for (int n = 0; n < PER; ++n) {
-            const int c = n * blockDim.x + threadIdx.x;
-            v[n] = c < part ? gated(c) : 0.0f;
-            sq += v[n] * v[n];
+            const int c = first + n * stride;
+            if (c < part) {
+                gated(c, v[n]);
+#pragma unroll
+                for (int i = 0; i < V; ++i) sq += v[n][i] * v[n][i];
+            }
         }
     } else {
-        for (int c = threadIdx.x; c < part; c += blockDim.x) {
-            const float y = gated(c);
-            sq += y * y;
+        for (int c = first; c < part; c += stride) {
+            gated(c, v[0]);
+#pragma unroll
+            for (int i = 0; i < V; ++i) sq += v[0][i] * v[0][i];
         }
     }
     const float inv = rsqrtf(block_sum(sq, scratch) / (float)part + eps);
-    T* to = out + t * size + col0;
     if constexpr (PER > 0) {
 #pragma unroll
-        for (int n = 0; n < PER; ++n) {
-            const int c = n * blockDim.x + threadIdx.x;
-            if (c < part) to[c] = from_f32<T>(v[n] * inv * w[col0 + c]);
-        }
+        for (int n = 0; n < PER; ++n)
+            if (first + n * stride < part) store(first + n * stride, v[n], inv);
     } else {
-        for (int c = threadIdx.x; c < part; c += blockDim.x) to[c] = from_f32<T>(gated(c) * inv * w[col0 + c]);
+        for (int c = first; c < part; c += stride) {
+            gated(c, v[0]);
+            store(c, v[0], inv);
+        }
     }
 }
 
@@ -445,9 +561,14 @@ int gate_group_norm_launch(const float* o, const T* gate, int64_t gate_row, cons
     auto launch = [&](auto kernel, int threads) {
         return (int)q3_launch(kernel, grid, dim3(threads), 0, stream, o, gate, gate_row, w, out, part, size, eps);
     };
-    if (part <= 512) return launch(gate_group_norm_kernel<T, 4>, (part + 127) / 128 * 32);
-    if (part <= 4096) return launch(gate_group_norm_kernel<T, 8>, (part + 255) / 256 * 32);
-    return launch(gate_group_norm_kernel<T, 0>, 512);
+    if (part % 4 == 0 && size % 4 == 0 && gate_row % 4 == 0 && aligned16(o) && aligned16(gate) && aligned16(out)) {
+        const int packets = part / 4;
+        if (packets <= 512) return launch(gate_group_norm_kernel<T, 4, 2>, (packets + 63) / 64 * 32);
+        if (packets <= 2048) return launch(gate_group_norm_kernel<T, 4, 4>, (packets + 127) / 128 * 32);
+        return launch(gate_group_norm_kernel<T, 4, 0>, 512);
+    }
+    if (part <= 4096) return launch(gate_group_norm_kernel<T, 1, 8>, (part + 255) / 256 * 32);
+    return launch(gate_group_norm_kernel<T, 1, 0>, 512);
 }
 
 }  // namespace
@@ -458,7 +579,7 @@ int gate_group_norm_launch(const float* o, const T* gate, int64_t gate_row, cons
                                          float q_scale, int ones, float* state, int64_t slot_stride, const int* seq_start,  \
                                          const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd,           \
                                          int share, const float* dt_bias, const float* a_log, const float* skip,           \
-                                         void* stream) {                                                                   \
+                                         int single, void* stream) {                                                                   \
         ScanArgs p;                                                                                                         \
         p.share = share; p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip;                                               \
         if ((dt_bias == nullptr) != (a_log == nullptr) || (dt_bias != nullptr && (keep == nullptr || ones)) ||              \
@@ -468,6 +589,7 @@ int gate_group_norm_launch(const float* o, const T* gate, int64_t gate_row, cons
         p.write = write; p.q_scale = q_scale; p.ones = ones; p.state = state; p.slot_stride = slot_stride;                  \
         p.seq_start = seq_start; p.seq_slots = seq_slots; p.out = out; p.H = heads; p.d = d; p.vd = vd;                     \
         p.vdx = vd + (ones ? 1 : 0);                                                                                        \
+        if (single) return state_step_launch<T>(p, n_seqs, (cudaStream_t)stream);                                           \
         if ((z == nullptr) == (keep == nullptr) || (keep != nullptr && write == nullptr && dt_bias == nullptr)) return Q3_ERR_BAD_SIZE;           \
         if (z != nullptr) return decay_scan_launch<T, true>(p, n_seqs, (cudaStream_t)stream);                               \
         return decay_scan_launch<T, false>(p, n_seqs, (cudaStream_t)stream);                                                \

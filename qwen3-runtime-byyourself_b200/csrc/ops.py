@@ -610,12 +610,12 @@ def head_gate(x: torch.Tensor, gate: torch.Tensor, heads: int, vd: int) -> torch
 
 
 def short_conv(u: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, token_seq, seq_start, seq_slots, out: torch.Tensor,
-               n_seqs: int, bias: Optional[torch.Tensor] = None, silu: bool = False) -> torch.Tensor:
+               n_seqs: int, bias: Optional[torch.Tensor] = None, silu: bool = False, single: bool = False) -> torch.Tensor:
     """Causal convolution over time on the first C columns of u [N, >= C]: out[t, c] = sum_j weight[j, c] u[t - taps + 1 + j, c]
     within every sequence, the rows before the step from `state` (a view [slots, (taps - 1) * C] of float32 rows, the
     oldest row first), which is moved on afterwards.  weight float32 [taps, C] (a checkpoint's [C, taps] transposed);
     out [N, C] in u's type.  `bias` (float32 [C]) is added to the sum; `silu`: the result goes through SiLU, both before the
-    rounding."""
+    rounding.  `single`: every sequence brings one token (one launch instead of two)."""
     N, (taps, C) = u.shape[0], weight.shape
     if out.shape != (N, C) or out.dtype != u.dtype or u.shape[1] < C or u.stride(1) != 1 or state.shape[1] != (taps - 1) * C \
             or state.dtype != torch.float32 or (taps > 1 and state.stride(1) != 1) or not out.is_contiguous() or out.data_ptr() == u.data_ptr() \
@@ -623,12 +623,12 @@ def short_conv(u: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, token
         raise KernelError("short_conv: shapes do not fit")
     fn = _fn("short_conv.cu", f"q3_short_conv_{_suffix(u)}",
              [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int64, c_int, c_void_p, c_int,
-              c_void_p])
+              c_int, c_void_p])
     _check(fn(u.data_ptr(), u.stride(0), _dev(weight, "weight", torch.float32), state.data_ptr(), state.stride(0),
               _dev(token_seq, "token_seq", torch.int32), _dev(seq_start, "seq_start", torch.int32),
               _dev(seq_slots, "seq_slots", torch.int32), out.data_ptr(), C, taps, N, int(n_seqs), _ptr(bias, "bias", torch.float32), int(bool(silu)),
-              _stream()), "short_conv")
-    if taps > 1:
+              int(bool(single)), _stream()), "short_conv")
+    if taps > 1 and not single:
         _count_extra(1)
     return out
 
@@ -766,23 +766,31 @@ def _check_dt(N, heads, dt_logits, dt_bias, a_log, skip):
         raise KernelError("step sizes: logits [N, heads] with a bias and a log decay rate per head")
 
 
+def state_step_fits(state: torch.Tensor, vd: int) -> bool:
+    """Whether the state's rows split into 16-byte packets, as the form of `decay_scan` for single tokens reads them."""
+    return vd % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0
+
+
 def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor, seq_slots: torch.Tensor,
                out: torch.Tensor, n_seqs: int, heads: int, d: int, vd: int, q_scale: float = 1.0, decay: Optional[torch.Tensor] = None,
                keep: Optional[torch.Tensor] = None, write: Optional[torch.Tensor] = None, ones: bool = False, share: int = 1,
                dt_logits: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None, a_log: Optional[torch.Tensor] = None,
-               skip: Optional[torch.Tensor] = None) -> torch.Tensor:
+               skip: Optional[torch.Tensor] = None, single: bool = False) -> torch.Tensor:
     """S_t = diag(a_t) S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T (q_t * q_scale) over the new tokens of every sequence, from and to
     the state rows (`state`: a view [slots, heads * d * vdx] of float32 rows).  q, k, v: column views of one projection
     output (same row stride).  With `decay` [N, heads * d] (float32, see `channel_decay`): a per channel, b = 1.  With
     `keep`, `write` [N, heads] (float32): a and b per head.  `ones`: vdx = vd + 1, the state's last column takes
     the value 1 (a normaliser); else vdx = vd.  `dt_logits` [N, heads] with `dt_bias`, `a_log` [heads] (float32) instead of
     `keep` and `write`: b = softplus(logit + dt_bias), a = exp(-exp(a_log) b).  `skip` [heads]: skip_h v_t is added to the output.
-    `share`: so many neighbouring heads read the same q and k.  out [N, heads * vdx] float32."""
+    `share`: so many neighbouring heads read the same q and k.  `single`: every sequence brings one token and the step sizes
+    come as logits (the form for decode steps where `state_step_fits`).  out [N, heads * vdx] float32."""
     vdx = vd + (1 if ones else 0)
     row = _scan_views(q, k, v, state, out, heads, d, vd, vdx, share)
     N = q.shape[0]
     z = decay
     _check_dt(N, heads, dt_logits, dt_bias, a_log, skip)
+    if single and (dt_logits is None or not state_step_fits(state, vd)):
+        raise KernelError("decay_scan: the form for single tokens takes step logits and state rows of 16-byte packets")
     if dt_logits is not None:
         if keep is not None or write is not None or ones:
             raise KernelError("decay_scan: step sizes come as logits or as gates per head, without a normaliser")
@@ -792,11 +800,11 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
         raise KernelError("decay_scan: a decay per channel or gates per head (keep, write)")
     fn = _fn("linear_scan.cu", f"q3_decay_scan_{_suffix(q)}",
              [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_int, c_void_p, c_int64,
-              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
+              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(fn(q.data_ptr(), k.data_ptr(), v.data_ptr(), row, _ptr(z, "decay", torch.float32), _ptr(keep, "keep", torch.float32), _ptr(write, "write", torch.float32), float(q_scale), int(bool(ones)),
               state.data_ptr(), state.stride(0), _dev(seq_start, "seq_start", torch.int32), _dev(seq_slots, "seq_slots", torch.int32),
               _dev(out, "out"), int(n_seqs), heads, d, vd, int(share), _ptr(dt_bias, "dt_bias", torch.float32),
-              _ptr(a_log, "a_log", torch.float32), _ptr(skip, "skip", torch.float32), _stream()), "decay_scan")
+              _ptr(a_log, "a_log", torch.float32), _ptr(skip, "skip", torch.float32), int(bool(single)), _stream()), "decay_scan")
     return out
 
 

@@ -10,6 +10,7 @@
 //                      token comes from the state [slot][taps - 1][C] (float32; the oldest row first), zeros for a new sequence.
 //                      The products are summed in 32-bit in ascending j whatever the step, so a token's output is the
 //                      same bits however the sequence was cut.
+//   short_conv_step  : steps of one token per sequence: a thread per (sequence, packet of channels) does both at once.
 //   short_conv_state : afterwards, one thread per (sequence, channel) moves the state on: the last taps - 1 rows of
 //                      (old state, the step's rows).
 //
@@ -90,27 +91,23 @@ __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, 
 #pragma unroll
         for (int k = 0; k < VEC; ++k) wt[j][k] = w[(int64_t)j * C + c + k];
     const int64_t t_begin = (int64_t)blockIdx.y * run, t_end = min(t_begin + run, n_tokens);
-    int cur = -1;
-    for (int64_t t = t_begin; t < t_end; ++t) {
-        const int seq = token_seq[t];
-        if (seq != cur) {                                      // the run's first token, or a sequence's first: fill the window
-            cur = seq;
-            const int64_t first = seq_start[seq];
-            const float* st = state + (int64_t)seq_slots[seq] * slot_stride;
+    auto fill = [&](int64_t t, int seq) {                      // the rows before token t
+        const int64_t first = seq_start[seq];
+        const float* st = state + (int64_t)seq_slots[seq] * slot_stride;
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; ++j) {
-                const int64_t src = t - (TAPS - 1) + j;
-                if (src >= first) {
-                    const Pack<T> pk = load_pack<T>(u + src * row_in + c);
+        for (int j = 0; j < TAPS - 1; ++j) {
+            const int64_t src = t - (TAPS - 1) + j;
+            if (src >= first) {
+                const Pack<T> pk = load_pack<T>(u + src * row_in + c);
 #pragma unroll
-                    for (int k = 0; k < VEC; ++k) win[j][k] = pk.get(k);
-                } else {
+                for (int k = 0; k < VEC; ++k) win[j][k] = pk.get(k);
+            } else {
 #pragma unroll
-                    for (int k = 0; k < VEC; ++k) win[j][k] = st[(int64_t)(TAPS - 1 + (src - first)) * C + c + k];
-                }
+                for (int k = 0; k < VEC; ++k) win[j][k] = st[(int64_t)(TAPS - 1 + (src - first)) * C + c + k];
             }
         }
-        const Pack<T> pk = load_pack<T>(u + t * row_in + c);
+    };
+    auto one = [&](int64_t t, const Pack<T>& pk) {
         float x[VEC], acc[VEC];
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
@@ -136,6 +133,73 @@ __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, 
 #pragma unroll
             for (int k = 0; k < VEC; ++k) win[TAPS - 2 > 0 ? TAPS - 2 : 0][k] = x[k];
         }
+    };
+    const int seq0 = token_seq[t_begin];
+    if (seq0 == token_seq[t_end - 1]) {                        // one sequence: the rows of several tokens are on their way together
+        constexpr int BATCH = 8;
+        fill(t_begin, seq0);
+        for (int64_t t0 = t_begin; t0 < t_end; t0 += BATCH) {
+            Pack<T> pk[BATCH];
+#pragma unroll
+            for (int n = 0; n < BATCH; ++n)
+                if (t0 + n < t_end) pk[n] = load_pack<T>(u + (t0 + n) * row_in + c);
+#pragma unroll
+            for (int n = 0; n < BATCH; ++n)
+                if (t0 + n < t_end) one(t0 + n, pk[n]);
+        }
+        return;
+    }
+    int cur = -1;
+    for (int64_t t = t_begin; t < t_end; ++t) {
+        const int seq = token_seq[t];
+        if (seq != cur) {                                      // the run's first token, or a sequence's first: fill the window
+            cur = seq;
+            fill(t, seq);
+        }
+        one(t, load_pack<T>(u + t * row_in + c));
+    }
+}
+
+template <typename T, int VEC>
+__global__ void short_conv_step_kernel(const T* __restrict__ u, int64_t row_in, const float* __restrict__ w, float* __restrict__ state,
+                                       int64_t slot_stride, const int* __restrict__ seq_start, const int* __restrict__ seq_slots,
+                                       T* __restrict__ y, int C, int taps, int n_seqs, const float* __restrict__ bias, int silu) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC, seq = blockIdx.y;
+    if (c >= C) return;
+    const int64_t t = seq_start[seq];
+    float* st = state + (int64_t)seq_slots[seq] * slot_stride + c;
+    float x[VEC], acc[VEC];
+    if constexpr (VEC == 1) {
+        x[0] = to_f32<T>(u[t * row_in + c]);
+    } else {
+        const Pack<T> pk = load_pack<T>(u + t * row_in + c);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) x[k] = pk.get(k);
+    }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) acc[k] = 0.0f;
+    for (int j = 0; j < taps - 1; ++j) {
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+            const float old = st[(int64_t)j * C + k];
+            acc[k] = fmaf(w[(int64_t)j * C + c + k], old, acc[k]);
+            if (j > 0) st[(int64_t)(j - 1) * C + k] = old;
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+        if (taps > 1) st[(int64_t)(taps - 2) * C + k] = x[k];
+        acc[k] = finish(fmaf(w[(int64_t)(taps - 1) * C + c + k], x[k], acc[k]), bias, c + k, silu);
+    }
+    if constexpr (VEC == 1) {
+        y[t * C + c] = from_f32<T>(acc[0]);
+    } else {
+        Pack<T> pk;
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) pk.set(k, acc[k]);
+        store_pack<T>(y + t * C + c, pk);
     }
 }
 
@@ -175,11 +239,17 @@ __global__ void short_conv_state_kernel(const T* __restrict__ u, int64_t row_in,
 template <typename T>
 int short_conv_launch(const T* u, int64_t row_in, const float* w, float* state, int64_t slot_stride, const int* token_seq, const int* seq_start,
                       const int* seq_slots, T* y, int C, int taps, int64_t n_tokens, int n_seqs, const float* bias, int silu,
-                      cudaStream_t stream) {
+                      int single, cudaStream_t stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return 0;
     if (C <= 0 || taps <= 0 || taps > 64 || row_in < C) return Q3_ERR_BAD_SIZE;
     constexpr int V = Pack<T>::N;
     const bool vec = C % V == 0 && row_in % V == 0 && aligned16(u) && aligned16(y);
+    if (single) {
+        if (n_tokens != n_seqs || n_seqs > 65535) return Q3_ERR_BAD_SIZE;
+        const int packets = C / (vec ? V : 1);
+        return (int)q3_launch(vec ? short_conv_step_kernel<T, V> : short_conv_step_kernel<T, 1>, dim3((packets + 63) / 64, n_seqs), dim3(64), 0,
+                              stream, u, row_in, w, state, slot_stride, seq_start, seq_slots, y, C, taps, n_seqs, bias, silu);
+    }
     int code;
     if (vec && taps >= 2 && taps <= 4 && (n_tokens + 15) / 16 <= 65535) {
         auto walk = [&](auto launch) {
@@ -204,9 +274,9 @@ int short_conv_launch(const T* u, int64_t row_in, const float* w, float* state, 
     Q3_EXPORT int q3_short_conv_##SUFFIX(const void* u, int64_t row_in, const float* w, float* state, int64_t slot_stride, \
                                          const int* token_seq, const int* seq_start, const int* seq_slots, void* y,      \
                                          int channels, int taps, int64_t n_tokens, int n_seqs, const float* bias,        \
-                                         int silu, void* stream) {                                                        \
+                                         int silu, int single, void* stream) {                                            \
         return short_conv_launch<T>((const T*)u, row_in, w, state, slot_stride, token_seq, seq_start, seq_slots, (T*)y,   \
-                                    channels, taps, n_tokens, n_seqs, bias, silu, (cudaStream_t)stream);                  \
+                                    channels, taps, n_tokens, n_seqs, bias, silu, single, (cudaStream_t)stream);          \
     }
 
 Q3_CONV_EXPORTS(f32, float)

@@ -81,7 +81,7 @@ class StateSpace(Part):
         conv_state = rows[:, self.cells():] if self.taps > 1 else s.get("ssm.no_state", (1, 0), torch.float32)
         u = s.get("ssm.conv", (N, self.channels), ctx.dtype)
         ops.short_conv(proj[:, inner:], self.conv, conv_state, ctx.token_seq, ctx.seq_start, ctx.seq_slots, u, ctx.n_seqs,
-                       bias=self.conv_bias, silu=True)
+                       bias=self.conv_bias, silu=True, single=ctx.is_decode)
         B, C = u[:, inner:inner + G * n], u[:, inner + G * n:]
         y = s.get("ssm.y", (N, inner), torch.float32)
         steps = dict(share=h // G, dt_logits=dt, dt_bias=self.dt_bias, a_log=self.a_log, skip=self.skip)
@@ -91,7 +91,7 @@ class StateSpace(Part):
             between = s.get("ssm.segments", (ctx.n_seqs * segments * h * (n * vd + 1),), torch.float32) if segments > 1 else None
             ops.ssd_prompt(*args, max_new=ctx.max_new, scratch=between, segments=segments, **steps)
         else:
-            ops.decay_scan(*args, **steps)
+            ops.decay_scan(*args, **steps, single=ctx.is_decode and ops.state_step_fits(args[3], vd))
         gated = s.get("ssm.gated", (N, inner), ctx.dtype)
         ops.gate_group_norm(y, proj[:, :inner], self.norm_weight, self.eps, gated, self.norm_groups)
         return linear(gated, self.w_o, s.get(self.out_name, (N, self.hidden_size), ctx.dtype))

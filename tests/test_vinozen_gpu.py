@@ -302,7 +302,7 @@ def test_convolution_with_a_bias_and_silu(dtype, C, taps, lead):
         u = dev(rng.standard_normal((int(start[-1]), lead + C + 8)), T)
         out = torch.empty((u.shape[0], C), dtype=T, device="cuda")
         ops.short_conv(u[:, lead:], dev(w.T.copy(), torch.float32), state, dev(seq, torch.int32), dev(start, torch.int32), dev(slots, torch.int32),
-                       out, 3, bias=dev(b, torch.float32), silu=True)
+                       out, 3, bias=dev(b, torch.float32), silu=True, single=max(lengths) == 1)
         got = f64(out)
         for s, n in enumerate(lengths):
             seen[s] = np.concatenate([seen[s], f64(u)[start[s]:start[s + 1], lead:lead + C]])
@@ -329,9 +329,10 @@ def test_state_space_over_unequal_sequences_and_from_its_state(dtype, H, G, n, v
     from qwen3_b200.csrc import ops
     rng = np.random.default_rng(H * 1000 + n + vd)
     T, cells, slots = torch_dtype(dtype), H * n * vd, [4, 0, 5, 2]
-    whole = torch.zeros((8, 3 + cells + 2), dtype=torch.float32, device="cuda")
-    whole[:, :3], whole[:, 3 + cells:] = 7.0, -7.0
-    state = whole[:, 3:3 + cells]
+    lead = 4 if chunks or n % 2 == 0 else 3                     # whether the rows split into 16-byte packets
+    whole = torch.zeros((8, lead + cells + 4 - cells % 4), dtype=torch.float32, device="cuda")
+    whole[:, :lead], whole[:, lead + cells:] = 7.0, -7.0
+    state = whole[:, lead:lead + cells]
     a_log, dt_bias = np.linspace(-4.0, 3.5, H), rng.standard_normal(H) - 1.0
     skip = rng.standard_normal(H)
     vectors = {k: dev(v, torch.float32) for k, v in (("a_log", a_log), ("dt_bias", dt_bias), ("skip", skip))}
@@ -345,8 +346,8 @@ def test_state_space_over_unequal_sequences_and_from_its_state(dtype, H, G, n, v
         args = (C, B, x, state, dev(start, torch.int32), dev(slots, torch.int32), out, 4, H, n, vd)
         if chunks and max(lengths) > 1:
             ops.ssd_prompt(*args, share=H // G, dt_logits=z, max_new=max(lengths), **vectors)
-        else:
-            ops.decay_scan(*args, share=H // G, dt_logits=z, **vectors)
+        else:                                                    # single tokens: also the form for them, where rows allow it
+            ops.decay_scan(*args, share=H // G, dt_logits=z, **vectors, single=max(lengths) == 1 and ops.state_step_fits(state, vd))
         got, dt = f64(out).reshape(N, H, vd), plain.softplus(f64(z) + f64(vectors["dt_bias"]))
         xs, Bs, Cs = f64(x).reshape(N, H, vd), f64(B).reshape(N, G, n), f64(C).reshape(N, G, n)
         rate = np.exp(f64(vectors["a_log"]))
@@ -359,8 +360,8 @@ def test_state_space_over_unequal_sequences_and_from_its_state(dtype, H, G, n, v
                     assert np.allclose(got[t, h], want, rtol=5e-4, atol=5e-4), (lengths, slot, t - start[i], h)
     final = f64(whole)
     for slot in slots:
-        assert np.allclose(final[slot, 3:-2].reshape(H, n, vd), S[slot], rtol=5e-4, atol=5e-4)
-    assert np.all(final[:, :3] == 7.0) and np.all(final[:, -2:] == -7.0) and np.all(final[[1, 3, 6, 7], 3:-2] == 0.0)
+        assert np.allclose(final[slot, lead:lead + cells].reshape(H, n, vd), S[slot], rtol=5e-4, atol=5e-4)
+    assert np.all(final[:, :lead] == 7.0) and np.all(final[:, lead + cells:] == -7.0) and np.all(final[[1, 3, 6, 7], lead:lead + cells] == 0.0)
 
 
 @pytest.mark.parametrize("H,G,n,vd", [(4, 2, 128, 64), (2, 1, 32, 48), (3, 3, 16, 128)])
