@@ -252,20 +252,26 @@ prefill_capped_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pag
             // the entries of this page that each row sees: from .. to (and the kept keys)
             const int from_lo = blocks ? 0 : c_lo, from_hi = blocks ? 0 : c_hi, to_lo = blocks ? b_lo - 1 : p_lo, to_hi = blocks ? b_hi - 1 : p_hi;
             float mx[2] = {-INFINITY, -INFINITY};
-            const bool far = BIAS && warp_first_pos - (key_base + PAGE - 1) >= bias.count - 1;   // one bias for the whole page
+            float s_bias[BIAS ? 8 : 1][4];
+            if constexpr (BIAS) {
+                if (warp_first_pos - (key_base + PAGE - 1) >= bias.count - 1) {               // one bias for the whole page
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) s_bias[j][0] = s_bias[j][1] = s_bias[j][2] = s_bias[j][3] = bias_far;
+                } else {
+                    const int back0 = p_lo - (key_base + tq * 2);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e)
+                            s_bias[j][e] = __ldg(bias_row + min(max(back0 + (e >> 1) * 8 - j * 8 - (e & 1), 0), bias.count - 1)) * LOG2E;
+                }
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     float v = score_log2(s[j][e], scale, cap, inv_cap);
-                    if constexpr (BIAS) {
-                        if (far) {
-                            v += bias_far;
-                        } else {
-                            const int back = ((e >> 1) ? p_hi : p_lo) - (key_base + j * 8 + tq * 2 + (e & 1));
-                            v = fmaf(__ldg(bias_row + min(max(back, 0), bias.count - 1)), LOG2E, v);
-                        }
-                    }
+                    if constexpr (BIAS) v += s_bias[j][e];
                     if (edge) {
                         const int key = key_base + j * 8 + tq * 2 + (e & 1);
                         const bool seen = (e >> 1) ? (key <= to_hi && (key >= from_hi || (!POOL && key < keep))) : (key <= to_lo && (key >= from_lo || (!POOL && key < keep)));

@@ -120,6 +120,13 @@ template <int GATED> __device__ __forceinline__ float gate_activation(float z) {
     return z / (1.0f + expf(-z));
 }
 
+// SiLU of a value that is rounded to T next: for bf16 the fast exponential and division (a few units in the last place of
+// 32-bit) are far below that rounding.
+template <typename T> __device__ __forceinline__ float silu_for(float z) {
+    if constexpr (sizeof(T) == 2) return __fdividef(z, 1.0f + __expf(fminf(-z, 80.0f)));
+    return z / (1.0f + expf(-z));
+}
+
 // What a product's epilogue does, beside 0 (nothing): 1 and 2 take pairs of gate and up columns (see above), 3 is the
 // square of relu on every value.
 template <int GATED> constexpr bool q3_paired = GATED == 1 || GATED == 2;

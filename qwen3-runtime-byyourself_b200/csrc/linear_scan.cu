@@ -502,7 +502,7 @@ __global__ void gate_group_norm_kernel(const float* __restrict__ o, const T* __r
             z[0] = to_f32<T>(g[c]);
         }
 #pragma unroll
-        for (int i = 0; i < V; ++i) v[i] *= z[i] / (1.0f + expf(-z[i]));
+        for (int i = 0; i < V; ++i) v[i] *= silu_for<T>(z[i]);
     };
     auto store = [&](int c, const float (&v)[V], float inv) {
         float y[V];

@@ -20,9 +20,9 @@
 
 namespace {
 
-__device__ __forceinline__ float finish(float acc, const float* __restrict__ bias, int c, int silu) {
+template <typename T> __device__ __forceinline__ float finish(float acc, const float* __restrict__ bias, int c, int silu) {
     if (bias != nullptr) acc += bias[c];
-    return silu ? acc / (1.0f + expf(-acc)) : acc;
+    return silu ? silu_for<T>(acc) : acc;
 }
 
 // VEC channels a thread (16 bytes of a row where the sizes allow it, else one).
@@ -63,11 +63,11 @@ __global__ void short_conv_kernel(const T* __restrict__ u, int64_t row_in, const
             for (int k = 0; k < VEC; ++k) acc[k] = fmaf(w[(int64_t)j * C + c + k], x[k], acc[k]);
         }
         if constexpr (VEC == 1) {
-            y[t * C + c] = from_f32<T>(finish(acc[0], bias, c, silu));
+            y[t * C + c] = from_f32<T>(finish<T>(acc[0], bias, c, silu));
         } else {
             Pack<T> pk;
 #pragma unroll
-            for (int k = 0; k < VEC; ++k) pk.set(k, finish(acc[k], bias, c + k, silu));
+            for (int k = 0; k < VEC; ++k) pk.set(k, finish<T>(acc[k], bias, c + k, silu));
             store_pack<T>(y + t * C + c, pk);
         }
     }
@@ -85,7 +85,9 @@ __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, 
     pdl_wait();
     const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
     if (c >= C) return;
-    float wt[TAPS][VEC], win[TAPS > 1 ? TAPS - 1 : 1][VEC];
+    float wt[TAPS][VEC], win[TAPS > 1 ? TAPS - 1 : 1][VEC], add[VEC];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) add[k] = bias != nullptr ? bias[c + k] : 0.0f;
 #pragma unroll
     for (int j = 0; j < TAPS; ++j)
 #pragma unroll
@@ -122,7 +124,9 @@ __global__ void short_conv_walk_kernel(const T* __restrict__ u, int64_t row_in, 
 #pragma unroll
         for (int k = 0; k < VEC; ++k) {
             acc[k] = fmaf(wt[TAPS - 1][k], x[k], acc[k]);
-            out.set(k, finish(acc[k], bias, c + k, silu));
+            acc[k] += add[k];
+            if (silu) acc[k] = silu_for<T>(acc[k]);
+            out.set(k, acc[k]);
         }
         store_pack<T>(y + t * C + c, out);
 #pragma unroll
@@ -191,7 +195,7 @@ __global__ void short_conv_step_kernel(const T* __restrict__ u, int64_t row_in, 
 #pragma unroll
     for (int k = 0; k < VEC; ++k) {
         if (taps > 1) st[(int64_t)(taps - 2) * C + k] = x[k];
-        acc[k] = finish(fmaf(w[(int64_t)(taps - 1) * C + c + k], x[k], acc[k]), bias, c + k, silu);
+        acc[k] = finish<T>(fmaf(w[(int64_t)(taps - 1) * C + c + k], x[k], acc[k]), bias, c + k, silu);
     }
     if constexpr (VEC == 1) {
         y[t * C + c] = from_f32<T>(acc[0]);

@@ -12,8 +12,8 @@
 //     state   S    = exp(c_last) S_0 + sum_j exp(c_last - c_j) dt_j B_j x_j^T
 //
 // x, B and C are bfloat16 (the convolution's output), so the first product is exact up to its 32-bit sum; in the others the
-// 32-bit factor (W, S, the weighted x) enters as a sum of bfloat16 terms, two for W (16 bits of mantissa) and three for S and
-// the weighted x (all 24).  The sums c run in 64-bit and are kept as two floats, so that a difference of two of them is right
+// 32-bit factor (W, S, the weighted x) enters as a sum of bfloat16 terms: three (all 24 bits of mantissa) for the weighted x,
+// whose sums are carried on in S, two (16 bits) for W and the S that is read out, which reach one output each.  The sums c run in 64-bit and are kept as two floats, so that a difference of two of them is right
 // to 32-bit rounding however long the sum is; no quotient of decays is ever formed.
 //
 // A block owns one head's state columns v0 .. v0 + VT - 1, a warp 16 of them, and keeps S^T in the accumulator registers of its
@@ -264,24 +264,20 @@ ssd_kernel(const Args p) {
                 float r[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) r[e] = S[2 * kt + (e >> 2)][e & 3];
-                uint32_t s0[4], s1[4], s2[4];
+                uint32_t s0[4], s1[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     s0[e] = take_term(r[2 * e], r[2 * e + 1]);
                     s1[e] = take_term(r[2 * e], r[2 * e + 1]);
-                    s2[e] = take_term(r[2 * e], r[2 * e + 1]);
                 }
+                uint32_t b[C / 16][4];
 #pragma unroll
-                for (int ib = 0; ib < C / 16; ++ib) {
-                    uint32_t b[4];
-                    ldmatrix_x4(b, c_s + (ib * 16 + krow) * N_ROW + (2 * kt + kcol) * 16);
+                for (int ib = 0; ib < C / 16; ++ib) ldmatrix_x4(b[ib], c_s + (ib * 16 + krow) * N_ROW + (2 * kt + kcol) * 16);
+                // term by term over all the tiles: the products of one accumulator do not wait for one another back to back
 #pragma unroll
-                    for (int h = 0; h < 2; ++h) {
-                        mma_bf16(y[2 * ib + h], s2, b[2 * h], b[2 * h + 1]);
-                        mma_bf16(y[2 * ib + h], s1, b[2 * h], b[2 * h + 1]);
-                        mma_bf16(y[2 * ib + h], s0, b[2 * h], b[2 * h + 1]);
-                    }
-                }
+                for (int it = 0; it < C / 8; ++it) mma_bf16(y[it], s1, b[it >> 1][2 * (it & 1)], b[it >> 1][2 * (it & 1) + 1]);
+#pragma unroll
+                for (int it = 0; it < C / 8; ++it) mma_bf16(y[it], s0, b[it >> 1][2 * (it & 1)], b[it >> 1][2 * (it & 1) + 1]);
             }
 #pragma unroll
             for (int it = 0; it < C / 8; ++it)
@@ -290,10 +286,10 @@ ssd_kernel(const Args p) {
 #pragma unroll
             for (int kt = 0; kt < C / 16; ++kt) {
 #pragma unroll
-                for (int ib = kt; ib < C / 16; ++ib) {
-                    uint32_t b[4];
+                for (int term = 1; term >= 0; --term) {
 #pragma unroll
-                    for (int term = 1; term >= 0; --term) {
+                    for (int ib = kt; ib < C / 16; ++ib) {
+                        uint32_t b[4];
                         ldmatrix_x4(b, (term ? w_lo : w_hi) + (ib * 16 + krow) * W_ROW + (2 * kt + kcol) * 16);
                         mma_bf16(y[2 * ib], xa[kt], b[0], b[1]);
                         mma_bf16(y[2 * ib + 1], xa[kt], b[2], b[3]);
@@ -325,16 +321,18 @@ ssd_kernel(const Args p) {
                 x1[e] = take_term(a, b);
                 x2[e] = take_term(a, b);
             }
+            constexpr int NB = NS / 16 % 4 == 0 ? 4 : (NS / 16 % 2 == 0 ? 2 : 1);    // 16-row blocks of B at a time
 #pragma unroll
-            for (int nb = 0; nb < NS / 16; ++nb) {
-                uint32_t b[4];
-                ldmatrix_x4_trans(b, b_s + (kt * 16 + vrow) * N_ROW + (2 * nb + vcol) * 16);
+            for (int nb = 0; nb < NS / 16; nb += NB) {
+                uint32_t b[NB][4];
 #pragma unroll
-                for (int h = 0; h < 2; ++h) {
-                    mma_bf16(S[2 * nb + h], x2, b[2 * h], b[2 * h + 1]);
-                    mma_bf16(S[2 * nb + h], x1, b[2 * h], b[2 * h + 1]);
-                    mma_bf16(S[2 * nb + h], x0, b[2 * h], b[2 * h + 1]);
-                }
+                for (int i = 0; i < NB; ++i) ldmatrix_x4_trans(b[i], b_s + (kt * 16 + vrow) * N_ROW + (2 * (nb + i) + vcol) * 16);
+#pragma unroll
+                for (int i = 0; i < 2 * NB; ++i) mma_bf16(S[2 * nb + i], x2, b[i >> 1][2 * (i & 1)], b[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+                for (int i = 0; i < 2 * NB; ++i) mma_bf16(S[2 * nb + i], x1, b[i >> 1][2 * (i & 1)], b[i >> 1][2 * (i & 1) + 1]);
+#pragma unroll
+                for (int i = 0; i < 2 * NB; ++i) mma_bf16(S[2 * nb + i], x0, b[i >> 1][2 * (i & 1)], b[i >> 1][2 * (i & 1) + 1]);
             }
         }
         if constexpr (WALK == STATES) __syncthreads();   // the sums and steps may be rewritten
@@ -376,11 +374,12 @@ __global__ void segment_starts_kernel(const Args p) {
     }
 }
 
-// The number of segments (1: none) for prompts of at most `max_new` tokens: enough blocks for two per multiprocessor, segments of
-// at least two chunks, at most 64 MB of states.
+// The number of segments (1: none) for prompts of at most `max_new` tokens: as many blocks as run at once, two per multiprocessor
+// (one block more and the last of them run alone: one prompt of 2,048 tokens with 128 heads took 226 us in 2 segments, 274 in 3),
+// segments of at least two chunks, at most 64 MB of states.
 int segment_count(int n_seqs, int max_new, int H) {
     const int64_t blocks = (int64_t)H * n_seqs * (VD / VT), bytes = (int64_t)n_seqs * H * NS * VD * 4;
-    const int64_t want = (2 * (int64_t)q3_device_sm_count() + blocks - 1) / blocks;
+    const int64_t want = 2 * (int64_t)q3_device_sm_count() / blocks;
     int64_t count = want < max_new / (2 * C) ? want : max_new / (2 * C);
     if (count > (64ll << 20) / bytes) count = (64ll << 20) / bytes;
     return count < 2 ? 1 : (int)count;
