@@ -29,4 +29,6 @@ def all_variants():
         ("latent.cu", ()),
         ("linear_scan.cu", ()),
         ("short_conv.cu", ()),
+        ("attention_prefill_tc.cu", ("Q3_HEAD_DIM=128", "Q3_CAPPED=2")),
+        ("ssd.cu", ("Q3_STATE=128", "Q3_VALUE_DIM=64")),
     ]

@@ -61,6 +61,12 @@ int q3_place_rows(const void* src, int src_kind, void* dst, int dst_kind, int64_
 /* out[t] = table[ids[t]] * scale */
 int q3_embedding_scaled_f32(const int* ids, const void* table, float* out, int64_t n_tokens, int hidden, int vocab, float scale, void* stream);
 int q3_embedding_scaled_bf16(const int* ids, const void* table, float* out, int64_t n_tokens, int hidden, int vocab, float scale, void* stream);
+/* the same plus, with p the token's position, sin(p f_i) in column 2i and cos(p f_i) in column 2i + 1; freq [2, (hidden + 1) / 2]:
+   every frequency f_i as a leading term and what its rounding dropped */
+int q3_embedding_sinusoid_f32(const int* ids, const int* positions, const void* table, const float* freq, float* out, int64_t n_tokens,
+                              int hidden, int vocab, float scale, void* stream);
+int q3_embedding_sinusoid_bf16(const int* ids, const int* positions, const void* table, const float* freq, float* out, int64_t n_tokens,
+                               int hidden, int vocab, float scale, void* stream);
 /* stream += RMSNorm(branch) * w_post (branch and w_post may both be null), then out = RMSNorm(stream) * w_pre (out and
    w_pre may both be null), one pass over a row; parts_post, parts_pre: a norm splits the row into that many equal
    consecutive parts, each with an rms of its own (1: the row as a whole) */
@@ -90,16 +96,18 @@ int q3_qkv_prepare_f32(const void* qkv, void* q_out, void* k_pages, void* v_page
                        const float* cos_tab, const float* sin_tab, const int* token_seq, const int* token_pos, const int* page_table,
                        int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d, float eps, int write_kv, int rotary_dim,
                        const float* bias, int value_dim, int value_heads, int64_t row, int tied_values, int norm_once,
-                       const float* v_cos, const float* v_sin, void* stream);
+                       const float* v_cos, const float* v_sin, float temp_coef, int temp_every, void* stream);
 int q3_qkv_prepare_bf16(const void* qkv, void* q_out, void* k_pages, void* v_pages, const float* q_norm_w, const float* k_norm_w,
                         const float* cos_tab, const float* sin_tab, const int* token_seq, const int* token_pos, const int* page_table,
                         int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d, float eps, int write_kv, int rotary_dim,
                        const float* bias, int value_dim, int value_heads, int64_t row, int tied_values, int norm_once,
-                       const float* v_cos, const float* v_sin, void* stream);
+                       const float* v_cos, const float* v_sin, float temp_coef, int temp_every, void* stream);
 /* (q3_qkv_prepare: value_heads 0 = nkv; fewer value heads than key heads: values that several key heads share; row 0 = the
    columns read, else values from one row of the projection to the next; tied_values: the values are the projected keys and
    have no columns; norm_once: a normed value is rounded once, when it is stored; v_cos, v_sin [positions, value_dim / 2], may
-   be null: the values are rotated by their position, over the whole head) */
+   be null: the values are rotated by their position, over the whole head; temp_coef, not 0: a query is multiplied by
+   1 + temp_coef ln((position + 1) / temp_every + 1), a whole quotient, after its norm; without write_kv `qkv` may hold the query
+   columns alone) */
 /* the pooled blocks that the step completes: block b of a sequence, its tokens b size .. b size + size - 1, gets the means of
    their cached keys and values as entry b of the sequence's pool pages (pool_table: as page_table) */
 int q3_pool_blocks_f32(const void* k_pages, const void* v_pages, const int* page_table, void* pool_k, void* pool_v,
@@ -121,17 +129,20 @@ int q3_turn_back_gate_bf16(void* x, const float* cos_tab, const float* sin_tab, 
    positions only; sink != 0: one more term exp(0) in the softmax's denominator, or exp(sink_values[head]) where sink_values
    (one float per query head) is given; keep_first (with window): the first so many keys of the sequence are seen too; pool_size
    (with window, without keep_first): every block of so many tokens that ends before the window is seen as the entry of the pool
-   pages that q3_pool_blocks wrote */
+   pages that q3_pool_blocks wrote; bias [nq, bias_count] (may be null): added to the scaled score by the distance between
+   query and key, the last column for all that is further (without pooled blocks) */
 int q3_attention_generic_f32(const void* q, const void* k_pages, const void* v_pages, void* out, const int* token_seq,
                              const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d,
                              float scale, int window, int value_dim, float softcap, int chunk, int sink, int value_heads, int out_f32,
                              const float* sink_values, int keep_first,
-                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, const float* bias, int bias_count,
+                             void* stream);
 int q3_attention_generic_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, const int* token_seq,
                               const int* token_pos, const int* page_table, int pages_per_seq, int64_t n_tokens, int nq, int nkv, int d,
                               float scale, int window, int value_dim, float softcap, int chunk, int sink, int value_heads, int out_f32,
                               const float* sink_values, int keep_first,
-                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, const float* bias, int bias_count,
+                             void* stream);
 
 /* the same from the q/k/v projection's output as it is: bias (may be null), rotation of the first rotary_dim values of q and k
    (tables may be null) and the write of the new key and value into their pages in the attention's own kernel */
@@ -141,11 +152,12 @@ int q3_attention_capped_decode_fused_bf16(const void* qkv, void* k_pages, void* 
                                           int nkv, float scale, float softcap, int chunk, int sink, int n_splits, void* stream);
 /* attention_prefill_tc.cu compiled with -DQ3_CAPPED=1: the tcgen05 prompt attention with capped scores, chunks and a sink
    (head sizes 64 and 128, values as wide as keys); arguments as q3_attention_prefill_tc_bf16 plus softcap, chunk, sink and
-   sink_values (one score per query head; may be null) */
+   sink_values (one score per query head; may be null).  Compiled with -DQ3_CAPPED=2: with biases by distance (see
+   q3_attention_generic) instead of a cap or chunks */
 int q3_attention_capped_prefill_tc_bf16(const void* q, const void* k_pages, const void* v_pages, void* out, const int* seq_start,
                                         const int* seq_pos0, const int* page_table, int pages_per_seq, int n_seqs, int max_new,
                                         int64_t n_tokens, int64_t n_cache_pages, int nq, int nkv, float scale, float softcap, int chunk,
-                                        int sink, const float* sink_values, int* status, void* stream);
+                                        int sink, const float* sink_values, const float* bias, int bias_count, int* status, void* stream);
 
 /* ---- attention_capped.cu (-DQ3_HEAD_DIM, -DQ3_VALUE_DIM): bfloat16 attention with scores capped by softcap * tanh(s / softcap)
    (0: none), chunked visibility (chunk 0: causal only), a sink term in the softmax's denominator, values of their own size */
@@ -155,10 +167,11 @@ int q3_attention_capped_prefill_bf16(const void* q, const void* k_pages, const v
                                      const int* seq_pos0, const int* page_table, int pages_per_seq, int n_seqs, int max_new, int nq,
                                      int nkv, float scale, float softcap, int chunk, int sink, int window, int value_heads,
                                      int out_f32, const float* sink_values, int keep_first,
-                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, void* stream);
+                             const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, const float* bias, int bias_count,
+                                     void* stream);
 /* (window > 0: a sliding window of that many keys instead of chunks, beside which the first keep_first keys of the sequence
    stay visible; value_heads 0 = nkv, else each value head serves nkv / value_heads key heads; out_f32: `out` is float;
-   sink_values (may be null): the sink's score per query head; pool_*: as for q3_attention_generic) */
+   sink_values (may be null): the sink's score per query head; pool_*, bias: as for q3_attention_generic) */
 /* one new token per sequence; scratch: n_tokens * nq * n_splits * (value_dim + 2) float32.  pool_write: the block that this token
    completes, if it does, is pooled here.  back_cos, back_sin [positions, value_dim / 2], may be null: every head of the output is
    turned back by the token's position; gate (may be null; rows gate_row apart): then multiplied by sigmoid(gate) (both for a
@@ -168,7 +181,8 @@ int q3_attention_capped_decode_bf16(const void* q, const void* k_pages, const vo
                                     int64_t n_tokens, int nq, int nkv, float scale, float softcap, int chunk, int sink, int n_splits,
                                     int window, int value_heads, int out_f32, const float* sink_values, int keep_first,
                              const void* pool_k, const void* pool_v, const int* pool_table, int pool_size, int pool_write,
-                                    const float* back_cos, const float* back_sin, const void* gate, int64_t gate_row, void* stream);
+                                    const float* back_cos, const float* back_sin, const void* gate, int64_t gate_row,
+                                    const float* bias, int bias_count, void* stream);
 
 /* ---- attention_decode.cu (-DQ3_HEAD_DIM): one new token per sequence, bfloat16 ---------------------------- */
 int q3_attention_decode_head_dim(void);
@@ -286,7 +300,7 @@ int q3_diff_combine_bf16(const float* a, void* out, int64_t n_tokens, int heads,
 /* ---- moe.cu: a routed feed-forward ---------------------------------------------------------------------------- */
 /* per token: float32 router logits, softmax, choice by score + correction within the kept groups, weights = scores;
    the outputs from n_real on are identity experts (their weights are summed into id_weight); by_logit: the largest logits
-   are chosen, weighted by the softmax over the chosen logits alone; gate_out (may be null): the router matrix has one more
+   are chosen, weighted by the softmax over the chosen logits alone (correction is then a bias on the logits); gate_out (may be null): the router matrix has one more
    row and gate_out[t] = sigmoid of its logit; by_logit 2: scores sigmoid(z) instead of the softmax; group_pair: a group's mark
    is the sum of its two best choice scores; the weights are multiplied by weight_scale; correction may be null */
 int q3_moe_route_f32(const void* h, const void* w_router, const float* correction, int* top_ids, float* top_w, float* id_weight,
@@ -318,7 +332,7 @@ int q3_moe_combine_bf16(const float* y, const void* h, const int* slot_of_pair, 
 
 /* ---- stream_shift.cu: a float32 hidden state with norms of several kinds, a token shift, a token side input ------ */
 /* one pass over the rows: stream += post(branch), out = pre(stream).  Norm kinds: 0 none, 1 unit rms times w, 2 dynamic tanh
-   tanh(alpha x) * w + b, 3 the rounded sum alone (pre only).  out_f32: `out` is float whatever the compute type.  With `rows`
+   tanh(alpha x) * w + b, 3 the rounded sum alone (pre only), 4 layer norm times w (no bias).  out_f32: `out` is float whatever the compute type.  With `rows`
    only those rows are read, nothing is written to the stream and out[r] belongs to rows[r] */
 int q3_settle_norm_f32(float* stream_rows, const void* branch, int post_kind, const float* post_w, const float* post_b,
                        float post_alpha, float post_eps, int pre_kind, const float* pre_w, const float* pre_b, float pre_alpha,
@@ -394,36 +408,57 @@ int q3_head_gate_bf16(void* x, const void* gate, int64_t gate_row, int heads, in
 
 /* ---- short_conv.cu ------------------------------------------------------------------------------------------- */
 /* y[t, c] = sum_j w[j, c] u[t - taps + 1 + j, c] (w [taps, channels]) within every sequence; rows before the step come from state
-   [slot][taps - 1][channels] (float32), which is moved on afterwards */
+   [slot][taps - 1][channels] (float32), which is moved on afterwards; bias [channels] (may be null) is added to the sum, silu: the
+   result goes through SiLU; single: every sequence brings one token (one launch instead of two) */
 int q3_short_conv_f32(const void* u, int64_t row_in, const float* w, float* state, int64_t slot_stride, const int* token_seq,
                       const int* seq_start, const int* seq_slots, void* y, int channels, int taps, int64_t n_tokens, int n_seqs,
-                      void* stream);
+                      const float* bias, int silu, int single, void* stream);
 int q3_short_conv_bf16(const void* u, int64_t row_in, const float* w, float* state, int64_t slot_stride, const int* token_seq,
                        const int* seq_start, const int* seq_slots, void* y, int channels, int taps, int64_t n_tokens, int n_seqs,
-                       void* stream);
+                      const float* bias, int silu, int single, void* stream);
 
 /* ---- linear_scan.cu: linear attention with keys ------------------------------------------------------------- */
 /* z <- sigmoid(z + bias)^inv_tau in place: the decays per key channel from their logits [n_tokens, width] */
 int q3_channel_decay(float* z, const float* bias, float inv_tau, int64_t n_tokens, int width, void* stream);
 /* S_t = diag(a_t) S_(t-1) + k_t (b_t v_t)^T, o_t = S_t^T (q_t q_scale); z given: the decays a per (token, channel), b = 1;
-   keep and write given: a and b per (token, head); ones: the state has a last column whose value is 1 */
+   keep and write given: a and b per (token, head); ones: the state has a last column whose value is 1.  dt_bias and a_log given
+   (state space): `keep` holds a logit z per (token, head), b = softplus(z + dt_bias), a = exp(-exp(a_log) b); skip (may be null):
+   skip_h v_t is added to the output; share: so many neighbouring heads read the same q and k; single: every sequence brings one
+   token (state rows of 16-byte packets) */
 int q3_decay_scan_f32(const void* q, const void* k, const void* v, int64_t row, const float* z,
                       const float* keep, const float* write, float q_scale, int ones, float* state, int64_t slot_stride,
-                      const int* seq_start, const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                      const int* seq_start, const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, int share,
+                       const float* dt_bias, const float* a_log, const float* skip, int single, void* stream);
 int q3_decay_scan_bf16(const void* q, const void* k, const void* v, int64_t row, const float* z,
                        const float* keep, const float* write, float q_scale, int ones, float* state, int64_t slot_stride,
-                       const int* seq_start, const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, void* stream);
+                       const int* seq_start, const int* seq_slots, float* out, int n_seqs, int heads, int d, int vd, int share,
+                       const float* dt_bias, const float* a_log, const float* skip, int single, void* stream);
 /* i = cap tanh((zi + bias_i) / cap), f = logsigmoid(cap tanh((zf + bias_f) / cap)), m_t = max(f_t + m_(t-1), i_t) from and to
    m_state; keep = exp(f + m_(t-1) - m_t), write = exp(i - m_t), low = exp(-m_t) */
 int q3_memory_gates(const float* zi, const float* zf, const float* bias_i, const float* bias_f, float cap, float* m_state,
                     int64_t slot_stride, const int* seq_start, const int* seq_slots, float* keep, float* write, float* low, int heads,
                     int64_t z_row, int n_seqs, void* stream);
+/* x = o * silu(gate), every one of `groups` equal parts of the row (size values) to unit rms by itself, times w */
+int q3_gate_group_norm_f32(const float* o, const void* gate, int64_t gate_row, const float* w, void* out, int64_t n_tokens, int size,
+                           int groups, float eps, void* stream);
+int q3_gate_group_norm_bf16(const float* o, const void* gate, int64_t gate_row, const float* w, void* out, int64_t n_tokens, int size,
+                            int groups, float eps, void* stream);
 /* per (token, head): x = o[:vd] (/ (max(|o[vd]|, low) + floor_add) if vdx > vd); out = x / sqrt(mean(x^2) + eps) * w * act(gate)
    (w null: no weight) */
 int q3_head_gated_norm_f32(const float* o, const float* low, float floor_add, const float* w, int w_per_head, const void* gate,
                            int64_t gate_row, void* out, int64_t n_tokens, int heads, int vd, int vdx, float eps, int act, void* stream);
 int q3_head_gated_norm_bf16(const float* o, const float* low, float floor_add, const float* w, int w_per_head, const void* gate,
                             int64_t gate_row, void* out, int64_t n_tokens, int heads, int vd, int vdx, float eps, int act, void* stream);
+
+/* ---- ssd.cu (-DQ3_STATE=n, -DQ3_VALUE_DIM=vd, multiples of 16 up to 256): a state space over bfloat16 prompts ---- */
+/* q3_decay_scan's state-space form (q = C, k = B, v = x) 64 tokens at a time on the tensor cores; segments > 1 (see
+   q3_ssd_segments): prompts of up to max_new tokens in so many stretches side by side, scratch then holds
+   n_seqs * segments * heads * (n * vd + 1) float32 */
+int q3_ssd_prompt_bf16(const void* x, const void* B, const void* C_rows, int64_t row, const float* z, const float* dt_bias,
+                       const float* a_log, const float* skip, float* state, int64_t slot_stride, const int* seq_start,
+                       const int* seq_slots, float* out, int n_seqs, int heads, int share, float* scratch, int max_new, int segments,
+                       void* stream);
+int q3_ssd_segments(int n_seqs, int max_new, int heads);
 
 /* ---- sampling.cu ------------------------------------------------------------------------------------------ */
 /* out[r] = index of the highest logit among the first `valid` (lowest id among equals, NaN as -inf) */
